@@ -155,8 +155,30 @@ typedef struct {
 } sptorch_gpt_config;
 #define SPT_ARCH_GPT 0
 #define SPT_ARCH_QWEN_LIKE 1
+#define SPT_ARCH_LAYERED 2      /* built from a list of layers: sptorch_ext_layered_create */
 
 void* sptorch_ext_gpt_create(const sptorch_gpt_config* cfg);       /* allocates weights + activations; NULL on failure */
+/* A decoder built from a list of layers that may differ in mixer, sizes and feed-forward.  The norm follows the sublayer:
+ * x += rms(mixer(x)) * w1, then (with a feed-forward) x += rms(mlp(x)) * w2; the residual stream is f32 in both dtypes, and f32 models
+ * run every product in f32.  The handle serves every sptorch_ext_gpt_* call except tensor parallelism and append = 0 decoding; any
+ * T >= 1 is accepted.  Of cfg, vocab, d_model, seq_len (positions a sequence may have), dtype, max_batch and eps are read.
+ * Parameter names: embed, l<i>.norm1, l<i>.norm2, l<i>.mix.*, l<i>.mlp.*, final.norm, head. */
+typedef struct {
+    int32_t mixer;                    /* SPT_MIXER_* */
+    int32_t heads, dim, vdim;         /* per head: query/key size (latent attention: its unrotated part) and value size */
+    int32_t decay_rank;               /* gated linear attention: rank of the decay projection */
+    float   tau;                      /* ... and the root of the sigmoid, alpha = sigmoid(z)^(1/tau) */
+    int32_t rot_dim, rope_dims;       /* latent attention: size of the rotated part, and how many of its dims rotate */
+    int32_t kv_rank, q_rank;          /* ... latent sizes of keys/values and of queries */
+    float   scale;                    /* ... factor of the scores */
+    double  rope_base;
+    int32_t mlp, d_ff;                /* SPT_MLP_* */
+} sptorch_layer_config;
+#define SPT_MIXER_GLA 0
+#define SPT_MIXER_LATENT 1
+#define SPT_MLP_NONE 0
+#define SPT_MLP_DENSE 1               /* down(up * silu(gate)), all three biased */
+void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const sptorch_layer_config* layers, int n_layers);
 void  sptorch_ext_gpt_destroy(void* gpt);
 /* name as in GPT::named_parameters (nn/src/lib.rs:1382-1392); host f32 values of the FULL
  * (unsharded) tensor; converted to the model dtype and sliced for this tp_rank on upload. */
@@ -197,6 +219,10 @@ int   sptorch_ext_gpt_cached_len(void* gpt);
 long long sptorch_ext_gpt_window_start(void* gpt);        /* absolute position of the oldest cached token (0 until the cache slides) */
 int   sptorch_ext_gpt_prefill(void* gpt, const void* ids_i32, int batch, int T, void* logits);
 int   sptorch_ext_gpt_decode(void* gpt, const void* last_ids_i32, int batch, int append, void* logits);
+/* The next portion of a prompt: ids [batch, T] continue the cached sequences (an empty cache: they start them), logits [batch*T, ld].
+ * Models built from a list of layers take any portion; the others a prefill first and then single tokens of one sequence. */
+int   sptorch_ext_gpt_extend(void* gpt, const void* ids_i32, int batch, int T, void* logits);
+int   sptorch_ext_gpt_reset_cache(void* gpt);             /* the cached sequences are finished: cache and state are free for the next ones */
 /* the attention of one new token over a cache (nn/src/lib.rs:706-760 without the projections): q [B, H*hd];
  * k_cache, v_cache [B, cache_positions, H*hd] of which the first n positions are valid; out [B, H*hd] */
 int   sptorch_ext_attention_last_token(const void* q, const void* k_cache, const void* v_cache, void* out, size_t B, size_t H, size_t hd,

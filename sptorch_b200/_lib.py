@@ -17,6 +17,12 @@ class GptConfig(C.Structure):
                 ("eps", C.c_float), ("tp_rank", C.c_int32), ("tp_size", C.c_int32), ("arch", C.c_int32), ("rope_base", C.c_float)]
 
 
+class LayerConfig(C.Structure):
+    _fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("decay_rank", C.c_int32), ("tau", C.c_float),
+                ("rot_dim", C.c_int32), ("rope_dims", C.c_int32), ("kv_rank", C.c_int32), ("q_rank", C.c_int32), ("scale", C.c_float),
+                ("rope_base", C.c_double), ("mlp", C.c_int32), ("d_ff", C.c_int32)]
+
+
 ALLREDUCE_FN = C.CFUNCTYPE(C.c_int, C.c_void_p, C.c_size_t, C.c_int, C.c_void_p, C.c_void_p)
 
 # name -> (restype, argtypes); the first 20 are the reference's C-ABI (include/sptorch_b200_hal.h)
@@ -89,6 +95,7 @@ EXT_SYMBOLS = {
     "sptorch_ext_attention_workspace": (_sz, [_sz, _sz, _sz, _sz, _i]),
     "sptorch_ext_attention_causal": (_i, [_vp, _vp, _vp, _vp, _vp, _sz, _sz, _sz, _sz, _sz, _i]),
     "sptorch_ext_gpt_create": (_vp, [C.POINTER(GptConfig)]),
+    "sptorch_ext_layered_create": (_vp, [C.POINTER(GptConfig), C.POINTER(LayerConfig), _i]),
     "sptorch_ext_gpt_destroy": (None, [_vp]),
     "sptorch_ext_gpt_set_param": (_i, [_vp, C.c_char_p, _vp, _sz]),
     "sptorch_ext_gpt_logits_ld": (_sz, [_vp]),
@@ -104,6 +111,8 @@ EXT_SYMBOLS = {
     "sptorch_ext_gpt_window_start": (C.c_longlong, [_vp]),
     "sptorch_ext_gpt_prefill": (_i, [_vp, _vp, _i, _i, _vp]),
     "sptorch_ext_gpt_decode": (_i, [_vp, _vp, _i, _i, _vp]),
+    "sptorch_ext_gpt_extend": (_i, [_vp, _vp, _i, _i, _vp]),
+    "sptorch_ext_gpt_reset_cache": (_i, [_vp]),
     "sptorch_ext_attention_last_token": (_i, [_vp, _vp, _vp, _vp, _sz, _sz, _sz, _sz, _sz, _i]),
     "sptorch_ext_gpt_launches": (_i, [_vp, _i, _i]),
     "sptorch_ext_gpt_enable_ln_fold": (_i, [_vp, _i]),

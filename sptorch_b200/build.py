@@ -62,10 +62,12 @@ def build(verbose: bool = False, force: bool = False) -> str:
         results = list(ex.map(compile_one, sources))
     objs = [o for o, _ in results]
     if force or any(changed for _, changed in results) or not os.path.exists(LIB):
-        cmd = [nvcc, *ARCH, "-shared", "-o", LIB, *objs, "-lcudart_static", "-ldl", "-lpthread", "-lrt"]
+        part = LIB + ".part"                     # a process that is killed here leaves no half-written library behind
+        cmd = [nvcc, *ARCH, "-shared", "-o", part, *objs, "-lcudart_static", "-ldl", "-lpthread", "-lrt"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+        os.replace(part, LIB)
     if verbose:
         for src, log in logs.items():
             sys.stdout.write(f"==== {src}\n{log}\n")

@@ -665,6 +665,9 @@ static int attn_npoly(int hd) {
     return hd == 64 ? e64 : e128;
 }
 
+bool attention_latent_supported(int D, int rot, int V, int kv_off, long long ld_q, long long ld_kv, int row) { (void)D; (void)rot; (void)V; (void)kv_off; (void)ld_q; (void)ld_kv; (void)row; return false; }
+int attention_latent(const void*, long long, const void*, const void*, long long, const void*, long long, long long, void*, long long, const void*, long long, int, int, int, int, int, int, int, int, float) { return fail("todo"); }
+
 // q, k, v: [B*T, ld] bf16, head h at columns h*hd (token-major: the layout the QKV projection writes);
 // out: [B*T, ld_out] bf16, head h at columns h*hd.
 int attention_fused(const void* q, const void* k, const void* v, void* out, int B, int T, int H, int hd, long long ld_q, long long ld_k,

@@ -819,14 +819,16 @@ int gemm_run(const GemmPlan& pl) {
 // ---------------- CUDA-core f32 matmul (exact-order mode and shapes TMA cannot express) ----------------
 // 64x64 output tile per CTA, 16x16 threads, 4x4 outputs per thread, K consumed in order p = 0..K-1 with
 // one fused multiply-add per product.
-__global__ void __launch_bounds__(256) simt_matmul_kernel(const float* __restrict__ A, const float* __restrict__ B, float* __restrict__ C,
+// Rows lda / ldb / ldc elements apart; batch z = z1 + nb1 * z2 with the strides of GemmDesc (R is laid out like C).
+struct SimtStrides { long long lda, ldb, ldc, sA1, sA2, sB1, sB2, sC1, sC2; int nb1; };
+__global__ void __launch_bounds__(256) simt_matmul_kernel(const float* __restrict__ A, const float* __restrict__ B, float* C,
                                                           int M, int N, int K, int b_is_kn, const float* __restrict__ bias,
-                                                          const float* __restrict__ R, float alpha, int epilogue) {
+                                                          const float* R, float alpha, int epilogue, const SimtStrides st) {
     __shared__ float As[16][64 + 1];
     __shared__ float Bs[16][64 + 1];
-    const int z = blockIdx.z;
-    A += (size_t)z * M * K; B += (size_t)z * N * K; C += (size_t)z * M * N;
-    if (R) R += (size_t)z * M * N;
+    const int z1 = blockIdx.z % st.nb1, z2 = blockIdx.z / st.nb1;
+    A += z1 * st.sA1 + z2 * st.sA2; B += z1 * st.sB1 + z2 * st.sB2; C += z1 * st.sC1 + z2 * st.sC2;
+    if (R) R += z1 * st.sC1 + z2 * st.sC2;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
     float acc[4][4] = {};
@@ -834,14 +836,14 @@ __global__ void __launch_bounds__(256) simt_matmul_kernel(const float* __restric
         for (int i = threadIdx.x; i < 64 * 16; i += 256) {
             int r = i / 16, c = i % 16;                 // A tile: 64 rows x 16 k
             int gm = m0 + r, gk = k0 + c;
-            As[c][r] = (gm < M && gk < K) ? A[(size_t)gm * K + gk] : 0.0f;
+            As[c][r] = (gm < M && gk < K) ? A[(size_t)gm * st.lda + gk] : 0.0f;
         }
         for (int i = threadIdx.x; i < 64 * 16; i += 256) {
             int gk, gn, kk, nn;
             if (b_is_kn) { kk = i / 64; nn = i % 64; } else { nn = i / 16; kk = i % 16; }
             gk = k0 + kk; gn = n0 + nn;
             float v = 0.0f;
-            if (gk < K && gn < N) v = b_is_kn ? B[(size_t)gk * N + gn] : B[(size_t)gn * K + gk];
+            if (gk < K && gn < N) v = b_is_kn ? B[(size_t)gk * st.ldb + gn] : B[(size_t)gn * st.ldb + gk];
             Bs[kk][nn] = v;
         }
         __syncthreads();
@@ -866,21 +868,33 @@ __global__ void __launch_bounds__(256) simt_matmul_kernel(const float* __restric
                 float v = acc[i][j] * alpha;
                 if (bias) v += bias[gn];
                 if (epilogue == EPI_GELU) v = gelu_exact(v);
-                if (epilogue == EPI_SWIGLU) { const float s_ = 1.0f / (1.0f + expf(-v)); v = R ? (R[(size_t)gm * N + gn] * v) * s_ : v * s_; }
-                else if (R) v += R[(size_t)gm * N + gn];
-                C[(size_t)gm * N + gn] = v;
+                if (epilogue == EPI_SWIGLU) { const float s_ = 1.0f / (1.0f + expf(-v)); v = R ? (R[(size_t)gm * st.ldc + gn] * v) * s_ : v * s_; }
+                else if (R) v += R[(size_t)gm * st.ldc + gn];
+                C[(size_t)gm * st.ldc + gn] = v;
             }
         }
 }
 
-int simt_matmul_f32(const float* A, const float* B, float* C, int batch, int M, int N, int K, bool b_is_kn, const float* bias,
-                    const float* R, float alpha, int epilogue) {
-    if (batch <= 0 || M <= 0 || N <= 0) return 0;
-    dim3 grid((unsigned)ceil_div(N, 64), (unsigned)ceil_div(M, 64), (unsigned)batch);
-    if (grid.y > 65535 || grid.z > 65535) return fail("simt_matmul: shape exceeds one launch (M tiles %u, batch %u)", grid.y, grid.z);
-    simt_matmul_kernel<<<grid, 256, 0, rt().stream>>>(A, B, C, M, N, K, b_is_kn ? 1 : 0, bias, R, alpha, epilogue);
+int simt_gemm_f32(const GemmDesc& d, bool b_is_kn) {
+    const long long batch = (long long)d.nb1 * d.nb2;
+    if (batch <= 0 || d.M <= 0 || d.N <= 0) return 0;
+    dim3 grid((unsigned)ceil_div(d.N, 64), (unsigned)ceil_div(d.M, 64), (unsigned)batch);
+    if (grid.y > 65535 || batch > 65535) return fail("simt_matmul: shape exceeds one launch (M tiles %u, batch %lld)", grid.y, batch);
+    const SimtStrides st = {d.lda, d.ldb, d.ldc, d.sA1, d.sA2, d.b_broadcast ? 0 : d.sB1, d.b_broadcast ? 0 : d.sB2, d.sC1, d.sC2, d.nb1};
+    simt_matmul_kernel<<<grid, 256, 0, rt().stream>>>((const float*)d.A, (const float*)d.B, (float*)d.C, d.M, d.N, d.K, b_is_kn ? 1 : 0, d.bias,
+                                                      (const float*)d.R, d.alpha, d.epilogue, st);
     SPT_LAUNCH_CHECK("simt_matmul");
     return 0;
+}
+
+int simt_matmul_f32(const float* A, const float* B, float* C, int batch, int M, int N, int K, bool b_is_kn, const float* bias,
+                    const float* R, float alpha, int epilogue) {
+    GemmDesc d;
+    d.A = A; d.B = B; d.C = C; d.bias = bias; d.R = R;
+    d.M = M; d.N = N; d.K = K; d.lda = K; d.ldb = b_is_kn ? N : K; d.ldc = N;
+    d.nb1 = batch; d.sA1 = (long long)M * K; d.sB1 = (long long)N * K; d.sC1 = (long long)M * N;
+    d.alpha = alpha; d.epilogue = epilogue; d.mode = MM_F32; d.out_dtype = F32;
+    return simt_gemm_f32(d, b_is_kn);
 }
 
 static std::atomic<int> g_abi_mode{MM_TF32};

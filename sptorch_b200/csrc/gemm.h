@@ -87,6 +87,9 @@ int norm_few_rows(const void* x, void* out, int rows, int K, const RowNorm& nrm,
 int simt_matmul_f32(const float* A, const float* B, float* C, int batch, int M, int N, int K, bool b_is_kn,
                     const float* bias, const float* R, float alpha, int epilogue);
 
+// the same for a GemmDesc with its strides and batch dims (f32 operands and output; b_is_kn: B is [K, N] with rows ldb apart)
+int simt_gemm_f32(const GemmDesc& d, bool b_is_kn = false);
+
 int layernorm_launch(const void* x, const void* gamma, const void* beta, void* out, size_t rows, size_t dim, float eps, int dtype);
 // LayerNorm folded into the following GEMM (GemmDesc::norm_axis): per-row statistics, and the folded weights / vectors
 bool layernorm_stats_supported(size_t dim, int dtype);

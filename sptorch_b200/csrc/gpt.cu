@@ -12,11 +12,8 @@
 // Tensor parallel (tp_size > 1): wq/wk/wv/ffn_up split by output rows (heads / d_ff columns), wo/ffn_down
 // split along K; each produces a partial [M,d] that a caller-supplied all-reduce sums.  Rank 0 alone folds
 // the residual and the ffn_down bias into its partial so that the reduced sum is the new residual stream.
-#include "gemm.h"
-#include "../../include/sptorch_b200_hal.h"
-#include "../../include/sptorch_b200_ext.h"
-#include <string>
-#include <vector>
+#include "gpt_model.h"
+#include "layered.h"
 #include <cstring>
 #include <cstdio>
 
@@ -41,76 +38,7 @@ int kv_append_launch(const void* qkv, void* kc, void* vc, int B, int dl, long lo
 int embedding_sum_launch(const void* tok_w, const void* pos_w, const void* ids, void* out, size_t n_tokens, size_t T, size_t vocab, size_t dim,
                          int dtype, const int* pos_row_dev);
 
-struct Layer {
-    float *ln1g, *ln1b, *ln2g, *ln2b, *b1, *b2;     // Qwen-like: ln1g / ln2g hold the RMSNorm weights, the betas are unused
-    void *wqkv;                                      // [Wq; Wk; Wv] of this rank, one [3*d_loc, d] matrix
-    void *wqk, *wv, *wo, *w1, *w2;                   // wqk = rows 0..2*d_loc of wqkv, wv = rows 2*d_loc..
-    void* wg = nullptr; float* bg = nullptr;         // Qwen-like: gate projection of the SwiGLU MLP
-    // LayerNorm folded into the GEMMs that consume it (bf16 GPT): weights times gamma, their row sums s, and c = W beta (+ bias)
-    void *wqkv_f = nullptr, *w1_f = nullptr;
-    float *s_qkv = nullptr, *c_qkv = nullptr, *s_1 = nullptr, *c_1 = nullptr;
-};
-
-struct Gpt {
-    sptorch_gpt_config c;
-    int es;                 // bytes per activation/weight element
-    int d_loc, H_loc, F_loc;
-    size_t ldl;             // logits row stride
-    void *tok, *pos, *head;
-    float *lnfg, *lnfb;
-    std::vector<Layer> L;
-    // activations for max_batch * seq_len tokens
-    void *x, *y, *h, *qkv, *ao, *f;                // qkv: [tokens, 3*d_loc] = [q | k | v] of every token
-    void *vt = nullptr, *scores = nullptr;          // materialised attention only (ensure_scores): V^T [d_loc, tokens], scores [batch, heads, T, T]
-    size_t scores_elems = 0, vt_elems = 0;
-    std::vector<void*> taps; bool taps_on = false;
-    sptorch_allreduce_fn ar = nullptr; void* ar_user = nullptr;
-    std::vector<void*> owned;
-    // pipelined host call
-    void* logits_dev[2] = {nullptr, nullptr}; int* ids_dev = nullptr; int ids_cap = 0; size_t logits_cap = 0;
-    cudaEvent_t ev_compute[2] = {nullptr, nullptr}, ev_copy[2] = {nullptr, nullptr};
-    cudaEvent_t ev_partial[2] = {nullptr, nullptr}, ev_reduced[2] = {nullptr, nullptr};     // tensor-parallel pipeline
-    // key/value cache for incremental decode: [layer][sequence][position][d_loc], allocated by gpt_enable_kv_cache
-    void *kcache = nullptr, *vcache = nullptr;
-    int cache_ctx = 0, cached_len = 0, cache_batch = 0;
-    long long window_start = 0;   // absolute position of the oldest cached token (grows once the cache is full and slides)
-    int* dstate = nullptr;        // device words of the current decode step: position, valid positions, ring slot, position-table row
-    struct DecodeKey {
-        const void* ids; void* logits; int batch, append; cudaStream_t stream; uint64_t epoch;
-        bool operator==(const DecodeKey& o) const { return ids == o.ids && logits == o.logits && batch == o.batch && append == o.append && stream == o.stream && epoch == o.epoch; }
-    };
-    DecodeKey dkey = {nullptr, nullptr, 0, 0, nullptr, 0};
-    cudaGraphExec_t dexec = nullptr; int d_eager = 0;
-    bool fill_cache = false;      // set while a prefill runs
-    void *dq = nullptr;                  // decode scratch: [max_batch, 3*d_loc] = [q | k | v] of the new tokens
-    // CUDA graph of one forward, keyed by everything that is baked into its kernel arguments
-    // (the config epoch covers the process-wide setters that change which kernels or grids a forward launches)
-    struct GraphKey {
-        const void* ids; void* logits; int batch, T; bool taps; cudaStream_t stream; uint64_t epoch;
-        const void *targets, *argmax, *row_loss; int has_ignore; long long ignore_index; bool reduce;      // fused LM head (HeadReduce)
-        bool operator==(const GraphKey& o) const {
-            return ids == o.ids && logits == o.logits && batch == o.batch && T == o.T && taps == o.taps && stream == o.stream && epoch == o.epoch &&
-                   targets == o.targets && argmax == o.argmax && row_loss == o.row_loss && has_ignore == o.has_ignore &&
-                   ignore_index == o.ignore_index && reduce == o.reduce;
-        }
-    };
-    // a few keys are kept so that callers alternating between buffers (double buffering) replay instead of re-capturing
-    struct GraphSlot { GraphKey key; cudaGraphExec_t exec = nullptr; int eager_runs = 0; uint64_t last_use = 0; };
-    static constexpr int kGraphSlots = 4;
-    GraphSlot gslots[kGraphSlots];
-    uint64_t guse = 0;
-    bool graphs = true;
-    // folded LayerNorm (see forward): per-token statistics, the head's folded copy, and whether the copies are stale
-    float2* ln_stats = nullptr; void* head_f = nullptr; float *s_h = nullptr, *c_h = nullptr;
-    bool ln_fold = false, fold_ready = false, fold_dirty = true;     // opt-in: measured neutral (see sptorch_ext_gpt_enable_ln_fold)
-    int tp_overlap = 2;        // tensor parallel: reduce one half of the batch while the other half computes: 0 never, 1 always, 2 from 4 ranks up
-    // LM head fused with the loss / greedy choice: per-row partial reductions of the head GEMM's tiles
-    float2* red_part = nullptr; int* red_arg = nullptr; float* red_tgt = nullptr; size_t red_rows = 0;
-    // host-buffer loss call: targets, greedy tokens and row losses of the whole batch on the device
-    long long* loss_targets = nullptr; int* loss_argmax = nullptr; float* loss_rows = nullptr; size_t loss_cap = 0;
-};
-
-static void drop_graphs(Gpt* g) {
+void drop_graphs(Gpt* g) {
     if (g->dexec) { cudaGraphExecDestroy(g->dexec); g->dexec = nullptr; }
     g->d_eager = 0;
     for (auto& sl : g->gslots) {
@@ -120,20 +48,20 @@ static void drop_graphs(Gpt* g) {
 }
 
 // returns a block of the model to the pool before the model itself goes (buffers that are re-allocated larger)
-static void gfree(Gpt* g, void* p) {
+void gfree(Gpt* g, void* p) {
     if (!p) return;
     for (auto it = g->owned.begin(); it != g->owned.end(); ++it)
         if (*it == p) { g->owned.erase(it); break; }
     sptorch_free(p);
 }
 
-static void* galloc(Gpt* g, size_t bytes) {
+void* galloc(Gpt* g, size_t bytes) {
     void* p = sptorch_ext_alloc_bytes(bytes);
     if (p) g->owned.push_back(p);
     return p;
 }
 
-static int upload_rows(Gpt* g, void* dst_model_dtype, const float* host, size_t n) {
+int upload_rows(Gpt* g, void* dst_model_dtype, const float* host, size_t n) {
     // host f32 -> device in the model dtype (bf16: round to nearest even on the device)
     if (g->c.dtype == SPT_F32) return sptorch_ext_copy_h2d_bytes(host, dst_model_dtype, n * 4);
     float* tmp = (float*)sptorch_ext_alloc_bytes(n * 4);
@@ -218,18 +146,23 @@ static int upload_shard(Gpt* g, void* dst, const char* name, const float* host, 
     return upload_rows(g, dst, src, n);
 }
 
+// one product timed as a projection: the tensor cores, or f32 multiply-adds on the CUDA cores for MM_F32
+int gemm_or_simt(const GemmDesc& d) {
+    ProfScope ps(PROF_LINEAR);
+    if (d.mode == MM_F32) return simt_gemm_f32(d);
+    GemmPlan pl;
+    return gemm_plan(d, &pl) || gemm_run(pl);
+}
+
 static int linear(Gpt* g, const void* x, const void* w, const float* bias, const void* res, void* out, int M, int K, int N,
                   long long ldo, int epi) {
     GemmDesc d;
     d.A = x; d.B = w; d.C = out; d.bias = bias; d.R = res;
     d.M = M; d.N = N; d.K = K; d.lda = K; d.ldb = K; d.ldc = ldo;
     d.epilogue = epi;
-    d.mode = g->c.dtype == SPT_BF16 ? MM_BF16 : MM_TF32;
+    d.mode = g->c.dtype == SPT_BF16 ? MM_BF16 : g->lay ? MM_F32 : MM_TF32;
     d.out_dtype = g->c.dtype;
-    GemmPlan pl;
-    if (gemm_plan(d, &pl)) return 1;
-    ProfScope ps(PROF_LINEAR);
-    return gemm_run(pl);
+    return gemm_or_simt(d);
 }
 
 static int ln(const void* x, const float* g_, const float* b_, void* out, size_t rows, size_t dim, float eps, int dt) {
@@ -367,10 +300,6 @@ static int attention_block(Gpt* g, const Layer& w, int l, const void* h, void* q
     return attention_materialized(qp, kp, g->vt, /*vt_ld*/ M, /*head*/ (long long)hd * M, /*batch*/ T, ao, g->scores, B, T, Hl, hd, 3 * dl, dl, dt);
 }
 
-// What replaces the logits when the LM head is fused with the step after it (cross_entropy_loss(_ignore_index), core-ops/src/lib.rs:1079-1194;
-// the greedy token = first candidate of sampling_candidates, nn/src/lib.rs:2381-2418): per-row loss and / or the column of the row maximum.
-struct HeadReduce { const long long* targets; int has_ignore; long long ignore_index; int* argmax; float* row_loss; };
-
 // partial-reduction buffers for `rows` tokens (grown outside any graph capture)
 static int ensure_reduce(Gpt* g, size_t rows) {
     if (rows <= g->red_rows) return 0;
@@ -386,13 +315,14 @@ static int ensure_reduce(Gpt* g, size_t rows) {
 }
 
 // logits = h head^T, or -- with hr -- the row reductions of that product without the [M, vocab] matrix ever reaching HBM
-static int lm_head(Gpt* g, const void* h, int M, void* logits, const HeadReduce* hr) {
+int lm_head(Gpt* g, const void* h, int M, void* logits, const HeadReduce* hr) {
     const sptorch_gpt_config& c = g->c;
-    if (!hr) return linear(g, h, g->head, nullptr, nullptr, logits, M, c.d_model, c.vocab, (long long)g->ldl, EPI_NONE);
+    const int K = g->lay ? g->lay->d8 : c.d_model;                  // models built from a list of layers pad their rows
+    if (!hr) return linear(g, h, g->head, nullptr, nullptr, logits, M, K, c.vocab, (long long)g->ldl, EPI_NONE);
     if ((size_t)M > g->red_rows) return fail("gpt: reduction buffers not prepared for %d rows", M);
     GemmDesc d;
     d.A = h; d.B = g->head; d.C = nullptr;
-    d.M = M; d.N = c.vocab; d.K = c.d_model; d.lda = c.d_model; d.ldb = c.d_model; d.ldc = (long long)g->ldl;
+    d.M = M; d.N = c.vocab; d.K = K; d.lda = K; d.ldb = K; d.ldc = (long long)g->ldl;
     d.mode = c.dtype == SPT_BF16 ? MM_BF16 : MM_TF32; d.out_dtype = c.dtype;
     d.reduce = 1; d.red_part = g->red_part; d.red_arg = g->red_arg; d.red_targets = hr->row_loss ? hr->targets : nullptr; d.red_tgt = g->red_tgt;
     GemmPlan pl;
@@ -527,6 +457,7 @@ static int forward_qwen(Gpt* g, const void* ids, int B, int T, void* logits, con
 }
 
 static int forward(Gpt* g, const void* ids, int B, int T, void* logits, const HeadReduce* hr = nullptr) {
+    if (g->lay) return layered_forward(g, ids, B, T, 0, false, logits, hr);
     if (g->c.arch == SPT_ARCH_QWEN_LIKE) return forward_qwen(g, ids, B, T, logits, hr);
     const bool overlap = g->tp_overlap == 1 || (g->tp_overlap == 2 && g->c.tp_size >= kTpOverlapFromRanks);
     if (g->c.tp_size > 1 && g->ar && overlap && !g->taps_on && !g->fill_cache && B >= 2 && B % 2 == 0 && model_uses_fused(g, T))
@@ -590,8 +521,8 @@ static int forward(Gpt* g, const void* ids, int B, int T, void* logits, const He
 }
 
 // GPT::named_parameters (nn/src/lib.rs:1382-1392) / QwenLikeGPT::named_parameters (:1483-1492) with the full (unsharded) shapes
-struct ParamInfo { std::string name; std::vector<size_t> shape; };
 std::vector<ParamInfo> gpt_param_table(void* gp) {
+    if (((Gpt*)gp)->lay) return layered_param_table((Gpt*)gp);
     const sptorch_gpt_config& c = ((Gpt*)gp)->c;
     const size_t d = c.d_model, V = c.vocab, S = c.seq_len, F = c.d_ff;
     const bool qwen = c.arch == SPT_ARCH_QWEN_LIKE;
@@ -630,6 +561,7 @@ void* sptorch_ext_gpt_create(const sptorch_gpt_config* cfg) {
         fail("gpt_create: non-positive dimension"); return nullptr;
     }
     if (c.dtype != SPT_F32 && c.dtype != SPT_BF16) { fail("gpt_create: unknown dtype %d", c.dtype); return nullptr; }
+    if (c.arch == SPT_ARCH_LAYERED) { fail("gpt_create: a model built from a list of layers is created by sptorch_ext_layered_create"); return nullptr; }
     if (c.arch != SPT_ARCH_GPT && c.arch != SPT_ARCH_QWEN_LIKE) { fail("gpt_create: unknown architecture %d", c.arch); return nullptr; }
     if (c.arch == SPT_ARCH_QWEN_LIKE && !(c.rope_base > 0.0f)) c.rope_base = 10000.0f;
     if (c.d_model % c.n_head) { fail("gpt_create: d_model %% n_head != 0"); return nullptr; }
@@ -680,6 +612,7 @@ void sptorch_ext_gpt_destroy(void* gp) {
             if (g->ev_reduced[i]) cudaEventDestroy(g->ev_reduced[i]);
         }
     }
+    layered_release(g);
     delete g;
 }
 
@@ -687,6 +620,7 @@ int sptorch_ext_gpt_set_param(void* gp, const char* name, const float* host, siz
     if (enter()) return 1;
     if (!gp || !name || !host) return fail("gpt_set_param: null argument");
     Gpt* g = (Gpt*)gp;
+    if (g->lay) return layered_set_param(g, name, host, n);
     const sptorch_gpt_config& c = g->c;
     const size_t d = c.d_model, V = c.vocab, S = c.seq_len, F = c.d_ff, dl = g->d_loc, Fl = g->F_loc, es = g->es;
     auto need = [&](size_t want) { return n == want ? 0 : fail("gpt_set_param(%s): got %zu values, expected %zu", name, n, want); };
@@ -736,6 +670,7 @@ static int check_shape(Gpt* g, int batch, int T) {
     if (batch <= 0 || T <= 0) return fail("gpt_forward: empty batch or sequence");
     if (T > g->c.seq_len) return fail("gpt_forward: T=%d exceeds seq_len=%d", T, g->c.seq_len);   // nn/src/lib.rs:1351 asserts the same
     if ((size_t)batch * T > (size_t)g->c.max_batch * g->c.seq_len) return fail("gpt_forward: batch*T exceeds the activation capacity");
+    if (g->lay) return layered_prepare(g, batch, T, 0, false);
     if (ensure_scores(g, batch, T)) return 1;      // outside any graph capture
     const int vec = 16 / g->es;
     if (T % vec) return fail("gpt_forward: T must be a multiple of %d for this dtype", vec);
@@ -798,6 +733,7 @@ int sptorch_ext_gpt_forward(void* gp, const void* ids, int batch, int T, void* l
 static int check_reduce(Gpt* g, const char* who) {
     if (g->c.vocab <= 128) return fail("%s: the fused LM head needs a vocabulary larger than 128", who);
     if (g->c.tp_size > 1) return fail("%s: not available with tensor parallel shards", who);
+    if (g->lay && g->c.dtype != SPT_BF16) return fail("%s: f32 models built from a list of layers take no reduced-precision product", who);
     return 0;
 }
 
@@ -881,6 +817,8 @@ int sptorch_ext_gpt_enable_kv_cache(void* gp, int max_context) {
     if (g->c.tp_size > 1) return fail("gpt_enable_kv_cache: not available with tensor parallel shards");
     if (max_context <= 0 || max_context > g->c.seq_len) max_context = g->c.seq_len;     // learned positions end at seq_len; forward_ids asserts it for both models
     if (g->kcache) return max_context == g->cache_ctx ? 0 : fail("gpt_enable_kv_cache: cache already allocated with %d positions", g->cache_ctx);
+    if (g->lay) return g->cache_ctx ? (max_context == g->cache_ctx ? 0 : fail("gpt_enable_kv_cache: cache already allocated with %d positions", g->cache_ctx))
+                                    : layered_enable_cache(g, max_context);
     const size_t bytes = (size_t)g->c.n_layer * g->c.max_batch * max_context * g->d_loc * g->es;
     g->kcache = galloc(g, bytes); g->vcache = galloc(g, bytes);
     g->dq = galloc(g, (size_t)g->c.max_batch * 3 * g->d_loc * g->es);
@@ -899,7 +837,8 @@ int sptorch_ext_gpt_prefill(void* gp, const void* ids, int batch, int T, void* l
     if (enter()) return 1;
     if (!gp || !ids || !logits) return fail("gpt_prefill: null argument");
     Gpt* g = (Gpt*)gp;
-    if (!g->kcache) return fail("gpt_prefill: call sptorch_ext_gpt_enable_kv_cache first");
+    if (!g->cache_ctx) return fail("gpt_prefill: call sptorch_ext_gpt_enable_kv_cache first");
+    if (g->lay) return layered_reset_cache(g) || sptorch_ext_gpt_extend(gp, ids, batch, T, logits);
     if (check_shape(g, batch, T)) return 1;
     if (T > g->cache_ctx) return fail("gpt_prefill: T=%d exceeds the cache of %d positions", T, g->cache_ctx);
     g->fill_cache = true;
@@ -907,6 +846,42 @@ int sptorch_ext_gpt_prefill(void* gp, const void* ids, int batch, int T, void* l
     g->fill_cache = false;
     if (rc) return rc;
     g->cached_len = T; g->cache_batch = batch; g->window_start = 0;
+    return 0;
+}
+
+int sptorch_ext_gpt_reset_cache(void* gp) {
+    if (enter()) return 1;
+    if (!gp) return fail("gpt_reset_cache: null model");
+    Gpt* g = (Gpt*)gp;
+    if (!g->cache_ctx) return fail("gpt_reset_cache: call sptorch_ext_gpt_enable_kv_cache first");
+    if (g->lay) return layered_reset_cache(g);
+    g->cached_len = 0; g->cache_batch = 0; g->window_start = 0;
+    return 0;
+}
+
+// The next portion of every sequence: T tokens each at positions cached_len .., which the cache or state then holds.
+int sptorch_ext_gpt_extend(void* gp, const void* ids, int batch, int T, void* logits) {
+    if (enter()) return 1;
+    if (!gp || !ids || !logits) return fail("gpt_extend: null argument");
+    Gpt* g = (Gpt*)gp;
+    if (!g->cache_ctx) return fail("gpt_extend: call sptorch_ext_gpt_enable_kv_cache first");
+    if (batch <= 0 || T <= 0) return fail("gpt_extend: empty batch or portion");
+    if (batch > g->c.max_batch) return fail("gpt_extend: batch %d exceeds max_batch %d", batch, g->c.max_batch);
+    if (g->cached_len > 0 && batch != g->cache_batch) return fail("gpt_extend: batch %d differs from the cached batch %d", batch, g->cache_batch);
+    if (!g->lay) {
+        // learned positions / rotated keys: the first portion is a prefill where its length allows, the rest goes token by token
+        if (g->cached_len == 0) return sptorch_ext_gpt_prefill(gp, ids, batch, T, logits);
+        if (batch != 1) return fail("gpt_extend: portions after the first take one sequence for this model");
+        for (int t = 0; t < T; t++)
+            if (sptorch_ext_gpt_decode(gp, (const int*)ids + t, 1, 1, (uint8_t*)logits + (size_t)t * g->ldl * g->es)) return 1;
+        return 0;
+    }
+    if (g->cached_len + T > g->cache_ctx) return fail("gpt_extend: %d cached positions and %d more exceed the cache of %d", g->cached_len, T, g->cache_ctx);
+    if (layered_prepare(g, batch, T, g->cached_len, true)) return 1;
+    const int rc = layered_takes_few_rows(g, batch * T, T) ? layered_few_rows(g, ids, batch, T, nullptr, g->cached_len, logits)
+                                                           : layered_forward(g, ids, batch, T, g->cached_len, true, logits, nullptr);
+    if (rc) return rc;
+    g->cached_len += T; g->cache_batch = batch;
     return 0;
 }
 
@@ -955,6 +930,8 @@ static int decode_linear(Gpt* g, const void* x, const RowNorm* nrm, const void* 
 }
 
 static int decode_launches(Gpt* g, const void* last_ids, int B, int append, void* logits) {
+    if (g->lay) return layered_takes_few_rows(g, B, 1) ? layered_few_rows(g, last_ids, B, 1, g->dstate, 0, logits)
+                                                       : layered_forward(g, last_ids, B, 1, g->cached_len, true, logits, nullptr);
     const sptorch_gpt_config& c = g->c;
     const int d = c.d_model, dl = g->d_loc, Fl = g->F_loc, hd = d / c.n_head, dt = c.dtype;
     const size_t es = g->es;
@@ -998,13 +975,19 @@ int sptorch_ext_gpt_decode(void* gp, const void* last_ids, int batch, int append
     if (!gp || !last_ids || !logits) return fail("gpt_decode: null argument");
     Gpt* g = (Gpt*)gp;
     const sptorch_gpt_config& c = g->c;
-    if (!g->kcache || g->cached_len <= 0) return fail("gpt_decode: the cache is empty (prefill first)");
+    if (!g->cache_ctx || g->cached_len <= 0) return fail("gpt_decode: the cache is empty (prefill first)");
     if (batch != g->cache_batch) return fail("gpt_decode: batch %d differs from the cached batch %d", batch, g->cache_batch);
     // The cache is a ring over absolute positions (slot = position % capacity): once it is full an appended token takes the slot
     // of the oldest one, which is how append_kv_tensor (nn/src/lib.rs:2165-2203) keeps the last max_context positions; the window
     // start then moves on by one (KvCacheWindowState::append, hal/src/lib.rs:129-239).  The attention reads the n valid slots;
     // their order in memory does not matter to a softmax-weighted sum.
     const bool full = g->cached_len >= g->cache_ctx;
+    if (g->lay) {
+        // every layer sees all earlier tokens and the recurrent state has already taken the last one in
+        if (!append) return fail("gpt_decode: this model cannot recompute the logits of a token its state already holds");
+        if (full) return fail("gpt_decode: the cache of %d positions is full", g->cache_ctx);
+        if (layered_prepare(g, batch, 1, g->cached_len, true)) return 1;
+    }
     const long long apos = append ? g->window_start + g->cached_len : g->window_start + g->cached_len - 1;   // absolute position of the token
     if (apos > INT32_MAX) return fail("gpt_decode: position overflow");
     const int pos = (int)apos;
@@ -1015,7 +998,7 @@ int sptorch_ext_gpt_decode(void* gp, const void* last_ids, int batch, int append
     // Replay: a decode step is about a hundred small launches, host-bound when issued one by one.  The first step of a key runs
     // eagerly, the second is captured, later ones are one cudaGraphLaunch.
     Gpt::DecodeKey key = {last_ids, logits, batch, append, rt().stream, config_epoch()};
-    const bool graph_ok = g->graphs && !prof_enabled();
+    const bool graph_ok = g->graphs && !prof_enabled() && !(g->lay && (g->taps_on || !layered_takes_few_rows(g, batch, 1)));
     int rc;
     if (!graph_ok) rc = decode_launches(g, last_ids, batch, append, logits);
     else {
@@ -1078,7 +1061,7 @@ int sptorch_ext_gpt_enable_taps(void* gp, int on) {
     if (!gp) return fail("gpt_enable_taps: null model");
     Gpt* g = (Gpt*)gp;
     if (on && g->taps.empty()) {
-        size_t bytes = (size_t)g->c.max_batch * g->c.seq_len * g->c.d_model * g->es;
+        size_t bytes = (size_t)g->c.max_batch * g->c.seq_len * g->c.d_model * (g->lay ? 4 : g->es);      // models built from a list of layers: the f32 residual stream
         for (int i = 0; i < g->c.n_layer + 2; i++) {
             void* p = galloc(g, bytes);
             if (!p) return 1;
@@ -1104,7 +1087,7 @@ int sptorch_ext_gpt_set_allreduce(void* gp, sptorch_allreduce_fn fn, void* user)
 int sptorch_ext_gpt_launches(void* gp, int batch, int T) {
     if (!gp) return 0;
     Gpt* g = (Gpt*)gp;
-    (void)batch;
+    if (g->lay) return layered_launches(g, batch, T);
     const bool fused = model_uses_fused(g, T);
     // embedding + per layer (LN1, QKV, attention [1 fused | V^T, S, softmax, PV], Wo, LN2, up, down) + ln_f + head;
     // the Qwen-like block adds the RoPE pass and the gate projection

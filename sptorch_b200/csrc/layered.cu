@@ -1,0 +1,539 @@
+// layered.cu -- driver of the models built from a list of layers.  Each layer has its own mixer (gated linear attention, latent
+// attention), sizes and optional feed-forward, and normalises the OUTPUT of a sublayer before it joins the residual stream:
+//   x <- x + rms(mixer(x)) w1;   x <- x + rms(mlp(x)) w2;   logits = head (rms(x) wf)
+// The residual stream x is f32; the sublayers read a copy of it in the model dtype (xb), which the kernel that updates x writes beside
+// it.  Launches of a prompt (bf16), per layer:
+//   gated linear attention: one GEMM for q, k, v, gate and decay latent | chunk kernels (gla.cu) | W_o | post-norm
+//   latent attention: one GEMM for query latent, key/value latent and head gates | latent norms and rotation | W_uq | rotation of q |
+//                     keys and values of every position from the latents (one GEMM) | fused attention | W_o | post-norm
+//   feed-forward: W_up (+bias) | W_gate (+bias, SwiGLU product) | W_down (+bias) | post-norm
+// A few tokens (a decode step, a short portion of a prompt) take the weight-streaming projections, the token-by-token recurrence and
+// attention over the cached latents themselves; all of these are programmatic dependents of one another.
+// f32 models run every product as f32 multiply-adds (MM_F32), the recurrence token by token and the latent attention unexpanded.
+#include "layered.h"
+#include "pdl.cuh"
+#include <cmath>
+#include <cstdio>
+#include <cstring>
+#include <map>
+
+namespace spt {
+
+bool attention_latent_supported(int D, int rot, int V, int kv_off, long long ld_q, long long ld_kv, int row);
+int attention_latent(const void* q, long long ld_q, const void* kn, const void* v, long long ld_kv, const void* kr, long long row, long long seq_stride,
+                     void* out, long long ld_out, const void* gate, long long ld_gate, int B, int T, int n, int H, int D, int rot, int V, int first, float scale);
+
+namespace {
+
+// x = embed[id] in f32 and in the model dtype; an id outside the vocabulary gives a zero row and raises the status word
+template <typename T>
+__global__ void __launch_bounds__(128) embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x, T* __restrict__ xb, int vocab,
+                                                         int ld, uint32_t* status) {
+    pdl_release();
+    pdl_acquire();
+    const int m = blockIdx.x, id = ids[m];
+    const bool ok = id >= 0 && id < vocab;
+    if (!ok && threadIdx.x == 0) atomicOr(status, 0x100u);
+    const T* src = table + (size_t)(ok ? id : 0) * ld;
+    for (int i = threadIdx.x; i < ld; i += 128) {
+        const T v = ok ? src[i] : (T)0.0f;
+        x[(size_t)m * ld + i] = (float)v;
+        xb[(size_t)m * ld + i] = v;
+    }
+}
+
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; i++) { const float2 f = bf16x2_to_float2(h[i]); v[2 * i] = f.x; v[2 * i + 1] = f.y; }
+}
+__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
+    uint4 raw;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; i++) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p) = raw;
+}
+
+template <int THREADS>
+__device__ __forceinline__ float row_sum(float v, float* sh) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    if (THREADS == 32) return v;
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.0f;
+#pragma unroll
+    for (int w = 0; w < THREADS / 32; w++) s += sh[w];
+    return s;
+}
+
+// One CTA per row, NV groups of eight elements per thread in registers.  HBM bytes per element: y + 4 (x in) + 4 (x out) + xb.
+template <typename T, int THREADS, int NV>
+__global__ void __launch_bounds__(THREADS) post_norm_kernel(const float* x, const T* __restrict__ y, const float* __restrict__ w, const float* __restrict__ w2,
+                                                            float* x_out, T* __restrict__ xb, int dim, int ld, float eps) {
+    __shared__ float sh[THREADS / 32];
+    pdl_release();
+    pdl_acquire();
+    const size_t base = (size_t)blockIdx.x * ld;
+    float xv[NV][8], yv[NV][8];
+    float sq = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int c = (i * THREADS + (int)threadIdx.x) * 8;
+        if (c < ld) {
+            load8(x + base + c, xv[i]);
+            if (y) {
+                load8(y + base + c, yv[i]);
+#pragma unroll
+                for (int j = 0; j < 8; j++) sq = fmaf(yv[i][j], yv[i][j], sq);
+            }
+        }
+    }
+    if (y) {
+        const float inv = 1.0f / sqrtf(row_sum<THREADS>(sq, sh) / (float)dim + eps);
+#pragma unroll
+        for (int i = 0; i < NV; i++) {
+            const int c = (i * THREADS + (int)threadIdx.x) * 8;
+            if (c < ld) {
+                float g[8];
+                load8(w + c, g);
+#pragma unroll
+                for (int j = 0; j < 8; j++) xv[i][j] += yv[i][j] * inv * g[j];
+            }
+        }
+    }
+    float inv2 = 1.0f;
+    if (w2) {
+        float s2 = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+            if ((i * THREADS + (int)threadIdx.x) * 8 < ld) {
+#pragma unroll
+                for (int j = 0; j < 8; j++) s2 = fmaf(xv[i][j], xv[i][j], s2);
+            }
+        inv2 = 1.0f / sqrtf(row_sum<THREADS>(s2, sh) / (float)dim + eps);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+        const int c = (i * THREADS + (int)threadIdx.x) * 8;
+        if (c < ld) {
+            if (x_out) store8(x_out + base + c, xv[i]);
+            if (w2) {
+                float g[8];
+                load8(w2 + c, g);
+#pragma unroll
+                for (int j = 0; j < 8; j++) xv[i][j] = xv[i][j] * inv2 * g[j];
+            }
+            store8(xb + base + c, xv[i]);
+        }
+    }
+}
+
+template <typename T>
+int post_norm_t(const float* x, const void* y, const float* w, const float* w2, float* x_out, void* xb, int rows, int dim, int ld, float eps, bool dependent) {
+    const int vecs = ld / 8;
+#define SPT_POST_NORM(TH_, NV_)                                                                                                                   \
+    SPT_CUDA(launch_dependent(post_norm_kernel<T, TH_, NV_>, dim3(rows), dim3(TH_), 0, dependent, 1, x, static_cast<const T*>(y), w, w2, x_out,       \
+                              static_cast<T*>(xb), dim, ld, eps))
+    if (vecs <= 32) SPT_POST_NORM(32, 1);
+    else if (vecs <= 128) SPT_POST_NORM(128, 1);
+    else if (vecs <= 256) SPT_POST_NORM(128, 2);
+    else if (vecs <= 512) SPT_POST_NORM(256, 2);
+    else if (vecs <= 2048) SPT_POST_NORM(512, 4);
+    else return fail("post_norm: width %d is larger than 16384", dim);
+#undef SPT_POST_NORM
+    note_submit();
+    return 0;
+}
+
+}  // namespace
+
+int post_norm_launch(const float* x, const void* y, const float* w, const float* w2, float* x_out, void* xb, int rows, int dim, int ld, float eps,
+                     int dtype, bool dependent) {
+    ProfScope ps(PROF_LAYERNORM);
+    return dtype == BF16 ? post_norm_t<__nv_bfloat16>(x, y, w, w2, x_out, xb, rows, dim, ld, eps, dependent)
+                         : post_norm_t<float>(x, y, w, w2, x_out, xb, rows, dim, ld, eps, dependent);
+}
+
+namespace {
+
+int ensure(Gpt* g, LayeredScratch* s, size_t bytes) {
+    if (bytes <= s->bytes) return 0;
+    if (s->p) { if (stream_wait()) return 1; drop_graphs(g); gfree(g, s->p); }
+    s->p = galloc(g, bytes);
+    s->bytes = s->p ? bytes : 0;
+    if (!s->p) return 1;
+    return sptorch_ext_memset(s->p, 0, bytes);
+}
+
+// out[M, N] = act(a W^T + bias) (* r for the SwiGLU product); rows of a are lda apart and read for K elements, W is [N, ldw]
+int product(Gpt* g, bool few, const void* a, long long lda, const void* w, long long ldw, int K, const float* bias, const void* r, void* out, long long ldo,
+            int M, int N, int epi) {
+    GemmDesc d;
+    d.A = a; d.B = w; d.C = out; d.bias = bias; d.R = r;
+    d.M = M; d.N = N; d.K = K; d.lda = lda; d.ldb = ldw; d.ldc = ldo;
+    d.epilogue = epi; d.mode = g->c.dtype == BF16 ? MM_BF16 : MM_F32; d.out_dtype = g->c.dtype;
+    if (few && linear_few_rows_supported(d)) { ProfScope ps(PROF_LINEAR); return linear_few_rows(d, nullptr, true); }
+    return gemm_or_simt(d);
+}
+
+GlaArgs gla_args(Gpt* g, const LayeredLayer& w, int B, int T, bool cached) {
+    GlaArgs a = {};
+    a.in = g->lay->in.p; a.ld = w.n_in;
+    a.c_q = w.c_q; a.c_k = w.c_k; a.c_v = w.c_v; a.c_g = w.c_g; a.c_a = w.c_a;
+    a.B = B; a.T = T; a.H = w.c.heads; a.D = w.c.dim; a.V = w.c.vdim; a.R = w.c.decay_rank;
+    a.a2 = w.a2; a.a2_b = w.a2_b; a.head_norm = w.head_norm;
+    a.tau = w.c.tau; a.eps = g->c.eps;
+    a.state = cached ? w.state : nullptr;
+    a.out = g->lay->ao.p; a.ld_out = w.o_ld();
+    a.dtype = g->c.dtype;
+    return a;
+}
+
+LatentArgs latent_args(Gpt* g, const LayeredLayer& w, int B, int T, int first, const int* pos_dev, bool cached) {
+    LatentArgs a = {};
+    a.in = g->lay->in.p; a.ld_in = w.n_in; a.c_dq = w.c_dq; a.c_dkv = w.c_dkv; a.c_g = w.c_g;
+    a.B = B; a.T = T; a.H = w.c.heads; a.D = w.c.dim; a.V = w.c.vdim; a.kv = w.c.kv_rank; a.rot = w.c.rot_dim; a.rope_dims = w.c.rope_dims; a.q_rank = w.c.q_rank;
+    a.first = first; a.pos_dev = pos_dev; a.scale = w.c.scale; a.eps = g->c.eps;
+    a.dq_norm = w.dq_norm; a.dkv_norm = w.dkv_norm; a.angles = w.angles;
+    a.row = w.row(); a.kv8 = w.kv8();
+    a.rows = cached ? w.rows : g->lay->rows.p;
+    a.seq_stride = (long long)(cached ? g->cache_ctx : T) * a.row;
+    a.cq = g->lay->cq.p; a.ld_cq = pad8(w.c.q_rank);
+    a.q = g->lay->q.p; a.ld_q = w.q_ld();
+    a.w_uk = w.w_ukv; a.w_uv = (const uint8_t*)w.w_ukv + (size_t)w.ukv_v() * a.kv8 * g->es; a.ld_w = a.kv8;
+    a.qabs = (float*)g->lay->qabs.p; a.olat = (float*)g->lay->olat.p;
+    a.out = g->lay->ao.p; a.ld_out = w.o_ld();
+    a.dtype = g->c.dtype;
+    return a;
+}
+
+// prompts of bf16 models whose head sizes fit expand the keys and values and run the fused kernel
+bool expands(const Gpt* g, const LayeredLayer& w) {
+    return g->c.dtype == BF16 && attention_latent_supported(w.c.dim, w.c.rot_dim, w.c.vdim, w.ukv_v(), w.q_ld(), w.ukv_ld(), w.row());
+}
+
+int gla_layer(Gpt* g, const LayeredLayer& w, int B, int T, bool few, bool cached) {
+    const GlaArgs a = gla_args(g, w, B, T, cached);
+    ProfScope ps(PROF_OTHER);
+    if (!few && gla_chunked_supported(a)) return gla_chunked(a, (float*)g->lay->gla_u.p, (float*)g->lay->gla_dec.p);
+    return gla_recurrent(a, (float*)g->lay->gla_o.p, few);
+}
+
+int latent_layer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
+    const LatentArgs a = latent_args(g, w, B, T, first, pos_dev, cached);
+    const int M = B * T;
+    { ProfScope ps(PROF_OTHER); if (latent_prep(a, few)) return 1; }
+    if (product(g, few, a.cq, a.ld_cq, w.w_uq, a.ld_cq, (int)a.ld_cq, nullptr, nullptr, a.q, a.ld_q, M, (int)a.ld_q, EPI_NONE)) return 1;
+    if (few || !expands(g, w)) { ProfScope ps(PROF_ATTN_FUSED); return latent_attention_absorbed(a, few); }
+    { ProfScope ps(PROF_OTHER); if (latent_rope_q(a)) return 1; }
+    // keys and values of positions 0 .. first + T - 1 of every sequence: [B][n][ukv_ld]
+    const int n = first + T;
+    GemmDesc d;
+    d.A = a.rows; d.B = w.w_ukv; d.C = g->lay->kv.p;
+    d.M = n; d.N = w.ukv_ld(); d.K = a.kv8; d.lda = a.row; d.ldb = a.kv8; d.ldc = d.N;
+    if (B > 1 && a.seq_stride == (long long)n * a.row) d.M = B * n;               // one product over all sequences
+    else if (B > 1) { d.nb1 = B; d.sA1 = a.seq_stride; d.sC1 = (long long)n * d.N; d.b_broadcast = 1; }
+    d.mode = MM_BF16; d.out_dtype = BF16;
+    if (gemm_or_simt(d)) return 1;
+    const uint8_t* kv = (const uint8_t*)g->lay->kv.p;
+    ProfScope ps(PROF_ATTN_FUSED);
+    return attention_latent(a.q, a.ld_q, kv, kv + (size_t)w.ukv_v() * 2, w.ukv_ld(), (const uint8_t*)a.rows + (size_t)a.kv8 * 2, a.row, a.seq_stride,
+                            a.out, a.ld_out, (const uint8_t*)a.in + (size_t)a.c_g * 2, a.ld_in, B, T, n, a.H, a.D, a.rot, a.V, first, a.scale);
+}
+
+// The launches of one step over B sequences of T new tokens at positions first .. (or pos_dev[0] ..).
+int run(Gpt* g, const void* ids, int B, int T, int first, const int* pos_dev, bool few, bool cached, void* logits, const HeadReduce* hr) {
+    const sptorch_gpt_config& c = g->c;
+    Layered& lay = *g->lay;
+    const int M = B * T, d8 = lay.d8, dt = c.dtype;
+    float* x = (float*)lay.x.p;
+    {
+        ProfScope ps(PROF_EMBED);
+        if (dt == BF16) SPT_CUDA(launch_dependent(embed_rows_kernel<__nv_bfloat16>, dim3(M), dim3(128), 0, few, 1, (const __nv_bfloat16*)lay.embed, (const int*)ids, x,
+                                                  (__nv_bfloat16*)lay.xb.p, c.vocab, d8, rt().dev_status));
+        else SPT_CUDA(launch_dependent(embed_rows_kernel<float>, dim3(M), dim3(128), 0, few, 1, (const float*)lay.embed, (const int*)ids, x, (float*)lay.xb.p, c.vocab, d8,
+                                       rt().dev_status));
+        note_submit();
+    }
+    auto tap = [&](int i) -> int {
+        if (!g->taps_on) return 0;
+        SPT_CUDA(cudaMemcpy2DAsync(g->taps[i], (size_t)c.d_model * 4, x, (size_t)d8 * 4, (size_t)c.d_model * 4, (size_t)M, cudaMemcpyDeviceToDevice, rt().stream));
+        return 0;
+    };
+    if (tap(0)) return 1;
+    const int nl = (int)lay.L.size();
+    if (nl == 0 && post_norm_launch(x, nullptr, nullptr, lay.final_norm, nullptr, lay.xb.p, M, c.d_model, d8, c.eps, dt, few)) return 1;
+    for (int l = 0; l < nl; l++) {
+        const LayeredLayer& w = lay.L[l];
+        const float* fin = l == nl - 1 ? lay.final_norm : nullptr;              // the last update of x also makes the head's input
+        if (product(g, few, lay.xb.p, d8, w.w_in, d8, d8, nullptr, nullptr, lay.in.p, w.n_in, M, w.n_in, EPI_NONE)) return 1;
+        if (w.c.mixer == SPT_MIXER_GLA ? gla_layer(g, w, B, T, few, cached) : latent_layer(g, w, B, T, first, pos_dev, few, cached)) return 1;
+        if (product(g, few, lay.ao.p, w.o_ld(), w.w_o, w.o_ld(), w.o_ld(), nullptr, nullptr, lay.y.p, d8, M, d8, EPI_NONE)) return 1;
+        const bool mlp = w.c.mlp == SPT_MLP_DENSE;
+        if (post_norm_launch(x, lay.y.p, w.norm1, mlp ? nullptr : fin, x, lay.xb.p, M, c.d_model, d8, c.eps, dt, few)) return 1;
+        if (mlp) {
+            const int f8 = pad8(w.c.d_ff);
+            if (product(g, few, lay.xb.p, d8, w.w_up, d8, d8, w.b_up, nullptr, lay.f.p, f8, M, f8, EPI_NONE)) return 1;
+            if (product(g, few, lay.xb.p, d8, w.w_gate, d8, d8, w.b_gate, lay.f.p, lay.f.p, f8, M, f8, EPI_SWIGLU)) return 1;
+            if (product(g, few, lay.f.p, f8, w.w_down, f8, f8, w.b_down, nullptr, lay.y.p, d8, M, d8, EPI_NONE)) return 1;
+            if (post_norm_launch(x, lay.y.p, w.norm2, fin, x, lay.xb.p, M, c.d_model, d8, c.eps, dt, few)) return 1;
+        }
+        if (tap(l + 1)) return 1;
+    }
+    if (few && !hr) return product(g, few, lay.xb.p, d8, g->head, d8, d8, nullptr, nullptr, logits, (long long)g->ldl, M, c.vocab, EPI_NONE);
+    return lm_head(g, lay.xb.p, M, logits, hr);
+}
+
+constexpr int kFewRows = 64, kFewTokens = 16;
+
+}  // namespace
+
+bool layered_takes_few_rows(const Gpt*, int rows, int T) { return rows <= kFewRows && T <= kFewTokens; }
+
+// scratch for B sequences of T tokens at positions first ..; outside any graph capture
+int layered_prepare(Gpt* g, int B, int T, int first, bool cached) {
+    Layered& lay = *g->lay;
+    const size_t M = (size_t)B * T, es = g->es, n = (size_t)first + T;
+    const bool few = cached && layered_takes_few_rows(g, (int)M, T);
+    size_t in = 0, ao = 0, cq = 0, q = 0, kv = 0, f = 0, rows = 0, qabs = 0, olat = 0, go = 0, gu = 0, gd = 0;
+    auto up = [](size_t& a, size_t b) { if (b > a) a = b; };
+    for (auto& w : lay.L) {
+        up(in, w.n_in); up(ao, w.o_ld());
+        if (w.c.mlp == SPT_MLP_DENSE) up(f, pad8(w.c.d_ff));
+        if (w.c.mixer == SPT_MIXER_GLA) {
+            const GlaArgs a = gla_args(g, w, B, T, cached);
+            if (!few && gla_chunked_supported(a)) { up(gu, gla_chunked_state_bytes(a)); up(gd, gla_chunked_decay_bytes(a)); }
+            else up(go, M * w.c.heads * w.c.vdim * 4);
+        } else {
+            up(cq, pad8(w.c.q_rank)); up(q, w.q_ld());
+            if (!cached) up(rows, w.row());
+            if (!few && expands(g, w)) up(kv, w.ukv_ld());
+            else { up(qabs, (size_t)w.c.heads * w.row()); up(olat, (size_t)w.c.heads * w.kv8()); }
+        }
+    }
+    const size_t d8 = lay.d8;
+    return ensure(g, &lay.x, M * d8 * 4) || ensure(g, &lay.x2, M * d8 * 4) || ensure(g, &lay.xb, M * d8 * es) || ensure(g, &lay.y, M * d8 * es) || ensure(g, &lay.in, M * in * es) ||
+           ensure(g, &lay.ao, M * ao * es) || ensure(g, &lay.cq, M * cq * es) || ensure(g, &lay.q, M * q * es) || ensure(g, &lay.kv, (size_t)B * n * kv * es) ||
+           ensure(g, &lay.f, M * f * es) || ensure(g, &lay.rows, M * rows * es) || ensure(g, &lay.qabs, M * qabs * 4) || ensure(g, &lay.olat, M * olat * 4) ||
+           ensure(g, &lay.gla_o, go) || ensure(g, &lay.gla_u, gu) || ensure(g, &lay.gla_dec, gd);
+}
+
+int layered_forward(Gpt* g, const void* ids, int B, int T, int first, bool cached, void* logits, const HeadReduce* hr) {
+    return run(g, ids, B, T, first, nullptr, false, cached, logits, hr);
+}
+int layered_few_rows(Gpt* g, const void* ids, int B, int T, const int* state, int first, void* logits) {
+    return run(g, ids, B, T, first, state, true, true, logits, nullptr);
+}
+
+int layered_enable_cache(Gpt* g, int max_context) {
+    for (auto& w : g->lay->L) {
+        if (w.c.mixer == SPT_MIXER_GLA) {
+            w.state = (float*)galloc(g, (size_t)g->c.max_batch * w.c.heads * w.c.dim * w.c.vdim * 4);
+            if (!w.state) return 1;
+        } else {
+            const size_t bytes = (size_t)g->c.max_batch * max_context * w.row() * g->es;
+            w.rows = galloc(g, bytes);
+            if (!w.rows || sptorch_ext_memset(w.rows, 0, bytes)) return 1;
+        }
+    }
+    g->dstate = (int*)galloc(g, 256);
+    if (!g->dstate) return 1;
+    g->cache_ctx = max_context;
+    return layered_reset_cache(g);
+}
+
+// Every sequence forgets what it has seen.  Cached rows need no clearing: a position is written before it is read.
+int layered_reset_cache(Gpt* g) {
+    for (auto& w : g->lay->L)
+        if (w.state && sptorch_ext_memset(w.state, 0, (size_t)g->c.max_batch * w.c.heads * w.c.dim * w.c.vdim * 4)) return 1;
+    g->cached_len = 0; g->cache_batch = 0; g->window_start = 0;
+    return 0;
+}
+
+int layered_launches(const Gpt* g, int B, int T) {
+    (void)B; (void)T;
+    int n = 2;                                                        // embedding, head
+    if (g->lay->L.empty()) n++;
+    for (auto& w : g->lay->L) {
+        n += 3;                                                       // input projection, W_o, post-norm
+        n += w.c.mixer == SPT_MIXER_GLA ? (g->c.dtype == BF16 && gla_chunked_supported(gla_args(const_cast<Gpt*>(g), w, B, T, false)) ? 3 : 2) : expands(g, w) ? 5 : 5;
+        if (w.c.mlp == SPT_MLP_DENSE) n += 4;
+    }
+    return n;
+}
+
+void layered_release(Gpt* g) { delete g->lay; g->lay = nullptr; }
+
+// ---------------- parameters ----------------
+namespace {
+
+// one entry per tensor: its name behind the layer's prefix, its shape, and where it goes
+struct Slot { std::string name; size_t rows, cols; void* dst; bool f32; int ld; size_t dst_row; };      // cols 0: a vector of `rows` values
+
+std::vector<Slot> layer_slots(const Gpt* g, const LayeredLayer& w) {
+    const size_t d = g->c.d_model;
+    const int d8 = g->lay->d8;
+    const sptorch_layer_config& c = w.c;
+    std::vector<Slot> s;
+    auto mat = [&](const char* n, size_t r, size_t k, void* dst, int ld, size_t row) { s.push_back({n, r, k, dst, false, ld, row}); };
+    auto vec = [&](const char* n, size_t r, float* dst) { s.push_back({n, r, 0, dst, true, 0, 0}); };
+    const bool mlp = c.mlp == SPT_MLP_DENSE;
+    vec("norm1", d, w.norm1);
+    if (mlp) vec("norm2", d, w.norm2);
+    if (c.mixer == SPT_MIXER_GLA) {
+        const size_t hd = (size_t)c.heads * c.dim, hv = (size_t)c.heads * c.vdim;
+        mat("mix.q", hd, d, w.w_in, d8, w.c_q); mat("mix.k", hd, d, w.w_in, d8, w.c_k); mat("mix.v", hv, d, w.w_in, d8, w.c_v); mat("mix.g", hv, d, w.w_in, d8, w.c_g);
+        mat("mix.o", d, hv, w.w_o, w.o_ld(), 0);
+        vec("mix.norm", c.vdim, w.head_norm);
+        mat("mix.a1", c.decay_rank, d, w.w_in, d8, w.c_a);
+        s.push_back({"mix.a2", hd, (size_t)c.decay_rank, w.a2, true, c.decay_rank, 0});
+        vec("mix.a2.b", hd, w.a2_b);
+    } else {
+        const int q8 = pad8(c.q_rank), kv8 = w.kv8();
+        mat("mix.dq", c.q_rank, d, w.w_in, d8, w.c_dq); vec("mix.dq.norm", c.q_rank, w.dq_norm);
+        mat("mix.uq", (size_t)c.heads * (c.dim + c.rot_dim), c.q_rank, w.w_uq, q8, 0);
+        mat("mix.dkv", (size_t)c.kv_rank + c.rot_dim, d, w.w_in, d8, w.c_dkv); vec("mix.dkv.norm", c.kv_rank, w.dkv_norm);
+        mat("mix.uk", (size_t)c.heads * c.dim, c.kv_rank, w.w_ukv, kv8, 0); mat("mix.uv", (size_t)c.heads * c.vdim, c.kv_rank, w.w_ukv, kv8, w.ukv_v());
+        mat("mix.g", c.heads, d, w.w_in, d8, w.c_g);
+        mat("mix.o", d, (size_t)c.heads * c.vdim, w.w_o, w.o_ld(), 0);
+    }
+    if (mlp) {
+        const int f8 = pad8(c.d_ff);
+        mat("mlp.gate", c.d_ff, d, w.w_gate, d8, 0); vec("mlp.gate.b", c.d_ff, w.b_gate);
+        mat("mlp.up", c.d_ff, d, w.w_up, d8, 0); vec("mlp.up.b", c.d_ff, w.b_up);
+        mat("mlp.down", d, c.d_ff, w.w_down, f8, 0); vec("mlp.down.b", d, w.b_down);
+    }
+    return s;
+}
+
+std::vector<Slot> model_slots(const Gpt* g) {
+    const size_t V = g->c.vocab, d = g->c.d_model;
+    std::vector<Slot> s;
+    s.push_back({"embed", V, d, g->lay->embed, false, g->lay->d8, 0});
+    for (size_t l = 0; l < g->lay->L.size(); l++)
+        for (auto& e : layer_slots(g, g->lay->L[l])) { s.push_back(e); s.back().name = "l" + std::to_string(l) + "." + e.name; }
+    s.push_back({"final.norm", d, 0, g->lay->final_norm, true, 0, 0});
+    s.push_back({"head", V, d, g->lay->head, false, g->lay->d8, 0});
+    return s;
+}
+
+}  // namespace
+
+std::vector<ParamInfo> layered_param_table(const Gpt* g) {
+    std::vector<ParamInfo> t;
+    for (auto& s : model_slots(g)) t.push_back({s.name, s.cols ? std::vector<size_t>{s.rows, s.cols} : std::vector<size_t>{s.rows}});
+    return t;
+}
+
+int layered_set_param(Gpt* g, const char* name, const float* host, size_t n) {
+    const std::string key(name);
+    for (auto& s : model_slots(g)) {
+        if (s.name != key) continue;
+        const size_t want = s.rows * (s.cols ? s.cols : 1);
+        if (n != want) return fail("gpt_set_param(%s): got %zu values, expected %zu", name, n, want);
+        if (s.f32) return sptorch_ext_copy_h2d_bytes(host, s.dst, n * 4) || stream_wait();
+        void* dst = (uint8_t*)s.dst + s.dst_row * s.ld * g->es;
+        if ((size_t)s.ld == s.cols) return upload_rows(g, dst, host, n) || stream_wait();
+        std::vector<float> padded(s.rows * s.ld, 0.0f);
+        for (size_t r = 0; r < s.rows; r++) memcpy(&padded[r * s.ld], host + r * s.cols, s.cols * 4);
+        return upload_rows(g, dst, padded.data(), padded.size()) || stream_wait();
+    }
+    return fail("gpt_set_param: unknown parameter name '%s'", name);
+}
+
+static int check_layer(const sptorch_layer_config& c, int i) {
+    if (c.mixer != SPT_MIXER_GLA && c.mixer != SPT_MIXER_LATENT) return fail("layered_create: layer %d: unknown mixer %d", i, c.mixer);
+    if (c.heads <= 0 || c.dim <= 0 || c.vdim <= 0) return fail("layered_create: layer %d: non-positive head count or size", i);
+    if (c.mixer == SPT_MIXER_GLA) {
+        if (c.decay_rank <= 0 || !(c.tau > 0.0f)) return fail("layered_create: layer %d: decay_rank and tau must be positive", i);
+        if (c.dim > 512) return fail("layered_create: layer %d: key size %d is larger than 512", i, c.dim);
+    } else {
+        if (c.kv_rank <= 0 || c.q_rank <= 0 || c.rot_dim < 0) return fail("layered_create: layer %d: latent sizes must be positive", i);
+        if (c.rope_dims < 0 || c.rope_dims > c.rot_dim || c.rope_dims % 2) return fail("layered_create: layer %d: %d rotated dims of %d", i, c.rope_dims, c.rot_dim);
+        if (c.rope_dims && !(c.rope_base > 0.0)) return fail("layered_create: layer %d: rope_base must be positive", i);
+        if (pad8(c.kv_rank) + pad8(c.rot_dim) > 1280) return fail("layered_create: layer %d: cached rows of %d + %d values are larger than 1280", i, c.kv_rank, c.rot_dim);
+    }
+    if (c.mlp != SPT_MLP_NONE && c.mlp != SPT_MLP_DENSE) return fail("layered_create: layer %d: unknown feed-forward %d", i, c.mlp);
+    if (c.mlp == SPT_MLP_DENSE && c.d_ff <= 0) return fail("layered_create: layer %d: non-positive d_ff", i);
+    return 0;
+}
+
+}  // namespace spt
+
+using namespace spt;
+
+extern "C" void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const sptorch_layer_config* layers, int n_layers) {
+    if (enter()) return nullptr;
+    if (!cfg || (n_layers > 0 && !layers)) { fail("layered_create: null config"); return nullptr; }
+    sptorch_gpt_config c = *cfg;
+    c.arch = SPT_ARCH_LAYERED; c.n_layer = n_layers; c.n_head = 1; c.d_ff = 1; c.tp_size = 1; c.tp_rank = 0;
+    if (cfg->tp_size > 1) { fail("layered_create: no tensor parallel shards"); return nullptr; }
+    if (c.vocab <= 0 || c.d_model <= 0 || n_layers < 0 || c.seq_len <= 0 || c.max_batch <= 0) { fail("layered_create: non-positive dimension"); return nullptr; }
+    if (c.dtype != SPT_F32 && c.dtype != SPT_BF16) { fail("layered_create: unknown dtype %d", c.dtype); return nullptr; }
+    for (int i = 0; i < n_layers; i++) if (check_layer(layers[i], i)) return nullptr;
+    Gpt* g = new Gpt();
+    g->c = c;
+    g->es = c.dtype == SPT_BF16 ? 2 : 4;
+    g->ldl = ((size_t)c.vocab + 63) / 64 * 64;
+    g->lay = new Layered();
+    Layered& lay = *g->lay;
+    lay.d8 = pad8(c.d_model);
+    const size_t d8 = lay.d8, es = g->es, V = c.vocab;
+    bool ok = true;
+    auto Z = [&](size_t bytes) { void* p = galloc(g, bytes); if (!p || sptorch_ext_memset(p, 0, bytes)) ok = false; return p; };
+    auto F = [&](size_t n) { return (float*)Z((size_t)pad8((int)n) * 4); };
+    lay.embed = Z(V * d8 * es); lay.head = Z(V * d8 * es); lay.final_norm = F(d8);
+    g->head = lay.head; g->tok = lay.embed;
+    std::map<std::pair<int, double>, float2*> angles;
+    for (int i = 0; i < n_layers && ok; i++) {
+        LayeredLayer w;
+        w.c = layers[i];
+        const sptorch_layer_config& lc = w.c;
+        auto at = [&](int& col, int width) { col = w.n_in; w.n_in += pad8(width); };
+        w.norm1 = F(d8); w.norm2 = F(d8);
+        if (lc.mixer == SPT_MIXER_GLA) {
+            at(w.c_q, lc.heads * lc.dim); at(w.c_k, lc.heads * lc.dim); at(w.c_v, lc.heads * lc.vdim); at(w.c_g, lc.heads * lc.vdim); at(w.c_a, lc.decay_rank);
+            w.a2 = F((size_t)lc.heads * lc.dim * lc.decay_rank); w.a2_b = F((size_t)lc.heads * lc.dim); w.head_norm = F(lc.vdim);
+        } else {
+            at(w.c_dq, lc.q_rank); at(w.c_dkv, lc.kv_rank + lc.rot_dim); at(w.c_g, lc.heads);
+            w.dq_norm = F(lc.q_rank); w.dkv_norm = F(lc.kv_rank);
+            w.w_uq = Z((size_t)w.q_ld() * pad8(lc.q_rank) * es); w.w_ukv = Z((size_t)w.ukv_ld() * w.kv8() * es);
+            if (lc.rope_dims) {
+                float2*& tab = angles[{lc.rope_dims, lc.rope_base}];
+                if (!tab) {
+                    const int half = lc.rope_dims / 2;
+                    std::vector<float2> host((size_t)c.seq_len * half);
+                    for (int k = 0; k < half; k++) {
+                        const double f = std::pow(lc.rope_base, -2.0 * k / lc.rope_dims);
+                        for (int p = 0; p < c.seq_len; p++) host[(size_t)p * half + k] = make_float2((float)std::cos(p * f), (float)std::sin(p * f));
+                    }
+                    tab = (float2*)galloc(g, host.size() * sizeof(float2));
+                    if (!tab || sptorch_ext_copy_h2d_bytes(host.data(), tab, host.size() * sizeof(float2)) || stream_wait()) { ok = false; break; }
+                }
+                w.angles = tab;
+            }
+        }
+        w.w_in = Z((size_t)w.n_in * d8 * es);
+        w.w_o = Z(d8 * w.o_ld() * es);
+        if (lc.mlp == SPT_MLP_DENSE) {
+            const size_t f8 = pad8(lc.d_ff);
+            w.w_gate = Z(f8 * d8 * es); w.w_up = Z(f8 * d8 * es); w.w_down = Z(d8 * f8 * es);
+            w.b_gate = F(f8); w.b_up = F(f8); w.b_down = F(d8);
+        }
+        lay.L.push_back(w);
+    }
+    if (!ok) { sptorch_ext_gpt_destroy(g); return nullptr; }
+    return g;
+}

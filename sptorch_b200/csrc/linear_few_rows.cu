@@ -18,6 +18,7 @@
 // A sum over k does not care about the order as long as both operands use the same one.
 #include "gemm.h"
 #include "epilogue_math.cuh"
+#include "pdl.cuh"
 #include <cooperative_groups.h>
 
 namespace spt {
@@ -47,13 +48,6 @@ __device__ __forceinline__ void mma_bf16_16x8x16(float (&d)[4], uint32_t a0, uin
 // (decode step of a 12-layer, 768-wide model at 64 sequences: 2.30 ms with, 1.0 ms without).
 constexpr int kNormMaxRows = 16;
 
-// Programmatic dependent launch: a kernel launched with launch_dependent() may start while its predecessor in the stream still
-// runs.  pdl_release() lets the successor's CTAs be scheduled as soon as every CTA of this grid has called it (or exited);
-// pdl_acquire() returns once the predecessor grid has completed and its writes are visible.  Everything a kernel does before
-// pdl_acquire() may only touch memory no earlier kernel of the stream writes (weights); both are no-ops in an ordinary launch.
-__device__ __forceinline__ void pdl_release() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
-__device__ __forceinline__ void pdl_acquire() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
-
 // MT: 16-row groups of A (M <= 16 MT); NT: 8-row groups of W per CTA; S: weight slices a warp has in flight.
 // NORM: A holds un-normalised rows; every CTA normalises them itself into shared memory (kind 1: LayerNorm, gamma * ((x - mean) *
 // inv) + beta with inv = 1 / sqrt(var + eps); kind 2: RMSNorm, x * inv * gamma with inv = 1 / sqrt(mean(x^2) + eps)), rounded to
@@ -70,8 +64,9 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
     // ksplit > 1: a cluster of ksplit CTAs shares the weight rows of one block, CTA r of it takes the r-th part of K
     const int krank = blockIdx.x % ksplit;
     const int n0 = (blockIdx.x / ksplit) * (NT * 8);
-    const int all_slices = K >> 5, per_cta = (all_slices + ksplit - 1) / ksplit;
+    const int all_slices = (K + 31) >> 5, per_cta = (all_slices + ksplit - 1) / ksplit;
     const int s_lo = krank * per_cta, slices = min(all_slices, s_lo + per_cta);
+    const int k_mine = K - 8 * t;               // a slice s holds elements of this lane while 32 s < k_mine (K is a multiple of 8)
     pdl_release();
 
     const __nv_bfloat16* wrow[NT];
@@ -91,7 +86,7 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
         for (int u = 0; u < S; u++) {
             const int s = s0 + u * kWarps;
 #pragma unroll
-            for (int j = 0; j < NT; j++) wv[u][j] = s < slices ? ld_stream(wrow[j] + 32 * s) : make_uint4(0, 0, 0, 0);
+            for (int j = 0; j < NT; j++) wv[u][j] = s < slices && 32 * s < k_mine ? ld_stream(wrow[j] + 32 * s) : make_uint4(0, 0, 0, 0);
         }
     };
     load_weights(s_lo + warp);       // the weights do not depend on the kernel before this one
@@ -207,8 +202,9 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
             for (int i = 0; i < MT; i++) {
                 const int r0 = 16 * i + g, r1 = r0 + 8;
                 uint4 a0 = make_uint4(0, 0, 0, 0), a1 = make_uint4(0, 0, 0, 0);
-                if (r0 < M) a0 = *reinterpret_cast<const uint4*>(a_base + (long long)r0 * a_ld + 32 * s + 8 * t);
-                if (r1 < M) a1 = *reinterpret_cast<const uint4*>(a_base + (long long)r1 * a_ld + 32 * s + 8 * t);
+                const bool live = 32 * s < k_mine;
+                if (live && r0 < M) a0 = *reinterpret_cast<const uint4*>(a_base + (long long)r0 * a_ld + 32 * s + 8 * t);
+                if (live && r1 < M) a1 = *reinterpret_cast<const uint4*>(a_base + (long long)r1 * a_ld + 32 * s + 8 * t);
 #pragma unroll
                 for (int j = 0; j < NT; j++) {
                     mma_bf16_16x8x16(acc[i][j], a0.x, a1.x, a0.y, a1.y, wv[u][j].x, wv[u][j].y);
@@ -412,7 +408,7 @@ bool linear_few_rows_supported(const GemmDesc& d) {
     // SPTORCH_B200_FEW_ROWS: the largest row count that takes this kernel (0 = never; experiments)
     static const int max_rows = [] { const char* e = getenv("SPTORCH_B200_FEW_ROWS"); const int v = e ? atoi(e) : kDefaultMaxRows; return v < 0 ? 0 : v > 64 ? 64 : v; }();
     const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    return d.mode == MM_BF16 && d.out_dtype == BF16 && d.M >= 1 && d.M <= max_rows && d.N >= 1 && d.K >= 32 && d.K % 32 == 0 && d.nb1 * d.nb2 == 1 &&
+    return d.mode == MM_BF16 && d.out_dtype == BF16 && d.M >= 1 && d.M <= max_rows && d.N >= 1 && d.K >= 8 && d.K % 8 == 0 && d.nb1 * d.nb2 == 1 &&
            !d.causal_lower && !d.causal_k && !d.norm_axis && !d.reduce && d.lda % 8 == 0 && d.ldb % 8 == 0 && d.lda >= d.K && d.ldb >= d.K &&
            d.ldc >= d.N && al16(d.A) && al16(d.B) && d.C != nullptr;
 }

@@ -10,8 +10,7 @@
 //                             F32 / F16 / BF16 converted to f32 exactly as f16_to_f32 / bf16_to_f32 there
 // The strictness of the reference is kept: wrong magic, version, schema, count, shape, dtype, duplicate or missing names are
 // errors, and nothing is uploaded unless every check has passed.
-#include "common.h"
-#include "../../include/sptorch_b200_ext.h"
+#include "gpt_model.h"
 #include <cerrno>
 #include <cstdio>
 #include <cstdlib>
@@ -339,7 +338,6 @@ static int check_manifest(const std::string& weights_path, const WeightFile& w, 
     return 0;
 }
 
-struct ParamInfo { std::string name; std::vector<size_t> shape; };
 // named_parameters of the model behind the handle (defined with the model in gpt.cu)
 std::vector<ParamInfo> gpt_param_table(void* gpt);
 

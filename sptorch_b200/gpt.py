@@ -193,6 +193,36 @@ class GPT:
         self.b._check(self.b.lib.sptorch_ext_gpt_prefill(self.h, d_ids.handle, B, T, d_log.handle), "gpt_prefill")
         return self._read_logits(d_log, B * T).reshape(B, T, -1)
 
+    def reset_cache(self):
+        """The cached sequences are finished; what they hold is free for the next ones."""
+        self.b._check(self.b.lib.sptorch_ext_gpt_reset_cache(self.h), "reset_cache")
+        self._gen_ctx = None
+
+    def extend_device(self, ids: np.ndarray):
+        """The next tokens [B, T] of the cached sequences (an empty cache: their first) -> device buffer of logits [B*T, ldl].  One
+        token per sequence behind a cached prefix is a decode step, anything longer a portion of a prompt."""
+        ids = np.asarray(ids)
+        B, T = ids.shape
+        d_ids, d_log = self.stage_ids(ids), self.logits_buffer(B * T)
+        if T == 1 and self.cached_len() > 0:
+            self.b._check(self.b.lib.sptorch_ext_gpt_decode(self.h, d_ids.handle, B, 1, d_log.handle), "gpt_decode")
+        else:
+            self.b._check(self.b.lib.sptorch_ext_gpt_extend(self.h, d_ids.handle, B, T, d_log.handle), "gpt_extend")
+        return d_log
+
+    def extend(self, ids: np.ndarray) -> np.ndarray:
+        """extend_device with the logits [B, T, V] on the host."""
+        B, T = np.asarray(ids).shape
+        return self._read_logits(self.extend_device(ids), B * T).reshape(B, T, -1)
+
+    def read_logit_rows(self, d_log, rows) -> np.ndarray:
+        """Some rows of a device buffer of logits on the host, [len(rows), V] float32."""
+        out = np.empty((len(rows), self.ldl), dtype=np.uint16 if self.dtype == BF16 else np.float32)
+        for i, r in enumerate(rows):
+            self.b._check(self.b.lib.sptorch_ext_copy_d2h_bytes(d_log.handle + int(r) * self.ldl * self.es, out[i].ctypes.data, out[i].nbytes), "logits d2h")
+        self.b.synchronize()
+        return (bf16_bits_to_f32(out) if self.dtype == BF16 else out)[:, :self.cfg["vocab"]].copy()
+
     def decode_logits_from_cache(self, last_ids) -> np.ndarray:
         """Logits [B, V] of the last cached token, recomputed from the cache (no append)."""
         return self._decode(last_ids, 0)

@@ -4,6 +4,7 @@ Reading needs no GPU; loading into a device model does."""
 from __future__ import annotations
 
 import ctypes as C
+from contextlib import nullcontext
 
 import numpy as np
 
@@ -50,6 +51,12 @@ class WeightFile:
         data = np.ctypeslib.as_array(L.sptorch_ext_weights_data(self.h, i), shape=(n,)).copy() if n else np.zeros(0, np.float32)
         return (L.sptorch_ext_weights_name(self.h, i).decode(), shape, L.sptorch_ext_weights_dtype(self.h, i).decode(), data)
 
+    def shapes(self) -> dict:
+        """{name: shape} without copying any data."""
+        L = self.lib
+        return {L.sptorch_ext_weights_name(self.h, i).decode():
+                tuple(int(L.sptorch_ext_weights_dim(self.h, i, k)) for k in range(L.sptorch_ext_weights_ndim(self.h, i))) for i in range(len(self))}
+
     def get(self, name: str):
         for i, n in enumerate(self.names()):
             if n == name:
@@ -57,10 +64,10 @@ class WeightFile:
         return None
 
 
-def load_into(model, path: str, fmt: int = AUTO, mapping=None):
-    """Checks the file against the model's named parameters with the reference's strictness and uploads it.
-    ``mapping`` (safetensors only): {model parameter name: name in the file}, as SafeTensorsFile::load_into."""
-    with WeightFile(path, fmt) as w:
+def load_into(model, path, fmt: int = AUTO, mapping=None):
+    """Checks the file (a path, or an opened WeightFile) against the model's named parameters with the reference's strictness and
+    uploads it.  ``mapping`` (safetensors only): {model parameter name: name in the file}, as SafeTensorsFile::load_into."""
+    with (nullcontext(path) if isinstance(path, WeightFile) else WeightFile(path, fmt)) as w:
         arr, n = None, 0
         if mapping:
             flat = []
