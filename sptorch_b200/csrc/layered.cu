@@ -454,19 +454,19 @@ int layered_set_param(Gpt* g, const char* name, const float* host, size_t n) {
 }
 
 static int check_layer(const sptorch_layer_config& c, int i) {
-    if (c.mixer != SPT_MIXER_GLA && c.mixer != SPT_MIXER_LATENT) return fail("layered_create: layer %d: unknown mixer %d", i, c.mixer);
-    if (c.heads <= 0 || c.dim <= 0 || c.vdim <= 0) return fail("layered_create: layer %d: non-positive head count or size", i);
+    if (c.mixer != SPT_MIXER_GLA && c.mixer != SPT_MIXER_LATENT) return fail_host("layered_create: layer %d: unknown mixer %d", i, c.mixer);
+    if (c.heads <= 0 || c.dim <= 0 || c.vdim <= 0) return fail_host("layered_create: layer %d: non-positive head count or size", i);
     if (c.mixer == SPT_MIXER_GLA) {
-        if (c.decay_rank <= 0 || !(c.tau > 0.0f)) return fail("layered_create: layer %d: decay_rank and tau must be positive", i);
-        if (c.dim > 512) return fail("layered_create: layer %d: key size %d is larger than 512", i, c.dim);
+        if (c.decay_rank <= 0 || !(c.tau > 0.0f)) return fail_host("layered_create: layer %d: decay_rank and tau must be positive", i);
+        if (c.dim > 512) return fail_host("layered_create: layer %d: key size %d is larger than 512", i, c.dim);
     } else {
-        if (c.kv_rank <= 0 || c.q_rank <= 0 || c.rot_dim < 0) return fail("layered_create: layer %d: latent sizes must be positive", i);
-        if (c.rope_dims < 0 || c.rope_dims > c.rot_dim || c.rope_dims % 2) return fail("layered_create: layer %d: %d rotated dims of %d", i, c.rope_dims, c.rot_dim);
-        if (c.rope_dims && !(c.rope_base > 0.0)) return fail("layered_create: layer %d: rope_base must be positive", i);
-        if (pad8(c.kv_rank) + pad8(c.rot_dim) > 1280) return fail("layered_create: layer %d: cached rows of %d + %d values are larger than 1280", i, c.kv_rank, c.rot_dim);
+        if (c.kv_rank <= 0 || c.q_rank <= 0 || c.rot_dim < 0) return fail_host("layered_create: layer %d: latent sizes must be positive", i);
+        if (c.rope_dims < 0 || c.rope_dims > c.rot_dim || c.rope_dims % 2) return fail_host("layered_create: layer %d: %d rotated dims of %d", i, c.rope_dims, c.rot_dim);
+        if (c.rope_dims && !(c.rope_base > 0.0)) return fail_host("layered_create: layer %d: rope_base must be positive", i);
+        if (pad8(c.kv_rank) + pad8(c.rot_dim) > 1280) return fail_host("layered_create: layer %d: cached rows of %d + %d values are larger than 1280", i, c.kv_rank, c.rot_dim);
     }
-    if (c.mlp != SPT_MLP_NONE && c.mlp != SPT_MLP_DENSE) return fail("layered_create: layer %d: unknown feed-forward %d", i, c.mlp);
-    if (c.mlp == SPT_MLP_DENSE && c.d_ff <= 0) return fail("layered_create: layer %d: non-positive d_ff", i);
+    if (c.mlp != SPT_MLP_NONE && c.mlp != SPT_MLP_DENSE) return fail_host("layered_create: layer %d: unknown feed-forward %d", i, c.mlp);
+    if (c.mlp == SPT_MLP_DENSE && c.d_ff <= 0) return fail_host("layered_create: layer %d: non-positive d_ff", i);
     return 0;
 }
 

@@ -78,3 +78,34 @@ def spec_of(model, max_context: int | None = None) -> KvCacheBufferSpec:
     c = model.cfg
     return KvCacheBufferSpec(("cuda", model.b.lib.sptorch_ext_device()), "BF16" if model.dtype == BF16 else "F32", c["n_layer"],
                              max_context or c["seq_len"], c["n_head"], c["d_model"] // c["n_head"])
+
+
+@dataclass(frozen=True)
+class LayerCacheSpec:
+    """What one layer of a model built from a list of layers keeps: a row per position ("rows") or a matrix per head ("state", f32)."""
+    layer: int
+    kind: str
+    shape: tuple           # rows: (sequences, positions, row); state: (sequences, heads, dim, vdim)
+    dtype: str
+
+    def elements(self) -> int:
+        n = 1
+        for s in self.shape:
+            n *= s
+        return n
+
+    def total_bytes(self) -> int:
+        return self.elements() * _DTYPE_BYTES[self.dtype]
+
+
+def layer_specs(model, max_context: int | None = None) -> list:
+    """Per layer, the device buffers that sptorch_ext_gpt_enable_kv_cache allocates for a model built from a list of layers."""
+    from .backend import BF16
+    ctx, out = max_context or model.cfg["seq_len"], []
+    for i, c in enumerate(model.layers):
+        if c.mixer == 0:
+            out.append(LayerCacheSpec(i, "state", (model.max_batch, c.heads, c.dim, c.vdim), "F32"))
+        else:
+            row = -(-c.kv_rank // 8) * 8 + -(-c.rot_dim // 8) * 8
+            out.append(LayerCacheSpec(i, "rows", (model.max_batch, ctx, row), "BF16" if model.dtype == BF16 else "F32"))
+    return out
