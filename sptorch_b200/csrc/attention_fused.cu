@@ -23,6 +23,11 @@
 // O_1 at 384 (512 columns, one CTA per SM).  Head size 64 (accumulators of 64 columns): THREE score buffers at 0 / 128 / 256
 // that the Q K^T products take in turn, O_0 at 384, O_1 at 448 -- a tile's next scores are ready before its softmax warps
 // have finished the current ones.
+// The same kernel serves latent attention (latent_attention.cu) once a prompt's keys and values are expanded: a score is then the sum of
+// two products over separately stored parts -- the head's own D columns and a rotated part all heads share -- queries may start at a
+// position `first` > 0 behind cached keys, values may be narrower or wider than the keys, and head h's output carries the factor
+// sigmoid(gate_h).  There the softmax weights enter P V as the sum of two bf16 numbers (PSPLIT: 16 mantissa bits instead of 8; the
+// second half sits in the score columns the first leaves free), so that the weights keep close to f32 precision.
 // Algorithmic work per (sequence, head): 2 * T(T+1) * hd FLOP; HBM traffic: Q, K, V read once per query tile
 // (K/V re-reads hit L2 thanks to the work schedule below), O written once.
 #include "gemm.h"
@@ -48,11 +53,15 @@ constexpr int kQPair = 2 * kQTile;          // query rows per work item
 struct AttnParams {
     __nv_bfloat16* out;
     long long ld_out;       // row stride of out in elements
-    int T, H, B;
+    int T, H, B;            // T query rows per sequence, at positions first .. first + T - 1
+    int n, first;           // keys 0 .. n - 1 per sequence
+    int V;                  // width of a head's output in memory (at most the template's VD)
     int n_ptiles;           // 256-row query tile pairs per sequence
-    float scale_log2;       // 1/sqrt(hd) * log2(e)
+    float scale_log2;       // factor of the scores * log2(e)
+    const __nv_bfloat16* gate;      // when given: head h of token m is multiplied by sigmoid(gate[m * ld_gate + h])
+    long long ld_gate;
     uint32_t* status;
-    const int* sched;       // work schedule [sched_len][gridDim.x]: item of CTA c at step k, -1 past the end of its list
+    const int* sched;       // work schedule [sched_len][gridDim.x]: item of CTA c at step k, -1 past the end of its list; null: items c, c + grid, ..
     int sched_len;
 };
 
@@ -83,6 +92,15 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
     float d;
     asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
     return d;
+}
+
+// two f32 as the sums of two bf16 each: hi and what hi misses (together 16 mantissa bits)
+__device__ __forceinline__ void split2(float2 e, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h2 = __floats2bfloat162_rn(e.x, e.y);
+    hi = *reinterpret_cast<const uint32_t*>(&h2);
+    const float2 f = bf16x2_to_float2(h2);
+    const __nv_bfloat162 l2 = __floats2bfloat162_rn(e.x - f.x, e.y - f.y);
+    lo = *reinterpret_cast<const uint32_t*>(&l2);
 }
 
 // 32 lanes x 16 consecutive 32-bit columns: thread i of the warp owns lane (base_lane + i)
@@ -126,49 +144,56 @@ __device__ __forceinline__ uint64_t make_mnmajor_sw128_desc(uint32_t smem_addr, 
     return d;
 }
 
-template <int HD>
+// KBN / KBR: 64-column blocks of the heads' own query/key part and of the shared part; VD: value columns
+template <int KBN, int KBR, int VD>
 struct AttnSmem {
-    static constexpr int kStages = HD == 64 ? 4 : 2;
-    static constexpr int kQTileBytes = kQTile * HD * 2;       // HD/64 k-blocks of [128 rows x 128 B]
-    static constexpr int kKBytes = kKvTile * HD * 2;          // HD/64 k-blocks of [128 keys x 128 B]
-    static constexpr int kVBytes = kKvTile * HD * 2;          // HD/64 chunks of [128 keys x 128 B] (64 head columns each)
-    static constexpr int kStageBytes = kKBytes + kVBytes;
+    static constexpr int KB = KBN + KBR;
+    static constexpr int kKStages = KB == 1 ? 4 : KB == 2 && VD == 64 && KBR == 1 ? 3 : 2;
+    static constexpr int kVStages = KB == 3 && VD == 128 ? 1 : kKStages;
+    static constexpr int kQTileBytes = KB * kQTile * 128;     // k-blocks of [128 rows x 128 B]
+    static constexpr int kKBytes = KB * kKvTile * 128;        // k-blocks of [128 keys x 128 B]
+    static constexpr int kVBytes = kKvTile * VD * 2;          // VD/64 chunks of [128 keys x 128 B] (64 head columns each)
     static constexpr int kQ = 0;
-    static constexpr int kKV = kQ + 2 * kQTileBytes;
-    static constexpr int kBars = kKV + kStages * kStageBytes; // mbarriers + TMEM slot + abort flag (256 B)
+    static constexpr int kK = kQ + 2 * kQTileBytes;
+    static constexpr int kV = kK + kKStages * kKBytes;
+    static constexpr int kBars = kV + kVStages * kVBytes;     // mbarriers + TMEM slot + abort flag (256 B)
     static constexpr int kTotal = kBars + 256;
+    static_assert(kTotal <= 227 * 1024, "shared memory");
 };
 
 // Persistent kernel: CTA c works through column c of a schedule built on the host (attention_schedule below), and all
 // roles run straight through item boundaries (barrier phases are driven by running counters), so the loads and the
 // first Q K^T of the next item are in flight while the current one drains.
-template <int HD, int NPOLY, bool ROTP = true>
+template <int KBN, int KBR, int VD, int NPOLY, bool ROTP, bool PSPLIT>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                  const __grid_constant__ CUtensorMap tmV, const AttnParams p) {
-    using L = AttnSmem<HD>;
+                  const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQr, const __grid_constant__ CUtensorMap tmKr,
+                  const AttnParams p) {
+    using L = AttnSmem<KBN, KBR, VD>;
     constexpr uint32_t TMEM_COLS = 512;
     constexpr uint32_t IDESC_S = make_idesc(false, 128, kKvTile);
-    constexpr uint32_t IDESC_O = make_idesc(false, 128, HD) | (1u << 16);      // B operand (V) is MN-major
-    constexpr int KB = HD / 64;                               // 128-byte blocks along head_dim
-    constexpr int NS = L::kStages;
+    constexpr uint32_t IDESC_O = make_idesc(false, 128, VD) | (1u << 16);      // B operand (V) is MN-major
+    constexpr int KB = L::KB;                                 // 128-byte blocks along the query/key width
+    constexpr int NSK = L::kKStages, NSV = L::kVStages;       // rings of key and of value tiles
 
     extern __shared__ __align__(1024) uint8_t smem[];
     const uint32_t base = smem_u32(smem);
     const uint32_t bar = base + L::kBars;
     const uint32_t q_full = bar;                    // 1
     const uint32_t q_free = q_full + 8;             // 1
-    const uint32_t kv_full = q_free + 8;            // NS
-    const uint32_t kv_empty = kv_full + 8 * NS;     // NS
+    const uint32_t k_full = q_free + 8;             // NSK
+    const uint32_t k_empty = k_full + 8 * NSK;      // NSK
+    const uint32_t v_full = k_empty + 8 * NSK;      // NSV
+    const uint32_t v_empty = v_full + 8 * NSV;      // NSV
     // Head size 64 leaves 128 TMEM columns free beside two score tiles and two 64-column accumulators: a THIRD score buffer.  The
     // three buffers go round robin to the Q K^T products in issue order (tile 0 / tile 1 alternating), so a query tile's next
     // scores are computed while its softmax warps are still on the current ones, and the softmax never waits for the tensor core
     // (ROT).  Head size 128 fills the 512 columns with two score tiles and two accumulators: buffer = query tile, as before.
-    constexpr bool ROT = HD == 64 && ROTP;
+    constexpr bool ROT = VD == 64 && ROTP;
     constexpr int NSB = ROT ? 3 : 2;                // score buffers
     constexpr uint32_t O_COL = ROT ? 384 : 256;     // first accumulator column
     constexpr uint32_t O_STRIDE = ROT ? 64 : 128;
-    const uint32_t s_full = kv_empty + 8 * NS;      // NSB (per score buffer)
+    const uint32_t s_full = v_empty + 8 * NSV;      // NSB (per score buffer)
     const uint32_t p_full = s_full + 8 * 3;         // NSB
     // P V products done: two barriers per query tile, taken in turn by the tile's steps (index step & 1, phase step >> 1).  With
     // rotating score buffers a tile's softmax can finish step j before P V of step j - 1 has completed, so its wait for the
@@ -178,11 +203,11 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const uint32_t o_free = pv_done + 32;           // 2
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + L::kBars + 240);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + L::kBars + 244);
-    static_assert(8 * (2 + 2 * NS + 12) <= 240, "barrier block overflows");
+    static_assert(8 * (2 + 2 * NSK + 2 * NSV + 12) <= 240, "barrier block overflows");
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int BH = p.B * p.H;
-    const int n_kv_seq = (p.T + kKvTile - 1) / kKvTile;
+    const int n_kv_seq = (p.n + kKvTile - 1) / kKvTile;
 
     if ((base & 1023u) != 0) {                                // swizzled tiles need 1024-byte alignment
         if (threadIdx.x == 0) atomicOr(p.status, 0x200u);
@@ -190,7 +215,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     }
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1); mbar_init(q_free, 1);
-        for (int s = 0; s < NS; s++) { mbar_init(kv_full + 8 * s, 1); mbar_init(kv_empty + 8 * s, 1); }
+        for (int s = 0; s < NSK; s++) { mbar_init(k_full + 8 * s, 1); mbar_init(k_empty + 8 * s, 1); }
+        for (int s = 0; s < NSV; s++) { mbar_init(v_full + 8 * s, 1); mbar_init(v_empty + 8 * s, 1); }
         for (int g = 0; g < 3; g++) {
             mbar_init(s_full + 8 * g, 1);
             mbar_init(p_full + 8 * g, 4);           // one arrival per softmax warp of the tile
@@ -207,20 +233,25 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const uint32_t tmem_base = *tmem_slot;
 
     // step k of this CTA's list; the entry of the next step is fetched while the current item runs
-    auto fetch = [&](int k) -> int { return k < p.sched_len ? __ldg(p.sched + (size_t)k * gridDim.x + blockIdx.x) : -1; };
+    auto fetch = [&](int k) -> int {
+        if (k >= p.sched_len) return -1;
+        const int at = k * (int)gridDim.x + (int)blockIdx.x;
+        return p.sched ? __ldg(p.sched + at) : at < p.n_ptiles * BH ? at : -1;
+    };
     // work item -> (first query row, sequence, head, key tiles of query tile 0 and of query tile 1)
     auto decode = [&](int item, int& q0, int& bb, int& hh, int& n0, int& n1) {
         const int pt = p.n_ptiles - 1 - item / BH;
         const int bh = item % BH;
         bb = bh / p.H; hh = bh % p.H;
         q0 = pt * kQPair;
-        n0 = min(q0 / kKvTile + 1, n_kv_seq);                             // causal: keys 0 .. q0+127
-        n1 = (q0 + kQTile < p.T) ? min(q0 / kKvTile + 2, n_kv_seq) : 0;   // second tile exists only inside the sequence
+        n0 = min((p.first + q0 + kQTile - 1) / kKvTile + 1, n_kv_seq);    // causal: keys 0 .. first+q0+127
+        n1 = (q0 + kQTile < p.T) ? min((p.first + q0 + 2 * kQTile - 1) / kKvTile + 1, n_kv_seq) : 0;   // second tile exists only inside the sequence
     };
 
     if (warp == 0) {
         // ---------------- TMA producer ----------------
         if (lane == 0) { tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV); }
+        if (KBR > 0 && lane == 0) { tma_prefetch_desc(&tmQr); tma_prefetch_desc(&tmKr); }
         bool ok = true;
         uint32_t g = 0, it = 0;
         for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
@@ -233,32 +264,57 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             if (!ok) break;
             if (lane == 0) {
                 mbar_expect_tx(q_full, 2 * L::kQTileBytes);
-                for (int t = 0; t < 2; t++)
-                    for (int kb = 0; kb < KB; kb++)
-                        tma_load_4d(base + L::kQ + t * L::kQTileBytes + kb * (kQTile * 128), &tmQ, q_full, kb * 64, q0 + t * kQTile, hh, bb);
-            }
-            for (int j = 0; j < nmax && ok; j++, g++) {
-                const uint32_t s = g % NS, u = (g / NS) & 1;
-                ok = mbar_wait(kv_empty + 8 * s, u ^ 1, abort_flag, p.status, kErrProducerWait);
-                if (!ok) break;
-                if (lane == 0) {
-                    const int k0 = j * kKvTile;
-                    const uint32_t dst = base + L::kKV + s * L::kStageBytes;
-                    mbar_expect_tx(kv_full + 8 * s, L::kStageBytes);
-                    for (int kb = 0; kb < KB; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, kv_full + 8 * s, kb * 64, k0, hh, bb);
-                    for (int kb = 0; kb < KB; kb++) tma_load_4d(dst + L::kKBytes + kb * (kKvTile * 128), &tmV, kv_full + 8 * s, kb * 64, k0, hh, bb);
+                for (int t = 0; t < 2; t++) {
+                    const uint32_t dst = base + L::kQ + t * L::kQTileBytes;
+                    for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kQTile * 128), &tmQ, q_full, kb * 64, q0 + t * kQTile, hh, bb);
+                    for (int kb = 0; kb < KBR; kb++) tma_load_4d(dst + (KBN + kb) * (kQTile * 128), &tmQr, q_full, kb * 64, q0 + t * kQTile, hh, bb);
                 }
-                __syncwarp();
             }
+            // keys run one tile ahead of the values: K_0, K_1, V_0, K_2, V_1, ... (the next scores are what the tensor core asks for first)
+            for (int j = 0; j <= nmax && ok; j++) {
+                if (j < nmax) {
+                    const uint32_t gk = g + j, s = gk % NSK;
+                    ok = mbar_wait(k_empty + 8 * s, ((gk / NSK) & 1) ^ 1, abort_flag, p.status, kErrProducerWait);
+                    if (!ok) break;
+                    if (lane == 0) {
+                        const uint32_t dst = base + L::kK + s * L::kKBytes;
+                        mbar_expect_tx(k_full + 8 * s, L::kKBytes);
+                        for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, k_full + 8 * s, kb * 64, j * kKvTile, hh, bb);
+                        for (int kb = 0; kb < KBR; kb++) tma_load_4d(dst + (KBN + kb) * (kKvTile * 128), &tmKr, k_full + 8 * s, kb * 64, j * kKvTile, 0, bb);
+                    }
+                    __syncwarp();
+                }
+                if (j > 0) {
+                    const uint32_t gv = g + j - 1, s = gv % NSV;
+                    ok = mbar_wait(v_empty + 8 * s, ((gv / NSV) & 1) ^ 1, abort_flag, p.status, kErrProducerWait);
+                    if (!ok) break;
+                    if (lane == 0) {
+                        const uint32_t dst = base + L::kV + s * L::kVBytes;
+                        mbar_expect_tx(v_full + 8 * s, L::kVBytes);
+                        for (int kb = 0; kb < VD / 64; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmV, v_full + 8 * s, kb * 64, (j - 1) * kKvTile, hh, bb);
+                    }
+                    __syncwarp();
+                }
+            }
+            g += nmax;
         }
     } else if (warp == 1) {
         // ---------------- MMA issuer ----------------
         bool ok = true;
         uint32_t g = 0, it = 0;                 // key tiles loaded so far (stage ring position); items so far
         uint32_t steps[2] = {0, 0};             // softmax steps of each query tile so far (phases of p_full)
+        // 16 keys per product: 8 columns of P, or with PSPLIT 8 columns of each half (a chunk of 32 keys is 16 + 16 columns)
+        auto mma_pv = [&](int t, uint32_t p_addr, uint64_t bdesc, bool accumulate) {
+#pragma unroll
+            for (int k = 0; k < kKvTile / 16; k++) {
+                const uint32_t o = tmem_base + O_COL + t * O_STRIDE, a = PSPLIT ? p_addr + 32 * (k / 2) + 8 * (k % 2) : p_addr + 8 * k;
+                mma_ts(o, a, bdesc + (uint64_t)(128 * k), IDESC_O, (accumulate || k != 0) ? 1u : 0u);
+                if (PSPLIT) mma_ts(o, a + 16, bdesc + (uint64_t)(128 * k), IDESC_O, 1u);
+            }
+        };
         // S_t = Q_t K^T with the key tile of ring position gg
         auto issue_s = [&](int t, uint32_t gg) {
-            const uint32_t kaddr = base + L::kKV + (gg % NS) * L::kStageBytes;
+            const uint32_t kaddr = base + L::kK + (gg % NSK) * L::kKBytes;
 #pragma unroll
             for (int kb = 0; kb < KB; kb++) {
                 const uint64_t adesc = make_kmajor_sw128_desc(base + L::kQ + t * L::kQTileBytes + kb * (kQTile * 128));
@@ -270,13 +326,12 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         };
         // O_t (+)= P_t V with the value tile of ring position gg; P is read from the TMEM columns of S_t
         auto issue_pv = [&](int t, uint32_t gg, bool accumulate, uint32_t pvidx) {      // pvidx: which product of this tile (over the whole kernel)
-            const uint64_t bdesc = make_mnmajor_sw128_desc(base + L::kKV + (gg % NS) * L::kStageBytes + L::kKBytes, kKvTile * 128);
-#pragma unroll
-            for (int k = 0; k < kKvTile / 16; k++)
-                mma_ts(tmem_base + O_COL + t * O_STRIDE, tmem_base + t * 128 + 8 * k, bdesc + (uint64_t)(128 * k), IDESC_O, (accumulate || k != 0) ? 1u : 0u);
+            const uint64_t bdesc = make_mnmajor_sw128_desc(base + L::kV + (gg % NSV) * L::kVBytes, kKvTile * 128);
+            mma_pv(t, tmem_base + t * 128, bdesc, accumulate);
             mma_commit(pv_done + 8 * (2 * t + (pvidx & 1)));
         };
-        auto kv_ready = [&](uint32_t gg) -> bool { return mbar_wait(kv_full + 8 * (gg % NS), (gg / NS) & 1, abort_flag, p.status, kErrMmaWait); };
+        auto k_ready = [&](uint32_t gg) -> bool { return mbar_wait(k_full + 8 * (gg % NSK), (gg / NSK) & 1, abort_flag, p.status, kErrMmaWait); };
+        auto v_ready = [&](uint32_t gg) -> bool { return mbar_wait(v_full + 8 * (gg % NSV), (gg / NSV) & 1, abort_flag, p.status, kErrMmaWait); };
         if constexpr (ROT) {
             // The products of an item in issue order ("entries"): key tile by key tile, query tile 0 before query tile 1 where both
             // still have that key tile.  Scores run up to two entries ahead of the P V product that is issued next; score number n
@@ -285,7 +340,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             uint32_t G = 0;                     // scores issued in earlier items
             auto issue_s3 = [&](int t, uint32_t gg, uint32_t n) {
                 const uint32_t buf = n % 3;
-                const uint32_t kaddr = base + L::kKV + (gg % NS) * L::kStageBytes;
+                const uint32_t kaddr = base + L::kK + (gg % NSK) * L::kKBytes;
 #pragma unroll
                 for (int kb = 0; kb < KB; kb++) {
                     const uint64_t adesc = make_kmajor_sw128_desc(base + L::kQ + t * L::kQTileBytes + kb * (kQTile * 128));
@@ -297,10 +352,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             };
             auto issue_pv3 = [&](int t, uint32_t gg, uint32_t n, bool accumulate, uint32_t pvidx) {
                 const uint32_t buf = n % 3;
-                const uint64_t bdesc = make_mnmajor_sw128_desc(base + L::kKV + (gg % NS) * L::kStageBytes + L::kKBytes, kKvTile * 128);
-#pragma unroll
-                for (int k = 0; k < kKvTile / 16; k++)
-                    mma_ts(tmem_base + O_COL + t * O_STRIDE, tmem_base + buf * 128 + 8 * k, bdesc + (uint64_t)(128 * k), IDESC_O, (accumulate || k != 0) ? 1u : 0u);
+                const uint64_t bdesc = make_mnmajor_sw128_desc(base + L::kV + (gg % NSV) * L::kVBytes, kKvTile * 128);
+                mma_pv(t, tmem_base + buf * 128, bdesc, accumulate);
                 mma_commit(pv_done + 8 * (2 * t + (pvidx & 1)));
             };
             for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
@@ -314,15 +367,18 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 };
                 ok = mbar_wait(q_full, it & 1, abort_flag, p.status, kErrMmaWait);
                 if (!ok) break;
-                int issued = 0, kv_seen = -1;
+                int issued = 0, k_seen = -1, v_seen = -1;
                 for (int e = 0; e < E && ok; e++) {
                     while (issued < min(E, e + 3)) {
                         int ts, js;
                         entry(issued, ts, js);
-                        if (js > kv_seen) { ok = kv_ready(g + js); kv_seen = js; if (!ok) break; }
+                        if (js > k_seen) { ok = k_ready(g + js); k_seen = js; if (!ok) break; }
                         tc_fence_after();
+                        int tn = 0, jn = -1;
+                        if (issued + 1 < E) entry(issued + 1, tn, jn);
                         if (elect_one_sync()) {
                             issue_s3(ts, g + js, G + issued);
+                            if (jn != js) mma_commit(k_empty + 8 * ((g + js) % NSK));            // every product that reads these keys has been issued
                             if (issued == E - 1) mma_commit(q_free);            // the item's last read of Q
                         }
                         __syncwarp();
@@ -335,13 +391,14 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     ok = mbar_wait(p_full + 8 * buf, (n / 3) & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
                     if (ok && j == 0) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j > v_seen) { ok = v_ready(g + j); v_seen = j; }
                     if (!ok) break;
                     tc_fence_after();
                     int tn = 0, jn = -1;
                     if (e + 1 < E) entry(e + 1, tn, jn);
                     if (elect_one_sync()) {
                         issue_pv3(t, g + j, n, j > 0, steps[t]);
-                        if (jn != j) mma_commit(kv_empty + 8 * ((g + j) % NS));     // every MMA that reads this stage has been issued
+                        if (jn != j) mma_commit(v_empty + 8 * ((g + j) % NSV));     // every MMA that reads these values has been issued
                     }
                     __syncwarp();
                     steps[t]++;
@@ -358,17 +415,19 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             const int nt[2] = {n0, n1};
             const int nmax = max(n0, n1);
             const int last_t = n1 > 0 ? 1 : 0;             // the tile whose last Q K^T is the item's last read of Q
-            ok = mbar_wait(q_full, it & 1, abort_flag, p.status, kErrMmaWait) && kv_ready(g);
+            ok = mbar_wait(q_full, it & 1, abort_flag, p.status, kErrMmaWait) && k_ready(g);
             if (!ok) break;
             tc_fence_after();
             if (elect_one_sync()) {
                 issue_s(0, g);
                 if (n1 > 0) issue_s(1, g);
                 if (nt[last_t] == 1) mma_commit(q_free);
+                mma_commit(k_empty + 8 * (g % NSK));
             }
             __syncwarp();
             for (int j = 0; j < nmax && ok; j++, g++) {
-                if (j + 1 < nmax) { ok = kv_ready(g + 1); if (!ok) break; }
+                ok = (j + 1 >= nmax || k_ready(g + 1)) && v_ready(g);
+                if (!ok) break;
                 for (int t = 0; t < 2 && ok; t++) {
                     if (j >= nt[t]) continue;
                     ok = mbar_wait(p_full + 8 * t, steps[t] & 1, abort_flag, p.status, kErrMmaWait);
@@ -388,7 +447,10 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     }
                     __syncwarp();
                 }
-                if (ok && elect_one_sync()) mma_commit(kv_empty + 8 * (g % NS));     // every MMA that reads this stage has been issued
+                if (ok && elect_one_sync()) {                   // every MMA that reads V_j, and K_(j+1), has been issued
+                    mma_commit(v_empty + 8 * (g % NSV));
+                    if (j + 1 < nmax) mma_commit(k_empty + 8 * ((g + 1) % NSK));
+                }
                 __syncwarp();
             }
         }
@@ -418,7 +480,9 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 ok = mbar_wait(s_full + 8 * sbuf, (ROT ? sn / 3 : sn) & 1, abort_flag, p.status, kErrEpilogueWait);
                 if (!ok) break;
                 tc_fence_after();
-                const bool diag = (j == n_kv - 1);               // the tile on the diagonal: keys q .. q+127 of rows q .. q+127
+                // row r of the tile sees the keys of this tile up to column r + delta
+                const int delta = p.first + q0 + t * kQTile - j * kKvTile;
+                const bool diag = delta < kKvTile - 1;
                 // The 128 scores of the row are taken in four chunks of 32: the load of chunk c + 1 is in flight while chunk c is
                 // worked on, and a chunk needs only 32 registers.  The reference maximum m of the row is allowed to lag the true
                 // maximum by up to 2^8 (lazy rescaling): a chunk whose maximum exceeds m by more moves m, and everything already
@@ -437,7 +501,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (c < 3) tmem_ld_32x32(s_addr + (c + 1) * 32, vnext);
                     if (DIAG) {
 #pragma unroll
-                        for (int i = 0; i < 32; i++) if (c * 32 + i > r) v[i] = 0xff800000u;       // -inf right of the diagonal
+                        for (int i = 0; i < 32; i++) if (c * 32 + i > r + delta) v[i] = 0xff800000u;       // -inf right of the diagonal
                     }
                     float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
 #pragma unroll
@@ -460,7 +524,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                             if (!mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait)) return false;
                             tc_fence_after();
 #pragma unroll
-                            for (int cc = 0; cc < HD / 32; cc++) {
+                            for (int cc = 0; cc < VD / 32; cc++) {
                                 uint32_t o[32];
                                 tmem_ld_32x32(o_addr + cc * 32, o);
                                 tmem_ld_wait();
@@ -469,7 +533,21 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                                 tmem_st_32x32(o_addr + cc * 32, o);
                             }
                         }
-                        if (c > 0) {
+                        if (c > 0 && PSPLIT) {
+                            uint32_t w[32];
+#pragma unroll
+                            for (int cc = 0; cc < c; cc++) {
+                                tmem_ld_32x32(s_addr + cc * 32, w);
+                                tmem_ld_wait();
+#pragma unroll
+                                for (int i = 0; i < 16; i++) {
+                                    const float lo = (__uint_as_float(w[i] << 16) + __uint_as_float(w[i + 16] << 16)) * alpha;
+                                    const float hi = (__uint_as_float(w[i] & 0xffff0000u) + __uint_as_float(w[i + 16] & 0xffff0000u)) * alpha;
+                                    split2(make_float2(lo, hi), w[i], w[i + 16]);
+                                }
+                                tmem_st_32x32(s_addr + cc * 32, w);
+                            }
+                        } else if (c > 0) {
                             // the chunks of P of this tile written so far: 16 columns (32 bf16) each
                             uint32_t w[16];
 #pragma unroll
@@ -490,7 +568,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     }
                     const float mb = m * p.scale_log2;
                     const float2 nmb2 = make_float2(-mb, -mb);
-                    uint32_t packed[16];
+                    uint32_t packed[PSPLIT ? 32 : 16];
 #pragma unroll
                     for (int i = 0; i < 16; i++) {
                         const float2 x = __ffma2_rn(make_float2(__uint_as_float(v[2 * i]), __uint_as_float(v[2 * i + 1])), c2, nmb2);
@@ -498,11 +576,16 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         if (i < NP) e = ex2_poly2(x);
                         else e = make_float2(ex2_approx(x.x), ex2_approx(x.y));
                         if (i & 1) sum_b = __fadd2_rn(sum_b, e); else sum_a = __fadd2_rn(sum_a, e);
-                        __nv_bfloat162 h2 = __floats2bfloat162_rn(e.x, e.y);
-                        packed[i] = *reinterpret_cast<uint32_t*>(&h2);
+                        if constexpr (PSPLIT) split2(e, packed[i], packed[i + 16]);
+                        else {
+                            __nv_bfloat162 h2 = __floats2bfloat162_rn(e.x, e.y);
+                            packed[i] = *reinterpret_cast<uint32_t*>(&h2);
+                        }
                     }
-                    // keys 32c .. 32c+31 of this row, two per column: columns 16c .. 16c+15, whose scores have been read (c' <= c)
-                    tmem_st_32x32b_x16(s_addr + c * 16, packed);
+                    // keys 32c .. 32c+31 of this row, two per column: columns 16c .. 16c+15, whose scores have been read (c' <= c);
+                    // the two halves of PSPLIT take the chunk's own 32 columns
+                    if constexpr (PSPLIT) tmem_st_32x32(s_addr + c * 32, packed);
+                    else tmem_st_32x32b_x16(s_addr + c * 16, packed);
                     return true;
                 };
                 auto tile = [&](auto npoly_tag, auto diag_tag) -> bool {
@@ -522,19 +605,21 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             G += (uint32_t)(n0 + n1);
             if (!ok) break;
             if (n_kv > 0) {
-                const float inv = 1.0f / l;
+                float inv = 1.0f / l;
+                if (p.gate && qrow < p.T) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[((long long)bb * p.T + qrow) * p.ld_gate + hh])));
                 ok = mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait);     // the item's last product
                 if (!ok) break;
                 tc_fence_after();
-                __nv_bfloat16* orow = p.out + ((long long)bb * p.T + qrow) * p.ld_out + (long long)hh * HD;
+                __nv_bfloat16* orow = p.out + ((long long)bb * p.T + qrow) * p.ld_out + (long long)hh * p.V;
 #pragma unroll
-                for (int c = 0; c < HD / 32; c++) {
+                for (int c = 0; c < VD / 32; c++) {
                     uint32_t o[32];
                     tmem_ld_32x32(o_addr + c * 32, o);
                     tmem_ld_wait();
                     if (qrow < p.T) {
 #pragma unroll
                         for (int i = 0; i < 32; i += 8) {
+                            if (KBR > 0 && c * 32 + i >= p.V) break;
                             uint4 w;
                             __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&w);
 #pragma unroll
@@ -578,11 +663,11 @@ static EncodeTiledFn attn_encode() {
 
 // bf16 rank-4 map over a token-major [B*T, ld] matrix seen as (head_dim, T, H, B): box (64, 128, 1, 1), 128-byte swizzle.
 // Rows past T read as zero (they belong to the next sequence in memory, but the T dimension of the map ends there).
-static int encode_heads(CUtensorMap* map, const void* ptr, int hd, int T, int H, int B, long long ld) {
+static int encode_heads(CUtensorMap* map, const void* ptr, int hd, int T, int H, int B, long long ld, long long head_stride, long long seq_stride) {
     EncodeTiledFn enc = attn_encode();
     if (!enc) return fail("cuTensorMapEncodeTiled is not available from this driver");
     cuuint64_t dims[4] = {(cuuint64_t)hd, (cuuint64_t)T, (cuuint64_t)H, (cuuint64_t)B};
-    cuuint64_t st[3] = {(cuuint64_t)ld * 2, (cuuint64_t)(H > 1 ? hd : ld) * 2, (cuuint64_t)(B > 1 ? (long long)T * ld : ld) * 2};
+    cuuint64_t st[3] = {(cuuint64_t)ld * 2, (cuuint64_t)(H > 1 ? head_stride : ld) * 2, (cuuint64_t)(B > 1 ? seq_stride : ld) * 2};
     cuuint32_t box[4] = {64, 128, 1, 1};
     cuuint32_t es[4] = {1, 1, 1, 1};
     CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(ptr), dims, st, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -665,9 +750,6 @@ static int attn_npoly(int hd) {
     return hd == 64 ? e64 : e128;
 }
 
-bool attention_latent_supported(int D, int rot, int V, int kv_off, long long ld_q, long long ld_kv, int row) { (void)D; (void)rot; (void)V; (void)kv_off; (void)ld_q; (void)ld_kv; (void)row; return false; }
-int attention_latent(const void*, long long, const void*, const void*, long long, const void*, long long, long long, void*, long long, const void*, long long, int, int, int, int, int, int, int, int, float) { return fail("todo"); }
-
 // q, k, v: [B*T, ld] bf16, head h at columns h*hd (token-major: the layout the QKV projection writes);
 // out: [B*T, ld_out] bf16, head h at columns h*hd.
 int attention_fused(const void* q, const void* k, const void* v, void* out, int B, int T, int H, int hd, long long ld_q, long long ld_k,
@@ -677,11 +759,11 @@ int attention_fused(const void* q, const void* k, const void* v, void* out, int 
         return fail("attention_fused: buffers must be 16-byte aligned");
     if (ld_out % 8) return fail("attention_fused: ld_out must be a multiple of 8");
     CUtensorMap tq, tk, tv;
-    if (encode_heads(&tq, q, hd, T, H, B, ld_q)) return 1;
-    if (encode_heads(&tk, k, hd, T, H, B, ld_k)) return 1;
-    if (encode_heads(&tv, v, hd, T, H, B, ld_v)) return 1;
+    if (encode_heads(&tq, q, hd, T, H, B, ld_q, hd, (long long)T * ld_q)) return 1;
+    if (encode_heads(&tk, k, hd, T, H, B, ld_k, hd, (long long)T * ld_k)) return 1;
+    if (encode_heads(&tv, v, hd, T, H, B, ld_v, hd, (long long)T * ld_v)) return 1;
     AttnParams prm;
-    prm.out = (__nv_bfloat16*)out; prm.ld_out = ld_out; prm.T = T; prm.H = H; prm.B = B;
+    prm.out = (__nv_bfloat16*)out; prm.ld_out = ld_out; prm.T = T; prm.H = H; prm.B = B; prm.n = T; prm.first = 0; prm.V = hd; prm.gate = nullptr; prm.ld_gate = 0;
     prm.n_ptiles = ceil_div(T, kQPair);
     prm.scale_log2 = (1.0f / sqrtf((float)hd)) * 1.4426950408889634f;
     prm.status = rt().dev_status;
@@ -693,25 +775,67 @@ int attention_fused(const void* q, const void* k, const void* v, void* out, int 
     ProfScope ps(PROF_ATTN_FUSED);
     auto launch = [&](auto kern, int smem_bytes) -> int {
         SPT_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes));
-        kern<<<(unsigned)grid, kAttnThreads, smem_bytes, rt().stream>>>(tq, tk, tv, prm);
+        kern<<<(unsigned)grid, kAttnThreads, smem_bytes, rt().stream>>>(tq, tk, tv, tq, tk, prm);
         return 0;
     };
     const int np = attn_npoly(hd);
     int lrc;
     if (hd == 64) {
         static const bool rot_off = getenv("SPTORCH_B200_ATTN_ROT") && atoi(getenv("SPTORCH_B200_ATTN_ROT")) == 0;
-        if (rot_off) lrc = launch(attn_fused_kernel<64, 0, false>, AttnSmem<64>::kTotal);
-        else if (np <= 0) lrc = launch(attn_fused_kernel<64, 0>, AttnSmem<64>::kTotal);
-        else if (np <= 4) lrc = launch(attn_fused_kernel<64, 4>, AttnSmem<64>::kTotal);
-        else if (np <= 5) lrc = launch(attn_fused_kernel<64, 5>, AttnSmem<64>::kTotal);
-        else if (np <= 6) lrc = launch(attn_fused_kernel<64, 6>, AttnSmem<64>::kTotal);
-        else lrc = launch(attn_fused_kernel<64, 8>, AttnSmem<64>::kTotal);
+        if (rot_off) lrc = launch(attn_fused_kernel<1, 0, 64, 0, false, false>, AttnSmem<1, 0, 64>::kTotal);
+        else if (np <= 0) lrc = launch(attn_fused_kernel<1, 0, 64, 0, true, false>, AttnSmem<1, 0, 64>::kTotal);
+        else if (np <= 4) lrc = launch(attn_fused_kernel<1, 0, 64, 4, true, false>, AttnSmem<1, 0, 64>::kTotal);
+        else if (np <= 5) lrc = launch(attn_fused_kernel<1, 0, 64, 5, true, false>, AttnSmem<1, 0, 64>::kTotal);
+        else if (np <= 6) lrc = launch(attn_fused_kernel<1, 0, 64, 6, true, false>, AttnSmem<1, 0, 64>::kTotal);
+        else lrc = launch(attn_fused_kernel<1, 0, 64, 8, true, false>, AttnSmem<1, 0, 64>::kTotal);
     } else {
-        if (np <= 0) lrc = launch(attn_fused_kernel<128, 0>, AttnSmem<128>::kTotal);
-        else lrc = launch(attn_fused_kernel<128, 4>, AttnSmem<128>::kTotal);
+        if (np <= 0) lrc = launch(attn_fused_kernel<2, 0, 128, 0, true, false>, AttnSmem<2, 0, 128>::kTotal);
+        else lrc = launch(attn_fused_kernel<2, 0, 128, 4, true, false>, AttnSmem<2, 0, 128>::kTotal);
     }
     if (lrc) return lrc;
     SPT_LAUNCH_CHECK("attn_fused");
+    return 0;
+}
+
+// ---- latent attention over expanded keys and values ----
+// q: [B*T, ld_q], head h at columns h*(D+rot): [D | rot]; kn, v: [B*n, ld_kv], head h at columns h*D / h*V; kr: the shared key part, rows
+// `row` elements apart, sequences seq_stride apart; gate: one logit per (token, head); out: [B*T, ld_out], head h at columns h*V.
+// Queries are at positions first .. first + T - 1, keys at 0 .. n - 1.
+bool attention_latent_supported(int D, int rot, int V, int kv_off, long long ld_q, long long ld_kv, int row) {
+    return D >= 8 && D <= 128 && D % 8 == 0 && rot >= 8 && rot <= 64 && rot % 8 == 0 && V >= 8 && V <= 128 && V % 8 == 0 && kv_off % 8 == 0 && ld_q % 8 == 0 &&
+           ld_kv % 8 == 0 && row % 8 == 0;
+}
+
+int attention_latent(const void* q, long long ld_q, const void* kn, const void* v, long long ld_kv, const void* kr, long long row, long long seq_stride,
+                     void* out, long long ld_out, const void* gate, long long ld_gate, int B, int T, int n, int H, int D, int rot, int V, int first, float scale) {
+    CUtensorMap tq, tqr, tk, tkr, tv;
+    if (encode_heads(&tq, q, D, T, H, B, ld_q, D + rot, (long long)T * ld_q)) return 1;
+    if (encode_heads(&tqr, (const __nv_bfloat16*)q + D, rot, T, H, B, ld_q, D + rot, (long long)T * ld_q)) return 1;
+    if (encode_heads(&tk, kn, D, n, H, B, ld_kv, D, (long long)n * ld_kv)) return 1;
+    if (encode_heads(&tv, v, V, n, H, B, ld_kv, V, (long long)n * ld_kv)) return 1;
+    if (encode_heads(&tkr, kr, rot, n, 1, B, row, row, seq_stride)) return 1;
+    AttnParams prm;
+    prm.out = (__nv_bfloat16*)out; prm.ld_out = ld_out; prm.T = T; prm.H = H; prm.B = B; prm.n = n; prm.first = first; prm.V = V;
+    prm.gate = (const __nv_bfloat16*)gate; prm.ld_gate = ld_gate;
+    prm.n_ptiles = ceil_div(T, kQPair);
+    prm.scale_log2 = scale * 1.4426950408889634f;
+    prm.status = rt().dev_status;
+    const long long items = (long long)B * H * prm.n_ptiles;
+    if (items > INT32_MAX) return fail("attention_latent: too many work items");
+    const long long slots = compute_sms(), grid = items < slots ? items : slots;
+    prm.sched = nullptr; prm.sched_len = ceil_div(items, grid);
+    // a prompt from position 0 uses a cached balanced schedule; a later portion, whose shape changes from call to call, the plain order
+    if (first == 0 && attention_schedule(B, H, T, (D + rot + V) / 2, prm.n_ptiles, (int)grid, &prm.sched, &prm.sched_len)) return 1;
+    auto launch = [&](auto kern, int smem_bytes) -> int {
+        SPT_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes));
+        kern<<<(unsigned)grid, kAttnThreads, smem_bytes, rt().stream>>>(tq, tk, tv, tqr, tkr, prm);
+        return 0;
+    };
+    int rc;
+    if (D <= 64) rc = V <= 64 ? launch(attn_fused_kernel<1, 1, 64, 0, true, true>, AttnSmem<1, 1, 64>::kTotal) : launch(attn_fused_kernel<1, 1, 128, 0, true, true>, AttnSmem<1, 1, 128>::kTotal);
+    else rc = V <= 64 ? launch(attn_fused_kernel<2, 1, 64, 0, true, true>, AttnSmem<2, 1, 64>::kTotal) : launch(attn_fused_kernel<2, 1, 128, 0, true, true>, AttnSmem<2, 1, 128>::kTotal);
+    if (rc) return rc;
+    SPT_LAUNCH_CHECK("attention_latent");
     return 0;
 }
 
