@@ -651,6 +651,126 @@ def sweep_decode(b, peaks, steps=32, emit=None, batches=(1, 8, 64)):
     return out
 
 
+# Layers of the size of real models': half gated linear attention, half latent attention, beside a Qwen-like model of equal width,
+# depth and feed-forward.  "prompt": (sequences, tokens) of a prefill; "decode": (sequences, cached positions).
+LAYERED_SIZES = {
+    "small": dict(width=768, n_layer=8, ff=3072, n_head=12, vocab=32000, gla=dict(heads=6, dim=64, vdim=128, tau=16.0, decay_rank=16),
+                  latent=dict(heads=12, dim=64, vdim=64, rot_dim=32, kv_rank=256, q_rank=384), prompts=((16, 1024), (1, 1024)), decodes=((1, 512), (8, 512), (64, 512))),
+    "large": dict(width=2048, n_layer=8, ff=5632, n_head=16, vocab=32000, gla=dict(heads=16, dim=64, vdim=128, tau=16.0, decay_rank=16),
+                  latent=dict(heads=16, dim=128, vdim=128, rot_dim=64, kv_rank=512, q_rank=1024), prompts=((8, 2048), (1, 2048)), decodes=((1, 2048), (8, 2048), (64, 1024))),
+    "wide_heads": dict(width=2048, n_layer=8, ff=5632, n_head=16, vocab=32000, gla=dict(heads=8, dim=128, vdim=256, tau=16.0, decay_rank=16),
+                       latent=dict(heads=16, dim=64, vdim=128, rot_dim=64, kv_rank=512, q_rank=512), prompts=((8, 2048),), decodes=((8, 2048),)),
+}
+
+
+def layered_config(z):
+    """config.json of a layered model of size z: gated linear attention without, latent attention with a feed-forward, alternating."""
+    la = dict(z["latent"], rot=dict(base=10000.0, dims=z["latent"]["rot_dim"]), scale=(z["latent"]["dim"] + z["latent"]["rot_dim"]) ** -0.5)
+    layers = [dict(type="gla", mixer=z["gla"], mlp=dict(kind="dense", ff=z["ff"])) if i % 2 == 0 else
+              dict(type="latent_attention", mixer=la, mlp=dict(kind="dense", ff=z["ff"])) for i in range(z["n_layer"])]
+    return dict(architecture="Tolevik", layers=layers, norm=dict(eps=1e-5), vocab=z["vocab"], width=z["width"])
+
+
+PROF_NAMES = ["linear_gemm", "attention_gemm", "causal_softmax", "norm", "embedding", "other", "attention", "gated_linear_attention", "latent_norms_rotation"]
+
+
+def _prof_pass(b, fn, reps):
+    lib = b.lib
+    lib.sptorch_ext_prof_enable(1); lib.sptorch_ext_prof_read(None, None, 0)
+    for _ in range(reps):
+        fn()
+    b.synchronize()
+    pm, pn = (C.c_float * 9)(), (C.c_uint32 * 9)()
+    lib.sptorch_ext_prof_read(pm, pn, 9); lib.sptorch_ext_prof_enable(0)
+    return {n: float(pm[i]) / reps for i, n in enumerate(PROF_NAMES) if pn[i]}
+
+
+def sweep_layered(b, peaks, iters, emit=None, sizes=None):
+    """Prefill and decode of a model built from a list of layers (random weights) beside the Qwen-like model of equal width, depth and
+    feed-forward.  Per kernel category: device time of a step (eager launches, CUDA events), and the fraction of its roofline --
+    algorithmic FLOP over the bf16 tensor peak or algorithmic bytes over the copy bandwidth, whichever takes longer.  Prompts of
+    (sequences x tokens) start at position 0; a decode step appends one token per sequence behind the given number of positions.
+    Inputs of a step (weights and activations) exceed L2."""
+    from sptorch_b200.backend import BF16
+    from sptorch_b200.gpt import QwenLikeGPT
+    from sptorch_b200.layered import LayeredGPT
+    out = []
+    for size in sizes or LAYERED_SIZES:
+        z = LAYERED_SIZES[size]
+        d, F, V, L, H = z["width"], z["ff"], z["vocab"], z["n_layer"], z["n_head"]
+        g, m = z["gla"], z["latent"]
+        max_tokens = max(B * (T + 64) for B, T in tuple(z["prompts"]) + tuple(z["decodes"]))
+        for kind in ("layered", "qwen_like"):
+            for phase, cases in (("prefill", z["prompts"]), ("decode", z["decodes"])):
+                for B, T in cases:
+                    cap = T + 64
+                    if kind == "layered":
+                        model = LayeredGPT(b, layered_config(z), cap, dtype=BF16, max_batch=B)
+                        cfg = dict(n_layer=L)
+                    else:
+                        model = QwenLikeGPT(b, V, d, H, L, F, cap, dtype=BF16, max_batch=B)
+                        cfg = dict(n_layer=L)
+                    _load_timing_weights(model, cfg)
+                    model.enable_kv_cache()
+                    ids = synth.randint(1, B * T, V).reshape(B, T).astype(np.int32)
+                    M = B * T if phase == "prefill" else B
+                    d_ids, d_log = model.stage_ids(ids), model.logits_buffer(B * T)
+                    prefill = lambda: b._check(b.lib.sptorch_ext_gpt_prefill(model.h, d_ids.handle, B, T, d_log.handle), "gpt_prefill")
+                    prefill()
+                    if phase == "prefill":
+                        step = prefill
+                    else:
+                        nxt = model.b.upload_bytes(synth.randint(2, B, V).astype(np.int32))
+                        step = lambda: b._check(b.lib.sptorch_ext_gpt_decode(model.h, nxt.handle, B, 1, d_log.handle), "gpt_decode")
+                    n = max(3, iters) if phase == "prefill" else 24
+                    for _ in range(4):
+                        step()
+                    b.synchronize()
+                    b.timer_begin()
+                    for _ in range(n):
+                        step()
+                    ms = b.timer_end() / n
+                    b.synchronize()
+                    parts = _prof_pass(b, step, 3)
+                    # algorithmic work per category
+                    half = L // 2
+                    w_mlp = 3 * d * F
+                    if kind == "layered":
+                        gw = d * (2 * g["heads"] * g["dim"] + 2 * g["heads"] * g["vdim"] + g["decay_rank"]) + d * g["heads"] * g["vdim"]
+                        lw = d * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + m["heads"]) + m["q_rank"] * m["heads"] * (m["dim"] + m["rot_dim"]) + d * m["heads"] * m["vdim"]
+                        up = m["kv_rank"] * m["heads"] * (m["dim"] + m["vdim"])
+                        w_lin = half * (gw + lw + 2 * w_mlp) + V * d + (half * up if phase == "prefill" else 0)
+                        dk, dv, ha, la_ = m["dim"] + m["rot_dim"], m["vdim"], m["heads"], half
+                        row = m["kv_rank"] + m["rot_dim"]
+                        if phase == "prefill":
+                            att = (B * ha * T * (T + 1.0) * (dk + dv) * la_, B * T * ha * (2 * dk + 2 * dv) * 2.0 * la_)
+                            gla = (M * g["heads"] * (4.0 * g["dim"] * g["vdim"] + 64 * (g["dim"] + g["vdim"])) * half, M * (g["heads"] * (2 * g["dim"] + 3 * g["vdim"]) + g["decay_rank"]) * 2.0 * half)
+                        else:
+                            att = (2.0 * B * ha * T * (row + m["kv_rank"]) * la_, (B * T * row + up) * 2.0 * la_)
+                            gla = (0.0, B * g["heads"] * g["dim"] * g["vdim"] * 8.0 * half)
+                        work = {"linear_gemm": (2.0 * M * w_lin, 2.0 * w_lin), "attention": att, "gated_linear_attention": gla,
+                                "norm": (0.0, M * d * 12.0 * 2 * L), "latent_norms_rotation": (0.0, 2.0 * 2 * M * (m["q_rank"] + row + (m["heads"] * m["rot_dim"] if phase == "prefill" else 0)) * half)}
+                    else:
+                        w_lin = L * (4 * d * d + w_mlp) + V * d
+                        att = (2.0 * B * T * (T + 1.0) * d * L, 8.0 * B * T * d * L) if phase == "prefill" else (0.0, 4.0 * B * T * d * L)
+                        work = {"linear_gemm": (2.0 * M * w_lin, 2.0 * w_lin), "attention": att, "norm": (0.0, M * d * 4.0 * (2 * L + 1)), "other": (0.0, M * 2 * d * 4.0 * L)}
+                    cats = {}
+                    for name, t in parts.items():
+                        e = {"ms": t}
+                        if name in work:
+                            fl, by = work[name]
+                            e["roofline_ms"] = max(fl / (peaks["tf"] * 1e12), by / (peaks["hbm"] * 1e9)) * 1e3
+                            e["frac"] = e["roofline_ms"] / t
+                        cats[name] = e
+                    rec = {"op": "layered", "size": size, "model": kind, "phase": phase, "batch": B, "tokens": T, "ms_per_step": ms,
+                           "tokens_per_s": M / (ms * 1e-3), "categories": cats, "peaks": [peaks["tf"], peaks["hbm"]]}
+                    out.append(rec)
+                    if emit:
+                        emit(rec)
+                    model.close()
+    return out
+
+
 def compact_sweeps(b, peaks, iters):
     """The three sweeps in the short form the bench line carries: one entry per case with its time and fraction of the roof
     (Linear and attention: measured burst bf16 tensor peak, TF32 against half of it; row ops: measured copy bandwidth)."""
@@ -687,6 +807,8 @@ def run_sweep(args):
         sweep_linear(b, peaks, args.iters, one if args.sweep == "linear" else None, emit)
     if args.sweep == "abi":
         sweep_abi(args, b)
+    if args.sweep == "layered":
+        sweep_layered(b, peaks, args.iters, emit, [args.size] if args.size else None)
     if args.sweep in ("attention", "all"):
         sweep_attention(b, peaks, args.iters, one if args.sweep == "attention" else None, emit)
     if args.sweep in ("rowops", "all"):
@@ -709,9 +831,9 @@ def _load_timing_weights(model, cfg, seed=0):
     rs = np.float32(1.0 / np.sqrt(2.0 * cfg["n_layer"]))
     for i, (name, shape) in enumerate(model.named_parameters()):
         n = int(np.prod(shape))
-        if name.endswith(".gamma"):
+        if name.endswith(".gamma") or "norm" in name:
             w = np.ones(n, np.float32)
-        elif name.endswith(".beta") or name.endswith(".bias"):
+        elif name.endswith(".beta") or name.endswith(".bias") or name.endswith(".b"):
             w = np.zeros(n, np.float32)
         else:
             w = np.resize(np.roll(block, 7919 * i), n)
@@ -858,8 +980,9 @@ def main():
     ap.add_argument("--chunk", type=int, default=8, help="sequences per micro-batch of the host-buffer call")
     ap.add_argument("--e2e-steps", type=int, default=3)
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
-    ap.add_argument("--sweep", default="", choices=["", "linear", "rowops", "attention", "decode", "abi", "all"], help="standalone op sweeps (the standalone Linear and row-op sweeps) instead of the GPT step")
+    ap.add_argument("--sweep", default="", choices=["", "linear", "rowops", "attention", "decode", "layered", "abi", "all"], help="standalone op sweeps (the standalone Linear and row-op sweeps) instead of the GPT step")
     ap.add_argument("--shape", default="", help="with --sweep linear: a single M,K,N; with --sweep decode: batch,steps")
+    ap.add_argument("--size", default="", choices=[""] + list(LAYERED_SIZES), help="with --sweep layered: one size")
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--workload", default=WORKLOAD, choices=[WORKLOAD, "c5_1p3b", "tp_check"],
                     help="c4_gpt2s: the bench line (batch sharding); c5_1p3b / tp_check: tensor parallel over the launched ranks")

@@ -226,7 +226,7 @@ bool expands(const Gpt* g, const LayeredLayer& w) {
 
 int gla_layer(Gpt* g, const LayeredLayer& w, int B, int T, bool few, bool cached) {
     const GlaArgs a = gla_args(g, w, B, T, cached);
-    ProfScope ps(PROF_OTHER);
+    ProfScope ps(PROF_RECURRENT);
     if (!few && gla_chunked_supported(a)) return gla_chunked(a, (float*)g->lay->gla_u.p, (float*)g->lay->gla_dec.p);
     return gla_recurrent(a, (float*)g->lay->gla_o.p, few);
 }
@@ -234,10 +234,10 @@ int gla_layer(Gpt* g, const LayeredLayer& w, int B, int T, bool few, bool cached
 int latent_layer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
     const LatentArgs a = latent_args(g, w, B, T, first, pos_dev, cached);
     const int M = B * T;
-    { ProfScope ps(PROF_OTHER); if (latent_prep(a, few)) return 1; }
+    { ProfScope ps(PROF_LATENT); if (latent_prep(a, few)) return 1; }
     if (product(g, few, a.cq, a.ld_cq, w.w_uq, a.ld_cq, (int)a.ld_cq, nullptr, nullptr, a.q, a.ld_q, M, (int)a.ld_q, EPI_NONE)) return 1;
     if (few || !expands(g, w)) { ProfScope ps(PROF_ATTN_FUSED); return latent_attention_absorbed(a, few); }
-    { ProfScope ps(PROF_OTHER); if (latent_rope_q(a)) return 1; }
+    { ProfScope ps(PROF_LATENT); if (latent_rope_q(a)) return 1; }
     // keys and values of positions 0 .. first + T - 1 of every sequence: [B][n][ukv_ld]
     const int n = first + T;
     GemmDesc d;
