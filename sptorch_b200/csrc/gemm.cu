@@ -572,6 +572,7 @@ bool gemm_supported(const GemmDesc& d, const char** why) {
     auto bad = [&](const char* w) { if (why) *why = w; return false; };
     if (d.mode != MM_TF32 && d.mode != MM_BF16) return bad("mode is not a tensor-core mode");
     if (d.M <= 0 || d.N <= 0 || d.K <= 0) return bad("empty problem");
+    if (d.group) return bad("block-diagonal products run on the weight-streaming kernel only");
     if ((reinterpret_cast<uintptr_t>(d.A) & 15) || (reinterpret_cast<uintptr_t>(d.B) & 15)) return bad("operand base not 16-byte aligned");
     if ((d.lda * es) % 16 || (d.ldb * es) % 16) return bad("operand row pitch not a multiple of 16 bytes");
     if (d.nb1 > 1 && ((d.sA1 * es) % 16 || (!d.b_broadcast && (d.sB1 * es) % 16))) return bad("batch stride not a multiple of 16 bytes");

@@ -48,6 +48,13 @@ struct GemmDesc {
     int* red_arg = nullptr;
     const long long* red_targets = nullptr;
     float* red_tgt = nullptr;
+    // Block-diagonal product of the weight-streaming kernel (heads): output columns come in groups of `group`; group i reads A from column
+    // i * group_a on and writes C from column i * group_c on.  gate: group i's outputs of row m are multiplied by
+    // sigmoid(gate[m * ld_gate + i]).  group is a multiple of 8 (0: an ordinary product).
+    int group = 0;
+    long long group_a = 0, group_c = 0;
+    const void* gate = nullptr;
+    long long ld_gate = 0;
 };
 inline int gemm_reduce_parts(int N) { return 2 * ((N + 255) / 256); }
 

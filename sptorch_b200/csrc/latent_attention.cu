@@ -9,6 +9,7 @@
 #include "layered.h"
 #include "pdl.cuh"
 #include <math.h>
+#include <cooperative_groups.h>
 
 namespace spt {
 
@@ -103,7 +104,7 @@ __global__ void __launch_bounds__(128) latent_absorb_kernel(const LatentArgs a) 
             v = (i & 1) ? v * cs.x + o * cs.y : v * cs.x - o * cs.y;
         }
     }
-    a.qabs[((size_t)m * a.H + h) * a.row + c] = v;
+    static_cast<float*>(a.qabs)[((size_t)m * a.H + h) * a.row + c] = v;
 }
 
 // One CTA per (head, token): four warps share the keys 0 .. pos, each with a running (maximum, sum, weighted latent); merged at the
@@ -117,7 +118,7 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const LatentArgs a) {
     pdl_acquire();
     const int n = (a.pos_dev ? a.pos_dev[0] : a.first) + (mt - b * a.T) + 1;
     const T* rows = static_cast<const T*>(a.rows) + (size_t)b * a.seq_stride;
-    const float* qp = a.qabs + ((size_t)mt * a.H + h) * a.row;
+    const float* qp = static_cast<const float*>(a.qabs) + ((size_t)mt * a.H + h) * a.row;
     float q[NV], o[NV];
 #pragma unroll
     for (int i = 0; i < NV; i++) { const int c = i * 32 + lane; q[i] = c < a.row ? qp[c] : 0.0f; o[i] = 0.0f; }
@@ -144,7 +145,7 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const LatentArgs a) {
 #pragma unroll
     for (int w = 0; w < 4; w++) { f[w] = m_sh[w] == -INFINITY ? 0.0f : expf(m_sh[w] - tm); tl += l_sh[w] * f[w]; }
     const float inv = 1.0f / tl;
-    float* out = a.olat + ((size_t)mt * a.H + h) * a.kv8;
+    float* out = static_cast<float*>(a.olat) + ((size_t)mt * a.H + h) * a.kv8;
     for (int c = threadIdx.x; c < a.kv8; c += 128) {
         float v = 0.0f;
 #pragma unroll
@@ -164,7 +165,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentArgs a) {
     if (i >= a.H * a.V) { if (lane == 0) out[i] = (T)0.0f; return; }
     const int h = i / a.V;
     const T* w = static_cast<const T*>(a.w_uv) + (size_t)i * a.ld_w;
-    const float* ol = a.olat + ((size_t)m * a.H + h) * a.kv8;
+    const float* ol = static_cast<const float*>(a.olat) + ((size_t)m * a.H + h) * a.kv8;
     float s = 0.0f;
     for (int c = lane; c < a.kv; c += 32) s = fmaf((float)w[c], ol[c], s);
 #pragma unroll
@@ -173,6 +174,224 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentArgs a) {
         const float g = (float)static_cast<const T*>(a.in)[(size_t)m * a.ld_in + a.c_g + h];
         out[i] = (T)(s * sigmoid_exact(g));
     }
+}
+
+// ---------------- few tokens, bf16: attention over the cached rows on the tensor cores ----------------
+// A cluster of `splits` CTAs owns one token and sixteen heads; each CTA walks its part of the positions in tiles of 64 cached rows
+// (cp.async, two tiles in flight).  Per tile: scores [16 heads x 64 keys] = Q rows^T, eight warps taking eight keys each; an online
+// softmax by 16 threads per head; O [16 x kv] += P rows, the warps taking kv / 8 columns each, with P as the sum of two bf16 numbers (16
+// mantissa bits).  The cluster's parts meet through distributed shared memory, every CTA merging a slice of the columns.  A row is read
+// from HBM once for all heads: 2 (kv + rot) bytes per position and sixteen heads.  mma.sync m16n8k16: sixteen heads are a sixteenth of a
+// tcgen05 tile's rows, and the kernel streams the cache at a few FLOP per byte.
+// NTW: 8-column tiles of the latent per warp (kv8 <= 64 NTW).
+constexpr int kLdThreads = 256, kLdKeys = 64, kLdP = 72, kLdS = 68;
+
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
+__device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+
+__host__ __device__ constexpr int ld_pitch(int row) { return (row + 31) / 32 * 32 + 8; }      // an odd number of 16-byte units: ldmatrix without conflicts
+inline size_t latent_decode_smem(int row) {
+    return (size_t)(2 * kLdKeys + 16) * ld_pitch(row) * 2 + 2 * 16 * kLdP * 2 + (size_t)16 * kLdS * 4 + 3 * 16 * 4;
+}
+
+template <int NTW>
+__global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const LatentArgs a, int splits, int groups) {
+    extern __shared__ __align__(16) uint8_t raw[];
+    const int pitch = ld_pitch(a.row), wide = pitch - 8;
+    __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(raw);                // [2][64][pitch]
+    __nv_bfloat16* qs = tile + 2 * kLdKeys * pitch;                             // [16][pitch]
+    __nv_bfloat16* ph = qs + 16 * pitch;                                        // [2][16][kLdP]: softmax weights, upper and lower half
+    float* ss = reinterpret_cast<float*>(ph + 2 * 16 * kLdP);                   // [16][kLdS]
+    float* corr_s = ss + 16 * kLdS;                                             // [16]
+    float* m_s = corr_s + 16;                                                   // [16]
+    float* l_s = m_s + 16;                                                      // [16]
+    float* o_s = reinterpret_cast<float*>(raw);                                 // [16][kv8 + 4], over the tiles once they are done
+    pdl_release();
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
+    const int rank = blockIdx.x % splits, item = blockIdx.x / splits, hg = item % groups, mt = item / groups, b = mt / a.T;
+    const int pos0 = a.pos_dev ? a.pos_dev[0] : a.first, n = pos0 + (mt - b * a.T) + 1;
+    const int part = ((n + splits - 1) / splits + kLdKeys - 1) / kLdKeys * kLdKeys, lo = min(n, rank * part), hi = min(n, lo + part);
+    const __nv_bfloat16* rows = static_cast<const __nv_bfloat16*>(a.rows) + (size_t)b * a.seq_stride;
+    const int per_row = a.row / 8;
+    auto load = [&](int stage, int k0) {
+        __nv_bfloat16* dst = tile + stage * kLdKeys * pitch;
+        for (int i = tid; i < kLdKeys * per_row; i += kLdThreads) {
+            const int k = i / per_row, c = (i - k * per_row) * 8;
+            if (k0 + k < hi) cp_async16(smem_addr(dst + k * pitch + c), rows + (size_t)(k0 + k) * a.row + c);
+            else *reinterpret_cast<uint4*>(dst + k * pitch + c) = make_uint4(0, 0, 0, 0);
+        }
+    };
+    // rows before this step's tokens were written by earlier steps: the first tile may be requested before the kernels ahead are done
+    const bool early = lo + kLdKeys <= pos0 && lo < hi;
+    if (early) load(0, lo);
+    for (int i = tid; i < (2 * kLdKeys + 16) * (wide - a.row); i += kLdThreads) {       // columns past the row: zero in every tile and in Q
+        const int r = i / (wide - a.row), c = a.row + i % (wide - a.row);
+        tile[r * pitch + c] = __float2bfloat16_rn(0.0f);
+    }
+    pdl_acquire();
+    if (!early && lo < hi) load(0, lo);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    // Q: absorbed part as it is, rotated part rotated to the token's position; missing heads of the last group are zero
+    for (int i = tid; i < 16 * per_row; i += kLdThreads) {
+        const int r = i / per_row, c = (i - r * per_row) * 8, h = hg * 16 + r;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (h < a.H) {
+            if (c < a.kv8) v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.qabs) + ((size_t)mt * a.H + h) * a.kv8 + c);
+            else {
+                const __nv_bfloat16* qr = static_cast<const __nv_bfloat16*>(a.q) + (size_t)mt * a.ld_q + (size_t)h * (a.D + a.rot) + a.D;
+                __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    const int e = c - a.kv8 + 2 * j;
+                    float x = e < a.rot ? __bfloat162float(qr[e]) : 0.0f, y = e + 1 < a.rot ? __bfloat162float(qr[e + 1]) : 0.0f;
+                    if (e < a.rope_dims) {
+                        const float2 cs = a.angles[(size_t)(n - 1) * (a.rope_dims / 2) + (e >> 1)];
+                        const float u = x * cs.x - y * cs.y;
+                        y = y * cs.x + x * cs.y; x = u;
+                    }
+                    o[j] = __floats2bfloat162_rn(x, y);
+                }
+            }
+        }
+        *reinterpret_cast<uint4*>(qs + r * pitch + c) = v;
+    }
+    float acc[NTW][4];
+#pragma unroll
+    for (int j = 0; j < NTW; j++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) acc[j][e] = 0.0f;
+    const float scale = a.scale * 1.4426950408889634f;
+    const int srow = tid >> 4, sk = (tid & 15) * 4;                             // softmax: 16 threads per head, four keys each
+    float m = -INFINITY, l = 0.0f;
+    int stage = 0;
+    for (int k0 = lo; k0 < hi; k0 += kLdKeys, stage ^= 1) {
+        if (k0 != lo) __syncthreads();                                          // the other stage's readers are done
+        if (k0 + kLdKeys < hi) load(stage ^ 1, k0 + kLdKeys);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();
+        const __nv_bfloat16* tl = tile + stage * kLdKeys * pitch;
+        {
+            float s0[4] = {0, 0, 0, 0}, s1[4] = {0, 0, 0, 0};
+            const uint32_t qa = smem_addr(qs + (lane & 15) * pitch + (lane >> 4) * 8), ka = smem_addr(tl + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 8);
+#pragma unroll 4
+            for (int k = 0; k < wide; k += 32) {
+                uint32_t x[4], y[4], kb[4];
+                ldsm4(x, qa + k * 2); ldsm4(y, qa + k * 2 + 32); ldsm4(kb, ka + k * 2);
+                mma_bf16(s0, x, kb[0], kb[1]);
+                mma_bf16(s1, y, kb[2], kb[3]);
+            }
+            const int c = warp * 8 + 2 * q4;
+            ss[g * kLdS + c] = (s0[0] + s1[0]) * scale; ss[g * kLdS + c + 1] = (s0[1] + s1[1]) * scale;
+            ss[(g + 8) * kLdS + c] = (s0[2] + s1[2]) * scale; ss[(g + 8) * kLdS + c + 1] = (s0[3] + s1[3]) * scale;
+        }
+        __syncthreads();
+        {
+            const float4 s4 = *reinterpret_cast<const float4*>(ss + srow * kLdS + sk);
+            float s[4] = {s4.x, s4.y, s4.z, s4.w}, mx = m, sum = 0.0f;
+#pragma unroll
+            for (int j = 0; j < 4; j++) { if (k0 + sk + j >= hi) s[j] = -INFINITY; mx = fmaxf(mx, s[j]); }
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            const float corr = ex2(m - mx);                                     // first tile: 2^(-inf) = 0
+            __nv_bfloat162 hi2[2], lo2[2];
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                const float e0 = ex2(s[2 * j] - mx), e1 = ex2(s[2 * j + 1] - mx);
+                sum += e0 + e1;
+                hi2[j] = __floats2bfloat162_rn(e0, e1);
+                const float2 f = bf16x2_to_float2(hi2[j]);
+                lo2[j] = __floats2bfloat162_rn(e0 - f.x, e1 - f.y);
+            }
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            l = l * corr + sum; m = mx;
+            *reinterpret_cast<uint2*>(ph + srow * kLdP + sk) = *reinterpret_cast<const uint2*>(hi2);
+            *reinterpret_cast<uint2*>(ph + (16 + srow) * kLdP + sk) = *reinterpret_cast<const uint2*>(lo2);
+            if ((tid & 15) == 0) corr_s[srow] = corr;
+        }
+        __syncthreads();
+        {
+            const float f0 = corr_s[g], f1 = corr_s[g + 8];
+#pragma unroll
+            for (int j = 0; j < NTW; j++) { acc[j][0] *= f0; acc[j][1] *= f0; acc[j][2] *= f1; acc[j][3] *= f1; }
+            const uint32_t pa = smem_addr(ph + (lane & 15) * kLdP + (lane >> 4) * 8), va = smem_addr(tl + (lane & 15) * pitch + warp * NTW * 8 + (lane >> 4) * 8);
+#pragma unroll
+            for (int k = 0; k < kLdKeys; k += 16) {
+                uint32_t x[4], y[4];
+                ldsm4(x, pa + k * 2); ldsm4(y, pa + 16 * kLdP * 2 + k * 2);
+#pragma unroll
+                for (int j = 0; j < NTW; j += 2) {
+                    if (warp * NTW * 8 + j * 8 < a.kv8) {
+                        uint32_t vb[4];
+                        ldsm4_trans(vb, va + (k * pitch + j * 8) * 2);
+                        mma_bf16(acc[j], x, vb[0], vb[1]); mma_bf16(acc[j], y, vb[0], vb[1]);
+                        mma_bf16(acc[j + 1], x, vb[2], vb[3]); mma_bf16(acc[j + 1], y, vb[2], vb[3]);
+                    }
+                }
+            }
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int lo_ = a.kv8 + 4;
+#pragma unroll
+    for (int j = 0; j < NTW; j++) {
+        const int c = (warp * NTW + j) * 8 + 2 * q4;
+        if (c < a.kv8) {
+            *reinterpret_cast<float2*>(o_s + g * lo_ + c) = make_float2(acc[j][0], acc[j][1]);
+            *reinterpret_cast<float2*>(o_s + (g + 8) * lo_ + c) = make_float2(acc[j][2], acc[j][3]);
+        }
+    }
+    if ((tid & 15) == 0) { m_s[srow] = m; l_s[srow] = l; }
+    namespace cg = cooperative_groups;
+    cg::cluster_group cluster = cg::this_cluster();
+    if (splits > 1) cluster.sync(); else __syncthreads();
+    // this CTA's slice of the columns, over all parts
+    const int slice = (a.kv8 / 8 + splits - 1) / splits * 8, c0 = rank * slice, c1 = min(a.kv8, c0 + slice);
+    const int w2 = max(0, c1 - c0) / 2;
+    for (int i = tid; i < 16 * w2; i += kLdThreads) {
+        const int r = i / w2, c = c0 + (i - r * w2) * 2, h = hg * 16 + r;
+        if (h >= a.H) continue;
+        float tm = -INFINITY, tl = 0.0f;
+        float2 t = make_float2(0.0f, 0.0f);
+        for (int s = 0; s < splits; s++) tm = fmaxf(tm, splits > 1 ? cluster.map_shared_rank(m_s, s)[r] : m_s[r]);
+        for (int s = 0; s < splits; s++) {
+            const float* om = splits > 1 ? cluster.map_shared_rank(o_s, s) : o_s;
+            const float ms = splits > 1 ? cluster.map_shared_rank(m_s, s)[r] : m_s[r], ls = splits > 1 ? cluster.map_shared_rank(l_s, s)[r] : l_s[r];
+            const float f = ms == -INFINITY ? 0.0f : ex2(ms - tm);
+            const float2 v = *reinterpret_cast<const float2*>(om + r * lo_ + c);
+            tl = fmaf(ls, f, tl); t.x = fmaf(v.x, f, t.x); t.y = fmaf(v.y, f, t.y);
+        }
+        const float inv = 1.0f / tl;
+        *reinterpret_cast<__nv_bfloat162*>(static_cast<__nv_bfloat16*>(a.olat) + ((size_t)mt * a.H + h) * a.kv8 + c) = __floats2bfloat162_rn(t.x * inv, t.y * inv);
+    }
+    if (splits > 1) cluster.sync();                     // no CTA leaves while its shared memory may still be read
+}
+
+template <int NTW>
+int launch_latent_decode(const LatentArgs& a, bool dependent) {
+    auto kern = latent_decode_kernel<NTW>;
+    const size_t smem = latent_decode_smem(a.row);
+    static size_t granted = 48 * 1024;
+    if (smem > granted) { SPT_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
+    const int groups = ceil_div(a.H, 16), items = a.B * a.T * groups;
+    int splits = 1;
+    while (splits < 8 && 2 * splits * items <= rt().sm_count && a.capacity > splits * kLdKeys) splits *= 2;
+    SPT_CUDA(launch_dependent(kern, dim3(items * splits), dim3(kLdThreads), smem, dependent, splits, a, splits, groups));
+    note_submit();
+    return 0;
 }
 
 template <typename T, int NV>
@@ -227,6 +446,15 @@ int latent_rope_q(const LatentArgs& a) {
 
 int latent_attention_absorbed(const LatentArgs& a, bool dependent) {
     return a.dtype == BF16 ? absorbed_t<__nv_bfloat16>(a, dependent) : absorbed_t<float>(a, dependent);
+}
+
+bool latent_decode_supported(const LatentArgs& a) {
+    return a.dtype == BF16 && a.kv8 <= 512 && latent_decode_smem(a.row) <= 227 * 1024;
+}
+
+int latent_decode(const LatentArgs& a, bool dependent) {
+    const int tiles = a.kv8 / 8;
+    return tiles <= 16 ? launch_latent_decode<2>(a, dependent) : tiles <= 32 ? launch_latent_decode<4>(a, dependent) : launch_latent_decode<8>(a, dependent);
 }
 
 }  // namespace spt

@@ -213,7 +213,8 @@ LatentArgs latent_args(Gpt* g, const LayeredLayer& w, int B, int T, int first, c
     a.cq = g->lay->cq.p; a.ld_cq = pad8(w.c.q_rank);
     a.q = g->lay->q.p; a.ld_q = w.q_ld();
     a.w_uk = w.w_ukv; a.w_uv = (const uint8_t*)w.w_ukv + (size_t)w.ukv_v() * a.kv8 * g->es; a.ld_w = a.kv8;
-    a.qabs = (float*)g->lay->qabs.p; a.olat = (float*)g->lay->olat.p;
+    a.qabs = g->lay->qabs.p; a.olat = g->lay->olat.p;
+    a.capacity = cached ? g->cache_ctx : T;
     a.out = g->lay->ao.p; a.ld_out = w.o_ld();
     a.dtype = g->c.dtype;
     return a;
@@ -236,6 +237,20 @@ int latent_layer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const i
     const int M = B * T;
     { ProfScope ps(PROF_LATENT); if (latent_prep(a, few)) return 1; }
     if (product(g, few, a.cq, a.ld_cq, w.w_uq, a.ld_cq, (int)a.ld_cq, nullptr, nullptr, a.q, a.ld_q, M, (int)a.ld_q, EPI_NONE)) return 1;
+    if (few && w.w_ukt && latent_decode_supported(a)) {
+        // queries absorbed head by head, attention over the cached rows, values head by head with the gates
+        GemmDesc d;
+        d.mode = MM_BF16; d.out_dtype = BF16; d.M = M;
+        d.A = a.q; d.lda = a.ld_q; d.B = w.w_ukt; d.K = a.D; d.ldb = a.D; d.N = a.H * a.kv8; d.C = a.qabs; d.ldc = d.N;
+        d.group = a.kv8; d.group_a = a.D + a.rot; d.group_c = a.kv8;
+        GemmDesc e = d;
+        e.A = a.olat; e.lda = d.N; e.B = a.w_uv; e.K = a.kv8; e.ldb = a.ld_w; e.N = a.H * a.V; e.C = a.out; e.ldc = a.ld_out;
+        e.group = a.V; e.group_a = a.kv8; e.group_c = a.V; e.gate = (const __nv_bfloat16*)a.in + a.c_g; e.ld_gate = a.ld_in;
+        if (linear_few_rows_supported(d) && linear_few_rows_supported(e)) {
+            ProfScope ps(PROF_ATTN_FUSED);
+            return linear_few_rows(d, nullptr, true) || latent_decode(a, true) || linear_few_rows(e, nullptr, true);
+        }
+    }
     if (few || !expands(g, w)) { ProfScope ps(PROF_ATTN_FUSED); return latent_attention_absorbed(a, few); }
     { ProfScope ps(PROF_LATENT); if (latent_rope_q(a)) return 1; }
     // keys and values of positions 0 .. first + T - 1 of every sequence: [B][n][ukv_ld]
@@ -261,9 +276,11 @@ int run(Gpt* g, const void* ids, int B, int T, int first, const int* pos_dev, bo
     float* x = (float*)lay.x.p;
     {
         ProfScope ps(PROF_EMBED);
-        if (dt == BF16) SPT_CUDA(launch_dependent(embed_rows_kernel<__nv_bfloat16>, dim3(M), dim3(128), 0, few, 1, (const __nv_bfloat16*)lay.embed, (const int*)ids, x,
+        // an ordinary launch: it starts when everything before this step is done, so the kernels behind it may read what earlier steps
+        // left in the cache before they wait for their predecessor
+        if (dt == BF16) SPT_CUDA(launch_dependent(embed_rows_kernel<__nv_bfloat16>, dim3(M), dim3(128), 0, false, 1, (const __nv_bfloat16*)lay.embed, (const int*)ids, x,
                                                   (__nv_bfloat16*)lay.xb.p, c.vocab, d8, rt().dev_status));
-        else SPT_CUDA(launch_dependent(embed_rows_kernel<float>, dim3(M), dim3(128), 0, few, 1, (const float*)lay.embed, (const int*)ids, x, (float*)lay.xb.p, c.vocab, d8,
+        else SPT_CUDA(launch_dependent(embed_rows_kernel<float>, dim3(M), dim3(128), 0, false, 1, (const float*)lay.embed, (const int*)ids, x, (float*)lay.xb.p, c.vocab, d8,
                                        rt().dev_status));
         note_submit();
     }
@@ -380,7 +397,18 @@ void layered_release(Gpt* g) { delete g->lay; g->lay = nullptr; }
 namespace {
 
 // one entry per tensor: its name behind the layer's prefix, its shape, and where it goes
-struct Slot { std::string name; size_t rows, cols; void* dst; bool f32; int ld; size_t dst_row; };      // cols 0: a vector of `rows` values
+struct Slot { std::string name; size_t rows, cols; void* dst; bool f32; int ld; size_t dst_row; const LayeredLayer* ukt = nullptr; };      // cols 0: a vector of `rows` values
+
+// uk [heads*dim, kv] -> its transpose per head, [heads][kv8][dim]
+int upload_ukt(Gpt* g, const Slot& s, const float* host) {
+    const LayeredLayer& w = *s.ukt;
+    const size_t H = w.c.heads, D = w.c.dim, kv = w.c.kv_rank, kv8 = w.kv8();
+    std::vector<float> t(H * kv8 * D, 0.0f);
+    for (size_t h = 0; h < H; h++)
+        for (size_t d = 0; d < D; d++)
+            for (size_t c = 0; c < kv; c++) t[(h * kv8 + c) * D + d] = host[(h * D + d) * kv + c];
+    return upload_rows(g, w.w_ukt, t.data(), t.size());
+}
 
 std::vector<Slot> layer_slots(const Gpt* g, const LayeredLayer& w) {
     const size_t d = g->c.d_model;
@@ -405,7 +433,9 @@ std::vector<Slot> layer_slots(const Gpt* g, const LayeredLayer& w) {
         mat("mix.dq", c.q_rank, d, w.w_in, d8, w.c_dq); vec("mix.dq.norm", c.q_rank, w.dq_norm);
         mat("mix.uq", (size_t)c.heads * (c.dim + c.rot_dim), c.q_rank, w.w_uq, q8, 0);
         mat("mix.dkv", (size_t)c.kv_rank + c.rot_dim, d, w.w_in, d8, w.c_dkv); vec("mix.dkv.norm", c.kv_rank, w.dkv_norm);
-        mat("mix.uk", (size_t)c.heads * c.dim, c.kv_rank, w.w_ukv, kv8, 0); mat("mix.uv", (size_t)c.heads * c.vdim, c.kv_rank, w.w_ukv, kv8, w.ukv_v());
+        mat("mix.uk", (size_t)c.heads * c.dim, c.kv_rank, w.w_ukv, kv8, 0);
+        if (w.w_ukt) s.back().ukt = &w;
+        mat("mix.uv", (size_t)c.heads * c.vdim, c.kv_rank, w.w_ukv, kv8, w.ukv_v());
         mat("mix.g", c.heads, d, w.w_in, d8, w.c_g);
         mat("mix.o", d, (size_t)c.heads * c.vdim, w.w_o, w.o_ld(), 0);
     }
@@ -445,6 +475,7 @@ int layered_set_param(Gpt* g, const char* name, const float* host, size_t n) {
         if (n != want) return fail("gpt_set_param(%s): got %zu values, expected %zu", name, n, want);
         if (s.f32) return sptorch_ext_copy_h2d_bytes(host, s.dst, n * 4) || stream_wait();
         void* dst = (uint8_t*)s.dst + s.dst_row * s.ld * g->es;
+        if (s.ukt && upload_ukt(g, s, host)) return 1;
         if ((size_t)s.ld == s.cols) return upload_rows(g, dst, host, n) || stream_wait();
         std::vector<float> padded(s.rows * s.ld, 0.0f);
         for (size_t r = 0; r < s.rows; r++) memcpy(&padded[r * s.ld], host + r * s.cols, s.cols * 4);
@@ -510,6 +541,7 @@ extern "C" void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const
             at(w.c_dq, lc.q_rank); at(w.c_dkv, lc.kv_rank + lc.rot_dim); at(w.c_g, lc.heads);
             w.dq_norm = F(lc.q_rank); w.dkv_norm = F(lc.kv_rank);
             w.w_uq = Z((size_t)w.q_ld() * pad8(lc.q_rank) * es); w.w_ukv = Z((size_t)w.ukv_ld() * w.kv8() * es);
+            if (c.dtype == SPT_BF16 && lc.dim % 8 == 0) w.w_ukt = Z((size_t)lc.heads * w.kv8() * lc.dim * es);
             if (lc.rope_dims) {
                 float2*& tab = angles[{lc.rope_dims, lc.rope_base}];
                 if (!tab) {

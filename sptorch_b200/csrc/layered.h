@@ -23,6 +23,7 @@ struct LayeredLayer {
     float* head_norm = nullptr;                  // [vdim]
     int c_dq = 0, c_dkv = 0;                     // latent attention: columns of the query latent and of [latent | rotated part]; c_g: the head gates
     float *dq_norm = nullptr, *dkv_norm = nullptr;
+    void* w_ukt = nullptr;                       // bf16, dim a multiple of 8: uk transposed per head, [heads][pad8(kv_rank)][dim] (few tokens)
     void *w_uq = nullptr, *w_ukv = nullptr;      // [heads*(dim+rot_dim), pad8(q_rank)]; [uk rows, then at row pad8(heads*dim) uv rows][pad8(kv_rank)]
     void* w_o = nullptr;                         // [pad8(width), pad8(heads*vdim)]
     float *norm1 = nullptr, *norm2 = nullptr;
@@ -104,7 +105,9 @@ struct LatentArgs {
     void* cq; long long ld_cq;                   // out of prep: normed query latent
     void* q; long long ld_q;                     // queries, head by head [D | rot]
     const void *w_uk, *w_uv; long long ld_w;
-    float *qabs, *olat;                          // per (token, head): absorbed query [row] and attended latent [kv8]
+    void *qabs, *olat;                           // per (token, head): absorbed query and attended latent.  Plain kernels: f32, [row] and
+                                                 // [kv8]; the tensor-core kernel: bf16, [kv8] (rotation applied as it loads) and [kv8]
+    int capacity;                                // positions the cache holds: what the split over CTAs is chosen for
     void* out; long long ld_out;
     int dtype;
 };
@@ -115,5 +118,8 @@ int latent_rope_q(const LatentArgs& a);
 // few tokens, or any tokens of a shape the fused kernel does not take: attention over the cached rows themselves, W_uk folded into
 // the query and W_uv applied to the attended latent
 int latent_attention_absorbed(const LatentArgs& a, bool dependent);
+// the attention of that path for bf16 on the tensor cores: qabs [M][H * kv8] without the rotated part -> olat [M][H * kv8]
+bool latent_decode_supported(const LatentArgs& a);
+int latent_decode(const LatentArgs& a, bool dependent);
 
 }  // namespace spt

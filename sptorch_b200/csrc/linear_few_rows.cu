@@ -48,6 +48,9 @@ __device__ __forceinline__ void mma_bf16_16x8x16(float (&d)[4], uint32_t a0, uin
 // (decode step of a 12-layer, 768-wide model at 64 sequences: 2.30 ms with, 1.0 ms without).
 constexpr int kNormMaxRows = 16;
 
+// GemmDesc's block-diagonal form
+struct FewRowsGroups { int group; long long group_a, group_c; const __nv_bfloat16* gate; long long ld_gate; };
+
 // MT: 16-row groups of A (M <= 16 MT); NT: 8-row groups of W per CTA; S: weight slices a warp has in flight.
 // NORM: A holds un-normalised rows; every CTA normalises them itself into shared memory (kind 1: LayerNorm, gamma * ((x - mean) *
 // inv) + beta with inv = 1 / sqrt(var + eps); kind 2: RMSNorm, x * inv * gamma with inv = 1 / sqrt(mean(x^2) + eps)), rounded to
@@ -57,7 +60,7 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
                                                                      const __nv_bfloat16* __restrict__ W, long long ldb,
                                                                      __nv_bfloat16* C, long long ldc, const float* __restrict__ bias,
                                                                      const __nv_bfloat16* R, int M, int N, int K, float alpha, int epilogue,
-                                                                     RowNorm nrm, int ksplit) {
+                                                                     RowNorm nrm, int ksplit, FewRowsGroups grp) {
     __shared__ float red[kWarps][MT * 16][NT * 8 + 1];
     extern __shared__ __align__(16) uint8_t dyn[];                       // NORM: M rows of (K + 8) bf16
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -66,6 +69,9 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
     const int n0 = (blockIdx.x / ksplit) * (NT * 8);
     const int all_slices = (K + 31) >> 5, per_cta = (all_slices + ksplit - 1) / ksplit;
     const int s_lo = krank * per_cta, slices = min(all_slices, s_lo + per_cta);
+    const int gi = grp.group ? n0 / grp.group : 0;          // a CTA's weight rows lie in one group
+    A += gi * grp.group_a;
+    C += gi * (grp.group_c - grp.group);
     const int k_mine = K - 8 * t;               // a slice s holds elements of this lane while 32 s < k_mine (K is a multiple of 8)
     pdl_release();
 
@@ -270,6 +276,7 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
         if (epilogue == EPI_GELU) v = gelu_fast2(make_float2(v, 0.0f)).x;
         else if (epilogue == EPI_SWIGLU) v = silu_fast(v);
         if (R) v = epilogue == EPI_SWIGLU ? v * rpre[it] : v + rpre[it];
+        if (grp.gate) v *= 1.0f / (1.0f + __expf(-__bfloat162float(grp.gate[(long long)m * grp.ld_gate + gi])));
         C[(long long)m * ldc + n] = __float2bfloat16_rn(v);
     }
 }
@@ -296,7 +303,8 @@ int launch(const GemmDesc& d, const RowNorm& nrm, bool dependent) {
     const int grid = ceil_div(d.N, NT * 8) * ksplit;
     SPT_CUDA(launch_dependent(kern, dim3(grid), dim3(kWarps * 32), smem, dependent, ksplit,
                               static_cast<const __nv_bfloat16*>(d.A), d.lda, static_cast<const __nv_bfloat16*>(d.B), d.ldb, static_cast<__nv_bfloat16*>(d.C), d.ldc,
-                              d.bias, static_cast<const __nv_bfloat16*>(d.R), d.M, d.N, d.K, d.alpha, d.epilogue, nrm, ksplit));
+                              d.bias, static_cast<const __nv_bfloat16*>(d.R), d.M, d.N, d.K, d.alpha, d.epilogue, nrm, ksplit,
+                              FewRowsGroups{d.group, d.group_a, d.group_c, static_cast<const __nv_bfloat16*>(d.gate), d.ld_gate}));
     note_submit();
     return 0;
 }
@@ -307,8 +315,8 @@ int dispatch(const GemmDesc& d, const RowNorm& nrm, bool dependent) {
     const long long want = 2ll * rt().sm_count;
     const int mt = d.M <= 16 ? 1 : d.M <= 32 ? 2 : 4;
     int nt = 1;
-    if (ceil_div(d.N, 16) >= want) nt = 2;
-    if (mt <= 2 && ceil_div(d.N, 32) >= want) nt = 4;
+    if (ceil_div(d.N, 16) >= want && d.group % 16 == 0) nt = 2;
+    if (mt <= 2 && ceil_div(d.N, 32) >= want && d.group % 32 == 0) nt = 4;
     if constexpr (NORM) {            // at most kNormMaxRows = 16 rows: one row group
         return nt == 1 ? launch<1, 1, true>(d, nrm, dependent) : nt == 2 ? launch<1, 2, true>(d, nrm, dependent) : launch<1, 4, true>(d, nrm, dependent);
     } else {
@@ -410,7 +418,7 @@ bool linear_few_rows_supported(const GemmDesc& d) {
     const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     return d.mode == MM_BF16 && d.out_dtype == BF16 && d.M >= 1 && d.M <= max_rows && d.N >= 1 && d.K >= 8 && d.K % 8 == 0 && d.nb1 * d.nb2 == 1 &&
            !d.causal_lower && !d.causal_k && !d.norm_axis && !d.reduce && d.lda % 8 == 0 && d.ldb % 8 == 0 && d.lda >= d.K && d.ldb >= d.K &&
-           d.ldc >= d.N && al16(d.A) && al16(d.B) && d.C != nullptr;
+           (d.group ? d.group > 0 && d.group % 8 == 0 && d.N % d.group == 0 && d.group_a % 8 == 0 && !d.R : d.ldc >= d.N) && al16(d.A) && al16(d.B) && d.C != nullptr;
 }
 
 bool linear_few_rows_norm_supported(const GemmDesc& d, const RowNorm& nrm) {
