@@ -125,9 +125,10 @@ __global__ void __launch_bounds__(256) gla_norm_gate_kernel(const GlaArgs a, con
 // Chunks are independent except through S, so three launches do a prompt: the chunks' own sums U = sum_s (k_s 2^(b_C - b_s)) v_s^T
 // (gla_chunk_state_kernel), a scan over the chunks that turns U into the state before each (gla_scan_kernel), and the outputs with head
 // norm and gate (gla_chunk_out_kernel).  (This is the chunkwise form of "Gated Linear Attention Transformers with Hardware-Efficient
-// Training", Yang, Wang, Shen, Panda, Kim.)  Every exponent that is evaluated is <= 0: A is taken in 16 x 16 blocks, off the diagonal
-// relative to the last token before the row block (2^(b_t - b_r) 2^(b_r - b_s)), on the diagonal pair by pair, so a strong decay
-// underflows where the product is nothing and never overflows.
+// Training", Yang, Wang, Shen, Panda, Kim.)  Every exponent that is evaluated is <= 0: A is taken as a binary tree of blocks -- rows
+// 32..63 against columns 0..31, then the two such halves of each 32, then of each 16 -- each relative to the last token r before its rows
+// (2^(b_t - b_r) 2^(b_r - b_s)), and pair by pair inside the 8 x 8 blocks on the diagonal, so a strong decay underflows where the product is
+// nothing and never overflows.
 // Products run as mma.sync on TF32 with each f32 operand split into two TF32 parts (hi hi + hi lo + lo hi: 21 mantissa bits); v comes
 // in bf16 and needs no split.  The tiles are 64 rows and the operands are scaled element by element on their way into the fragments,
 // so there is no operand for tcgen05 to fetch from shared memory as it lies there; the kernels are bound by that work and by HBM.
@@ -147,277 +148,350 @@ __device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], 
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-__host__ __device__ constexpr int round_up(int n, int m) { return (n + m - 1) / m * m; }
-// row pitches of shared-memory tiles: = 4 (mod 32) where fragments take rows by lane / 4 and columns by lane % 4, = 8 where the other way round
-__host__ __device__ constexpr int pitch4(int n) { return round_up(n, 32) + 4; }
-__host__ __device__ constexpr int pitch8(int n) { return round_up(n, 32) + 8; }
-
 struct ChunkArgs { GlaArgs a; float *u, *dec; int nc; };
 
-// rows of bf16 -> f32 tile [kChunk][pitch], zero outside n rows and w columns (up to wp columns); eight columns at a time where aligned
-__device__ __forceinline__ void load_tile(float* dst, int pitch, const __nv_bfloat16* src, long long ld, int n, int w, int wp, float f, bool vec) {
+// rows of bf16 -> f32 tile [kChunk][PITCH], zero outside n rows and w columns (up to WP columns); eight columns at a time where aligned
+template <int PITCH, int WP>
+__device__ __forceinline__ void load_tile(float* dst, const __nv_bfloat16* src, long long ld, int n, int w, float f, bool vec) {
     if (vec) {
-        const int per = wp / 8;
-        for (int i = threadIdx.x; i < kChunk * per; i += kChunkThreads) {
-            const int t = i / per, c = (i - t * per) * 8;
-            uint4 raw = make_uint4(0, 0, 0, 0);
-            if (t < n && c < w) raw = *reinterpret_cast<const uint4*>(src + (size_t)t * ld + c);
-            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        constexpr int PER = WP / 8;
 #pragma unroll
-            for (int j = 0; j < 4; j += 2) {
-                const float2 x = bf16x2_to_float2(h[j]), y = bf16x2_to_float2(h[j + 1]);
-                *reinterpret_cast<float4*>(dst + t * pitch + c + 2 * j) = make_float4(x.x * f, x.y * f, y.x * f, y.y * f);
+        for (int i0 = 0; i0 < kChunk * PER; i0 += kChunkThreads) {
+            const int i = i0 + (int)threadIdx.x;
+            if (kChunk * PER % kChunkThreads == 0 || i < kChunk * PER) {
+                const int t = i / PER, c = (i % PER) * 8;
+                uint4 raw = make_uint4(0, 0, 0, 0);
+                if (t < n && c < w) raw = *reinterpret_cast<const uint4*>(src + (size_t)t * ld + c);
+                const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+                for (int j = 0; j < 4; j += 2) {
+                    const float2 x = bf16x2_to_float2(h[j]), y = bf16x2_to_float2(h[j + 1]);
+                    *reinterpret_cast<float4*>(dst + t * PITCH + c + 2 * j) = make_float4(x.x * f, x.y * f, y.x * f, y.y * f);
+                }
             }
         }
     } else {
-        for (int i = threadIdx.x; i < kChunk * wp; i += kChunkThreads) {
-            const int t = i / wp, c = i - t * wp;
-            dst[t * pitch + c] = t < n && c < w ? (float)src[(size_t)t * ld + c] * f : 0.0f;
+        for (int i = threadIdx.x; i < kChunk * WP; i += kChunkThreads) {
+            const int t = i / WP, c = i % WP;
+            dst[t * PITCH + c] = t < n && c < w ? (float)src[(size_t)t * ld + c] * f : 0.0f;
         }
     }
 }
 
+// log2 of the decay: 1 + e with e = exp(-|z|) loses e's low bits, so a small e takes the series of log(1 + e) (next term e^5 / 5)
+__device__ __forceinline__ float log2_decay(float z, float inv_tau) {
+    const float e = exp2_fast(-1.4426950408889634f * fabsf(z));
+    float lg;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(lg) : "f"(1.0f + e));
+    const float series = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 0.33333334f), -0.5f), 1.0f) * 1.4426950408889634f;
+    return (fminf(z, 0.0f) * 1.4426950408889634f - (e < 0.03f ? series : lg)) * inv_tau;
+}
+
+// DP / VP: dim and vdim rounded up to the sizes the kernels are built for; padding columns are zeros
+template <int DP, int VP>
+struct ChunkSmem {
+    static constexpr int LDK = DP + 8, LDQ = DP + 4, LDV = VP + 8, LDA = 68;      // = 8 / 4 / 8 / 4 (mod 32)
+    static constexpr int kStateFloats = kChunk * (2 * LDK + LDV) + 4 * DP;        // + R (kChunk + DP) for the decay projection
+    static constexpr int kOutFloats = kChunk * (3 * LDQ + LDV + LDA) + 4 * kChunk;
+};
+
+template <int DP, int VP>
 __global__ void __launch_bounds__(kChunkThreads) gla_chunk_state_kernel(const ChunkArgs p) {
     extern __shared__ __align__(16) float sm[];
+    using L = ChunkSmem<DP, VP>;
+    constexpr int LDK = L::LDK, LDV = L::LDV;
     const GlaArgs& a = p.a;
-    const int D = a.D, V = a.V, R = a.R, Dp = round_up(D, 16), Vp = round_up(V, 8);
-    const int ldk = pitch8(Dp), ldv = pitch8(Vp);
-    float* bs = sm;                               // [kChunk][ldk]: log2 decays, then their running sums
-    float* ks = bs + kChunk * ldk;                // [kChunk][ldk]
-    float* vs = ks + kChunk * ldk;                // [kChunk][ldv]
-    float* a1s = vs + kChunk * ldv;               // [kChunk][R]
-    float* a2s = a1s + kChunk * R;                // [R][Dp]
-    float* seg = a2s + R * Dp;                    // [4][Dp]
+    const int D = a.D, V = a.V, R = a.R;
+    float* bs = sm;                               // [kChunk][LDK]: log2 decays, then their running sums
+    float* ks = bs + kChunk * LDK;                // [kChunk][LDK]
+    float* vs = ks + kChunk * LDK;                // [kChunk][LDV]
+    float* seg = vs + kChunk * LDV;               // [4][DP]
+    float* a1s = seg + 4 * DP;                    // [R][kChunk]
+    float* a2s = a1s + R * kChunk;                // [R][DP]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
     const int chunk = blockIdx.x, bh = blockIdx.y, b = bh / a.H, h = bh - b * a.H;
     const int t0 = chunk * kChunk, n = min(kChunk, a.T - t0);
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + ((size_t)b * a.T + t0) * a.ld;
     const bool vec = D % 8 == 0 && V % 8 == 0;
-    for (int i = tid; i < kChunk * R; i += kChunkThreads) { const int t = i / R; a1s[i] = t < n ? (float)in[(size_t)t * a.ld + a.c_a + (i - t * R)] : 0.0f; }
-    for (int i = tid; i < D * R; i += kChunkThreads) { const int d = i / R, r = i - d * R; a2s[r * Dp + d] = a.a2[(size_t)(h * D) * R + i]; }
-    load_tile(ks, ldk, in + a.c_k + h * D, a.ld, n, D, Dp, 1.0f, vec);
-    load_tile(vs, ldv, in + a.c_v + h * V, a.ld, n, V, Vp, 1.0f, vec);
+    for (int i = tid; i < kChunk * R; i += kChunkThreads) { const int t = i % kChunk, r = i / kChunk; a1s[i] = t < n ? (float)in[(size_t)t * a.ld + a.c_a + r] : 0.0f; }
+    for (int i = tid; i < DP * R; i += kChunkThreads) { const int d = i % DP, r = i / DP; a2s[i] = d < D ? __ldg(a.a2 + (size_t)(h * D + d) * R + r) : 0.0f; }
+    load_tile<LDK, DP>(ks, in + a.c_k + h * D, a.ld, n, D, 1.0f, vec);
+    load_tile<LDV, VP>(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
     __syncthreads();
     // log2 alpha of four tokens per turn of a thread; padding tokens and channels decay by nothing
-    const float to_log2 = 1.4426950408889634f, inv_tau = 1.0f / a.tau;
-    for (int i = tid; i < kChunk / 4 * Dp; i += kChunkThreads) {
-        const int d = i % Dp, t = i / Dp * 4;
-        float z[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        if (d < D) {
-            const float bias = a.a2_b[h * D + d];
-#pragma unroll
-            for (int j = 0; j < 4; j++) z[j] = bias;
-            for (int r = 0; r < R; r++) {
-                const float w = a2s[r * Dp + d];
-#pragma unroll
-                for (int j = 0; j < 4; j++) z[j] = fmaf(a1s[(t + j) * R + r], w, z[j]);
-            }
+    const float inv_tau = 1.0f / a.tau;
+#pragma unroll 1
+    for (int i = tid; i < kChunk / 4 * DP; i += kChunkThreads) {
+        const int d = i % DP, t = i / DP * 4;
+        const float bias = d < D ? a.a2_b[h * D + d] : 0.0f;
+        float z[4] = {bias, bias, bias, bias};
+#pragma unroll 4
+        for (int r = 0; r < R; r++) {
+            const float w = a2s[r * DP + d];
+            const float4 x = *reinterpret_cast<const float4*>(a1s + r * kChunk + t);
+            z[0] = fmaf(x.x, w, z[0]); z[1] = fmaf(x.y, w, z[1]); z[2] = fmaf(x.z, w, z[2]); z[3] = fmaf(x.w, w, z[3]);
         }
 #pragma unroll
-        for (int j = 0; j < 4; j++) bs[(t + j) * ldk + d] = d < D && t + j < n ? log_decay(z[j], inv_tau) * to_log2 : 0.0f;
+        for (int j = 0; j < 4; j++) bs[(t + j) * LDK + d] = d < D && t + j < n ? log2_decay(z[j], inv_tau) : 0.0f;
     }
     __syncthreads();
     // running sums: four segments of 16 tokens side by side, then the segments' totals on top
-    for (int i = tid; i < 4 * Dp; i += kChunkThreads) {
-        const int d = i % Dp, s = i / Dp;
+    for (int i = tid; i < 4 * DP; i += kChunkThreads) {
+        const int d = i % DP, s = i / DP;
         float sum = 0.0f;
 #pragma unroll
-        for (int t = 0; t < 16; t++) { float& x = bs[(s * 16 + t) * ldk + d]; sum += x; x = sum; }
-        seg[s * Dp + d] = sum;
+        for (int t = 0; t < 16; t++) { float& x = bs[(s * 16 + t) * LDK + d]; sum += x; x = sum; }
+        seg[i] = sum;
     }
     __syncthreads();
-    for (int i = tid; i < kChunk * Dp; i += kChunkThreads) {
-        const int d = i % Dp, t = i / Dp, s = t >> 4;
-        float off = 0.0f, tot = 0.0f;
+    {
+        float* dec = p.dec + ((size_t)bh * p.nc + chunk) * kChunk * D;
+        constexpr int STEP = kChunkThreads / DP;                       // tokens per turn; a thread keeps its channel
+        const int d = tid % DP;
+        float off[5];
+        off[0] = 0.0f;
 #pragma unroll
-        for (int j = 0; j < 4; j++) { const float x = seg[j * Dp + d]; if (j < s) off += x; tot += x; }
-        const float bt = bs[t * ldk + d] + off;
-        if (d < D) p.dec[(((size_t)bh * p.nc + chunk) * kChunk + t) * D + d] = bt;
-        ks[t * ldk + d] *= exp2_fast(fminf(tot - bt, 0.0f));
+        for (int j = 0; j < 4; j++) off[j + 1] = off[j] + seg[j * DP + d];
+#pragma unroll
+        for (int t1 = 0; t1 < kChunk; t1 += STEP) {
+            const int t = t1 + tid / DP;
+            const float bt = bs[t * LDK + d] + off[t1 >> 4];           // STEP divides 16: the segment does not depend on the thread
+            if (d < D) dec[(size_t)t * D + d] = bt;
+            ks[t * LDK + d] *= exp2_fast(fminf(off[4] - bt, 0.0f));
+        }
     }
     __syncthreads();
     // U[d][v] = sum_t ks[t][d] vs[t][v]: blocks of 16 channels x 64 values dealt over the warps
     float* u = p.u + ((size_t)bh * p.nc + chunk) * D * V;
-    const int mb = Dp / 16, nt = Vp / 8, nb = (nt + 7) / 8;
-    for (int blk = warp; blk < mb * nb; blk += kChunkThreads / 32) {
-        const int m0 = blk % mb * 16, n0 = blk / mb * 64;
+    constexpr int MB = DP / 16, NB = VP / 64;
+    for (int blk = warp; blk < MB * NB; blk += kChunkThreads / 32) {
+        const int m0 = blk % MB * 16, n0 = blk / MB * 64;
+        if (m0 >= D || n0 >= V) continue;
         float acc[8][4] = {};
-        for (int k = 0; k < kChunk; k += 8) {
+        const float *kp = ks + q4 * LDK + m0 + g, *vp = vs + q4 * LDV + n0 + g;
+#pragma unroll 2
+        for (int k = 0; k < kChunk; k += 8, kp += 8 * LDK, vp += 8 * LDV) {
             uint32_t hi[4], lo[4];
-            split_tf32(ks[(k + q4) * ldk + m0 + g], hi[0], lo[0]);
-            split_tf32(ks[(k + q4) * ldk + m0 + g + 8], hi[1], lo[1]);
-            split_tf32(ks[(k + q4 + 4) * ldk + m0 + g], hi[2], lo[2]);
-            split_tf32(ks[(k + q4 + 4) * ldk + m0 + g + 8], hi[3], lo[3]);
+            split_tf32(kp[0], hi[0], lo[0]);
+            split_tf32(kp[8], hi[1], lo[1]);
+            split_tf32(kp[4 * LDK], hi[2], lo[2]);
+            split_tf32(kp[4 * LDK + 8], hi[3], lo[3]);
 #pragma unroll
             for (int j = 0; j < 8; j++) {
-                const int c = n0 + 8 * j;
-                if (c < Vp) {
-                    const uint32_t b0 = __float_as_uint(vs[(k + q4) * ldv + c + g]), b1 = __float_as_uint(vs[(k + q4 + 4) * ldv + c + g]);
-                    mma_tf32(acc[j], hi, b0, b1);
-                    mma_tf32(acc[j], lo, b0, b1);
-                }
+                const uint32_t b0 = __float_as_uint(vp[8 * j]), b1 = __float_as_uint(vp[4 * LDV + 8 * j]);
+                mma_tf32(acc[j], lo, b0, b1);
+                mma_tf32(acc[j], hi, b0, b1);
             }
         }
+        const bool even = V % 2 == 0;
 #pragma unroll
         for (int j = 0; j < 8; j++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-                const int d = m0 + g + (e >> 1) * 8, v = n0 + 8 * j + 2 * q4 + (e & 1);
-                if (d < D && v < V) u[(size_t)d * V + v] = acc[j][e];
+            for (int e = 0; e < 2; e++) {
+                const int d = m0 + g + e * 8, v = n0 + 8 * j + 2 * q4;
+                if (d < D && v < V) {
+                    if (even) *reinterpret_cast<float2*>(u + (size_t)d * V + v) = make_float2(acc[j][2 * e], acc[j][2 * e + 1]);
+                    else { u[(size_t)d * V + v] = acc[j][2 * e]; if (v + 1 < V) u[(size_t)d * V + v + 1] = acc[j][2 * e + 1]; }
+                }
             }
     }
 }
 
-// u[c] <- the state before chunk c; state <- the state behind the last one.  One thread per element, eight chunks in flight.
+// u[c] <- the state before chunk c; state <- the state behind the last one.  A thread owns W neighbouring values (W = 4 where V is a
+// multiple of four), eight chunks in flight.
+template <int W>
 __global__ void __launch_bounds__(256) gla_scan_kernel(const ChunkArgs p) {
+    struct alignas(4 * W) Vec { float v[W]; };
     const GlaArgs& a = p.a;
     const int DV = a.D * a.V;
-    const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+    const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * W;
     if (i >= (long long)a.B * a.H * DV) return;
     const int bh = (int)(i / DV), e = (int)(i - (long long)bh * DV), d = e / a.V;
     float* u = p.u + (size_t)bh * p.nc * DV + e;
     const float* last = p.dec + ((size_t)bh * p.nc * kChunk + kChunk - 1) * a.D + d;
-    float s = a.state ? a.state[i] : 0.0f;
+    Vec s;
+#pragma unroll
+    for (int w = 0; w < W; w++) s.v[w] = 0.0f;
+    if (a.state) s = *reinterpret_cast<const Vec*>(a.state + i);
     for (int c0 = 0; c0 < p.nc; c0 += 8) {
-        float x[8], f[8];
+        Vec x[8];
+        float f[8];
 #pragma unroll
         for (int j = 0; j < 8; j++)
-            if (c0 + j < p.nc) { x[j] = u[(size_t)(c0 + j) * DV]; f[j] = last[(size_t)(c0 + j) * kChunk * a.D]; }
+            if (c0 + j < p.nc) { x[j] = *reinterpret_cast<const Vec*>(u + (size_t)(c0 + j) * DV); f[j] = last[(size_t)(c0 + j) * kChunk * a.D]; }
 #pragma unroll
         for (int j = 0; j < 8; j++)
-            if (c0 + j < p.nc) { u[(size_t)(c0 + j) * DV] = s; s = fmaf(s, exp2_fast(f[j]), x[j]); }
+            if (c0 + j < p.nc) {
+                *reinterpret_cast<Vec*>(u + (size_t)(c0 + j) * DV) = s;
+                const float g = exp2_fast(f[j]);
+#pragma unroll
+                for (int w = 0; w < W; w++) s.v[w] = fmaf(s.v[w], g, x[j].v[w]);
+            }
     }
-    if (a.state) a.state[i] = s;
+    if (a.state) *reinterpret_cast<Vec*>(a.state + i) = s;
 }
 
-// Warps are 2 (halves of the rows) x 4 (quarters of the values); NT: the most 8-column tiles a warp owns (V <= 32 NT).
-template <int NT>
+// One block of A: rows r0 .. r0 + 15 (ROWS8: only the lower eight of the fragment, rows r0 .. r0 + 7), columns c0 .. c0 + 8 NTILES - 1, all
+// before row `ref + 1`; exponents relative to token ref.
+template <int DP, int NTILES, bool ROWS8>
+__device__ __forceinline__ void a_block(const float* qs, const float* ks, const float* bs, float* as, int r0, int c0, int ref, int g, int q4) {
+    constexpr int LD = DP + 4, LDA = 68;
+    float acc[NTILES][4] = {};
+    const float *qp = qs + (r0 + g) * LD + q4, *bq = bs + (r0 + g) * LD + q4, *br = bs + ref * LD + q4, *kp = ks + (c0 + g) * LD + q4, *bk = bs + (c0 + g) * LD + q4;
+#pragma unroll 2
+    for (int k = 0; k < DP; k += 8) {
+        const float f0 = br[k], f1 = br[k + 4];
+        uint32_t ah[4] = {0, 0, 0, 0}, al[4] = {0, 0, 0, 0};
+        split_tf32(qp[k] * exp2_fast(bq[k] - f0), ah[0], al[0]);
+        split_tf32(qp[k + 4] * exp2_fast(bq[k + 4] - f1), ah[2], al[2]);
+        if (!ROWS8) {
+            split_tf32(qp[8 * LD + k] * exp2_fast(bq[8 * LD + k] - f0), ah[1], al[1]);
+            split_tf32(qp[8 * LD + k + 4] * exp2_fast(bq[8 * LD + k + 4] - f1), ah[3], al[3]);
+        }
+#pragma unroll
+        for (int j = 0; j < NTILES; j++) {
+            uint32_t h0, l0, h1, l1;
+            split_tf32(kp[8 * j * LD + k] * exp2_fast(f0 - bk[8 * j * LD + k]), h0, l0);
+            split_tf32(kp[8 * j * LD + k + 4] * exp2_fast(f1 - bk[8 * j * LD + k + 4]), h1, l1);
+            mma_tf32(acc[j], al, h0, h1);
+            mma_tf32(acc[j], ah, l0, l1);
+            mma_tf32(acc[j], ah, h0, h1);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NTILES; j++) {
+        float* o = as + (r0 + g) * LDA + c0 + 8 * j + 2 * q4;
+        o[0] = acc[j][0]; o[1] = acc[j][1];
+        if (!ROWS8) { o[8 * LDA] = acc[j][2]; o[8 * LDA + 1] = acc[j][3]; }
+    }
+}
+
+// Warps are 2 (halves of the rows) x 4 (quarters of the values), NT 8-column tiles each.
+template <int DP, int VP>
 __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const ChunkArgs p) {
     extern __shared__ __align__(16) float sm[];
+    using L = ChunkSmem<DP, VP>;
+    constexpr int LD = L::LDQ, LDV = L::LDV, LDA = L::LDA, NT = VP / 32;
     const GlaArgs& a = p.a;
-    const int D = a.D, V = a.V, Dp = round_up(D, 16), Vp = round_up(V, 8);
-    const int ld = pitch4(Dp), ldv = pitch8(Vp);
-    constexpr int lda = 68;
-    float* bs = sm;                               // [kChunk][ld]: running sums of the log2 decays
-    float* qs = bs + kChunk * ld;                 // [kChunk][ld]: q D^(-1/2), later times 2^b
-    float* ks = qs + kChunk * ld;
-    float* vs = ks + kChunk * ld;                 // [kChunk][ldv]
-    float* as = vs + kChunk * ldv;                // [kChunk][lda]: A
-    float* red = as + kChunk * lda;               // [4][kChunk]
+    const int D = a.D, V = a.V;
+    float* bs = sm;                               // [kChunk][LD]: running sums of the log2 decays
+    float* qs = bs + kChunk * LD;                 // [kChunk][LD]: q D^(-1/2), later times 2^b
+    float* ks = qs + kChunk * LD;
+    float* vs = ks + kChunk * LD;                 // [kChunk][LDV]
+    float* as = vs + kChunk * LDV;                // [kChunk][LDA]: A
+    float* red = as + kChunk * LDA;               // [4][kChunk]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
     const int chunk = blockIdx.x, bh = blockIdx.y, b = bh / a.H, h = bh - b * a.H;
     const int t0 = chunk * kChunk, n = min(kChunk, a.T - t0);
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + ((size_t)b * a.T + t0) * a.ld;
     const bool vec = D % 8 == 0 && V % 8 == 0;
     const float* dec = p.dec + ((size_t)bh * p.nc + chunk) * kChunk * D;
-    for (int i = tid; i < kChunk * Dp; i += kChunkThreads) { const int t = i / Dp, d = i - t * Dp; bs[t * ld + d] = d < D ? dec[(size_t)t * D + d] : 0.0f; }
-    load_tile(qs, ld, in + a.c_q + h * D, a.ld, n, D, Dp, 1.0f / sqrtf((float)D), vec);
-    load_tile(ks, ld, in + a.c_k + h * D, a.ld, n, D, Dp, 1.0f, vec);
-    load_tile(vs, ldv, in + a.c_v + h * V, a.ld, n, V, Vp, 1.0f, vec);
-    for (int i = tid; i < kChunk * lda; i += kChunkThreads) as[i] = 0.0f;
+    if (D % 4 == 0) {
+#pragma unroll
+        for (int i0 = 0; i0 < kChunk * DP / 4; i0 += kChunkThreads) {
+            const int i = i0 + tid, t = i / (DP / 4), d = i % (DP / 4) * 4;
+            *reinterpret_cast<float4*>(bs + t * LD + d) = d < D ? *reinterpret_cast<const float4*>(dec + (size_t)t * D + d) : make_float4(0, 0, 0, 0);
+        }
+    } else
+        for (int i = tid; i < kChunk * DP; i += kChunkThreads) { const int t = i / DP, d = i % DP; bs[t * LD + d] = d < D ? dec[(size_t)t * D + d] : 0.0f; }
+    load_tile<LD, DP>(qs, in + a.c_q + h * D, a.ld, n, D, 1.0f / sqrtf((float)D), vec);
+    load_tile<LD, DP>(ks, in + a.c_k + h * D, a.ld, n, D, 1.0f, vec);
+    load_tile<LDV, VP>(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
+    for (int i = tid; i < kChunk * LDA / 4; i += kChunkThreads) reinterpret_cast<float4*>(as)[i] = make_float4(0, 0, 0, 0);
     __syncthreads();
 
+    // A: four tasks of the 32-row block and two of the 16-row blocks (16 rows x 16 columns each), four 8 x 8 blocks, and the 288 pairs of
+    // the diagonal blocks in nine turns of a warp
+    int pair_turn, pair_last;                     // this warp's turns
     if (warp < 4) {
-        // diagonal block `warp`: its 136 pairs (t, s <= t) one by one, four channels at a time
-        const int r0 = warp * 16;
-#pragma unroll 1
-        for (int pr = lane; pr < 136; pr += 32) {
-            int t = (int)((sqrtf(8.0f * pr + 1.0f) - 1.0f) * 0.5f);
-            while ((t + 1) * (t + 2) / 2 <= pr) t++;
-            while (t * (t + 1) / 2 > pr) t--;
-            const int s = pr - t * (t + 1) / 2;
-            const float *qt = qs + (r0 + t) * ld, *bt = bs + (r0 + t) * ld, *kt = ks + (r0 + s) * ld, *bk = bs + (r0 + s) * ld;
-            float acc = 0.0f;
-            for (int d = 0; d < Dp; d += 4) {
-                const float4 x = *reinterpret_cast<const float4*>(qt + d), y = *reinterpret_cast<const float4*>(kt + d);
-                const float4 u = *reinterpret_cast<const float4*>(bt + d), w = *reinterpret_cast<const float4*>(bk + d);
-                acc = fmaf(x.x * y.x, exp2_fast(u.x - w.x), acc); acc = fmaf(x.y * y.y, exp2_fast(u.y - w.y), acc);
-                acc = fmaf(x.z * y.z, exp2_fast(u.z - w.z), acc); acc = fmaf(x.w * y.w, exp2_fast(u.w - w.w), acc);
-            }
-            as[(r0 + t) * lda + r0 + s] = acc;
-        }
+        a_block<DP, 2, false>(qs, ks, bs, as, 32 + 16 * (warp >> 1), 16 * (warp & 1), 31, g, q4);
+        a_block<DP, 1, true>(qs, ks, bs, as, 16 * warp + 8, 16 * warp, 16 * warp + 7, g, q4);
+        pair_turn = 0; pair_last = warp == 0 ? 1 : 0;
     } else {
-        // the six blocks below the diagonal, each as two halves of eight columns: twelve tasks over four warps
+        if (warp < 6) a_block<DP, 2, false>(qs, ks, bs, as, warp == 4 ? 16 : 48, warp == 4 ? 0 : 32, warp == 4 ? 15 : 47, g, q4);
+        pair_turn = warp == 4 ? 1 : warp == 5 ? 2 : warp == 6 ? 3 : 6; pair_last = warp == 4 ? 2 : warp == 5 ? 3 : warp == 6 ? 6 : 9;
+    }
 #pragma unroll 1
-        for (int task = warp - 4; task < 12; task += 4) {
-            const int blk = task >> 1, i = blk == 0 ? 1 : blk < 3 ? 2 : 3, j = blk == 0 ? 0 : blk < 3 ? blk - 1 : blk - 3;
-            const int r0 = 16 * i, c0 = 16 * j + 8 * (task & 1);
-            const float* br = bs + (r0 - 1) * ld;                       // the last token before the row block
-            float acc[4] = {};
-            for (int k = 0; k < Dp; k += 8) {
-                uint32_t ah[4], al[4], bh_[2], bl[2];
-#pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    const int t = r0 + g + (e & 1) * 8, d = k + q4 + (e >> 1) * 4;
-                    split_tf32(qs[t * ld + d] * exp2_fast(bs[t * ld + d] - br[d]), ah[e], al[e]);
-                }
-#pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    const int s = c0 + g, d = k + q4 + e * 4;
-                    split_tf32(ks[s * ld + d] * exp2_fast(br[d] - bs[s * ld + d]), bh_[e], bl[e]);
-                }
-                mma_tf32(acc, al, bh_[0], bh_[1]);
-                mma_tf32(acc, ah, bl[0], bl[1]);
-                mma_tf32(acc, ah, bh_[0], bh_[1]);
-            }
-#pragma unroll
-            for (int e = 0; e < 4; e++) as[(r0 + g + (e >> 1) * 8) * lda + c0 + 2 * q4 + (e & 1)] = acc[e];
+    for (; pair_turn < pair_last; pair_turn++) {
+        // turn i covers pairs 32 i ..: pair e of the eight diagonal blocks' 8 * 36, row-major inside a block's triangle
+        const int e = pair_turn * 32 + lane, blk = e / 36, f = e - blk * 36;
+        const int t = f < 1 ? 0 : f < 3 ? 1 : f < 6 ? 2 : f < 10 ? 3 : f < 15 ? 4 : f < 21 ? 5 : f < 28 ? 6 : 7, s = f - t * (t + 1) / 2;
+        const int rt = (blk * 8 + t) * LD, rs = (blk * 8 + s) * LD;
+        float acc = 0.0f;
+#pragma unroll 4
+        for (int d = 0; d < DP; d += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(qs + rt + d), y = *reinterpret_cast<const float4*>(ks + rs + d);
+            const float4 u = *reinterpret_cast<const float4*>(bs + rt + d), w = *reinterpret_cast<const float4*>(bs + rs + d);
+            acc = fmaf(x.x * y.x, exp2_fast(u.x - w.x), acc); acc = fmaf(x.y * y.y, exp2_fast(u.y - w.y), acc);
+            acc = fmaf(x.z * y.z, exp2_fast(u.z - w.z), acc); acc = fmaf(x.w * y.w, exp2_fast(u.w - w.w), acc);
         }
+        as[(blk * 8 + t) * LDA + blk * 8 + s] = acc;
+    }
+    const int wm = warp >> 2, wn = warp & 3, first = wn * NT;
+    float acc[2][NT][4] = {};
+    const bool carried = chunk > 0 || a.state;
+    const float* u = p.u + ((size_t)bh * p.nc + chunk) * D * V;
+    float cur[NT][2];
+    auto fetch = [&](int k, float (&x)[NT][2]) {
+#pragma unroll
+        for (int j = 0; j < NT; j++) {
+            const int v = (first + j) * 8 + g;
+#pragma unroll
+            for (int e = 0; e < 2; e++) { const int d = k + q4 + 4 * e; x[j][e] = v < V && d < D ? __ldcs(u + (size_t)d * V + v) : 0.0f; }
+        }
+    };
+    if (carried) fetch(0, cur);
+    __syncthreads();
+#pragma unroll
+    for (int i0 = 0; i0 < kChunk * DP / 4; i0 += kChunkThreads) {
+        const int i = i0 + tid, o = i / (DP / 4) * LD + i % (DP / 4) * 4;
+        float4 x = *reinterpret_cast<const float4*>(qs + o);
+        const float4 e = *reinterpret_cast<const float4*>(bs + o);
+        x.x *= exp2_fast(e.x); x.y *= exp2_fast(e.y); x.z *= exp2_fast(e.z); x.w *= exp2_fast(e.w);
+        *reinterpret_cast<float4*>(qs + o) = x;
     }
     __syncthreads();
-    for (int i = tid; i < kChunk * Dp; i += kChunkThreads) { const int t = i / Dp, d = i - t * Dp; qs[t * ld + d] *= exp2_fast(bs[t * ld + d]); }
-    __syncthreads();
-
-    const int wm = warp >> 2, wn = warp & 3, nt_all = Vp / 8, per = (nt_all + 3) / 4, first = wn * per, mine = max(0, min(per, nt_all - first));
-    float acc[2][NT][4] = {};
-    if (chunk > 0 || a.state) {
+    if (carried) {
         // (q 2^b) S: S straight from global memory into the fragments, the next eight channels in flight
-        const float* u = p.u + ((size_t)bh * p.nc + chunk) * D * V;
-        float cur[NT][2], nxt[NT][2];
-        auto fetch = [&](int k, float (&x)[NT][2]) {
-#pragma unroll
-            for (int j = 0; j < NT; j++) {
-                const int v = (first + j) * 8 + g;
-#pragma unroll
-                for (int e = 0; e < 2; e++) { const int d = k + q4 + 4 * e; x[j][e] = j < mine && v < V && d < D ? u[(size_t)d * V + v] : 0.0f; }
-            }
-        };
-        fetch(0, cur);
-        for (int k = 0; k < Dp; k += 8) {
-            if (k + 8 < Dp) fetch(k + 8, nxt);
+        const float* qp = qs + (wm * 32 + g) * LD + q4;
+#pragma unroll 2
+        for (int k = 0; k < DP; k += 8) {
+            float nxt[NT][2];
+            if (k + 8 < DP) fetch(k + 8, nxt);
             uint32_t ah[2][4], al[2][4];
 #pragma unroll
             for (int i = 0; i < 2; i++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) split_tf32(qs[(wm * 32 + i * 16 + g + (e & 1) * 8) * ld + k + q4 + (e >> 1) * 4], ah[i][e], al[i][e]);
+                for (int e = 0; e < 4; e++) split_tf32(qp[(i * 16 + (e & 1) * 8) * LD + k + (e >> 1) * 4], ah[i][e], al[i][e]);
 #pragma unroll
             for (int j = 0; j < NT; j++) {
-                if (j < mine) {
-                    uint32_t h0, l0, h1, l1;
-                    split_tf32(cur[j][0], h0, l0); split_tf32(cur[j][1], h1, l1);
+                uint32_t h0, l0, h1, l1;
+                split_tf32(cur[j][0], h0, l0); split_tf32(cur[j][1], h1, l1);
 #pragma unroll
-                    for (int i = 0; i < 2; i++) { mma_tf32(acc[i][j], al[i], h0, h1); mma_tf32(acc[i][j], ah[i], l0, l1); mma_tf32(acc[i][j], ah[i], h0, h1); }
-                }
+                for (int i = 0; i < 2; i++) { mma_tf32(acc[i][j], al[i], h0, h1); mma_tf32(acc[i][j], ah[i], l0, l1); mma_tf32(acc[i][j], ah[i], h0, h1); }
             }
+            if (k + 8 < DP) {
 #pragma unroll
-            for (int j = 0; j < NT; j++) { cur[j][0] = nxt[j][0]; cur[j][1] = nxt[j][1]; }
+                for (int j = 0; j < NT; j++) { cur[j][0] = nxt[j][0]; cur[j][1] = nxt[j][1]; }
+            }
         }
     }
     // A v up to the diagonal
-    for (int k = 0; k < wm * 32 + 32; k += 8) {
-        uint32_t ah[2][4], al[2][4];
+    {
+        const float *ap = as + (wm * 32 + g) * LDA + q4, *vp = vs + q4 * LDV + first * 8 + g;
+#pragma unroll 2
+        for (int k = 0; k < wm * 32 + 32; k += 8) {
+            uint32_t ah[2][4], al[2][4];
 #pragma unroll
-        for (int i = 0; i < 2; i++)
+            for (int i = 0; i < 2; i++)
 #pragma unroll
-            for (int e = 0; e < 4; e++) split_tf32(as[(wm * 32 + i * 16 + g + (e & 1) * 8) * lda + k + q4 + (e >> 1) * 4], ah[i][e], al[i][e]);
+                for (int e = 0; e < 4; e++) split_tf32(ap[(i * 16 + (e & 1) * 8) * LDA + k + (e >> 1) * 4], ah[i][e], al[i][e]);
+            const bool upper = k < wm * 32 + 16;          // the first 16 rows see no further columns
 #pragma unroll
-        for (int j = 0; j < NT; j++) {
-            if (j < mine) {
-                const int c = (first + j) * 8 + g;
-                const uint32_t b0 = __float_as_uint(vs[(k + q4) * ldv + c]), b1 = __float_as_uint(vs[(k + q4 + 4) * ldv + c]);
-#pragma unroll
-                for (int i = 0; i < 2; i++)
-                    if (k < wm * 32 + i * 16 + 16) { mma_tf32(acc[i][j], al[i], b0, b1); mma_tf32(acc[i][j], ah[i], b0, b1); }
+            for (int j = 0; j < NT; j++) {
+                const uint32_t b0 = __float_as_uint(vp[k * LDV + 8 * j]), b1 = __float_as_uint(vp[(k + 4) * LDV + 8 * j]);
+                if (upper) { mma_tf32(acc[0][j], al[0], b0, b1); mma_tf32(acc[0][j], ah[0], b0, b1); }
+                mma_tf32(acc[1][j], al[1], b0, b1); mma_tf32(acc[1][j], ah[1], b0, b1);
             }
         }
     }
@@ -437,6 +511,12 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + ((size_t)b * a.T + t0) * a.ld_out + h * V;
     const __nv_bfloat16* gate = in + a.c_g + h * V;
     const bool even = V % 2 == 0;
+    float hn[NT][2];
+#pragma unroll
+    for (int j = 0; j < NT; j++) {
+        const int v = (first + j) * 8 + 2 * q4;
+        hn[j][0] = v < V ? __ldg(a.head_norm + v) : 0.0f; hn[j][1] = v + 1 < V ? __ldg(a.head_norm + v + 1) : 0.0f;
+    }
 #pragma unroll
     for (int i = 0; i < 2; i++)
 #pragma unroll
@@ -444,18 +524,19 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
             const int t = wm * 32 + i * 16 + r * 8 + g;
             if (t >= n) continue;
             const float inv = 1.0f / sqrtf((red[t] + red[kChunk + t] + red[2 * kChunk + t] + red[3 * kChunk + t]) / (float)V + a.eps);
+            const __nv_bfloat16* gr = gate + (size_t)t * a.ld;
+            __nv_bfloat16* orow = out + (size_t)t * a.ld_out;
 #pragma unroll
             for (int j = 0; j < NT; j++) {
                 const int v = (first + j) * 8 + 2 * q4;
-                if (j >= mine || v >= V) continue;
-                const float x = acc[i][j][2 * r] * inv * a.head_norm[v];
+                if (v >= V) continue;
+                const float x = acc[i][j][2 * r] * inv * hn[j][0], y = acc[i][j][2 * r + 1] * inv * hn[j][1];
                 if (even) {
-                    const float y = acc[i][j][2 * r + 1] * inv * a.head_norm[v + 1];
-                    const float2 gg = bf16x2_to_float2(*reinterpret_cast<const __nv_bfloat162*>(gate + (size_t)t * a.ld + v));
-                    *reinterpret_cast<__nv_bfloat162*>(out + (size_t)t * a.ld_out + v) = __floats2bfloat162_rn(x * silu_fast(gg.x), y * silu_fast(gg.y));
+                    const float2 gg = bf16x2_to_float2(*reinterpret_cast<const __nv_bfloat162*>(gr + v));
+                    *reinterpret_cast<__nv_bfloat162*>(orow + v) = __floats2bfloat162_rn(x * silu_fast(gg.x), y * silu_fast(gg.y));
                 } else {
-                    out[(size_t)t * a.ld_out + v] = __float2bfloat16_rn(x * silu_fast((float)gate[(size_t)t * a.ld + v]));
-                    if (v + 1 < V) out[(size_t)t * a.ld_out + v + 1] = __float2bfloat16_rn(acc[i][j][2 * r + 1] * inv * a.head_norm[v + 1] * silu_fast((float)gate[(size_t)t * a.ld + v + 1]));
+                    orow[v] = __float2bfloat16_rn(x * silu_fast((float)gr[v]));
+                    if (v + 1 < V) orow[v + 1] = __float2bfloat16_rn(y * silu_fast((float)gr[v + 1]));
                 }
             }
         }
@@ -463,25 +544,32 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
         for (int i = tid; i < n * 8; i += kChunkThreads) { const int c = V + (i & 7); if (h * V + c < a.ld_out) out[(size_t)(i >> 3) * a.ld_out + c] = __float2bfloat16_rn(0.0f); }
 }
 
-size_t chunk_state_smem(const GlaArgs& a) {
-    const int Dp = round_up(a.D, 16), Vp = round_up(a.V, 8);
-    return ((size_t)kChunk * (2 * pitch8(Dp) + pitch8(Vp) + a.R) + (size_t)a.R * Dp + 4 * Dp) * sizeof(float);
-}
-size_t chunk_out_smem(const GlaArgs& a) {
-    const int Dp = round_up(a.D, 16), Vp = round_up(a.V, 8);
-    return ((size_t)kChunk * (3 * pitch4(Dp) + pitch8(Vp) + 68) + 4 * kChunk) * sizeof(float);
-}
 constexpr size_t kMaxSmem = 227 * 1024;
 
-template <int NT>
-int launch_chunk_out(const ChunkArgs& p) {
-    auto kern = gla_chunk_out_kernel<NT>;
-    const size_t smem = chunk_out_smem(p.a);
-    static size_t granted = 48 * 1024;
-    if (smem > granted) { SPT_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
-    kern<<<dim3(p.nc, p.a.B * p.a.H), kChunkThreads, smem, rt().stream>>>(p);
+template <int DP, int VP>
+int launch_chunked(const ChunkArgs& p) {
+    using L = ChunkSmem<DP, VP>;
+    static size_t granted = 0;
+    const size_t s1 = (L::kStateFloats + (size_t)p.a.R * (kChunk + DP)) * sizeof(float), s2 = L::kOutFloats * sizeof(float);
+    if (s1 > granted) {
+        SPT_CUDA(cudaFuncSetAttribute(gla_chunk_state_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1));
+        SPT_CUDA(cudaFuncSetAttribute(gla_chunk_out_kernel<DP, VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2));
+        granted = s1;
+    }
+    const dim3 grid(p.nc, p.a.B * p.a.H);
+    gla_chunk_state_kernel<DP, VP><<<grid, kChunkThreads, s1, rt().stream>>>(p);
+    SPT_LAUNCH_CHECK("gla_chunk_state");
+    const long long elems = (long long)p.a.B * p.a.H * p.a.D * p.a.V;
+    if (p.a.V % 4 == 0) gla_scan_kernel<4><<<(unsigned)((elems / 4 + 255) / 256), 256, 0, rt().stream>>>(p);
+    else gla_scan_kernel<1><<<(unsigned)((elems + 255) / 256), 256, 0, rt().stream>>>(p);
+    SPT_LAUNCH_CHECK("gla_scan");
+    gla_chunk_out_kernel<DP, VP><<<grid, kChunkThreads, s2, rt().stream>>>(p);
     SPT_LAUNCH_CHECK("gla_chunk_out");
     return 0;
+}
+template <int DP>
+int launch_chunked_v(const ChunkArgs& p) {
+    return p.a.V <= 64 ? launch_chunked<DP, 64>(p) : p.a.V <= 128 ? launch_chunked<DP, 128>(p) : launch_chunked<DP, 256>(p);
 }
 
 template <typename T, int DPW>
@@ -524,25 +612,14 @@ int gla_recurrent(const GlaArgs& a, float* o_scratch, bool dependent) {
     return gla_norm_gate(a, o_scratch, dependent);
 }
 
-bool gla_chunked_supported(const GlaArgs& a) {
-    return a.dtype == BF16 && a.D <= 128 && a.V <= 256 && a.B * a.H <= 65535 && chunk_state_smem(a) <= kMaxSmem && chunk_out_smem(a) <= kMaxSmem;
-}
+bool gla_chunked_supported(const GlaArgs& a) { return a.dtype == BF16 && a.D <= 128 && a.V <= 256 && a.R <= 64 && a.B * a.H <= 65535; }
 static size_t chunks_of(const GlaArgs& a) { return (size_t)a.B * a.H * ceil_div(a.T, kChunk); }
 size_t gla_chunked_state_bytes(const GlaArgs& a) { return chunks_of(a) * a.D * a.V * sizeof(float); }
 size_t gla_chunked_decay_bytes(const GlaArgs& a) { return chunks_of(a) * kChunk * a.D * sizeof(float); }
 
 int gla_chunked(const GlaArgs& a, float* u_scratch, float* dec_scratch) {
     const ChunkArgs p = {a, u_scratch, dec_scratch, ceil_div(a.T, kChunk)};
-    const size_t smem = chunk_state_smem(a);
-    static size_t granted = 48 * 1024;
-    if (smem > granted) { SPT_CUDA(cudaFuncSetAttribute(gla_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
-    gla_chunk_state_kernel<<<dim3(p.nc, a.B * a.H), kChunkThreads, smem, rt().stream>>>(p);
-    SPT_LAUNCH_CHECK("gla_chunk_state");
-    const long long elems = (long long)a.B * a.H * a.D * a.V;
-    gla_scan_kernel<<<(unsigned)((elems + 255) / 256), 256, 0, rt().stream>>>(p);
-    SPT_LAUNCH_CHECK("gla_scan");
-    const int nt = ceil_div(ceil_div(a.V, 8), 4);
-    return nt <= 2 ? launch_chunk_out<2>(p) : nt <= 4 ? launch_chunk_out<4>(p) : launch_chunk_out<8>(p);
+    return a.D <= 32 ? launch_chunked_v<32>(p) : a.D <= 64 ? launch_chunked_v<64>(p) : launch_chunked_v<128>(p);
 }
 
 }  // namespace spt
