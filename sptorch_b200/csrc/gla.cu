@@ -8,6 +8,7 @@
 #include "epilogue_math.cuh"
 #include "pdl.cuh"
 #include <math.h>
+#include <cooperative_groups.h>
 
 namespace spt {
 
@@ -21,8 +22,11 @@ __device__ __forceinline__ float log_decay(float z, float inv_tau) { return (fmi
 
 // A CTA owns 32 columns of one (sequence, head)'s state: lane = column, warp w the DPW rows w * DPW ...  Each warp sums its rows'
 // share of o; the eight shares are added in warp order once per block of staged tokens.
-template <typename T, int DPW>
+// FUSED (at most kRecTokens tokens): the CTAs of a (sequence, head) are one cluster; they exchange their columns' sums of squares through
+// distributed shared memory and write the normed, gated heads themselves instead of o.
+template <typename T, int DPW, bool FUSED>
 __global__ void __launch_bounds__(kRecWarps * 32) gla_recurrent_kernel(const GlaArgs a, float* __restrict__ o) {
+    __shared__ float sq_sh[kRecTokens];
     extern __shared__ float sm[];
     const int D = a.D, V = a.V, R = a.R;
     float* qs = sm;                                   // [tokens][D]
@@ -83,7 +87,13 @@ __global__ void __launch_bounds__(kRecWarps * 32) gla_recurrent_kernel(const Gla
 #pragma unroll
             for (int w = 0; w < kRecWarps; w++) sum += part[w * kRecTokens * 32 + i];
             const int t = i >> 5, c = v0 + (i & 31);
-            if (c < V) o[((size_t)b * a.T + t0 + t) * a.H * V + h * V + c] = sum;
+            if constexpr (FUSED) {                         // a warp holds the 32 columns of one token
+                vs[i] = sum;                               // v of this element has been used up (the barrier above)
+                float sq = sum * sum;                      // columns past V are zero
+#pragma unroll
+                for (int w = 16; w > 0; w >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, w);
+                if (lane == 0) sq_sh[t] = sq;
+            } else if (c < V) o[((size_t)b * a.T + t0 + t) * a.H * V + h * V + c] = sum;
         }
         // the next block's staging writes as / vs / qs only after every warp is past its token loop (the barrier above)
     }
@@ -93,6 +103,24 @@ __global__ void __launch_bounds__(kRecWarps * 32) gla_recurrent_kernel(const Gla
             const int d = warp * DPW + i;
             if (d < D && col < V) st[(size_t)d * V + col] = s[i];
         }
+    }
+    if constexpr (FUSED) {
+        namespace cg = cooperative_groups;
+        cg::cluster_group cluster = cg::this_cluster();
+        const int parts = gridDim.x;
+        if (parts > 1) cluster.sync(); else __syncthreads();
+        T* out = static_cast<T*>(a.out) + (size_t)b * a.T * a.ld_out;
+        for (int i = tid; i < a.T * 32; i += blockDim.x) {
+            const int t = i >> 5, c = v0 + (i & 31);
+            float sq = 0.0f;
+            for (int r = 0; r < parts; r++) sq += parts > 1 ? cluster.map_shared_rank(sq_sh, r)[t] : sq_sh[t];
+            const float inv = 1.0f / sqrtf(sq / (float)V + a.eps);
+            if (c < V) out[(size_t)t * a.ld_out + h * V + c] = (T)(vs[i] * inv * a.head_norm[c] * silu_exact((float)in[(size_t)t * a.ld + a.c_g + h * V + c]));
+            else if (h == a.H - 1 && h * V + c < a.ld_out) out[(size_t)t * a.ld_out + h * V + c] = (T)0.0f;
+        }
+        if (h == a.H - 1 && v0 + 32 >= V)              // padding of the output row that lies past this CTA's columns
+            for (int i = tid; i < a.T * 8; i += blockDim.x) { const int c = h * V + v0 + 32 + (i & 7); if (c < a.ld_out) out[(size_t)(i >> 3) * a.ld_out + c] = (T)0.0f; }
+        if (parts > 1) cluster.sync();                  // no CTA leaves while its sums may still be read
     }
 }
 
@@ -150,33 +178,42 @@ __device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], 
 
 struct ChunkArgs { GlaArgs a; float *u, *dec; int nc; };
 
-// rows of bf16 -> f32 tile [kChunk][PITCH], zero outside n rows and w columns (up to WP columns); eight columns at a time where aligned
+// rows of bf16 -> f32 tile [kChunk][PITCH], zero outside n rows and w columns (up to WP columns).  Eight columns at a time where aligned:
+// request() starts the loads (all tiles of a kernel before the first is stored), store() widens them into shared memory.
 template <int PITCH, int WP>
-__device__ __forceinline__ void load_tile(float* dst, const __nv_bfloat16* src, long long ld, int n, int w, float f, bool vec) {
-    if (vec) {
-        constexpr int PER = WP / 8;
+struct TileLoad {
+    static constexpr int PER = WP / 8, TURNS = (kChunk * PER + kChunkThreads - 1) / kChunkThreads;
+    uint4 raw[TURNS];
+    __device__ __forceinline__ void request(const __nv_bfloat16* src, long long ld, int n, int w, bool vec) {
 #pragma unroll
-        for (int i0 = 0; i0 < kChunk * PER; i0 += kChunkThreads) {
-            const int i = i0 + (int)threadIdx.x;
-            if (kChunk * PER % kChunkThreads == 0 || i < kChunk * PER) {
-                const int t = i / PER, c = (i % PER) * 8;
-                uint4 raw = make_uint4(0, 0, 0, 0);
-                if (t < n && c < w) raw = *reinterpret_cast<const uint4*>(src + (size_t)t * ld + c);
-                const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-                for (int j = 0; j < 4; j += 2) {
-                    const float2 x = bf16x2_to_float2(h[j]), y = bf16x2_to_float2(h[j + 1]);
-                    *reinterpret_cast<float4*>(dst + t * PITCH + c + 2 * j) = make_float4(x.x * f, x.y * f, y.x * f, y.y * f);
-                }
-            }
-        }
-    } else {
-        for (int i = threadIdx.x; i < kChunk * WP; i += kChunkThreads) {
-            const int t = i / WP, c = i % WP;
-            dst[t * PITCH + c] = t < n && c < w ? (float)src[(size_t)t * ld + c] * f : 0.0f;
+        for (int i0 = 0; i0 < TURNS; i0++) {
+            const int i = i0 * kChunkThreads + (int)threadIdx.x, t = i / PER, c = (i % PER) * 8;
+            raw[i0] = make_uint4(0, 0, 0, 0);
+            if (vec && t < n && c < w) raw[i0] = __ldg(reinterpret_cast<const uint4*>(src + (size_t)t * ld + c));
         }
     }
-}
+    __device__ __forceinline__ void store(float* dst, const __nv_bfloat16* src, long long ld, int n, int w, float f, bool vec) const {
+        if (vec) {
+#pragma unroll
+            for (int i0 = 0; i0 < TURNS; i0++) {
+                const int i = i0 * kChunkThreads + (int)threadIdx.x, t = i / PER, c = (i % PER) * 8;
+                if (kChunk * PER % kChunkThreads == 0 || i < kChunk * PER) {
+                    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw[i0]);
+#pragma unroll
+                    for (int j = 0; j < 4; j += 2) {
+                        const float2 x = bf16x2_to_float2(h[j]), y = bf16x2_to_float2(h[j + 1]);
+                        *reinterpret_cast<float4*>(dst + t * PITCH + c + 2 * j) = make_float4(x.x * f, x.y * f, y.x * f, y.y * f);
+                    }
+                }
+            }
+        } else {
+            for (int i = threadIdx.x; i < kChunk * WP; i += kChunkThreads) {
+                const int t = i / WP, c = i % WP;
+                dst[t * PITCH + c] = t < n && c < w ? (float)src[(size_t)t * ld + c] * f : 0.0f;
+            }
+        }
+    }
+};
 
 // log2 of the decay: 1 + e with e = exp(-|z|) loses e's low bits, so a small e takes the series of log(1 + e) (next term e^5 / 5)
 __device__ __forceinline__ float log2_decay(float z, float inv_tau) {
@@ -213,10 +250,14 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_state_kernel(const Ch
     const int t0 = chunk * kChunk, n = min(kChunk, a.T - t0);
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + ((size_t)b * a.T + t0) * a.ld;
     const bool vec = D % 8 == 0 && V % 8 == 0;
+    TileLoad<LDK, DP> tk;
+    TileLoad<LDV, VP> tv;
+    tk.request(in + a.c_k + h * D, a.ld, n, D, vec);
+    tv.request(in + a.c_v + h * V, a.ld, n, V, vec);
     for (int i = tid; i < kChunk * R; i += kChunkThreads) { const int t = i % kChunk, r = i / kChunk; a1s[i] = t < n ? (float)in[(size_t)t * a.ld + a.c_a + r] : 0.0f; }
     for (int i = tid; i < DP * R; i += kChunkThreads) { const int d = i % DP, r = i / DP; a2s[i] = d < D ? __ldg(a.a2 + (size_t)(h * D + d) * R + r) : 0.0f; }
-    load_tile<LDK, DP>(ks, in + a.c_k + h * D, a.ld, n, D, 1.0f, vec);
-    load_tile<LDV, VP>(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
+    tk.store(ks, in + a.c_k + h * D, a.ld, n, D, 1.0f, vec);
+    tv.store(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
     __syncthreads();
     // log2 alpha of four tokens per turn of a thread; padding tokens and channels decay by nothing
     const float inv_tau = 1.0f / a.tau;
@@ -386,17 +427,29 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + ((size_t)b * a.T + t0) * a.ld;
     const bool vec = D % 8 == 0 && V % 8 == 0;
     const float* dec = p.dec + ((size_t)bh * p.nc + chunk) * kChunk * D;
-    if (D % 4 == 0) {
+    {
+        constexpr int TURNS = kChunk * DP / 4 / kChunkThreads;
+        TileLoad<LD, DP> tq, tk;
+        TileLoad<LDV, VP> tv;
+        float4 bd[TURNS];
 #pragma unroll
-        for (int i0 = 0; i0 < kChunk * DP / 4; i0 += kChunkThreads) {
-            const int i = i0 + tid, t = i / (DP / 4), d = i % (DP / 4) * 4;
-            *reinterpret_cast<float4*>(bs + t * LD + d) = d < D ? *reinterpret_cast<const float4*>(dec + (size_t)t * D + d) : make_float4(0, 0, 0, 0);
+        for (int i0 = 0; i0 < TURNS; i0++) {
+            const int i = i0 * kChunkThreads + tid, t = i / (DP / 4), d = i % (DP / 4) * 4;
+            bd[i0] = D % 4 == 0 && d < D ? __ldg(reinterpret_cast<const float4*>(dec + (size_t)t * D + d)) : make_float4(0, 0, 0, 0);
         }
-    } else
-        for (int i = tid; i < kChunk * DP; i += kChunkThreads) { const int t = i / DP, d = i % DP; bs[t * LD + d] = d < D ? dec[(size_t)t * D + d] : 0.0f; }
-    load_tile<LD, DP>(qs, in + a.c_q + h * D, a.ld, n, D, 1.0f / sqrtf((float)D), vec);
-    load_tile<LD, DP>(ks, in + a.c_k + h * D, a.ld, n, D, 1.0f, vec);
-    load_tile<LDV, VP>(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
+        tq.request(in + a.c_q + h * D, a.ld, n, D, vec);
+        tk.request(in + a.c_k + h * D, a.ld, n, D, vec);
+        tv.request(in + a.c_v + h * V, a.ld, n, V, vec);
+#pragma unroll
+        for (int i0 = 0; i0 < TURNS; i0++) {
+            const int i = i0 * kChunkThreads + tid;
+            if (D % 4 == 0) *reinterpret_cast<float4*>(bs + i / (DP / 4) * LD + i % (DP / 4) * 4) = bd[i0];
+        }
+        if (D % 4) for (int i = tid; i < kChunk * DP; i += kChunkThreads) { const int t = i / DP, d = i % DP; bs[t * LD + d] = d < D ? dec[(size_t)t * D + d] : 0.0f; }
+        tq.store(qs, in + a.c_q + h * D, a.ld, n, D, 1.0f / sqrtf((float)D), vec);
+        tk.store(ks, in + a.c_k + h * D, a.ld, n, D, 1.0f, vec);
+        tv.store(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
+    }
     for (int i = tid; i < kChunk * LDA / 4; i += kChunkThreads) reinterpret_cast<float4*>(as)[i] = make_float4(0, 0, 0, 0);
     __syncthreads();
 
@@ -431,16 +484,16 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     float acc[2][NT][4] = {};
     const bool carried = chunk > 0 || a.state;
     const float* u = p.u + ((size_t)bh * p.nc + chunk) * D * V;
-    float cur[NT][2];
+    float cur[NT][2], nxt[NT][2];
     auto fetch = [&](int k, float (&x)[NT][2]) {
 #pragma unroll
         for (int j = 0; j < NT; j++) {
             const int v = (first + j) * 8 + g;
 #pragma unroll
-            for (int e = 0; e < 2; e++) { const int d = k + q4 + 4 * e; x[j][e] = v < V && d < D ? __ldcs(u + (size_t)d * V + v) : 0.0f; }
+            for (int e = 0; e < 2; e++) { const int d = k + q4 + 4 * e; x[j][e] = v < V && d < D ? __ldg(u + (size_t)d * V + v) : 0.0f; }
         }
     };
-    if (carried) fetch(0, cur);
+    if (carried) { fetch(0, cur); fetch(8, nxt); }
     __syncthreads();
 #pragma unroll
     for (int i0 = 0; i0 < kChunk * DP / 4; i0 += kChunkThreads) {
@@ -456,8 +509,8 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
         const float* qp = qs + (wm * 32 + g) * LD + q4;
 #pragma unroll 2
         for (int k = 0; k < DP; k += 8) {
-            float nxt[NT][2];
-            if (k + 8 < DP) fetch(k + 8, nxt);
+            float far[NT][2];                              // S two steps ahead
+            if (k + 16 < DP) fetch(k + 16, far);
             uint32_t ah[2][4], al[2][4];
 #pragma unroll
             for (int i = 0; i < 2; i++)
@@ -472,7 +525,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
             }
             if (k + 8 < DP) {
 #pragma unroll
-                for (int j = 0; j < NT; j++) { cur[j][0] = nxt[j][0]; cur[j][1] = nxt[j][1]; }
+                for (int j = 0; j < NT; j++) { cur[j][0] = nxt[j][0]; cur[j][1] = nxt[j][1]; nxt[j][0] = far[j][0]; nxt[j][1] = far[j][1]; }
             }
         }
     }
@@ -532,7 +585,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
                 if (v >= V) continue;
                 const float x = acc[i][j][2 * r] * inv * hn[j][0], y = acc[i][j][2 * r + 1] * inv * hn[j][1];
                 if (even) {
-                    const float2 gg = bf16x2_to_float2(*reinterpret_cast<const __nv_bfloat162*>(gr + v));
+                    const float2 gg = bf16x2_to_float2(__ldg(reinterpret_cast<const __nv_bfloat162*>(gr + v)));
                     *reinterpret_cast<__nv_bfloat162*>(orow + v) = __floats2bfloat162_rn(x * silu_fast(gg.x), y * silu_fast(gg.y));
                 } else {
                     orow[v] = __float2bfloat16_rn(x * silu_fast((float)gr[v]));
@@ -572,14 +625,24 @@ int launch_chunked_v(const ChunkArgs& p) {
     return p.a.V <= 64 ? launch_chunked<DP, 64>(p) : p.a.V <= 128 ? launch_chunked<DP, 128>(p) : launch_chunked<DP, 256>(p);
 }
 
+// few tokens and at most eight CTAs (a portable cluster) per head: norm and gate in the same launch
+// ... while the launch is short: with many CTAs the clusters hold their SMs longer than the second launch costs (64 sequences x 16 heads of
+// 64 x 128: 57 us fused, 37 us in two launches; 8 sequences: 13 and 14)
+bool recurrent_fuses(const GlaArgs& a) { return a.T <= kRecTokens && a.V <= 256 && (long long)a.B * a.H * ceil_div(a.V, 32) <= 8ll * rt().sm_count; }
+
 template <typename T, int DPW>
 int launch_recurrent(const GlaArgs& a, float* o, bool dependent) {
     const size_t smem = (size_t)kRecTokens * (3 * a.D + 32 + kRecWarps * 32 + a.R) * sizeof(float);
     if (smem > 200 * 1024) return fail("gla: key size %d with a decay rank of %d does not fit shared memory", a.D, a.R);
-    auto kern = gla_recurrent_kernel<T, DPW>;
+    const bool fused = recurrent_fuses(a);
+    auto kern = fused ? gla_recurrent_kernel<T, DPW, true> : gla_recurrent_kernel<T, DPW, false>;
     static size_t granted = 48 * 1024;
-    if (smem > granted) { SPT_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
-    SPT_CUDA(launch_dependent(kern, dim3(ceil_div(a.V, 32), a.B * a.H), dim3(kRecWarps * 32), smem, dependent, 1, a, o));
+    if (smem > granted) {
+        SPT_CUDA(cudaFuncSetAttribute(gla_recurrent_kernel<T, DPW, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        SPT_CUDA(cudaFuncSetAttribute(gla_recurrent_kernel<T, DPW, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        granted = smem;
+    }
+    SPT_CUDA(launch_dependent(kern, dim3(ceil_div(a.V, 32), a.B * a.H), dim3(kRecWarps * 32), smem, dependent, fused ? ceil_div(a.V, 32) : 1, a, o));
     note_submit();
     return 0;
 }
@@ -609,7 +672,7 @@ int gla_norm_gate(const GlaArgs& a, const float* o, bool dependent) {
 int gla_recurrent(const GlaArgs& a, float* o_scratch, bool dependent) {
     if (a.B * a.H > 65535) return fail("gla: batch x heads exceeds one launch");
     if (a.dtype == BF16 ? recurrent_t<__nv_bfloat16>(a, o_scratch, dependent) : recurrent_t<float>(a, o_scratch, dependent)) return 1;
-    return gla_norm_gate(a, o_scratch, dependent);
+    return recurrent_fuses(a) ? 0 : gla_norm_gate(a, o_scratch, dependent);
 }
 
 bool gla_chunked_supported(const GlaArgs& a) { return a.dtype == BF16 && a.D <= 128 && a.V <= 256 && a.R <= 64 && a.B * a.H <= 65535; }

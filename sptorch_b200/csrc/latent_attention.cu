@@ -178,13 +178,13 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LatentArgs a) {
 
 // ---------------- few tokens, bf16: attention over the cached rows on the tensor cores ----------------
 // A cluster of `splits` CTAs owns one token and sixteen heads; each CTA walks its part of the positions in tiles of 64 cached rows
-// (cp.async, two tiles in flight).  Per tile: scores [16 heads x 64 keys] = Q rows^T, eight warps taking eight keys each; an online
-// softmax by 16 threads per head; O [16 x kv] += P rows, the warps taking kv / 8 columns each, with P as the sum of two bf16 numbers (16
+// (cp.async, two tiles in flight).  Per tile: scores [16 heads x 64 keys] = Q rows^T, sixteen warps taking eight keys and half of
+// the columns each; an online softmax by one warp per head; O [16 x kv] += P rows, the warps taking kv / 16 columns each, with P as the sum of two bf16 numbers (16
 // mantissa bits).  The cluster's parts meet through distributed shared memory, every CTA merging a slice of the columns.  A row is read
 // from HBM once for all heads: 2 (kv + rot) bytes per position and sixteen heads.  mma.sync m16n8k16: sixteen heads are a sixteenth of a
 // tcgen05 tile's rows, and the kernel streams the cache at a few FLOP per byte.
-// NTW: 8-column tiles of the latent per warp (kv8 <= 64 NTW).
-constexpr int kLdThreads = 256, kLdKeys = 64, kLdP = 72, kLdS = 68;
+// NTW: 8-column tiles of the latent per warp (kv8 <= 128 NTW).
+constexpr int kLdThreads = 512, kLdKeys = 64, kLdP = 72, kLdS = 68;
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
@@ -202,7 +202,7 @@ __device__ __forceinline__ float ex2(float x) { float y; asm("ex2.approx.ftz.f32
 
 __host__ __device__ constexpr int ld_pitch(int row) { return (row + 31) / 32 * 32 + 8; }      // an odd number of 16-byte units: ldmatrix without conflicts
 inline size_t latent_decode_smem(int row) {
-    return (size_t)(2 * kLdKeys + 16) * ld_pitch(row) * 2 + 2 * 16 * kLdP * 2 + (size_t)16 * kLdS * 4 + 3 * 16 * 4;
+    return (size_t)(2 * kLdKeys + 16) * ld_pitch(row) * 2 + 2 * 16 * kLdP * 2 + (size_t)2 * 16 * kLdS * 4 + 3 * 16 * 4;
 }
 
 template <int NTW>
@@ -212,8 +212,8 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     __nv_bfloat16* tile = reinterpret_cast<__nv_bfloat16*>(raw);                // [2][64][pitch]
     __nv_bfloat16* qs = tile + 2 * kLdKeys * pitch;                             // [16][pitch]
     __nv_bfloat16* ph = qs + 16 * pitch;                                        // [2][16][kLdP]: softmax weights, upper and lower half
-    float* ss = reinterpret_cast<float*>(ph + 2 * 16 * kLdP);                   // [16][kLdS]
-    float* corr_s = ss + 16 * kLdS;                                             // [16]
+    float* ss = reinterpret_cast<float*>(ph + 2 * 16 * kLdP);                   // [2][16][kLdS]: scores over either half of the columns
+    float* corr_s = ss + 2 * 16 * kLdS;                                             // [16]
     float* m_s = corr_s + 16;                                                   // [16]
     float* l_s = m_s + 16;                                                      // [16]
     float* o_s = reinterpret_cast<float*>(raw);                                 // [16][kv8 + 4], over the tiles once they are done
@@ -272,7 +272,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
 #pragma unroll
         for (int e = 0; e < 4; e++) acc[j][e] = 0.0f;
     const float scale = a.scale * 1.4426950408889634f;
-    const int srow = tid >> 4, sk = (tid & 15) * 4;                             // softmax: 16 threads per head, four keys each
+    const int srow = warp, sk = lane * 2;                                       // softmax: one warp per head, two keys per lane
     float m = -INFINITY, l = 0.0f;
     int stage = 0;
     for (int k0 = lo; k0 < hi; k0 += kLdKeys, stage ^= 1) {
@@ -284,42 +284,38 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
         const __nv_bfloat16* tl = tile + stage * kLdKeys * pitch;
         {
             float s0[4] = {0, 0, 0, 0}, s1[4] = {0, 0, 0, 0};
-            const uint32_t qa = smem_addr(qs + (lane & 15) * pitch + (lane >> 4) * 8), ka = smem_addr(tl + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 8);
+            const int nt = warp & 7, half = warp >> 3, kmid = (wide / 32 + 1) / 2 * 32;
+            const uint32_t qa = smem_addr(qs + (lane & 15) * pitch + (lane >> 4) * 8), ka = smem_addr(tl + (nt * 8 + (lane & 7)) * pitch + (lane >> 3) * 8);
 #pragma unroll 4
-            for (int k = 0; k < wide; k += 32) {
+            for (int k = half ? kmid : 0; k < (half ? wide : kmid); k += 32) {
                 uint32_t x[4], y[4], kb[4];
                 ldsm4(x, qa + k * 2); ldsm4(y, qa + k * 2 + 32); ldsm4(kb, ka + k * 2);
                 mma_bf16(s0, x, kb[0], kb[1]);
                 mma_bf16(s1, y, kb[2], kb[3]);
             }
-            const int c = warp * 8 + 2 * q4;
-            ss[g * kLdS + c] = (s0[0] + s1[0]) * scale; ss[g * kLdS + c + 1] = (s0[1] + s1[1]) * scale;
-            ss[(g + 8) * kLdS + c] = (s0[2] + s1[2]) * scale; ss[(g + 8) * kLdS + c + 1] = (s0[3] + s1[3]) * scale;
+            float* so = ss + (half * 16 + g) * kLdS + nt * 8 + 2 * q4;
+            *reinterpret_cast<float2*>(so) = make_float2((s0[0] + s1[0]) * scale, (s0[1] + s1[1]) * scale);
+            *reinterpret_cast<float2*>(so + 8 * kLdS) = make_float2((s0[2] + s1[2]) * scale, (s0[3] + s1[3]) * scale);
         }
         __syncthreads();
         {
-            const float4 s4 = *reinterpret_cast<const float4*>(ss + srow * kLdS + sk);
-            float s[4] = {s4.x, s4.y, s4.z, s4.w}, mx = m, sum = 0.0f;
+            const float2 sa = *reinterpret_cast<const float2*>(ss + srow * kLdS + sk), sb = *reinterpret_cast<const float2*>(ss + (16 + srow) * kLdS + sk);
+            const float x = k0 + sk < hi ? sa.x + sb.x : -INFINITY, y = k0 + sk + 1 < hi ? sa.y + sb.y : -INFINITY;
+            float mx = fmaxf(m, fmaxf(x, y));
 #pragma unroll
-            for (int j = 0; j < 4; j++) { if (k0 + sk + j >= hi) s[j] = -INFINITY; mx = fmaxf(mx, s[j]); }
-#pragma unroll
-            for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
             const float corr = ex2(m - mx);                                     // first tile: 2^(-inf) = 0
-            __nv_bfloat162 hi2[2], lo2[2];
+            const float e0 = ex2(x - mx), e1 = ex2(y - mx);
+            const __nv_bfloat162 hi2 = __floats2bfloat162_rn(e0, e1);
+            const float2 f = bf16x2_to_float2(hi2);
+            const __nv_bfloat162 lo2 = __floats2bfloat162_rn(e0 - f.x, e1 - f.y);
+            float sum = e0 + e1;
 #pragma unroll
-            for (int j = 0; j < 2; j++) {
-                const float e0 = ex2(s[2 * j] - mx), e1 = ex2(s[2 * j + 1] - mx);
-                sum += e0 + e1;
-                hi2[j] = __floats2bfloat162_rn(e0, e1);
-                const float2 f = bf16x2_to_float2(hi2[j]);
-                lo2[j] = __floats2bfloat162_rn(e0 - f.x, e1 - f.y);
-            }
-#pragma unroll
-            for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
             l = l * corr + sum; m = mx;
-            *reinterpret_cast<uint2*>(ph + srow * kLdP + sk) = *reinterpret_cast<const uint2*>(hi2);
-            *reinterpret_cast<uint2*>(ph + (16 + srow) * kLdP + sk) = *reinterpret_cast<const uint2*>(lo2);
-            if ((tid & 15) == 0) corr_s[srow] = corr;
+            *reinterpret_cast<__nv_bfloat162*>(ph + srow * kLdP + sk) = hi2;
+            *reinterpret_cast<__nv_bfloat162*>(ph + (16 + srow) * kLdP + sk) = lo2;
+            if (lane == 0) corr_s[srow] = corr;
         }
         __syncthreads();
         {
@@ -354,7 +350,7 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
             *reinterpret_cast<float2*>(o_s + (g + 8) * lo_ + c) = make_float2(acc[j][2], acc[j][3]);
         }
     }
-    if ((tid & 15) == 0) { m_s[srow] = m; l_s[srow] = l; }
+    if (lane == 0) { m_s[srow] = m; l_s[srow] = l; }
     namespace cg = cooperative_groups;
     cg::cluster_group cluster = cg::this_cluster();
     if (splits > 1) cluster.sync(); else __syncthreads();
@@ -387,8 +383,26 @@ int launch_latent_decode(const LatentArgs& a, bool dependent) {
     static size_t granted = 48 * 1024;
     if (smem > granted) { SPT_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); granted = smem; }
     const int groups = ceil_div(a.H, 16), items = a.B * a.T * groups;
+    // the widest split whose clusters are all resident at once and leave every CTA a tile: a CTA fills its SM, and how many clusters of 2,
+    // 4, 8 such CTAs fit depends on how the SMs are grouped
+    static int fits[4] = {0, -1, -1, -1};
+    static size_t fits_smem = 0;
+    if (fits_smem != smem) {
+        fits_smem = smem;
+        for (int k = 1; k < 4; k++) {
+            cudaLaunchConfig_t cfg = {};
+            cfg.gridDim = dim3(8 * 148); cfg.blockDim = dim3(kLdThreads); cfg.dynamicSmemBytes = smem;
+            cudaLaunchAttribute at[1];
+            at[0].id = cudaLaunchAttributeClusterDimension; at[0].val.clusterDim.x = 1u << k; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+            cfg.attrs = at; cfg.numAttrs = 1;
+            int c = 0;
+            if (cudaOccupancyMaxActiveClusters(&c, kern, &cfg) != cudaSuccess) { cudaGetLastError(); c = 0; }
+            fits[k] = c;
+        }
+    }
     int splits = 1;
-    while (splits < 8 && 2 * splits * items <= rt().sm_count && a.capacity > splits * kLdKeys) splits *= 2;
+    for (int k = 1; k < 4; k++)
+        if (items <= fits[k] && a.capacity > (1 << (k - 1)) * kLdKeys) splits = 1 << k;
     SPT_CUDA(launch_dependent(kern, dim3(items * splits), dim3(kLdThreads), smem, dependent, splits, a, splits, groups));
     note_submit();
     return 0;
@@ -454,7 +468,7 @@ bool latent_decode_supported(const LatentArgs& a) {
 
 int latent_decode(const LatentArgs& a, bool dependent) {
     const int tiles = a.kv8 / 8;
-    return tiles <= 16 ? launch_latent_decode<2>(a, dependent) : tiles <= 32 ? launch_latent_decode<4>(a, dependent) : launch_latent_decode<8>(a, dependent);
+    return tiles <= 32 ? launch_latent_decode<2>(a, dependent) : launch_latent_decode<4>(a, dependent);
 }
 
 }  // namespace spt
