@@ -416,10 +416,15 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     const GlaArgs& a = p.a;
     const int D = a.D, V = a.V;
     float* bs = sm;                               // [kChunk][LD]: running sums of the log2 decays
-    float* qs = bs + kChunk * LD;                 // [kChunk][LD]: q D^(-1/2), later times 2^b
-    float* ks = qs + kChunk * LD;
-    float* vs = ks + kChunk * LD;                 // [kChunk][LDV]
-    float* as = vs + kChunk * LDV;                // [kChunk][LDA]: A
+    float* ks = bs + kChunk * LD;                 // [kChunk][LD]
+    float* qs = ks + kChunk * LD;                 // [kChunk][LD]: q D^(-1/2), later times 2^b
+    // SS: the state's tile fits the values' place.  S is then copied there while A is computed, and v -- kept in registers meanwhile --
+    // goes where b and k lay.  Otherwise S comes straight from global memory into the fragments.  Either way the place next to A holds
+    // the normed output at the end.
+    constexpr bool SS = DP <= kChunk && LDV <= 2 * LD;
+    float* xs = qs + kChunk * LD;                 // [kChunk][LDV]: S or v, then the output
+    float* vs = SS ? sm : xs;
+    float* as = xs + kChunk * LDV;                // [kChunk][LDA]: A
     float* red = as + kChunk * LDA;               // [4][kChunk]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, q4 = lane & 3;
     const int chunk = blockIdx.x, bh = blockIdx.y, b = bh / a.H, h = bh - b * a.H;
@@ -427,10 +432,12 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + ((size_t)b * a.T + t0) * a.ld;
     const bool vec = D % 8 == 0 && V % 8 == 0;
     const float* dec = p.dec + ((size_t)bh * p.nc + chunk) * kChunk * D;
+    const bool carried = chunk > 0 || a.state;
+    const float* u = p.u + ((size_t)bh * p.nc + chunk) * D * V;
+    TileLoad<LDV, VP> tv;
     {
         constexpr int TURNS = kChunk * DP / 4 / kChunkThreads;
         TileLoad<LD, DP> tq, tk;
-        TileLoad<LDV, VP> tv;
         float4 bd[TURNS];
 #pragma unroll
         for (int i0 = 0; i0 < TURNS; i0++) {
@@ -448,7 +455,19 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
         if (D % 4) for (int i = tid; i < kChunk * DP; i += kChunkThreads) { const int t = i / DP, d = i % DP; bs[t * LD + d] = d < D ? dec[(size_t)t * D + d] : 0.0f; }
         tq.store(qs, in + a.c_q + h * D, a.ld, n, D, 1.0f / sqrtf((float)D), vec);
         tk.store(ks, in + a.c_k + h * D, a.ld, n, D, 1.0f, vec);
-        tv.store(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
+        if (!SS) tv.store(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);
+        if (SS && carried) {
+            if (V % 4 == 0) {
+                for (int i = tid; i < DP * (VP / 4); i += kChunkThreads) {
+                    const int d = i / (VP / 4), v = i % (VP / 4) * 4;
+                    float* dst = xs + d * LDV + v;
+                    if (d < D && v < V) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(u + (size_t)d * V + v) : "memory");
+                    else *reinterpret_cast<float4*>(dst) = make_float4(0, 0, 0, 0);
+                }
+                asm volatile("cp.async.commit_group;" ::: "memory");
+            } else
+                for (int i = tid; i < DP * VP; i += kChunkThreads) { const int d = i / VP, v = i % VP; xs[d * LDV + v] = d < D && v < V ? u[(size_t)d * V + v] : 0.0f; }
+        }
     }
     for (int i = tid; i < kChunk * LDA / 4; i += kChunkThreads) reinterpret_cast<float4*>(as)[i] = make_float4(0, 0, 0, 0);
     __syncthreads();
@@ -482,8 +501,6 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     }
     const int wm = warp >> 2, wn = warp & 3, first = wn * NT;
     float acc[2][NT][4] = {};
-    const bool carried = chunk > 0 || a.state;
-    const float* u = p.u + ((size_t)bh * p.nc + chunk) * D * V;
     float cur[NT][2], nxt[NT][2];
     auto fetch = [&](int k, float (&x)[NT][2]) {
 #pragma unroll
@@ -493,7 +510,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
             for (int e = 0; e < 2; e++) { const int d = k + q4 + 4 * e; x[j][e] = v < V && d < D ? __ldg(u + (size_t)d * V + v) : 0.0f; }
         }
     };
-    if (carried) { fetch(0, cur); fetch(8, nxt); }
+    if (!SS && carried) { fetch(0, cur); fetch(8, nxt); }
     __syncthreads();
 #pragma unroll
     for (int i0 = 0; i0 < kChunk * DP / 4; i0 += kChunkThreads) {
@@ -503,14 +520,21 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
         x.x *= exp2_fast(e.x); x.y *= exp2_fast(e.y); x.z *= exp2_fast(e.z); x.w *= exp2_fast(e.w);
         *reinterpret_cast<float4*>(qs + o) = x;
     }
+    if (SS) asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
+    if (SS) tv.store(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);          // over b and k, which are done; read behind the next barrier
     if (carried) {
-        // (q 2^b) S: S straight from global memory into the fragments, the next eight channels in flight
+        // (q 2^b) S
         const float* qp = qs + (wm * 32 + g) * LD + q4;
 #pragma unroll 2
         for (int k = 0; k < DP; k += 8) {
             float far[NT][2];                              // S two steps ahead
-            if (k + 16 < DP) fetch(k + 16, far);
+            if (!SS && k + 16 < DP) fetch(k + 16, far);
+            if (SS) {
+                const float* sp = xs + (k + q4) * LDV + first * 8 + g;
+#pragma unroll
+                for (int j = 0; j < NT; j++) { cur[j][0] = sp[8 * j]; cur[j][1] = sp[4 * LDV + 8 * j]; }
+            }
             uint32_t ah[2][4], al[2][4];
 #pragma unroll
             for (int i = 0; i < 2; i++)
@@ -523,12 +547,13 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
 #pragma unroll
                 for (int i = 0; i < 2; i++) { mma_tf32(acc[i][j], al[i], h0, h1); mma_tf32(acc[i][j], ah[i], l0, l1); mma_tf32(acc[i][j], ah[i], h0, h1); }
             }
-            if (k + 8 < DP) {
+            if (!SS && k + 8 < DP) {
 #pragma unroll
                 for (int j = 0; j < NT; j++) { cur[j][0] = nxt[j][0]; cur[j][1] = nxt[j][1]; nxt[j][0] = far[j][0]; nxt[j][1] = far[j][1]; }
             }
         }
     }
+    if (SS) __syncthreads();
     // A v up to the diagonal
     {
         const float *ap = as + (wm * 32 + g) * LDA + q4, *vp = vs + q4 * LDV + first * 8 + g;
@@ -561,43 +586,46 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
             if (q4 == 0) red[wn * kChunk + wm * 32 + i * 16 + r * 8 + g] = sq;
         }
     __syncthreads();
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + ((size_t)b * a.T + t0) * a.ld_out + h * V;
-    const __nv_bfloat16* gate = in + a.c_g + h * V;
-    const bool even = V % 2 == 0;
-    float hn[NT][2];
-#pragma unroll
-    for (int j = 0; j < NT; j++) {
-        const int v = (first + j) * 8 + 2 * q4;
-        hn[j][0] = v < V ? __ldg(a.head_norm + v) : 0.0f; hn[j][1] = v + 1 < V ? __ldg(a.head_norm + v + 1) : 0.0f;
-    }
+    // normed rows through shared memory, so that gate and output are read and written sixteen bytes at a time
 #pragma unroll
     for (int i = 0; i < 2; i++)
 #pragma unroll
         for (int r = 0; r < 2; r++) {
             const int t = wm * 32 + i * 16 + r * 8 + g;
-            if (t >= n) continue;
             const float inv = 1.0f / sqrtf((red[t] + red[kChunk + t] + red[2 * kChunk + t] + red[3 * kChunk + t]) / (float)V + a.eps);
-            const __nv_bfloat16* gr = gate + (size_t)t * a.ld;
-            __nv_bfloat16* orow = out + (size_t)t * a.ld_out;
 #pragma unroll
-            for (int j = 0; j < NT; j++) {
-                const int v = (first + j) * 8 + 2 * q4;
-                if (v >= V) continue;
-                const float x = acc[i][j][2 * r] * inv * hn[j][0], y = acc[i][j][2 * r + 1] * inv * hn[j][1];
-                if (even) {
-                    const float2 gg = bf16x2_to_float2(__ldg(reinterpret_cast<const __nv_bfloat162*>(gr + v)));
-                    *reinterpret_cast<__nv_bfloat162*>(orow + v) = __floats2bfloat162_rn(x * silu_fast(gg.x), y * silu_fast(gg.y));
-                } else {
-                    orow[v] = __float2bfloat16_rn(x * silu_fast((float)gr[v]));
-                    if (v + 1 < V) orow[v + 1] = __float2bfloat16_rn(y * silu_fast((float)gr[v + 1]));
-                }
+            for (int j = 0; j < NT; j++)
+                *reinterpret_cast<float2*>(xs + t * LDV + (first + j) * 8 + 2 * q4) = make_float2(acc[i][j][2 * r] * inv, acc[i][j][2 * r + 1] * inv);
+        }
+    __syncthreads();
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + ((size_t)b * a.T + t0) * a.ld_out + h * V;
+    const __nv_bfloat16* gate = in + a.c_g + h * V;
+    if (vec) {
+        constexpr int PER = VP / 8;
+#pragma unroll 2
+        for (int i = tid; i < kChunk * PER; i += kChunkThreads) {
+            const int t = i / PER, c = i % PER * 8;
+            if (t >= n || c >= V) continue;
+            const uint4 gr = __ldg(reinterpret_cast<const uint4*>(gate + (size_t)t * a.ld + c));
+            const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&gr);
+            const float* xr = xs + t * LDV + c;
+            uint4 o4;
+            __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o4);
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const float2 gg = bf16x2_to_float2(gh[j]), x = *reinterpret_cast<const float2*>(xr + 2 * j), w = __ldg(reinterpret_cast<const float2*>(a.head_norm + c + 2 * j));
+                oh[j] = __floats2bfloat162_rn(x.x * w.x * silu_fast(gg.x), x.y * w.y * silu_fast(gg.y));
             }
+            *reinterpret_cast<uint4*>(out + (size_t)t * a.ld_out + c) = o4;
+        }
+    } else
+        for (int i = tid; i < n * V; i += kChunkThreads) {
+            const int t = i / V, c = i - t * V;
+            out[(size_t)t * a.ld_out + c] = __float2bfloat16_rn(xs[t * LDV + c] * a.head_norm[c] * silu_fast((float)gate[(size_t)t * a.ld + c]));
         }
     if (h == a.H - 1)                             // the padding of the output rows
         for (int i = tid; i < n * 8; i += kChunkThreads) { const int c = V + (i & 7); if (h * V + c < a.ld_out) out[(size_t)(i >> 3) * a.ld_out + c] = __float2bfloat16_rn(0.0f); }
 }
-
-constexpr size_t kMaxSmem = 227 * 1024;
 
 template <int DP, int VP>
 int launch_chunked(const ChunkArgs& p) {
