@@ -161,7 +161,7 @@ __global__ void __launch_bounds__(256) gla_norm_gate_kernel(const GlaArgs a, con
 // in bf16 and needs no split.  The tiles are 64 rows and the operands are scaled element by element on their way into the fragments,
 // so there is no operand for tcgen05 to fetch from shared memory as it lies there; the kernels are bound by that work and by HBM.
 constexpr int kChunk = 64;
-constexpr int kChunkThreads = 256;
+constexpr int kChunkThreads = 512;    // sixteen warps: the phases are chains of dependent work, two such CTAs an SM keep it busy
 
 __device__ __forceinline__ float exp2_fast(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
@@ -287,7 +287,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_state_kernel(const Ch
     __syncthreads();
     {
         float* dec = p.dec + ((size_t)bh * p.nc + chunk) * kChunk * D;
-        constexpr int STEP = kChunkThreads / DP;                       // tokens per turn; a thread keeps its channel
+        constexpr int STEP = kChunkThreads / DP;                       // tokens per turn (4, 8 or 16); a thread keeps its channel
         const int d = tid % DP;
         float off[5];
         off[0] = 0.0f;
@@ -302,13 +302,13 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_state_kernel(const Ch
         }
     }
     __syncthreads();
-    // U[d][v] = sum_t ks[t][d] vs[t][v]: blocks of 16 channels x 64 values dealt over the warps
+    // U[d][v] = sum_t ks[t][d] vs[t][v]: blocks of 16 channels x 32 values dealt over the warps
     float* u = p.u + ((size_t)bh * p.nc + chunk) * D * V;
-    constexpr int MB = DP / 16, NB = VP / 64;
+    constexpr int MB = DP / 16, NB = VP / 32;
     for (int blk = warp; blk < MB * NB; blk += kChunkThreads / 32) {
-        const int m0 = blk % MB * 16, n0 = blk / MB * 64;
+        const int m0 = blk % MB * 16, n0 = blk / MB * 32;
         if (m0 >= D || n0 >= V) continue;
-        float acc[8][4] = {};
+        float acc[4][4] = {};
         const float *kp = ks + q4 * LDK + m0 + g, *vp = vs + q4 * LDV + n0 + g;
 #pragma unroll 2
         for (int k = 0; k < kChunk; k += 8, kp += 8 * LDK, vp += 8 * LDV) {
@@ -318,7 +318,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_state_kernel(const Ch
             split_tf32(kp[4 * LDK], hi[2], lo[2]);
             split_tf32(kp[4 * LDK + 8], hi[3], lo[3]);
 #pragma unroll
-            for (int j = 0; j < 8; j++) {
+            for (int j = 0; j < 4; j++) {
                 const uint32_t b0 = __float_as_uint(vp[8 * j]), b1 = __float_as_uint(vp[4 * LDV + 8 * j]);
                 mma_tf32(acc[j], lo, b0, b1);
                 mma_tf32(acc[j], hi, b0, b1);
@@ -326,7 +326,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_state_kernel(const Ch
         }
         const bool even = V % 2 == 0;
 #pragma unroll
-        for (int j = 0; j < 8; j++)
+        for (int j = 0; j < 4; j++)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int d = m0 + g + e * 8, v = n0 + 8 * j + 2 * q4;
@@ -407,9 +407,9 @@ __device__ __forceinline__ void a_block(const float* qs, const float* ks, const 
     }
 }
 
-// Warps are 2 (halves of the rows) x 4 (quarters of the values), NT 8-column tiles each.
+// Warps are 4 (16 rows each) x 4 (quarters of the values), NT 8-column tiles each.
 template <int DP, int VP>
-__global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const ChunkArgs p) {
+__global__ void __launch_bounds__(kChunkThreads, ChunkSmem<DP, VP>::kOutFloats * 4 <= 113 * 1024 ? 2 : 1) gla_chunk_out_kernel(const ChunkArgs p) {
     extern __shared__ __align__(16) float sm[];
     using L = ChunkSmem<DP, VP>;
     constexpr int LD = L::LDQ, LDV = L::LDV, LDA = L::LDA, NT = VP / 32;
@@ -441,7 +441,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
         float4 bd[TURNS];
 #pragma unroll
         for (int i0 = 0; i0 < TURNS; i0++) {
-            const int i = i0 * kChunkThreads + tid, t = i / (DP / 4), d = i % (DP / 4) * 4;
+            const int i = i0 * kChunkThreads + tid, t = i / (DP / 4), d = i % (DP / 4) * 4;      // DP >= 32: the turns are full
             bd[i0] = D % 4 == 0 && d < D ? __ldg(reinterpret_cast<const float4*>(dec + (size_t)t * D + d)) : make_float4(0, 0, 0, 0);
         }
         tq.request(in + a.c_q + h * D, a.ld, n, D, vec);
@@ -474,15 +474,11 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
 
     // A: four tasks of the 32-row block and two of the 16-row blocks (16 rows x 16 columns each), four 8 x 8 blocks, and the 288 pairs of
     // the diagonal blocks in nine turns of a warp
-    int pair_turn, pair_last;                     // this warp's turns
-    if (warp < 4) {
-        a_block<DP, 2, false>(qs, ks, bs, as, 32 + 16 * (warp >> 1), 16 * (warp & 1), 31, g, q4);
-        a_block<DP, 1, true>(qs, ks, bs, as, 16 * warp + 8, 16 * warp, 16 * warp + 7, g, q4);
-        pair_turn = 0; pair_last = warp == 0 ? 1 : 0;
-    } else {
-        if (warp < 6) a_block<DP, 2, false>(qs, ks, bs, as, warp == 4 ? 16 : 48, warp == 4 ? 0 : 32, warp == 4 ? 15 : 47, g, q4);
-        pair_turn = warp == 4 ? 1 : warp == 5 ? 2 : warp == 6 ? 3 : 6; pair_last = warp == 4 ? 2 : warp == 5 ? 3 : warp == 6 ? 6 : 9;
-    }
+    int pair_turn = 0, pair_last = 0;             // this warp's turns
+    if (warp < 4) a_block<DP, 2, false>(qs, ks, bs, as, 32 + 16 * (warp >> 1), 16 * (warp & 1), 31, g, q4);
+    else if (warp < 6) a_block<DP, 2, false>(qs, ks, bs, as, warp == 4 ? 16 : 48, warp == 4 ? 0 : 32, warp == 4 ? 15 : 47, g, q4);
+    else if (warp < 10) a_block<DP, 1, true>(qs, ks, bs, as, 16 * (warp - 6) + 8, 16 * (warp - 6), 16 * (warp - 6) + 7, g, q4);
+    else { const int w = warp - 10; pair_turn = w < 3 ? 2 * w : w + 3; pair_last = w < 3 ? pair_turn + 2 : pair_turn + 1; }
 #pragma unroll 1
     for (; pair_turn < pair_last; pair_turn++) {
         // turn i covers pairs 32 i ..: pair e of the eight diagonal blocks' 8 * 36, row-major inside a block's triangle
@@ -500,7 +496,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
         as[(blk * 8 + t) * LDA + blk * 8 + s] = acc;
     }
     const int wm = warp >> 2, wn = warp & 3, first = wn * NT;
-    float acc[2][NT][4] = {};
+    float acc[NT][4] = {};
     float cur[NT][2], nxt[NT][2];
     auto fetch = [&](int k, float (&x)[NT][2]) {
 #pragma unroll
@@ -525,7 +521,7 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     if (SS) tv.store(vs, in + a.c_v + h * V, a.ld, n, V, 1.0f, vec);          // over b and k, which are done; read behind the next barrier
     if (carried) {
         // (q 2^b) S
-        const float* qp = qs + (wm * 32 + g) * LD + q4;
+        const float* qp = qs + (wm * 16 + g) * LD + q4;
 #pragma unroll 2
         for (int k = 0; k < DP; k += 8) {
             float far[NT][2];                              // S two steps ahead
@@ -535,17 +531,14 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
 #pragma unroll
                 for (int j = 0; j < NT; j++) { cur[j][0] = sp[8 * j]; cur[j][1] = sp[4 * LDV + 8 * j]; }
             }
-            uint32_t ah[2][4], al[2][4];
+            uint32_t ah[4], al[4];
 #pragma unroll
-            for (int i = 0; i < 2; i++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) split_tf32(qp[(i * 16 + (e & 1) * 8) * LD + k + (e >> 1) * 4], ah[i][e], al[i][e]);
+            for (int e = 0; e < 4; e++) split_tf32(qp[(e & 1) * 8 * LD + k + (e >> 1) * 4], ah[e], al[e]);
 #pragma unroll
             for (int j = 0; j < NT; j++) {
                 uint32_t h0, l0, h1, l1;
                 split_tf32(cur[j][0], h0, l0); split_tf32(cur[j][1], h1, l1);
-#pragma unroll
-                for (int i = 0; i < 2; i++) { mma_tf32(acc[i][j], al[i], h0, h1); mma_tf32(acc[i][j], ah[i], l0, l1); mma_tf32(acc[i][j], ah[i], h0, h1); }
+                mma_tf32(acc[j], al, h0, h1); mma_tf32(acc[j], ah, l0, l1); mma_tf32(acc[j], ah, h0, h1);
             }
             if (!SS && k + 8 < DP) {
 #pragma unroll
@@ -556,47 +549,39 @@ __global__ void __launch_bounds__(kChunkThreads) gla_chunk_out_kernel(const Chun
     if (SS) __syncthreads();
     // A v up to the diagonal
     {
-        const float *ap = as + (wm * 32 + g) * LDA + q4, *vp = vs + q4 * LDV + first * 8 + g;
+        const float *ap = as + (wm * 16 + g) * LDA + q4, *vp = vs + q4 * LDV + first * 8 + g;
 #pragma unroll 2
-        for (int k = 0; k < wm * 32 + 32; k += 8) {
-            uint32_t ah[2][4], al[2][4];
+        for (int k = 0; k < wm * 16 + 16; k += 8) {
+            uint32_t ah[4], al[4];
 #pragma unroll
-            for (int i = 0; i < 2; i++)
-#pragma unroll
-                for (int e = 0; e < 4; e++) split_tf32(ap[(i * 16 + (e & 1) * 8) * LDA + k + (e >> 1) * 4], ah[i][e], al[i][e]);
-            const bool upper = k < wm * 32 + 16;          // the first 16 rows see no further columns
+            for (int e = 0; e < 4; e++) split_tf32(ap[(e & 1) * 8 * LDA + k + (e >> 1) * 4], ah[e], al[e]);
 #pragma unroll
             for (int j = 0; j < NT; j++) {
                 const uint32_t b0 = __float_as_uint(vp[k * LDV + 8 * j]), b1 = __float_as_uint(vp[(k + 4) * LDV + 8 * j]);
-                if (upper) { mma_tf32(acc[0][j], al[0], b0, b1); mma_tf32(acc[0][j], ah[0], b0, b1); }
-                mma_tf32(acc[1][j], al[1], b0, b1); mma_tf32(acc[1][j], ah[1], b0, b1);
+                mma_tf32(acc[j], al, b0, b1); mma_tf32(acc[j], ah, b0, b1);
             }
         }
     }
     // head norm over V and gate; a row's values lie with four warps
 #pragma unroll
-    for (int i = 0; i < 2; i++)
+    for (int r = 0; r < 2; r++) {
+        float sq = 0.0f;
 #pragma unroll
-        for (int r = 0; r < 2; r++) {
-            float sq = 0.0f;
-#pragma unroll
-            for (int j = 0; j < NT; j++) { sq = fmaf(acc[i][j][2 * r], acc[i][j][2 * r], sq); sq = fmaf(acc[i][j][2 * r + 1], acc[i][j][2 * r + 1], sq); }
-            sq += __shfl_xor_sync(0xffffffffu, sq, 1);
-            sq += __shfl_xor_sync(0xffffffffu, sq, 2);
-            if (q4 == 0) red[wn * kChunk + wm * 32 + i * 16 + r * 8 + g] = sq;
-        }
+        for (int j = 0; j < NT; j++) { sq = fmaf(acc[j][2 * r], acc[j][2 * r], sq); sq = fmaf(acc[j][2 * r + 1], acc[j][2 * r + 1], sq); }
+        sq += __shfl_xor_sync(0xffffffffu, sq, 1);
+        sq += __shfl_xor_sync(0xffffffffu, sq, 2);
+        if (q4 == 0) red[wn * kChunk + wm * 16 + r * 8 + g] = sq;
+    }
     __syncthreads();
     // normed rows through shared memory, so that gate and output are read and written sixteen bytes at a time
 #pragma unroll
-    for (int i = 0; i < 2; i++)
+    for (int r = 0; r < 2; r++) {
+        const int t = wm * 16 + r * 8 + g;
+        const float inv = 1.0f / sqrtf((red[t] + red[kChunk + t] + red[2 * kChunk + t] + red[3 * kChunk + t]) / (float)V + a.eps);
 #pragma unroll
-        for (int r = 0; r < 2; r++) {
-            const int t = wm * 32 + i * 16 + r * 8 + g;
-            const float inv = 1.0f / sqrtf((red[t] + red[kChunk + t] + red[2 * kChunk + t] + red[3 * kChunk + t]) / (float)V + a.eps);
-#pragma unroll
-            for (int j = 0; j < NT; j++)
-                *reinterpret_cast<float2*>(xs + t * LDV + (first + j) * 8 + 2 * q4) = make_float2(acc[i][j][2 * r] * inv, acc[i][j][2 * r + 1] * inv);
-        }
+        for (int j = 0; j < NT; j++)
+            *reinterpret_cast<float2*>(xs + t * LDV + (first + j) * 8 + 2 * q4) = make_float2(acc[j][2 * r] * inv, acc[j][2 * r + 1] * inv);
+    }
     __syncthreads();
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + ((size_t)b * a.T + t0) * a.ld_out + h * V;
     const __nv_bfloat16* gate = in + a.c_g + h * V;
