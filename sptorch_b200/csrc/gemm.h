@@ -81,7 +81,16 @@ bool gemm_supported(const GemmDesc& d, const char** why);
 // nrm: the rows of A are normalised on the fly (kind 1: LayerNorm with gamma / beta, kind 2: RMSNorm with gamma), which saves the
 // stand-alone normalisation launch in front of a projection.  dependent: launched as a programmatic dependent of the previous
 // kernel in the stream (see launch_dependent in common.h).
-struct RowNorm { int kind = 0; const float* gamma = nullptr; const float* beta = nullptr; float eps = 0.0f; };
+// kind 3: the rows are a residual stream that still lacks the sublayer output before it, a = x + y / sqrt(mean(y^2) + eps) * gamma (x
+// f32, y bf16, rows of K elements, the mean over `dim` of them); a goes to x_out (f32, not x) and xb (bf16) too, for those who come after.
+struct RowNorm {
+    int kind = 0;
+    const float* gamma = nullptr; const float* beta = nullptr;
+    float eps = 0.0f;
+    int dim = 0;
+    const float* x = nullptr; const __nv_bfloat16* y = nullptr;
+    float* x_out = nullptr; __nv_bfloat16* xb = nullptr;
+};
 bool linear_few_rows_supported(const GemmDesc& d);
 bool linear_few_rows_norm_supported(const GemmDesc& d, const RowNorm& nrm);
 int linear_few_rows(const GemmDesc& d, const RowNorm* nrm = nullptr, bool dependent = false);

@@ -61,6 +61,101 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentArgs a) {
     }
 }
 
+// eight bf16 at a time
+struct Eight { float v[8]; };
+__device__ __forceinline__ Eight load_eight(const __nv_bfloat16* p) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+    Eight e;
+#pragma unroll
+    for (int i = 0; i < 4; i++) { const float2 f = bf16x2_to_float2(h[i]); e.v[2 * i] = f.x; e.v[2 * i + 1] = f.y; }
+    return e;
+}
+__device__ __forceinline__ void store_eight(__nv_bfloat16* p, const Eight& e) {
+    uint4 raw;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; i++) h[i] = __floats2bfloat162_rn(e.v[2 * i], e.v[2 * i + 1]);
+    *reinterpret_cast<uint4*>(p) = raw;
+}
+__device__ __forceinline__ void rotate_eight(Eight& e, const float2* cs) {      // four pairs by four angles (16-byte aligned)
+#pragma unroll
+    for (int i = 0; i < 4; i += 2) {
+        const float4 c = __ldg(reinterpret_cast<const float4*>(cs + i));
+        const float u0 = e.v[2 * i] * c.x - e.v[2 * i + 1] * c.y, v0 = e.v[2 * i + 1] * c.x + e.v[2 * i] * c.y;
+        const float u1 = e.v[2 * i + 2] * c.z - e.v[2 * i + 3] * c.w, v1 = e.v[2 * i + 3] * c.z + e.v[2 * i + 2] * c.w;
+        e.v[2 * i] = u0; e.v[2 * i + 1] = v0; e.v[2 * i + 2] = u1; e.v[2 * i + 3] = v1;
+    }
+}
+
+// The same as latent_prep_kernel for bf16 sizes that are multiples of eight: one warp per token, the row in registers.  NQ / NK: groups
+// of eight per lane of the query latent and of the latent.
+template <int NQ, int NK>
+__global__ void __launch_bounds__(128) latent_prep_vec_kernel(const LatentArgs a) {
+    pdl_release();
+    const int m = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, b = m / a.T;
+    pdl_acquire();
+    if (m >= a.B * a.T) return;
+    const int pos = (a.pos_dev ? a.pos_dev[0] : a.first) + (m - b * a.T);
+    const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + (size_t)m * a.ld_in;
+    const int nq = a.q_rank / 8, nk = a.kv / 8, nr = a.rot / 8;
+    Eight q[NQ], c[NK], r = {};
+    float sq = 0.0f, sc = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NQ; i++) if (i * 32 + lane < nq) q[i] = load_eight(in + a.c_dq + (i * 32 + lane) * 8);
+#pragma unroll
+    for (int i = 0; i < NK; i++) if (i * 32 + lane < nk) c[i] = load_eight(in + a.c_dkv + (i * 32 + lane) * 8);
+    if (lane < nr) r = load_eight(in + a.c_dkv + a.kv + lane * 8);
+#pragma unroll
+    for (int i = 0; i < NQ; i++) if (i * 32 + lane < nq) {
+#pragma unroll
+        for (int j = 0; j < 8; j++) sq = fmaf(q[i].v[j], q[i].v[j], sq);
+    }
+#pragma unroll
+    for (int i = 0; i < NK; i++) if (i * 32 + lane < nk) {
+#pragma unroll
+        for (int j = 0; j < 8; j++) sc = fmaf(c[i].v[j], c[i].v[j], sc);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) { sq += __shfl_xor_sync(0xffffffffu, sq, o); sc += __shfl_xor_sync(0xffffffffu, sc, o); }
+    const float iq = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps), ic = 1.0f / sqrtf(sc / (float)a.kv + a.eps);
+    __nv_bfloat16* cq = static_cast<__nv_bfloat16*>(a.cq) + (size_t)m * a.ld_cq;
+    __nv_bfloat16* row = static_cast<__nv_bfloat16*>(a.rows) + (size_t)b * a.seq_stride + (size_t)pos * a.row;
+    auto scaled = [](Eight e, float inv, const float* w) {
+        const float4 w0 = __ldg(reinterpret_cast<const float4*>(w)), w1 = __ldg(reinterpret_cast<const float4*>(w + 4));
+        const float ww[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+        for (int j = 0; j < 8; j++) e.v[j] = e.v[j] * inv * ww[j];
+        return e;
+    };
+#pragma unroll
+    for (int i = 0; i < NQ; i++) if (i * 32 + lane < nq) store_eight(cq + (i * 32 + lane) * 8, scaled(q[i], iq, a.dq_norm + (i * 32 + lane) * 8));
+#pragma unroll
+    for (int i = 0; i < NK; i++) if (i * 32 + lane < nk) store_eight(row + (i * 32 + lane) * 8, scaled(c[i], ic, a.dkv_norm + (i * 32 + lane) * 8));
+    if (lane < nr) {
+        if (lane * 8 < a.rope_dims) rotate_eight(r, a.angles + (size_t)pos * (a.rope_dims / 2) + lane * 4);
+        store_eight(row + a.kv8 + lane * 8, r);
+    }
+}
+
+bool vec_sizes(const LatentArgs& a) {
+    return a.dtype == BF16 && a.q_rank % 8 == 0 && a.kv % 8 == 0 && a.rot % 8 == 0 && a.rope_dims % 8 == 0 && a.D % 8 == 0 && a.rot <= 256;
+}
+
+// rotation of every head's rot part in place, four pairs per thread
+__global__ void __launch_bounds__(256) latent_rope_q_vec_kernel(const LatentArgs a) {
+    const int per = a.rope_dims / 8;
+    const long long idx = (long long)blockIdx.x * 256 + threadIdx.x;
+    if (idx >= (long long)a.B * a.T * a.H * per) return;
+    const int e = (int)(idx % per);
+    const long long mh = idx / per, m = mh / a.H;
+    const int h = (int)(mh - m * a.H), pos = (a.pos_dev ? a.pos_dev[0] : a.first) + (int)(m % a.T);
+    __nv_bfloat16* p = static_cast<__nv_bfloat16*>(a.q) + m * a.ld_q + (long long)h * (a.D + a.rot) + a.D + 8 * e;
+    Eight v = load_eight(p);
+    rotate_eight(v, a.angles + (size_t)pos * (a.rope_dims / 2) + 4 * e);
+    store_eight(p, v);
+}
+
 // rotation of neighbouring pairs of every head's rot part, in place
 template <typename T>
 __global__ void __launch_bounds__(256) latent_rope_q_kernel(const LatentArgs a) {
@@ -442,6 +537,15 @@ int absorbed_t(const LatentArgs& a, bool dependent) {
 
 int latent_prep(const LatentArgs& a, bool dependent) {
     const dim3 grid(a.B * a.T), block(128);
+    const int nq = ceil_div(a.q_rank, 256), nk = ceil_div(a.kv, 256);
+    if (vec_sizes(a) && nq <= 8 && nk <= 4) {
+        const dim3 rows(ceil_div(a.B * a.T, 4));
+        if (nq <= 2 && nk <= 1) SPT_CUDA(launch_dependent(latent_prep_vec_kernel<2, 1>, rows, block, 0, dependent, 1, a));
+        else if (nq <= 4 && nk <= 2) SPT_CUDA(launch_dependent(latent_prep_vec_kernel<4, 2>, rows, block, 0, dependent, 1, a));
+        else SPT_CUDA(launch_dependent(latent_prep_vec_kernel<8, 4>, rows, block, 0, dependent, 1, a));
+        note_submit();
+        return 0;
+    }
     if (a.dtype == BF16) SPT_CUDA(launch_dependent(latent_prep_kernel<__nv_bfloat16>, grid, block, 0, dependent, 1, a));
     else SPT_CUDA(launch_dependent(latent_prep_kernel<float>, grid, block, 0, dependent, 1, a));
     note_submit();
@@ -451,6 +555,11 @@ int latent_prep(const LatentArgs& a, bool dependent) {
 int latent_rope_q(const LatentArgs& a) {
     const long long work = (long long)a.B * a.T * a.H * (a.rope_dims / 2);
     if (work == 0) return 0;
+    if (vec_sizes(a)) {
+        latent_rope_q_vec_kernel<<<(unsigned)((work / 4 + 255) / 256), 256, 0, rt().stream>>>(a);
+        SPT_LAUNCH_CHECK("latent_rope_q");
+        return 0;
+    }
     const unsigned grid = (unsigned)((work + 255) / 256);
     if (a.dtype == BF16) latent_rope_q_kernel<__nv_bfloat16><<<grid, 256, 0, rt().stream>>>(a);
     else latent_rope_q_kernel<float><<<grid, 256, 0, rt().stream>>>(a);

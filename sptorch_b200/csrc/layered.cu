@@ -8,7 +8,8 @@
 //                     keys and values of every position from the latents (one GEMM) | fused attention | W_o | post-norm
 //   feed-forward: W_up (+bias) | W_gate (+bias, SwiGLU product) | W_down (+bias) | post-norm
 // A few tokens (a decode step, a short portion of a prompt) take the weight-streaming projections, the token-by-token recurrence and
-// attention over the cached latents themselves; all of these are programmatic dependents of one another.
+// attention over the cached latents themselves; all of these are programmatic dependents of one another, and with one or two rows the
+// projection behind a sublayer does the post-norm on the way.
 // f32 models run every product as f32 multiply-adds (MM_F32), the recurrence token by token and the latent attention unexpanded.
 #include "layered.h"
 #include "pdl.cuh"
@@ -178,12 +179,20 @@ int ensure(Gpt* g, LayeredScratch* s, size_t bytes) {
 }
 
 // out[M, N] = act(a W^T + bias) (* r for the SwiGLU product); rows of a are lda apart and read for K elements, W is [N, ldw]
+// pend (few rows only, may be null): a is the residual stream completed on the fly; *fused tells whether that was possible, otherwise
+// nothing was launched
 int product(Gpt* g, bool few, const void* a, long long lda, const void* w, long long ldw, int K, const float* bias, const void* r, void* out, long long ldo,
-            int M, int N, int epi) {
+            int M, int N, int epi, const RowNorm* pend = nullptr, bool* fused = nullptr) {
     GemmDesc d;
     d.A = a; d.B = w; d.C = out; d.bias = bias; d.R = r;
     d.M = M; d.N = N; d.K = K; d.lda = lda; d.ldb = ldw; d.ldc = ldo;
     d.epilogue = epi; d.mode = g->c.dtype == BF16 ? MM_BF16 : MM_F32; d.out_dtype = g->c.dtype;
+    if (pend) {
+        *fused = few && linear_few_rows_norm_supported(d, *pend);
+        if (!*fused) return 0;
+        ProfScope ps(PROF_LINEAR);
+        return linear_few_rows(d, pend, true);
+    }
     if (few && linear_few_rows_supported(d)) { ProfScope ps(PROF_LINEAR); return linear_few_rows(d, nullptr, true); }
     return gemm_or_simt(d);
 }
@@ -290,25 +299,44 @@ int run(Gpt* g, const void* ids, int B, int T, int first, const int* pos_dev, bo
         return 0;
     };
     if (tap(0)) return 1;
+    // y holds a sublayer's output that has not joined the stream yet: its norm weight.  With few rows the next projection completes the
+    // stream while it reads it (x and x2 taken in turn: every CTA reads the old one); otherwise the post-norm kernel does.
+    const float* pending = nullptr;
+    float* x_other = (float*)lay.x2.p;
+    auto settle = [&](const float* fin) -> int {
+        if (!pending && !fin) return 0;
+        if (post_norm_launch(x, pending ? lay.y.p : nullptr, pending, fin, x, lay.xb.p, M, c.d_model, d8, c.eps, dt, few)) return 1;
+        pending = nullptr;
+        return 0;
+    };
+    auto project = [&](const void* w, const float* bias, void* out, int N) -> int {              // a projection of the completed stream
+        if (pending && few && !g->taps_on) {
+            RowNorm n;
+            n.kind = 3; n.gamma = pending; n.eps = c.eps; n.dim = c.d_model; n.x = x; n.y = (const __nv_bfloat16*)lay.y.p; n.x_out = x_other; n.xb = (__nv_bfloat16*)lay.xb.p;
+            bool fused = false;
+            if (product(g, few, lay.xb.p, d8, w, d8, d8, bias, nullptr, out, N, M, N, EPI_NONE, &n, &fused)) return 1;
+            if (fused) { std::swap(x, x_other); pending = nullptr; return 0; }
+        }
+        return settle(nullptr) || product(g, few, lay.xb.p, d8, w, d8, d8, bias, nullptr, out, N, M, N, EPI_NONE);
+    };
     const int nl = (int)lay.L.size();
-    if (nl == 0 && post_norm_launch(x, nullptr, nullptr, lay.final_norm, nullptr, lay.xb.p, M, c.d_model, d8, c.eps, dt, few)) return 1;
     for (int l = 0; l < nl; l++) {
         const LayeredLayer& w = lay.L[l];
-        const float* fin = l == nl - 1 ? lay.final_norm : nullptr;              // the last update of x also makes the head's input
-        if (product(g, few, lay.xb.p, d8, w.w_in, d8, d8, nullptr, nullptr, lay.in.p, w.n_in, M, w.n_in, EPI_NONE)) return 1;
+        if (project(w.w_in, nullptr, lay.in.p, w.n_in)) return 1;
         if (w.c.mixer == SPT_MIXER_GLA ? gla_layer(g, w, B, T, few, cached) : latent_layer(g, w, B, T, first, pos_dev, few, cached)) return 1;
         if (product(g, few, lay.ao.p, w.o_ld(), w.w_o, w.o_ld(), w.o_ld(), nullptr, nullptr, lay.y.p, d8, M, d8, EPI_NONE)) return 1;
-        const bool mlp = w.c.mlp == SPT_MLP_DENSE;
-        if (post_norm_launch(x, lay.y.p, w.norm1, mlp ? nullptr : fin, x, lay.xb.p, M, c.d_model, d8, c.eps, dt, few)) return 1;
-        if (mlp) {
+        pending = w.norm1;
+        if (w.c.mlp == SPT_MLP_DENSE) {
             const int f8 = pad8(w.c.d_ff);
-            if (product(g, few, lay.xb.p, d8, w.w_up, d8, d8, w.b_up, nullptr, lay.f.p, f8, M, f8, EPI_NONE)) return 1;
+            if (project(w.w_up, w.b_up, lay.f.p, f8)) return 1;
             if (product(g, few, lay.xb.p, d8, w.w_gate, d8, d8, w.b_gate, lay.f.p, lay.f.p, f8, M, f8, EPI_SWIGLU)) return 1;
             if (product(g, few, lay.f.p, f8, w.w_down, f8, f8, w.b_down, nullptr, lay.y.p, d8, M, d8, EPI_NONE)) return 1;
-            if (post_norm_launch(x, lay.y.p, w.norm2, fin, x, lay.xb.p, M, c.d_model, d8, c.eps, dt, few)) return 1;
+            pending = w.norm2;
         }
-        if (tap(l + 1)) return 1;
+        if (g->taps_on && l < nl - 1 && (settle(nullptr) || tap(l + 1))) return 1;
     }
+    if (settle(lay.final_norm)) return 1;                              // the last update of x also makes the head's input
+    if (nl > 0 && tap(nl)) return 1;
     if (few && !hr) return product(g, few, lay.xb.p, d8, g->head, d8, d8, nullptr, nullptr, logits, (long long)g->ldl, M, c.vocab, EPI_NONE);
     return lm_head(g, lay.xb.p, M, logits, hr);
 }

@@ -47,6 +47,9 @@ __device__ __forceinline__ void mma_bf16_16x8x16(float (&d)[4], uint32_t a0, uin
 // Every CTA normalises all M rows itself: for a few rows that is noise, at 64 rows it cost more than the launch it saves
 // (decode step of a 12-layer, 768-wide model at 64 sequences: 2.30 ms with, 1.0 ms without).
 constexpr int kNormMaxRows = 16;
+// Completing the residual stream reads six bytes per element in every CTA where a finished row is two: one or two rows.  (Decode step of
+// an 8-layer, 2048-wide model: one row 0.540 ms with, 0.544 without; eight rows 0.679 against 0.620.)
+constexpr int kPostNormMaxRows = 2;
 
 // GemmDesc's block-diagonal form
 struct FewRowsGroups { int group; long long group_a, group_c; const __nv_bfloat16* gate; long long ld_gate; };
@@ -54,8 +57,9 @@ struct FewRowsGroups { int group; long long group_a, group_c; const __nv_bfloat1
 // MT: 16-row groups of A (M <= 16 MT); NT: 8-row groups of W per CTA; S: weight slices a warp has in flight.
 // NORM: A holds un-normalised rows; every CTA normalises them itself into shared memory (kind 1: LayerNorm, gamma * ((x - mean) *
 // inv) + beta with inv = 1 / sqrt(var + eps); kind 2: RMSNorm, x * inv * gamma with inv = 1 / sqrt(mean(x^2) + eps)), rounded to
-// bf16 as the stand-alone kernels store them.  M rows of K values per CTA is little work next to the launch it saves.
-template <int MT, int NT, int S, bool NORM>
+// bf16 as the stand-alone kernels store them.  M rows of K values per CTA is little work next to the launch it saves.  NORM 2: RowNorm
+// kind 3, the residual stream completed on the fly.
+template <int MT, int NT, int S, int NORM>
 __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv_bfloat16* __restrict__ A, long long lda,
                                                                      const __nv_bfloat16* __restrict__ W, long long ldb,
                                                                      __nv_bfloat16* C, long long ldc, const float* __restrict__ bias,
@@ -113,7 +117,54 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
 
     const long long a_ld = NORM ? (long long)(K + 8) : lda;
     const __nv_bfloat16* a_base = NORM ? reinterpret_cast<const __nv_bfloat16*>(dyn) : A;
-    if constexpr (NORM) {
+    if constexpr (NORM == 2) {
+        __shared__ float part[kPostNormMaxRows][kWarps];
+        const int P = M >= 8 ? 1 : M >= 4 ? 2 : M >= 2 ? 4 : 8, RP = kWarps / P, my_p = warp % P, my_r = warp / P;
+        const int nvec = K >> 3, per = (nvec + P - 1) / P, c_begin = my_p * per, c_end = min(nvec, c_begin + per);
+        for (int r = my_r; r < M; r += RP) {
+            const uint4* src = reinterpret_cast<const uint4*>(nrm.y + (size_t)r * K);
+            float sq = 0.0f;
+            for (int c = c_begin + lane; c < c_end; c += 32) {
+                const uint4 d = src[c];
+                const uint32_t wd[4] = {d.x, d.y, d.z, d.w};
+#pragma unroll
+                for (int j = 0; j < 4; j++) { const float lo = __uint_as_float(wd[j] << 16), hi = __uint_as_float(wd[j] & 0xffff0000u); sq += lo * lo + hi * hi; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+            if (lane == 0) part[r][my_p] = sq;
+        }
+        __syncthreads();
+        for (int r = my_r; r < M; r += RP) {
+            float tot = 0.0f;
+            for (int q = 0; q < P; q++) tot += part[r][q];
+            const float inv = 1.0f / sqrtf(tot / (float)nrm.dim + nrm.eps);
+            for (int c = c_begin + lane; c < c_end; c += 32) {
+                const uint4 d = reinterpret_cast<const uint4*>(nrm.y + (size_t)r * K)[c];
+                const uint32_t wd[4] = {d.x, d.y, d.z, d.w};
+                const float4 x0 = reinterpret_cast<const float4*>(nrm.x + (size_t)r * K)[2 * c], x1 = reinterpret_cast<const float4*>(nrm.x + (size_t)r * K)[2 * c + 1];
+                const float4 g0 = __ldg(reinterpret_cast<const float4*>(nrm.gamma + 8 * c)), g1 = __ldg(reinterpret_cast<const float4*>(nrm.gamma + 8 * c + 4));
+                float v[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
+                const float gg[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+                uint4 o;
+                __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    v[2 * j] += __uint_as_float(wd[j] << 16) * inv * gg[2 * j];
+                    v[2 * j + 1] += __uint_as_float(wd[j] & 0xffff0000u) * inv * gg[2 * j + 1];
+                    oh[j] = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+                }
+                reinterpret_cast<uint4*>(dyn + (size_t)r * (K + 8) * 2)[c] = o;
+                if (blockIdx.x == 0) {
+                    reinterpret_cast<float4*>(nrm.x_out + (size_t)r * K)[2 * c] = make_float4(v[0], v[1], v[2], v[3]);
+                    reinterpret_cast<float4*>(nrm.x_out + (size_t)r * K)[2 * c + 1] = make_float4(v[4], v[5], v[6], v[7]);
+                    reinterpret_cast<uint4*>(nrm.xb + (size_t)r * K)[c] = o;
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if constexpr (NORM == 1) {
         // Warps are dealt over (row, part of the row): eight rows or more, one warp per row; a single row, eight warps on its eighths.
         // The partial sums of a row's parts meet in shared memory.
         __shared__ float part[kNormMaxRows][kWarps], part2[kNormMaxRows][kWarps];
@@ -284,12 +335,12 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
 constexpr size_t kNormSmemLimit = 160 * 1024;
 size_t norm_smem(const GemmDesc& d) { return (size_t)d.M * (d.K + 8) * 2; }
 
-template <int MT, int NT, bool NORM>
+template <int MT, int NT, int NORM>
 int launch(const GemmDesc& d, const RowNorm& nrm, bool dependent) {
     // Few weight rows and a long K (the projections back to the model width): clusters of 2 or 4 CTAs split K, so that the launch
     // still covers the SMs and a warp's share of K is one round of loads.
     int ksplit = 1;
-    if constexpr (!NORM) {
+    if constexpr (NORM == 0) {
         const long long blocks = ceil_div(d.N, NT * 8);
         while (ksplit < 4 && blocks * ksplit * 2 <= 3ll * rt().sm_count && d.K / (ksplit * 2) >= 32 * kWarps) ksplit *= 2;
     }
@@ -309,7 +360,7 @@ int launch(const GemmDesc& d, const RowNorm& nrm, bool dependent) {
     return 0;
 }
 
-template <bool NORM>
+template <int NORM>
 int dispatch(const GemmDesc& d, const RowNorm& nrm, bool dependent) {
     // CTAs: 8, 16 or 32 weight rows each, the widest that still gives every SM two CTAs (a short kernel: spread first)
     const long long want = 2ll * rt().sm_count;
@@ -317,18 +368,18 @@ int dispatch(const GemmDesc& d, const RowNorm& nrm, bool dependent) {
     int nt = 1;
     if (ceil_div(d.N, 16) >= want && d.group % 16 == 0) nt = 2;
     if (mt <= 2 && ceil_div(d.N, 32) >= want && d.group % 32 == 0) nt = 4;
-    if constexpr (NORM) {            // at most kNormMaxRows = 16 rows: one row group
-        return nt == 1 ? launch<1, 1, true>(d, nrm, dependent) : nt == 2 ? launch<1, 2, true>(d, nrm, dependent) : launch<1, 4, true>(d, nrm, dependent);
+    if constexpr (NORM != 0) {       // at most kNormMaxRows = 16 rows: one row group
+        return nt == 1 ? launch<1, 1, NORM>(d, nrm, dependent) : nt == 2 ? launch<1, 2, NORM>(d, nrm, dependent) : launch<1, 4, NORM>(d, nrm, dependent);
     } else {
         switch (mt * 10 + nt) {
-            case 11: return launch<1, 1, false>(d, nrm, dependent);
-            case 12: return launch<1, 2, false>(d, nrm, dependent);
-            case 14: return launch<1, 4, false>(d, nrm, dependent);
-            case 21: return launch<2, 1, false>(d, nrm, dependent);
-            case 22: return launch<2, 2, false>(d, nrm, dependent);
-            case 24: return launch<2, 4, false>(d, nrm, dependent);
-            case 41: return launch<4, 1, false>(d, nrm, dependent);
-            default: return launch<4, 2, false>(d, nrm, dependent);
+            case 11: return launch<1, 1, 0>(d, nrm, dependent);
+            case 12: return launch<1, 2, 0>(d, nrm, dependent);
+            case 14: return launch<1, 4, 0>(d, nrm, dependent);
+            case 21: return launch<2, 1, 0>(d, nrm, dependent);
+            case 22: return launch<2, 2, 0>(d, nrm, dependent);
+            case 24: return launch<2, 4, 0>(d, nrm, dependent);
+            case 41: return launch<4, 1, 0>(d, nrm, dependent);
+            default: return launch<4, 2, 0>(d, nrm, dependent);
         }
     }
 }
@@ -423,6 +474,9 @@ bool linear_few_rows_supported(const GemmDesc& d) {
 
 bool linear_few_rows_norm_supported(const GemmDesc& d, const RowNorm& nrm) {
     const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    if (nrm.kind == 3)
+        return linear_few_rows_supported(d) && nrm.gamma && nrm.x && nrm.y && nrm.x_out && nrm.x_out != nrm.x && nrm.xb && nrm.dim > 0 && nrm.dim <= d.K && !d.group &&
+               al16(nrm.gamma) && al16(nrm.x) && al16(nrm.y) && al16(nrm.x_out) && al16(nrm.xb) && d.M <= kPostNormMaxRows && norm_smem(d) <= kNormSmemLimit;
     return linear_few_rows_supported(d) && (nrm.kind == 1 || nrm.kind == 2) && nrm.gamma && al16(nrm.gamma) && (nrm.kind == 2 || (nrm.beta && al16(nrm.beta))) &&
            d.M <= kNormMaxRows && norm_smem(d) <= kNormSmemLimit;
 }
@@ -449,10 +503,10 @@ int norm_few_rows(const void* x, void* out, int rows, int K, const RowNorm& nrm,
 int linear_few_rows(const GemmDesc& d, const RowNorm* nrm, bool dependent) {
     if (nrm && nrm->kind) {
         if (!linear_few_rows_norm_supported(d, *nrm)) return fail("linear_few_rows: unsupported problem (normalised rows)");
-        return dispatch<true>(d, *nrm, dependent);
+        return nrm->kind == 3 ? dispatch<2>(d, *nrm, dependent) : dispatch<1>(d, *nrm, dependent);
     }
     if (!linear_few_rows_supported(d)) return fail("linear_few_rows: unsupported problem");
-    return dispatch<false>(d, RowNorm{}, dependent);
+    return dispatch<0>(d, RowNorm{}, dependent);
 }
 
 }  // namespace spt

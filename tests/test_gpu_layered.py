@@ -10,7 +10,7 @@ import pytest
 from conftest import parity_record
 from layered_models import bf16, config, gla, latent, params, row_errors, shapes_of
 from oracle.layered import LayeredOracle
-from sptorch_b200 import trace, weights
+from sptorch_b200 import generate, trace, weights
 from sptorch_b200.backend import BF16, F32, HalError
 from sptorch_b200.gpt import GPT
 from sptorch_b200.kv_cache import layer_specs
@@ -246,7 +246,7 @@ def _save(folder, cfg, p):
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
-def test_model_folder_generation_and_replay(backend, dtype, tmp_path):
+def test_model_folder_generation_and_replay(backend, dtype, tmp_path, capsys):
     """config.json + safetensors through the registry, greedy generation through the framework's own loop, and the same tokens replayed."""
     cfg = MIXED
     p = params(cfg, 41)
@@ -266,6 +266,9 @@ def test_model_folder_generation_and_replay(backend, dtype, tmp_path):
             agreed += 1
     assert agreed >= 10
     assert m.generate(prompt, 40, top_k=1) == out                    # a second request on the same model
+    assert generate.main(["--model", str(tmp_path), "--tokens", ",".join(map(str, prompt)), "--max-new-tokens", "40", "--max-context", "128",
+                          "--dtype", "float32" if dtype == F32 else "bfloat16"]) == 0
+    assert [int(t) for t in capsys.readouterr().out.strip().split(",")] == out
     said = []
     steps = [{"step": 0, "entries": [{"id": "r", "tokens": out[:50], "want": [20, 49]}], "end": []}] + \
             [{"step": i + 1, "entries": [{"id": "r", "tokens": [out[50 + i]], "want": [0]}], "end": []} for i in range(11)]
