@@ -198,7 +198,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     // P V products done: two barriers per query tile, taken in turn by the tile's steps (index step & 1, phase step >> 1).  With
     // rotating score buffers a tile's softmax can finish step j before P V of step j - 1 has completed, so its wait for the
     // product of step j on a single barrier would be two phases ahead -- which a parity wait cannot tell from none; on the
-    // barrier of its own parity class it is never more than one phase ahead (the product of step j + 2 needs this thread's P).
+    // barrier of its own parity class it is never more than one phase ahead (the product of step j + 2 needs this thread's P).  With one
+    // query tile in the item the softmax can be a step further ahead; its end has a wait of its own for that (below).
     const uint32_t pv_done = p_full + 8 * 3;        // 4: [query tile][step & 1]
     const uint32_t o_free = pv_done + 32;           // 2
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + L::kBars + 240);
@@ -515,6 +516,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (j == 0 && c == 0) m = mx;                    // the first chunk of a row always holds key 0: finite
                     const bool grow = (mx - m) * p.scale_log2 > 8.0f;
                     if (__any_sync(0xffffffffu, grow)) {
+                        tmem_ld_wait();                          // the next chunk's registers may be moved below: they must have arrived
                         float alpha = 1.0f;
                         if (grow) { alpha = ex2_approx((m - mx) * p.scale_log2); m = mx; }
                         l *= alpha;
@@ -522,6 +524,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         if (j > 0) {
                             // every product accumulated so far is in place (the commit of step - 1; the next one needs this thread's P)
                             if (!mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait)) return false;
+                            __syncwarp();                        // the wait's lanes leave it one by one, the loads below are warp-wide
                             tc_fence_after();
 #pragma unroll
                             for (int cc = 0; cc < VD / 32; cc++) {
@@ -533,6 +536,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                                 tmem_st_32x32(o_addr + cc * 32, o);
                             }
                         }
+                        if (c > 0) tmem_st_wait();               // P's chunks have landed before they are read back
                         if (c > 0 && PSPLIT) {
                             uint32_t w[32];
 #pragma unroll
@@ -607,8 +611,13 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             if (n_kv > 0) {
                 float inv = 1.0f / l;
                 if (p.gate && qrow < p.T) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[((long long)bb * p.T + qrow) * p.ld_gate + hh])));
-                ok = mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait);     // the item's last product
+                // The item's last product -- after the one before it: scores run up to two ahead, so with a single query tile only the product of
+                // step - 4 is sure to be done here, and a parity wait for step - 1 could not tell step - 3 (same barrier, the phase before)
+                // from step - 1.  The product of step - 2 waits on the other barrier, one phase ahead of step - 4, and brings step - 3 with it.
+                ok = (n_kv < 2 || mbar_wait(pv_done + 8 * (2 * t + (step & 1)), ((step - 2) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait)) &&
+                     mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait);
                 if (!ok) break;
+                __syncwarp();
                 tc_fence_after();
                 __nv_bfloat16* orow = p.out + ((long long)bb * p.T + qrow) * p.ld_out + (long long)hh * p.V;
 #pragma unroll

@@ -244,3 +244,22 @@ def test_fused_attention_with_steeply_rising_scores(backend, oracle, T, hd):
     fused2 = backend.attention_causal(q, k2, v, H, dtype=BF16)
     ref2 = _mha_core(oracle, q[0], k2[0], v[0], H)[None]
     assert relerr(fused2, ref2) <= 1.5 * 2 ** -8
+@pytest.mark.parametrize("T", [264, 320, 384, 640, 896])
+def test_fused_attention_when_the_last_query_tile_is_alone(backend, oracle, T):
+    """T = 256 n + 1 .. 128: the last work item has one query tile, whose scores run two key tiles ahead of P V.  The first warp's rows are
+    slow (their maximum moves at every chunk), the other warps' rows are not, so the fast warps ask for the last product long before it --
+    or the ones before it -- is done; none of them may read the output early."""
+    rng = np.random.default_rng(T)
+    B, H, hd = 2, 8, 64
+    u = np.where(rng.random(hd) < 0.5, -0.125, 0.125).astype(np.float32)
+    q = _bf16(0.02 * rng.standard_normal((B, T, H * hd)).astype(np.float32))
+    last = (T - 1) // 128 * 128
+    q[:, last:last + 32] = np.tile(u, H)
+    k = np.concatenate([(8.0 * (j // 4)) * np.tile(u, H)[None, :] for j in range(T)])[None].repeat(B, 0).astype(np.float32)
+    k = _bf16(k)
+    v = _bf16(rng.standard_normal((B, T, H * hd)).astype(np.float32))
+    ref = np.stack([_mha_core(oracle, q[i], k[i], v[i], H) for i in range(B)])
+    for _ in range(5):
+        assert relerr(backend.attention_causal(q, k, v, H, dtype=BF16), ref) <= 2e-2
+
+

@@ -102,6 +102,42 @@ def test_other_sizes(backend, dtype, width, vocab, layers, rank):
     m.close()
 
 
+@pytest.mark.parametrize("layer", [
+    latent(heads=2, dim=96, vdim=40, rot_dim=48, sharp=2.0), latent(heads=3, dim=32, vdim=104, rot_dim=64, sharp=2.0), latent(heads=2, dim=128, vdim=128, rot_dim=64, sharp=2.0),
+    latent(heads=20, dim=24, vdim=16, kv_rank=400, q_rank=64, rot_dim=24, sharp=2.0), latent(heads=17, dim=16, vdim=32, kv_rank=512, rot_dim=64), latent(heads=1, dim=64, vdim=64, kv_rank=24, rot_dim=8),
+    gla(heads=1, dim=32, vdim=120), gla(heads=2, dim=20, vdim=250), gla(heads=2, dim=64, vdim=128), gla(heads=1, dim=60, vdim=200), gla(heads=2, dim=100, vdim=64), gla(heads=1, dim=112, vdim=144)])
+def test_every_kernel_shape(backend, layer):
+    """bf16: every tile shape the fused attention, the cached-row attention and the chunk kernels are built for, on several tiles of keys
+    and chunks, as one prompt, behind a cached prefix and in decoding."""
+    cfg = config([layer], width=80)
+    p = params(cfg, 53)
+    ids = _ids(cfg, 560)
+    ref = LayeredOracle(cfg, p).feed(ids)
+    m = _model(backend, cfg, p, BF16, seq_len=560)
+    for cuts in ([560], [300, 200, 2, 3, 16, 33, 1, 1, 1, 1, 1, 1], [129, 383, 48]):
+        _check(_feed(m, ids, cuts), ref, BF16, f"portions {cuts}")
+    m.close()
+
+
+@pytest.mark.parametrize("layer", [latent(heads=20, dim=24, vdim=16, kv_rank=400, q_rank=64, rot_dim=24, sharp=2.0), latent(heads=4, dim=64, vdim=64, rot_dim=32, sharp=3.0),
+                                   latent(heads=4, dim=64, vdim=128, rot_dim=32, sharp=3.0), latent(heads=4, dim=128, vdim=64, rot_dim=32, sharp=3.0), latent(heads=4, dim=128, vdim=128, rot_dim=64, sharp=3.0)])
+def test_short_portions_behind_long_prefixes(backend, layer):
+    """A portion of at most one query tile behind several key tiles, with scores peaked enough that some warps rescale and others do not:
+    every position of every portion, none far off."""
+    cfg = config([layer], width=80)
+    p = params(cfg, 53)
+    ids = _ids(cfg, 800)
+    ref = LayeredOracle(cfg, p).feed(ids)
+    m = _model(backend, cfg, p, BF16, seq_len=800)
+    for first in (128, 256, 384, 521, 640):
+        for T in (17, 33, 48, 64, 90, 128, 150):
+            m.reset_cache()
+            m.extend(ids[:first].reshape(1, -1))
+            e = row_errors(m.extend(ids[first:first + T].reshape(1, -1))[0], ref[first:first + T])
+            assert e.max() <= 2 * TOL[BF16], f"{T} tokens at {first}: {e.max():.3e} at row {int(e.argmax())}"
+    m.close()
+
+
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
 def test_prompt_portions_and_decoding_agree(backend, dtype):
     """The same tokens as one prompt, token by token and in portions of several sizes: each against the oracle at every position."""
