@@ -3,7 +3,8 @@
 // followed by an RMS norm of each head's o over V and the gate silu(W_g h).  q carries the factor D^(-1/2).  The recurrence, its
 // decays and the norm are f32 whatever the model's dtype; q, k, v, the gate and A1 h come from the layer's input projection.
 //
-// gla_recurrent walks the tokens one by one (any sizes, both dtypes; a decode step is T = 1); gla_chunked takes bf16 prompts in chunks.
+// gla_recurrent walks the tokens one by one (any sizes, both dtypes; one token per sequence has a kernel of
+// its own); gla_chunked takes bf16 prompts in chunks.
 #include "layered.h"
 #include "epilogue_math.cuh"
 #include "pdl.cuh"
@@ -122,6 +123,78 @@ __global__ void __launch_bounds__(kRecWarps * 32) gla_recurrent_kernel(const Gla
             for (int i = tid; i < a.T * 8; i += blockDim.x) { const int c = h * V + v0 + 32 + (i & 7); if (c < a.ld_out) out[(size_t)(i >> 3) * a.ld_out + c] = (T)0.0f; }
         if (parts > 1) cluster.sync();                  // no CTA leaves while its sums may still be read
     }
+}
+
+// One token per sequence, V a multiple of four: a CTA owns a whole head.  Thread = (row group, four columns); its rows of the state are
+// requested before the programmatic-launch wait (the step before wrote them), pass through registers once and go back; the row groups'
+// shares of o meet in shared memory, where norm and gate finish the head.  HBM bytes: 8 D V per head.
+template <typename T, int NR>
+__global__ void __launch_bounds__(NR > 16 ? 512 : 256) gla_step_kernel(const GlaArgs a) {
+    extern __shared__ float sm[];
+    __shared__ float red[16];
+    pdl_release();
+    const int D = a.D, V = a.V, R = a.R, c4n = V / 4, rgs = blockDim.x / c4n;
+    const int D4 = (D + 3) / 4 * 4;
+    float* qs = sm;                                   // [D4]
+    float* ks = qs + D4;
+    float* al = ks + D4;
+    float* as = al + D4;                              // [R]
+    float* part = as + (R + 3) / 4 * 4;               // [row groups][V]
+    const int tid = threadIdx.x, bh = blockIdx.x, b = bh / a.H, h = bh - b * a.H, rg = tid / c4n, c = (tid - rg * c4n) * 4;
+    const bool mine = rg < rgs;
+    float* st = a.state + (size_t)bh * D * V + c;
+    float4 s[NR];
+#pragma unroll
+    for (int i = 0; i < NR; i++) { const int d = rg + i * rgs; if (mine && d < D) s[i] = *reinterpret_cast<const float4*>(st + (size_t)d * V); }
+    pdl_acquire();
+    const T* in = static_cast<const T*>(a.in) + (size_t)b * a.ld;
+    const float qsc = 1.0f / sqrtf((float)D), inv_tau = 1.0f / a.tau;
+    for (int r = tid; r < R; r += blockDim.x) as[r] = (float)in[a.c_a + r];
+    for (int d = tid; d < D; d += blockDim.x) { qs[d] = (float)in[a.c_q + h * D + d] * qsc; ks[d] = (float)in[a.c_k + h * D + d]; }
+    float v[4] = {0, 0, 0, 0};
+    if (mine) {
+#pragma unroll
+        for (int j = 0; j < 4; j++) v[j] = (float)in[a.c_v + h * V + c + j];
+    }
+    __syncthreads();
+    for (int d = tid; d < D; d += blockDim.x) {
+        const float* w = a.a2 + (size_t)(h * D + d) * R;
+        float z = a.a2_b[h * D + d];
+#pragma unroll 8
+        for (int r = 0; r < R; r++) z = fmaf(as[r], __ldg(w + r), z);
+        al[d] = expf(log_decay(z, inv_tau));
+    }
+    __syncthreads();
+    float4 acc = make_float4(0, 0, 0, 0);
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int d = rg + i * rgs;
+        if (mine && d < D) {
+            const float f = al[d], k = ks[d], q = qs[d];
+            s[i].x = fmaf(s[i].x, f, k * v[0]); s[i].y = fmaf(s[i].y, f, k * v[1]); s[i].z = fmaf(s[i].z, f, k * v[2]); s[i].w = fmaf(s[i].w, f, k * v[3]);
+            *reinterpret_cast<float4*>(st + (size_t)d * V) = s[i];
+            acc.x = fmaf(s[i].x, q, acc.x); acc.y = fmaf(s[i].y, q, acc.y); acc.z = fmaf(s[i].z, q, acc.z); acc.w = fmaf(s[i].w, q, acc.w);
+        }
+    }
+    if (mine) *reinterpret_cast<float4*>(part + rg * V + c) = acc;
+    __syncthreads();
+    float sq = 0.0f;
+    for (int i = tid; i < V; i += blockDim.x) {
+        float o = 0.0f;
+        for (int r = 0; r < rgs; r++) o += part[r * V + i];
+        part[i] = o;                                  // only this thread reads column i
+        sq = fmaf(o, o, sq);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    if ((tid & 31) == 0) red[tid >> 5] = sq;
+    __syncthreads();
+    float tot = 0.0f;
+    for (int w = 0; w < (int)blockDim.x / 32; w++) tot += red[w];
+    const float inv = 1.0f / sqrtf(tot / (float)V + a.eps);
+    T* out = static_cast<T*>(a.out) + (size_t)b * a.ld_out;
+    for (int i = tid; i < V; i += blockDim.x) out[h * V + i] = (T)(part[i] * inv * a.head_norm[i] * silu_exact((float)in[a.c_g + h * V + i]));
+    if (h == a.H - 1) for (int i = a.H * V + tid; i < a.ld_out; i += blockDim.x) out[i] = (T)0.0f;
 }
 
 // out = o / sqrt(mean(o^2) + eps) * w * silu(g): one warp per (token, head); the last head's warp zeroes the row's padding
@@ -660,6 +733,29 @@ int launch_recurrent(const GlaArgs& a, float* o, bool dependent) {
     return 0;
 }
 
+// rows of the state per thread of the one-token kernel with `threads` threads; 0: it does not take this layer
+int step_rows(const GlaArgs& a, int threads) {
+    if (a.T != 1 || !a.state || a.V % 4 || a.V > 1024 || a.V / 4 > threads) return 0;
+    return ceil_div(a.D, threads / (a.V / 4));
+}
+
+template <typename T>
+int step_t(const GlaArgs& a, bool dependent) {
+    const int small = step_rows(a, 256), threads = small <= 16 ? 256 : 512, rows = threads == 256 ? small : step_rows(a, 512);
+    const size_t smem = ((size_t)3 * ((a.D + 3) / 4 * 4) + (a.R + 3) / 4 * 4 + (size_t)threads / (a.V / 4) * a.V) * sizeof(float);
+    const dim3 grid(a.B * a.H), block(threads);
+    if (rows <= 4) SPT_CUDA(launch_dependent(gla_step_kernel<T, 4>, grid, block, smem, dependent, 1, a));
+    else if (rows <= 8) SPT_CUDA(launch_dependent(gla_step_kernel<T, 8>, grid, block, smem, dependent, 1, a));
+    else if (rows <= 16 && threads == 256) SPT_CUDA(launch_dependent(gla_step_kernel<T, 16>, grid, block, smem, dependent, 1, a));
+    else SPT_CUDA(launch_dependent(gla_step_kernel<T, 24>, grid, block, smem, dependent, 1, a));
+    note_submit();
+    return 0;
+}
+bool step_takes(const GlaArgs& a) {
+    const int small = step_rows(a, 256), wide = step_rows(a, 512);
+    return (small > 0 && small <= 16) || (wide > 8 && wide <= 24);
+}
+
 template <typename T>
 int recurrent_t(const GlaArgs& a, float* o, bool dependent) {
     const int per = ceil_div(a.D, kRecWarps);
@@ -684,11 +780,12 @@ int gla_norm_gate(const GlaArgs& a, const float* o, bool dependent) {
 
 int gla_recurrent(const GlaArgs& a, float* o_scratch, bool dependent) {
     if (a.B * a.H > 65535) return fail("gla: batch x heads exceeds one launch");
+    if (step_takes(a)) return a.dtype == BF16 ? step_t<__nv_bfloat16>(a, dependent) : step_t<float>(a, dependent);
     if (a.dtype == BF16 ? recurrent_t<__nv_bfloat16>(a, o_scratch, dependent) : recurrent_t<float>(a, o_scratch, dependent)) return 1;
     return recurrent_fuses(a) ? 0 : gla_norm_gate(a, o_scratch, dependent);
 }
 
-bool gla_chunked_supported(const GlaArgs& a) { return a.dtype == BF16 && a.D <= 128 && a.V <= 256 && a.R <= 64 && a.B * a.H <= 65535; }
+bool gla_chunked_supported(const GlaArgs& a) { return a.dtype == BF16 && a.T > kRecTokens && a.D <= 128 && a.V <= 256 && a.R <= 64 && a.B * a.H <= 65535; }
 static size_t chunks_of(const GlaArgs& a) { return (size_t)a.B * a.H * ceil_div(a.T, kChunk); }
 size_t gla_chunked_state_bytes(const GlaArgs& a) { return chunks_of(a) * a.D * a.V * sizeof(float); }
 size_t gla_chunked_decay_bytes(const GlaArgs& a) { return chunks_of(a) * kChunk * a.D * sizeof(float); }

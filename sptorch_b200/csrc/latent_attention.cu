@@ -321,10 +321,16 @@ __global__ void __launch_bounds__(kLdThreads, 1) latent_decode_kernel(const Late
     const int per_row = a.row / 8;
     auto load = [&](int stage, int k0) {
         __nv_bfloat16* dst = tile + stage * kLdKeys * pitch;
-        for (int i = tid; i < kLdKeys * per_row; i += kLdThreads) {
-            const int k = i / per_row, c = (i - k * per_row) * 8;
-            if (k0 + k < hi) cp_async16(smem_addr(dst + k * pitch + c), rows + (size_t)(k0 + k) * a.row + c);
-            else *reinterpret_cast<uint4*>(dst + k * pitch + c) = make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int r = 0; r < kLdKeys / 16; r++) {                                // a warp copies four rows
+            const int k = warp + 16 * r;
+            const bool live = k0 + k < hi;
+            const __nv_bfloat16* src = rows + (size_t)(k0 + k) * a.row;
+            const uint32_t d = smem_addr(dst + k * pitch);
+            for (int c = lane * 8; c < a.row; c += 256) {
+                if (live) cp_async16(d + c * 2, src + c);
+                else *reinterpret_cast<uint4*>(dst + k * pitch + c) = make_uint4(0, 0, 0, 0);
+            }
         }
     };
     // rows before this step's tokens were written by earlier steps: the first tile may be requested before the kernels ahead are done
