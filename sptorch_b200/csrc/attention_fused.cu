@@ -15,9 +15,8 @@
 //   warps 2..5  softmax of query tile 0, warps 6..9 of query tile 1: ONE THREAD PER QUERY ROW.  A thread reads
 //               its 128 scores from TMEM in four chunks of 32 (the next chunk's load in flight while one is worked on;
 //               the running row maximum is the thread's own business, no other thread has a part in it), evaluates
-//               2^(s*c - m*c) (part on the special-function unit, part as a cubic polynomial on the FMA pipe,
-//               because the 16-per-clock exponential unit would otherwise be the limit), and writes P as bf16
-//               back into the TMEM columns the scores came from
+//               2^(s*c - m*c) on the special-function unit, and writes P as bf16 back into the TMEM columns the scores
+//               came from
 // O accumulates in TMEM over the key tiles of an item and is rescaled in place only when a row maximum grows by
 // more than 2^8 (lazy rescaling).  TMEM, head size 128: S/P of tile 0 at columns 0..127, of tile 1 at 128..255, O_0 at 256,
 // O_1 at 384 (512 columns, one CTA per SM).  Head size 64 (accumulators of 64 columns): THREE score buffers at 0 / 128 / 256
@@ -70,22 +69,6 @@ __device__ __forceinline__ float ex2_approx(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
-}
-
-// 2^x for two values on the FMA pipe: x = n + f with n = round(x), f in [-0.5, 0.5]; 2^f by a cubic (relative error
-// 7.5e-5 = 2^-13.7, far below the 2^-9 of the bf16 rounding that follows); n goes straight into the exponent field.
-// x is clamped at -125 so that the exponent arithmetic cannot wrap (the result is then 2^-125, nothing in any sum).
-__device__ __forceinline__ float2 ex2_poly2(float2 x) {
-    const float kMagic = 12582912.0f;               // 1.5 * 2^23: adding it leaves round(x) in the low mantissa bits
-    x.x = fmaxf(x.x, -125.0f); x.y = fmaxf(x.y, -125.0f);
-    const float2 r = __fadd2_rn(x, make_float2(kMagic, kMagic));
-    const float2 n = __fadd2_rn(r, make_float2(-kMagic, -kMagic));
-    const float2 f = __ffma2_rn(n, make_float2(-1.0f, -1.0f), x);
-    float2 p = __ffma2_rn(f, make_float2(0.055171654f, 0.055171654f), make_float2(0.24261113f, 0.24261113f));
-    p = __ffma2_rn(p, f, make_float2(0.69326097f, 0.69326097f));
-    p = __ffma2_rn(p, f, make_float2(0.99992806f, 0.99992806f));
-    return make_float2(__int_as_float(__float_as_int(p.x) + (__float_as_int(r.x) << 23)),
-                       __int_as_float(__float_as_int(p.y) + (__float_as_int(r.y) << 23)));
 }
 
 __device__ __forceinline__ float max3(float a, float b, float c) {
@@ -164,7 +147,7 @@ struct AttnSmem {
 // Persistent kernel: CTA c works through column c of a schedule built on the host (attention_schedule below), and all
 // roles run straight through item boundaries (barrier phases are driven by running counters), so the loads and the
 // first Q K^T of the next item are in flight while the current one drains.
-template <int KBN, int KBR, int VD, int NPOLY, bool ROTP, bool PSPLIT>
+template <int KBN, int KBR, int VD, bool ROTP, bool PSPLIT>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQr, const __grid_constant__ CUtensorMap tmKr,
@@ -494,9 +477,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 const float2 c2 = make_float2(p.scale_log2, p.scale_log2);
                 uint32_t va[32], vb[32];
                 tmem_ld_32x32(s_addr, va);
-                auto chunk = [&](auto c_tag, uint32_t (&v)[32], uint32_t (&vnext)[32], auto npoly_tag, auto diag_tag) -> bool {
+                auto chunk = [&](auto c_tag, uint32_t (&v)[32], uint32_t (&vnext)[32], auto diag_tag) -> bool {
                     constexpr int c = decltype(c_tag)::value;
-                    constexpr int NP = decltype(npoly_tag)::value;
                     constexpr bool DIAG = decltype(diag_tag)::value;
                     tmem_ld_wait();
                     if (c < 3) tmem_ld_32x32(s_addr + (c + 1) * 32, vnext);
@@ -576,9 +558,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
                     for (int i = 0; i < 16; i++) {
                         const float2 x = __ffma2_rn(make_float2(__uint_as_float(v[2 * i]), __uint_as_float(v[2 * i + 1])), c2, nmb2);
-                        float2 e;
-                        if (i < NP) e = ex2_poly2(x);
-                        else e = make_float2(ex2_approx(x.x), ex2_approx(x.y));
+                        const float2 e = make_float2(ex2_approx(x.x), ex2_approx(x.y));
                         if (i & 1) sum_b = __fadd2_rn(sum_b, e); else sum_a = __fadd2_rn(sum_a, e);
                         if constexpr (PSPLIT) split2(e, packed[i], packed[i + 16]);
                         else {
@@ -592,13 +572,13 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     else tmem_st_32x32b_x16(s_addr + c * 16, packed);
                     return true;
                 };
-                auto tile = [&](auto npoly_tag, auto diag_tag) -> bool {
-                    return chunk(std::integral_constant<int, 0>(), va, vb, npoly_tag, diag_tag) &&
-                           chunk(std::integral_constant<int, 1>(), vb, va, npoly_tag, diag_tag) &&
-                           chunk(std::integral_constant<int, 2>(), va, vb, npoly_tag, diag_tag) &&
-                           chunk(std::integral_constant<int, 3>(), vb, va, npoly_tag, diag_tag);
+                auto tile = [&](auto diag_tag) -> bool {
+                    return chunk(std::integral_constant<int, 0>(), va, vb, diag_tag) &&
+                           chunk(std::integral_constant<int, 1>(), vb, va, diag_tag) &&
+                           chunk(std::integral_constant<int, 2>(), va, vb, diag_tag) &&
+                           chunk(std::integral_constant<int, 3>(), vb, va, diag_tag);
                 };
-                ok = diag ? tile(std::integral_constant<int, 0>(), std::true_type()) : tile(std::integral_constant<int, NPOLY>(), std::false_type());
+                ok = diag ? tile(std::true_type()) : tile(std::false_type());
                 if (!ok) break;
                 tmem_st_wait();
                 tc_fence_before();
@@ -752,13 +732,6 @@ bool attention_fused_supported(int T, int hd, long long ld_q, long long ld_kv) {
     return (hd == 64 || hd == 128) && T > 0 && ld_q % 8 == 0 && ld_kv % 8 == 0;
 }
 
-// share of the exponentials evaluated on the FMA pipe (of every 16 pairs), per head size; tunable for experiments
-static int attn_npoly(int hd) {
-    static const int e64 = getenv("SPTORCH_B200_ATTN_NPOLY64") ? atoi(getenv("SPTORCH_B200_ATTN_NPOLY64")) : 0;
-    static const int e128 = getenv("SPTORCH_B200_ATTN_NPOLY128") ? atoi(getenv("SPTORCH_B200_ATTN_NPOLY128")) : 0;
-    return hd == 64 ? e64 : e128;
-}
-
 // q, k, v: [B*T, ld] bf16, head h at columns h*hd (token-major: the layout the QKV projection writes);
 // out: [B*T, ld_out] bf16, head h at columns h*hd.
 int attention_fused(const void* q, const void* k, const void* v, void* out, int B, int T, int H, int hd, long long ld_q, long long ld_k,
@@ -787,20 +760,11 @@ int attention_fused(const void* q, const void* k, const void* v, void* out, int 
         kern<<<(unsigned)grid, kAttnThreads, smem_bytes, rt().stream>>>(tq, tk, tv, tq, tk, prm);
         return 0;
     };
-    const int np = attn_npoly(hd);
     int lrc;
     if (hd == 64) {
         static const bool rot_off = getenv("SPTORCH_B200_ATTN_ROT") && atoi(getenv("SPTORCH_B200_ATTN_ROT")) == 0;
-        if (rot_off) lrc = launch(attn_fused_kernel<1, 0, 64, 0, false, false>, AttnSmem<1, 0, 64>::kTotal);
-        else if (np <= 0) lrc = launch(attn_fused_kernel<1, 0, 64, 0, true, false>, AttnSmem<1, 0, 64>::kTotal);
-        else if (np <= 4) lrc = launch(attn_fused_kernel<1, 0, 64, 4, true, false>, AttnSmem<1, 0, 64>::kTotal);
-        else if (np <= 5) lrc = launch(attn_fused_kernel<1, 0, 64, 5, true, false>, AttnSmem<1, 0, 64>::kTotal);
-        else if (np <= 6) lrc = launch(attn_fused_kernel<1, 0, 64, 6, true, false>, AttnSmem<1, 0, 64>::kTotal);
-        else lrc = launch(attn_fused_kernel<1, 0, 64, 8, true, false>, AttnSmem<1, 0, 64>::kTotal);
-    } else {
-        if (np <= 0) lrc = launch(attn_fused_kernel<2, 0, 128, 0, true, false>, AttnSmem<2, 0, 128>::kTotal);
-        else lrc = launch(attn_fused_kernel<2, 0, 128, 4, true, false>, AttnSmem<2, 0, 128>::kTotal);
-    }
+        lrc = rot_off ? launch(attn_fused_kernel<1, 0, 64, false, false>, AttnSmem<1, 0, 64>::kTotal) : launch(attn_fused_kernel<1, 0, 64, true, false>, AttnSmem<1, 0, 64>::kTotal);
+    } else lrc = launch(attn_fused_kernel<2, 0, 128, true, false>, AttnSmem<2, 0, 128>::kTotal);
     if (lrc) return lrc;
     SPT_LAUNCH_CHECK("attn_fused");
     return 0;
@@ -841,8 +805,8 @@ int attention_latent(const void* q, long long ld_q, const void* kn, const void* 
         return 0;
     };
     int rc;
-    if (D <= 64) rc = V <= 64 ? launch(attn_fused_kernel<1, 1, 64, 0, true, true>, AttnSmem<1, 1, 64>::kTotal) : launch(attn_fused_kernel<1, 1, 128, 0, true, true>, AttnSmem<1, 1, 128>::kTotal);
-    else rc = V <= 64 ? launch(attn_fused_kernel<2, 1, 64, 0, true, true>, AttnSmem<2, 1, 64>::kTotal) : launch(attn_fused_kernel<2, 1, 128, 0, true, true>, AttnSmem<2, 1, 128>::kTotal);
+    if (D <= 64) rc = V <= 64 ? launch(attn_fused_kernel<1, 1, 64, true, true>, AttnSmem<1, 1, 64>::kTotal) : launch(attn_fused_kernel<1, 1, 128, true, true>, AttnSmem<1, 1, 128>::kTotal);
+    else rc = V <= 64 ? launch(attn_fused_kernel<2, 1, 64, true, true>, AttnSmem<2, 1, 64>::kTotal) : launch(attn_fused_kernel<2, 1, 128, true, true>, AttnSmem<2, 1, 128>::kTotal);
     if (rc) return rc;
     SPT_LAUNCH_CHECK("attention_latent");
     return 0;
