@@ -159,11 +159,16 @@ typedef struct {
 #define SPT_ARCH_LAYERED 2      /* built from a list of layers: sptorch_ext_layered_create */
 
 void* sptorch_ext_gpt_create(const sptorch_gpt_config* cfg);       /* allocates weights + activations; NULL on failure */
-/* A decoder built from a list of layers that may differ in mixer, sizes and feed-forward.  The norm follows the sublayer:
- * x += rms(mixer(x)) * w1, then (with a feed-forward) x += rms(mlp(x)) * w2; the residual stream is f32 in both dtypes, and f32 models
- * run every product in f32.  The handle serves every sptorch_ext_gpt_* call except tensor parallelism and append = 0 decoding; any
- * T >= 1 is accepted.  Of cfg, vocab, d_model, seq_len (positions a sequence may have), dtype, max_batch and eps are read.
- * Parameter names: embed, l<i>.norm1, l<i>.norm2, l<i>.mix.*, l<i>.mlp.*, final.norm, head. */
+/* A decoder built from a list of layers that may differ in mixer, sizes and feed-forward.  opt->block says how a layer joins the f32
+ * residual stream (norms are RMS norms):
+ *   SPT_BLOCK_POST_NORM  x += rms(mixer(x)) * norm1, then (with a feed-forward) x += rms(mlp(x)) * norm2
+ *   SPT_BLOCK_PARALLEL   h = rms(x) * norm1;  x += mixer(h) + mlp(h); then, with side_dim > 0, the per-layer token input
+ *                        x += rms(proj (gelu(gate x) * e)) * norm, e = this layer's side_dim values of the token's row in side.embed
+ * The stream starts as embed[token] * embed_scale; logits = head (rms(x) final.norm), where with tied_head the head is embed itself.
+ * f32 models run every product in f32.  The handle serves every sptorch_ext_gpt_* call except tensor parallelism and append = 0
+ * decoding; any T >= 1 is accepted.  Of cfg, vocab, d_model, seq_len (positions a sequence may have), dtype, max_batch and eps are read.
+ * Parameter names: embed, side.embed, l<i>.norm1, l<i>.norm2, l<i>.mix.*, l<i>.mlp.*, l<i>.side.*, final.norm, head.
+ * Zero-initialise both structures: a field a layer does not use is ignored. */
 typedef struct {
     int32_t mixer;                    /* SPT_MIXER_* */
     int32_t heads, dim, vdim;         /* per head: query/key size (latent attention: its unrotated part) and value size */
@@ -171,15 +176,34 @@ typedef struct {
     float   tau;                      /* ... and the root of the sigmoid, alpha = sigmoid(z)^(1/tau) */
     int32_t rot_dim, rope_dims;       /* latent attention: size of the rotated part, and how many of its dims rotate */
     int32_t kv_rank, q_rank;          /* ... latent sizes of keys/values and of queries */
-    float   scale;                    /* ... factor of the scores */
+    float   scale;                    /* ... and window attention: factor of the scores */
     double  rope_base;
     int32_t mlp, d_ff;                /* SPT_MLP_* */
+    int32_t mlp_act, mlp_bias;        /* SPT_ACT_* of the gate; whether the three projections have biases */
+    int32_t kv_heads;                 /* window attention: key/value heads, a divisor of heads; query head h reads head h / (heads / kv_heads) */
+    int32_t kv_shared, kv_from;       /* ... kv_shared 1: reads the keys and values of layer kv_from, an earlier one with its own */
+    int32_t window;                   /* ... position i sees positions i - window + 1 .. i (0: all up to i) */
+    int32_t conv_taps;                /* ... causal convolution over time on every channel of q, k and v, behind the projection (0: none) */
+    int32_t distance_bias;            /* ... 1: score - 2^(-8 (h + 1) / heads) * (i - j) */
+    int32_t out_gate;                 /* ... 1: the heads are multiplied element by element with sigmoid(g x) */
+    double  q_temp_coef, q_temp_every;/* ... every > 0: the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) */
 } sptorch_layer_config;
 #define SPT_MIXER_GLA 0
 #define SPT_MIXER_LATENT 1
+#define SPT_MIXER_WINDOW 2            /* softmax attention over cached keys and values (window_attention.cu) */
 #define SPT_MLP_NONE 0
-#define SPT_MLP_DENSE 1               /* down(up * silu(gate)), all three biased */
-void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const sptorch_layer_config* layers, int n_layers);
+#define SPT_MLP_DENSE 1               /* down(up * act(gate)) */
+#define SPT_ACT_SILU 0
+#define SPT_ACT_RELU 1
+typedef struct {
+    int32_t block;                    /* SPT_BLOCK_* */
+    int32_t tied_head;
+    int32_t side_dim;                 /* width of a layer's per-layer token input (0: none) */
+    float   embed_scale;
+} sptorch_layered_options;
+#define SPT_BLOCK_POST_NORM 0
+#define SPT_BLOCK_PARALLEL 1
+void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const sptorch_layer_config* layers, int n_layers, const sptorch_layered_options* opt);
 void  sptorch_ext_gpt_destroy(void* gpt);
 /* name as in GPT::named_parameters (nn/src/lib.rs:1382-1392); host f32 values of the FULL
  * (unsharded) tensor; converted to the model dtype and sliced for this tp_rank on upload. */

@@ -1,8 +1,10 @@
-"""Plain restatement of the models built from a list of layers (architecture "Tolevik"): one function per mechanism, numpy, one
-token after the other wherever the definition is a recurrence.  Test infrastructure only; it shares nothing with the product path.
+"""Plain restatement of the models built from a list of layers (architectures "Tolevik" and "Bulidra"): one function per mechanism,
+numpy, one token after the other wherever the definition is a recurrence.  Test infrastructure only; it shares nothing with the
+product path.
 
 Notation.  A sequence is a matrix of row vectors x[t].  Every weight is [out, in].  ``st`` arguments carry what a sequence keeps
-between calls (GLA: the state matrices; latent attention: the latents and rotated keys), so a prompt may be fed in portions.
+between calls (GLA: the state matrices; latent attention: the latents and rotated keys; attention: keys, values and the last
+projected rows before its convolutions), so a prompt may be fed in portions.
 """
 from __future__ import annotations
 
@@ -113,6 +115,75 @@ def dense_mlp(h, p):
     return (silu(h @ p["gate"].T + p["gate.b"]) * (h @ p["up"].T + p["up.b"])) @ p["down"].T + p["down.b"]
 
 
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + np.tanh(np.sqrt(2.0 / np.pi) * (z + 0.044715 * z ** 3)))
+
+
+def short_convolution(u, w, tail):
+    """u [T, C] projected rows, w [C, K], tail [K - 1, C] the rows before u (zeros in front of a sequence): y[t] = sum_j w[:, j] *
+    u[t - (K - 1) + j].  Returns (y, the new tail)."""
+    taps = w.shape[1]
+    line = np.concatenate([tail, u])
+    y = np.zeros_like(u)
+    for t in range(u.shape[0]):
+        for j in range(taps):
+            y[t] += w[:, j] * line[t + j]
+    return y, line[line.shape[0] - (taps - 1):]
+
+
+def query_temperature(positions, coef, every):
+    return 1.0 + coef * np.log(np.floor((np.asarray(positions, np.float64) + 1.0) / every) + 1.0)
+
+
+def distance_slopes(heads):
+    return 2.0 ** (-8.0 * (np.arange(heads) + 1.0) / heads)
+
+
+def window_attention(q, k, v, first, window, scale, slopes):
+    """q [T, H, D] at positions first, first + 1, ...; k [n, G, D], v [n, G, V] of positions 0 .. n - 1; head h reads key/value head
+    h // (H / G).  Position i sees the last ``window`` positions up to i itself; score = q . k * scale - slope_h * (i - j)."""
+    H, G = q.shape[1], k.shape[1]
+    out = np.zeros((q.shape[0], H, v.shape[2]), q.dtype)
+    for t in range(q.shape[0]):
+        i = first + t
+        seen = np.arange(max(0, i - window + 1), i + 1)
+        for h in range(H):
+            g = h // (H // G)
+            s = k[seen, g] @ q[t, h] * scale - slopes[h] * (i - seen)
+            w = np.exp(s - s.max())
+            out[t, h] = (w / w.sum()) @ v[seen, g]
+    return out
+
+
+def attention_mixer(h, p, m, st, source):
+    """st: {"n": positions seen, "tails": {"q" | "k" | "v": rows}, "k": [n, G, D], "v": [n, G, V]}; source: the state whose keys and
+    values are read (st itself, or that of the layer named by "kv_from", which has run on the same tokens)."""
+    T, H, G, D, V = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+    first = st["n"]
+
+    def projected(name):
+        y, st["tails"][name] = short_convolution(h @ p[name].T, p[name + ".conv"], st["tails"][name])
+        return y
+
+    q = projected("q").reshape(T, H, D) * query_temperature(first + np.arange(T), m["q_temp"]["coef"], m["q_temp"]["every"])[:, None, None]
+    if source is st:
+        st["k"] = np.concatenate([st["k"], projected("k").reshape(T, G, D)])
+        st["v"] = np.concatenate([st["v"], projected("v").reshape(T, G, V)])
+    st["n"] = first + T
+    o = window_attention(q, source["k"], source["v"], first, m["mask"]["size"], m["scale"], distance_slopes(H))
+    return (o.reshape(T, H * V) * sigmoid(h @ p["g"].T)) @ p["o"].T
+
+
+def relu_mlp(h, p):
+    return (np.maximum(h @ p["gate"].T, 0.0) * (h @ p["up"].T)) @ p["down"].T
+
+
+def token_side(x, e, p, eps):
+    """The per-layer token input: e [T, dim] is the layer's part of the tokens' rows in the side table."""
+    y = (gelu_tanh(x @ p["gate"].T) * e) @ p["proj"].T
+    return x + rms_norm(y, p["norm"], eps)
+
+
 class LayeredOracle:
     """config: the dictionary of config.json; params: {tensor name: array}.  ``feed`` runs the next tokens of the sequence."""
 
@@ -127,6 +198,10 @@ class LayeredOracle:
             m = la["mixer"]
             if la["type"] == "gla":
                 self.states.append(np.zeros((m["heads"], m["dim"], m["vdim"]), self.dtype))
+            elif la["type"] == "attention":
+                G, D, V = m["kv_heads"], m["dim"], m["vdim"]
+                self.states.append({"n": 0, "k": np.zeros((0, G, D), self.dtype), "v": np.zeros((0, G, V), self.dtype),
+                                    "tails": {n: np.zeros((m["conv"] - 1, c), self.dtype) for n, c in (("q", m["heads"] * D), ("k", G * D), ("v", G * V))}})
             elif la["type"] == "latent_attention":
                 self.states.append({"c": np.zeros((0, m["kv_rank"]), self.dtype), "kr": np.zeros((0, m["rot_dim"]), self.dtype)})
             else:
@@ -137,6 +212,23 @@ class LayeredOracle:
         return {k[n:]: v for k, v in self.p.items() if k.startswith(prefix)}
 
     def feed(self, tokens, taps=None):
+        return self._feed_bulidra(np.asarray(tokens), taps) if self.c["architecture"] == "Bulidra" else self._feed_tolevik(tokens, taps)
+
+    def _feed_bulidra(self, tokens, taps):
+        eps, dim = self.c["norm"]["eps"], self.c["token_side"]["dim"]
+        x = self.p["embed"][tokens] * self.c["embedding"]["scale"]
+        for i, la in enumerate(self.c["layers"]):
+            m, st = la["mixer"], self.states[i]
+            h = rms_norm(x, self.p[f"l{i}.norm1"], eps)
+            y = attention_mixer(h, self._sub(f"l{i}.mix."), m, st, self.states[m["kv_from"]] if "kv_from" in m else st)
+            if la["mlp"] is not None:
+                y = y + relu_mlp(h, self._sub(f"l{i}.mlp."))
+            x = token_side(x + y, self.p["side.embed"][tokens][:, i * dim:(i + 1) * dim], self._sub(f"l{i}.side."), eps)
+            if taps is not None:
+                taps.append(x)
+        return rms_norm(x, self.p["final.norm"], eps) @ self.p["embed"].T
+
+    def _feed_tolevik(self, tokens, taps):
         eps = self.c["norm"]["eps"]
         x = self.p["embed"][np.asarray(tokens)]
         for i, la in enumerate(self.c["layers"]):

@@ -20,7 +20,13 @@ class GptConfig(C.Structure):
 class LayerConfig(C.Structure):
     _fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("decay_rank", C.c_int32), ("tau", C.c_float),
                 ("rot_dim", C.c_int32), ("rope_dims", C.c_int32), ("kv_rank", C.c_int32), ("q_rank", C.c_int32), ("scale", C.c_float),
-                ("rope_base", C.c_double), ("mlp", C.c_int32), ("d_ff", C.c_int32)]
+                ("rope_base", C.c_double), ("mlp", C.c_int32), ("d_ff", C.c_int32),
+                ("mlp_act", C.c_int32), ("mlp_bias", C.c_int32), ("kv_heads", C.c_int32), ("kv_shared", C.c_int32), ("kv_from", C.c_int32), ("window", C.c_int32),
+                ("conv_taps", C.c_int32), ("distance_bias", C.c_int32), ("out_gate", C.c_int32), ("q_temp_coef", C.c_double), ("q_temp_every", C.c_double)]
+
+
+class LayeredOptions(C.Structure):
+    _fields_ = [("block", C.c_int32), ("tied_head", C.c_int32), ("side_dim", C.c_int32), ("embed_scale", C.c_float)]
 
 
 ALLREDUCE_FN = C.CFUNCTYPE(C.c_int, C.c_void_p, C.c_size_t, C.c_int, C.c_void_p, C.c_void_p)
@@ -95,7 +101,7 @@ EXT_SYMBOLS = {
     "sptorch_ext_attention_workspace": (_sz, [_sz, _sz, _sz, _sz, _i]),
     "sptorch_ext_attention_causal": (_i, [_vp, _vp, _vp, _vp, _vp, _sz, _sz, _sz, _sz, _sz, _i]),
     "sptorch_ext_gpt_create": (_vp, [C.POINTER(GptConfig)]),
-    "sptorch_ext_layered_create": (_vp, [C.POINTER(GptConfig), C.POINTER(LayerConfig), _i]),
+    "sptorch_ext_layered_create": (_vp, [C.POINTER(GptConfig), C.POINTER(LayerConfig), _i, C.POINTER(LayeredOptions)]),
     "sptorch_ext_gpt_destroy": (None, [_vp]),
     "sptorch_ext_gpt_set_param": (_i, [_vp, C.c_char_p, _vp, _sz]),
     "sptorch_ext_gpt_logits_ld": (_sz, [_vp]),

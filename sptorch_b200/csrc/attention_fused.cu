@@ -27,6 +27,9 @@
 // position `first` > 0 behind cached keys, values may be narrower or wider than the keys, and head h's output carries the factor
 // sigmoid(gate_h).  There the softmax weights enter P V as the sum of two bf16 numbers (PSPLIT: 16 mantissa bits instead of 8; the
 // second half sits in the score columns the first leaves free), so that the weights keep close to f32 precision.
+// And window attention (WIN; window_attention.cu): several query heads read one key/value head, row i sees the last `window` keys up to
+// its own, a score carries the distance bias - slope_h (i - j), and the output is multiplied element by element with a sigmoid.  A work
+// item then starts at the first key tile that query tile 0 sees; query tile 1 starts one tile later when it sees nothing of that one.
 // Algorithmic work per (sequence, head): 2 * T(T+1) * hd FLOP; HBM traffic: Q, K, V read once per query tile
 // (K/V re-reads hit L2 thanks to the work schedule below), O written once.
 #include "gemm.h"
@@ -57,8 +60,10 @@ struct AttnParams {
     int V;                  // width of a head's output in memory (at most the template's VD)
     int n_ptiles;           // 256-row query tile pairs per sequence
     float scale_log2;       // factor of the scores * log2(e)
-    const __nv_bfloat16* gate;      // when given: head h of token m is multiplied by sigmoid(gate[m * ld_gate + h])
-    long long ld_gate;
+    const __nv_bfloat16* gate;      // when given: head h of token m is multiplied by sigmoid(gate[m * ld_gate + h]); WIN: element by
+    long long ld_gate;              // element, laid out like out (and may be out)
+    int group, window;              // WIN: query heads per key/value head; keys a row sees
+    const float* slopes;            // WIN: [H] or null
     uint32_t* status;
     const int* sched;       // work schedule [sched_len][gridDim.x]: item of CTA c at step k, -1 past the end of its list; null: items c, c + grid, ..
     int sched_len;
@@ -147,7 +152,7 @@ struct AttnSmem {
 // Persistent kernel: CTA c works through column c of a schedule built on the host (attention_schedule below), and all
 // roles run straight through item boundaries (barrier phases are driven by running counters), so the loads and the
 // first Q K^T of the next item are in flight while the current one drains.
-template <int KBN, int KBR, int VD, bool ROTP, bool PSPLIT>
+template <int KBN, int KBR, int VD, bool ROTP, bool PSPLIT, bool WIN = false>
 __global__ void __launch_bounds__(kAttnThreads, 1)
 attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQr, const __grid_constant__ CUtensorMap tmKr,
@@ -222,14 +227,21 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const int at = k * (int)gridDim.x + (int)blockIdx.x;
         return p.sched ? __ldg(p.sched + at) : at < p.n_ptiles * BH ? at : -1;
     };
-    // work item -> (first query row, sequence, head, key tiles of query tile 0 and of query tile 1)
-    auto decode = [&](int item, int& q0, int& bb, int& hh, int& n0, int& n1) {
+    // work item -> (first query row, sequence, head, key tiles of query tile 0 and of query tile 1).  WIN: js is the item's first key tile,
+    // n0 and n1 count from there, and d1 is 1 when query tile 1 has no part in tile js.
+    auto decode = [&](int item, int& q0, int& bb, int& hh, int& n0, int& n1, int& js, int& d1) {
         const int pt = p.n_ptiles - 1 - item / BH;
         const int bh = item % BH;
         bb = bh / p.H; hh = bh % p.H;
         q0 = pt * kQPair;
         n0 = min((p.first + q0 + kQTile - 1) / kKvTile + 1, n_kv_seq);    // causal: keys 0 .. first+q0+127
         n1 = (q0 + kQTile < p.T) ? min((p.first + q0 + 2 * kQTile - 1) / kKvTile + 1, n_kv_seq) : 0;   // second tile exists only inside the sequence
+        js = 0; d1 = 0;
+        if constexpr (WIN) {
+            js = max(0, p.first + q0 - p.window + 1) / kKvTile;
+            n0 -= js;
+            if (n1 > 0) { n1 -= js; d1 = max(0, p.first + q0 + kQTile - p.window + 1) / kKvTile > js ? 1 : 0; }
+        }
     };
 
     if (warp == 0) {
@@ -240,10 +252,10 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         uint32_t g = 0, it = 0;
         for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
             const int item_next = fetch(k + 1);
-            int q0, bb, hh, n0, n1;
-            decode(item, q0, bb, hh, n0, n1);
+            int q0, bb, hh, n0, n1, js, d1;
+            decode(item, q0, bb, hh, n0, n1, js, d1);
             item = item_next;
-            const int nmax = max(n0, n1);
+            const int nmax = max(n0, n1), kh = WIN ? hh / p.group : hh;
             ok = mbar_wait(q_free, (it & 1) ^ 1, abort_flag, p.status, kErrProducerWait);
             if (!ok) break;
             if (lane == 0) {
@@ -263,7 +275,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (lane == 0) {
                         const uint32_t dst = base + L::kK + s * L::kKBytes;
                         mbar_expect_tx(k_full + 8 * s, L::kKBytes);
-                        for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, k_full + 8 * s, kb * 64, j * kKvTile, hh, bb);
+                        for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, k_full + 8 * s, kb * 64, (js + j) * kKvTile, kh, bb);
                         for (int kb = 0; kb < KBR; kb++) tma_load_4d(dst + (KBN + kb) * (kKvTile * 128), &tmKr, k_full + 8 * s, kb * 64, j * kKvTile, 0, bb);
                     }
                     __syncwarp();
@@ -275,7 +287,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (lane == 0) {
                         const uint32_t dst = base + L::kV + s * L::kVBytes;
                         mbar_expect_tx(v_full + 8 * s, L::kVBytes);
-                        for (int kb = 0; kb < VD / 64; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmV, v_full + 8 * s, kb * 64, (j - 1) * kKvTile, hh, bb);
+                        for (int kb = 0; kb < VD / 64; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmV, v_full + 8 * s, kb * 64, (js + j - 1) * kKvTile, kh, bb);
                     }
                     __syncwarp();
                 }
@@ -342,11 +354,12 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             };
             for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
                 const int item_next = fetch(k + 1);
-                int q0, bb, hh, n0, n1;
-                decode(item, q0, bb, hh, n0, n1);
+                int q0, bb, hh, n0, n1, js, d1;
+                decode(item, q0, bb, hh, n0, n1, js, d1);
                 item = item_next;
-                const int E = n0 + n1, nmin = min(n0, n1), t_long = n1 > n0 ? 1 : 0;
+                const int E = n0 + n1 - d1, nmin = min(n0, n1), t_long = n1 > n0 ? 1 : 0;
                 auto entry = [&](int e, int& t, int& j) {
+                    if (WIN && e > 0) e += d1;              // (tile 1, key tile 0) is left out
                     if (e < 2 * nmin) { j = e >> 1; t = e & 1; } else { j = nmin + (e - 2 * nmin); t = t_long; }
                 };
                 ok = mbar_wait(q_full, it & 1, abort_flag, p.status, kErrMmaWait);
@@ -374,14 +387,14 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     const uint32_t n = G + e, buf = n % 3;
                     ok = mbar_wait(p_full + 8 * buf, (n / 3) & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == 0) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == (t ? d1 : 0)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
                     if (ok && j > v_seen) { ok = v_ready(g + j); v_seen = j; }
                     if (!ok) break;
                     tc_fence_after();
                     int tn = 0, jn = -1;
                     if (e + 1 < E) entry(e + 1, tn, jn);
                     if (elect_one_sync()) {
-                        issue_pv3(t, g + j, n, j > 0, steps[t]);
+                        issue_pv3(t, g + j, n, j > (t ? d1 : 0), steps[t]);
                         if (jn != j) mma_commit(v_empty + 8 * ((g + j) % NSV));     // every MMA that reads these values has been issued
                     }
                     __syncwarp();
@@ -393,8 +406,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         } else
         for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
             const int item_next = fetch(k + 1);
-            int q0, bb, hh, n0, n1;
-            decode(item, q0, bb, hh, n0, n1);
+            int q0, bb, hh, n0, n1, js, d1;
+            decode(item, q0, bb, hh, n0, n1, js, d1);
             item = item_next;
             const int nt[2] = {n0, n1};
             const int nmax = max(n0, n1);
@@ -404,7 +417,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             tc_fence_after();
             if (elect_one_sync()) {
                 issue_s(0, g);
-                if (n1 > 0) issue_s(1, g);
+                if (n1 > 0 && d1 == 0) issue_s(1, g);
                 if (nt[last_t] == 1) mma_commit(q_free);
                 mma_commit(k_empty + 8 * (g % NSK));
             }
@@ -414,14 +427,23 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 if (!ok) break;
                 for (int t = 0; t < 2 && ok; t++) {
                     if (j >= nt[t]) continue;
+                    if (WIN && t == 1 && j < d1) {             // nothing of this key tile: only the scores of the next one
+                        if (elect_one_sync()) {
+                            tc_fence_after();
+                            issue_s(1, g + 1);
+                            if (last_t == 1 && nt[1] == 2) mma_commit(q_free);
+                        }
+                        __syncwarp();
+                        continue;
+                    }
                     ok = mbar_wait(p_full + 8 * t, steps[t] & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == 0) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == (t ? d1 : 0)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
                     if (!ok) break;
                     steps[t]++;
                     tc_fence_after();
                     if (elect_one_sync()) {
-                        issue_pv(t, g, j > 0, steps[t] - 1);
+                        issue_pv(t, g, j > (t ? d1 : 0), steps[t] - 1);
                         // the next scores of this tile go into the columns P was just read from: the tensor pipe runs the
                         // MMAs of one thread in order, so the product above has consumed P before these overwrite it
                         if (j + 1 < nt[t]) {
@@ -450,23 +472,28 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         uint32_t G = 0;                                          // ROT: scores of earlier items (both tiles), as the MMA warp counts them
         for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
             const int item_next = fetch(k + 1);
-            int q0, bb, hh, n0, n1;
-            decode(item, q0, bb, hh, n0, n1);
+            int q0, bb, hh, n0, n1, js, d1;
+            decode(item, q0, bb, hh, n0, n1, js, d1);
             item = item_next;
             const int n_kv = t == 0 ? n0 : n1;
             const int qrow = q0 + t * kQTile + r;
-            float m = -INFINITY, l = 0.0f;
-            for (int j = 0; j < n_kv && ok; j++, step++) {
+            // WIN: kUnseen until the row's first visible key (masked scores are -inf: their weights and sums are then zeros)
+            constexpr float kUnseen = -1e30f;
+            float m = WIN ? kUnseen : -INFINITY, l = 0.0f;
+            const int j_first = t == 1 ? d1 : 0;
+            const float slope = WIN && p.slopes ? __ldg(p.slopes + hh) * 1.4426950408889634f : 0.0f;
+            for (int j = j_first; j < n_kv && ok; j++, step++) {
                 // ROT: this step's scores are number G + (entries of the item before (t, j)) of the kernel, in buffer number % 3
-                const uint32_t sn = ROT ? G + (uint32_t)(min(j, n0) + min(j, n1) + ((t == 1 && j < n0) ? 1 : 0)) : step;
+                const uint32_t sn = ROT ? G + (uint32_t)(min(j, n0) + min(j, n1) + ((t == 1 && j < n0) ? 1 : 0) - (WIN && j > 0 ? d1 : 0)) : step;
                 const uint32_t sbuf = ROT ? sn % 3 : (uint32_t)t;
                 const uint32_t s_addr = tmem_base + lane_off + sbuf * 128;          // scores, and P over their first 64 columns
                 ok = mbar_wait(s_full + 8 * sbuf, (ROT ? sn / 3 : sn) & 1, abort_flag, p.status, kErrEpilogueWait);
                 if (!ok) break;
                 tc_fence_after();
                 // row r of the tile sees the keys of this tile up to column r + delta
-                const int delta = p.first + q0 + t * kQTile - j * kKvTile;
-                const bool diag = delta < kKvTile - 1;
+                const int delta = p.first + q0 + t * kQTile - (js + j) * kKvTile;
+                // ... and (WIN) from column r + delta - window + 1 on
+                const bool diag = delta < kKvTile - 1 || (WIN && delta > p.window - kQTile);
                 // The 128 scores of the row are taken in four chunks of 32: the load of chunk c + 1 is in flight while chunk c is
                 // worked on, and a chunk needs only 32 registers.  The reference maximum m of the row is allowed to lag the true
                 // maximum by up to 2^8 (lazy rescaling): a chunk whose maximum exceeds m by more moves m, and everything already
@@ -474,7 +501,9 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 // written -- is multiplied by 2^(old - new) at that moment.  tcgen05.ld / st are warp-wide, so a warp rescales when any
                 // of its rows does (the others multiply by one).
                 float2 sum_a = make_float2(0.0f, 0.0f), sum_b = make_float2(0.0f, 0.0f);
-                const float2 c2 = make_float2(p.scale_log2, p.scale_log2);
+                // WIN: the scores become scale * s - slope * (r + delta - column) (times log2 e) before anything else is done with them
+                const float mul = WIN ? 1.0f : p.scale_log2;
+                const float2 c2 = make_float2(mul, mul);
                 uint32_t va[32], vb[32];
                 tmem_ld_32x32(s_addr, va);
                 auto chunk = [&](auto c_tag, uint32_t (&v)[32], uint32_t (&vnext)[32], auto diag_tag) -> bool {
@@ -482,9 +511,20 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     constexpr bool DIAG = decltype(diag_tag)::value;
                     tmem_ld_wait();
                     if (c < 3) tmem_ld_32x32(s_addr + (c + 1) * 32, vnext);
+                    if constexpr (WIN) {
+                        const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), sl2 = make_float2(slope, slope);
+                        const float b0 = slope * (float)(c * 32 - r - delta);
+                        const float2 b2 = make_float2(b0, b0);
+#pragma unroll
+                        for (int i = 0; i < 32; i += 2) {
+                            const float2 x = __ffma2_rn(make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), sc2, __ffma2_rn(sl2, make_float2((float)i, (float)(i + 1)), b2));
+                            v[i] = __float_as_uint(x.x); v[i + 1] = __float_as_uint(x.y);
+                        }
+                    }
                     if (DIAG) {
 #pragma unroll
-                        for (int i = 0; i < 32; i++) if (c * 32 + i > r + delta) v[i] = 0xff800000u;       // -inf right of the diagonal
+                        for (int i = 0; i < 32; i++)
+                            if (c * 32 + i > r + delta || (WIN && c * 32 + i <= r + delta - p.window)) v[i] = 0xff800000u;       // -inf right of the diagonal
                     }
                     float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
 #pragma unroll
@@ -495,15 +535,16 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         m3 = max3(m3, __uint_as_float(v[i + 6]), __uint_as_float(v[i + 7]));
                     }
                     const float mx = fmaxf(max3(m0, m1, m2), m3);
-                    if (j == 0 && c == 0) m = mx;                    // the first chunk of a row always holds key 0: finite
-                    const bool grow = (mx - m) * p.scale_log2 > 8.0f;
+                    if constexpr (WIN) { if (m == kUnseen) m = fmaxf(mx, kUnseen); }     // everything accumulated so far is zero: nothing to rescale
+                    else if (j == 0 && c == 0) m = mx;               // the first chunk of a row always holds key 0: finite
+                    const bool grow = (mx - m) * mul > 8.0f;
                     if (__any_sync(0xffffffffu, grow)) {
                         tmem_ld_wait();                          // the next chunk's registers may be moved below: they must have arrived
                         float alpha = 1.0f;
-                        if (grow) { alpha = ex2_approx((m - mx) * p.scale_log2); m = mx; }
+                        if (grow) { alpha = ex2_approx((m - mx) * mul); m = mx; }
                         l *= alpha;
                         sum_a.x *= alpha; sum_a.y *= alpha; sum_b.x *= alpha; sum_b.y *= alpha;
-                        if (j > 0) {
+                        if (j > j_first) {
                             // every product accumulated so far is in place (the commit of step - 1; the next one needs this thread's P)
                             if (!mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait)) return false;
                             __syncwarp();                        // the wait's lanes leave it one by one, the loads below are warp-wide
@@ -552,7 +593,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         tmem_st_wait();
                         // the load of the next chunk was issued before this branch: the wait of the next chunk() call still covers it
                     }
-                    const float mb = m * p.scale_log2;
+                    const float mb = m * mul;
                     const float2 nmb2 = make_float2(-mb, -mb);
                     uint32_t packed[PSPLIT ? 32 : 16];
 #pragma unroll
@@ -586,15 +627,15 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 if (lane == 0) mbar_arrive(p_full + 8 * sbuf);
                 l += (sum_a.x + sum_a.y) + (sum_b.x + sum_b.y);
             }
-            G += (uint32_t)(n0 + n1);
+            G += (uint32_t)(n0 + n1 - d1);
             if (!ok) break;
             if (n_kv > 0) {
                 float inv = 1.0f / l;
-                if (p.gate && qrow < p.T) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[((long long)bb * p.T + qrow) * p.ld_gate + hh])));
+                if (!WIN && p.gate && qrow < p.T) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[((long long)bb * p.T + qrow) * p.ld_gate + hh])));
                 // The item's last product -- after the one before it: scores run up to two ahead, so with a single query tile only the product of
                 // step - 4 is sure to be done here, and a parity wait for step - 1 could not tell step - 3 (same barrier, the phase before)
                 // from step - 1.  The product of step - 2 waits on the other barrier, one phase ahead of step - 4, and brings step - 3 with it.
-                ok = (n_kv < 2 || mbar_wait(pv_done + 8 * (2 * t + (step & 1)), ((step - 2) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait)) &&
+                ok = (n_kv - j_first < 2 || mbar_wait(pv_done + 8 * (2 * t + (step & 1)), ((step - 2) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait)) &&
                      mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait);
                 if (!ok) break;
                 __syncwarp();
@@ -608,7 +649,19 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (qrow < p.T) {
 #pragma unroll
                         for (int i = 0; i < 32; i += 8) {
-                            if (KBR > 0 && c * 32 + i >= p.V) break;
+                            if ((KBR > 0 || WIN) && c * 32 + i >= p.V) break;
+                            if constexpr (WIN) {
+                                if (p.gate) {
+                                    const uint4 graw = *reinterpret_cast<const uint4*>(p.gate + ((long long)bb * p.T + qrow) * p.ld_gate + (long long)hh * p.V + c * 32 + i);
+                                    const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&graw);
+#pragma unroll
+                                    for (int q = 0; q < 4; q++) {
+                                        const float2 gv = bf16x2_to_float2(gh[q]);
+                                        o[i + 2 * q] = __float_as_uint(__uint_as_float(o[i + 2 * q]) * (1.0f / (1.0f + __expf(-gv.x))));
+                                        o[i + 2 * q + 1] = __float_as_uint(__uint_as_float(o[i + 2 * q + 1]) * (1.0f / (1.0f + __expf(-gv.y))));
+                                    }
+                                }
+                            }
                             uint4 w;
                             __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&w);
 #pragma unroll
@@ -745,7 +798,7 @@ int attention_fused(const void* q, const void* k, const void* v, void* out, int 
     if (encode_heads(&tk, k, hd, T, H, B, ld_k, hd, (long long)T * ld_k)) return 1;
     if (encode_heads(&tv, v, hd, T, H, B, ld_v, hd, (long long)T * ld_v)) return 1;
     AttnParams prm;
-    prm.out = (__nv_bfloat16*)out; prm.ld_out = ld_out; prm.T = T; prm.H = H; prm.B = B; prm.n = T; prm.first = 0; prm.V = hd; prm.gate = nullptr; prm.ld_gate = 0;
+    prm.out = (__nv_bfloat16*)out; prm.ld_out = ld_out; prm.T = T; prm.H = H; prm.B = B; prm.n = T; prm.first = 0; prm.V = hd; prm.gate = nullptr; prm.ld_gate = 0; prm.group = 1; prm.window = 0; prm.slopes = nullptr;
     prm.n_ptiles = ceil_div(T, kQPair);
     prm.scale_log2 = (1.0f / sqrtf((float)hd)) * 1.4426950408889634f;
     prm.status = rt().dev_status;
@@ -789,7 +842,7 @@ int attention_latent(const void* q, long long ld_q, const void* kn, const void* 
     if (encode_heads(&tkr, kr, rot, n, 1, B, row, row, seq_stride)) return 1;
     AttnParams prm;
     prm.out = (__nv_bfloat16*)out; prm.ld_out = ld_out; prm.T = T; prm.H = H; prm.B = B; prm.n = n; prm.first = first; prm.V = V;
-    prm.gate = (const __nv_bfloat16*)gate; prm.ld_gate = ld_gate;
+    prm.gate = (const __nv_bfloat16*)gate; prm.ld_gate = ld_gate; prm.group = 1; prm.window = 0; prm.slopes = nullptr;
     prm.n_ptiles = ceil_div(T, kQPair);
     prm.scale_log2 = scale * 1.4426950408889634f;
     prm.status = rt().dev_status;
@@ -809,6 +862,46 @@ int attention_latent(const void* q, long long ld_q, const void* kn, const void* 
     else rc = V <= 64 ? launch(attn_fused_kernel<2, 1, 64, true, true>, AttnSmem<2, 1, 64>::kTotal) : launch(attn_fused_kernel<2, 1, 128, true, true>, AttnSmem<2, 1, 128>::kTotal);
     if (rc) return rc;
     SPT_LAUNCH_CHECK("attention_latent");
+    return 0;
+}
+
+// ---- window attention over cached keys and values ----
+// q: [B*T, H*D]; rows: [B][positions][row] with key head g at columns g*D and value head g at columns G*D + g*V, sequences seq_stride
+// apart, of which positions 0 .. n - 1 are there; gate (null: none) and out: [B*T, ld_out], head h at columns h*V, may be the same.
+bool attention_window_supported(int D, int V, int row, long long ld_out) {
+    return D >= 8 && D <= 128 && D % 8 == 0 && V >= 8 && V <= 128 && V % 8 == 0 && row % 8 == 0 && ld_out % 8 == 0;
+}
+
+int attention_window(const void* q, const void* rows, int row, long long seq_stride, void* out, long long ld_out, const void* gate, int B, int T, int n, int H, int G,
+                     int D, int V, int first, int window, const float* slopes, float scale) {
+    CUtensorMap tq, tk, tv;
+    if (encode_heads(&tq, q, D, T, H, B, (long long)H * D, D, (long long)T * H * D)) return 1;
+    if (encode_heads(&tk, rows, D, n, G, B, row, D, seq_stride)) return 1;
+    if (encode_heads(&tv, (const __nv_bfloat16*)rows + (size_t)G * D, V, n, G, B, row, V, seq_stride)) return 1;
+    AttnParams prm;
+    prm.out = (__nv_bfloat16*)out; prm.ld_out = ld_out; prm.T = T; prm.H = H; prm.B = B; prm.n = n; prm.first = first; prm.V = V;
+    prm.gate = (const __nv_bfloat16*)gate; prm.ld_gate = ld_out; prm.group = H / G; prm.slopes = slopes;
+    const bool all = window <= 0 || window >= n;
+    prm.window = all ? n : window;
+    prm.n_ptiles = ceil_div(T, kQPair);
+    prm.scale_log2 = scale * 1.4426950408889634f;
+    prm.status = rt().dev_status;
+    const long long items = (long long)B * H * prm.n_ptiles;
+    if (items > INT32_MAX) return fail("attention_window: too many work items");
+    const long long slots = compute_sms(), grid = items < slots ? items : slots;
+    prm.sched = nullptr; prm.sched_len = ceil_div(items, grid);
+    // with a window that cuts, the items are nearly alike and the plain order does; otherwise as for latent attention
+    if (all && first == 0 && attention_schedule(B, H, T, (D + V) / 2, prm.n_ptiles, (int)grid, &prm.sched, &prm.sched_len)) return 1;
+    auto launch = [&](auto kern, int smem_bytes) -> int {
+        SPT_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes));
+        kern<<<(unsigned)grid, kAttnThreads, smem_bytes, rt().stream>>>(tq, tk, tv, tq, tk, prm);
+        return 0;
+    };
+    int rc;
+    if (D <= 64) rc = V <= 64 ? launch(attn_fused_kernel<1, 0, 64, true, true, true>, AttnSmem<1, 0, 64>::kTotal) : launch(attn_fused_kernel<1, 0, 128, true, true, true>, AttnSmem<1, 0, 128>::kTotal);
+    else rc = V <= 64 ? launch(attn_fused_kernel<2, 0, 64, true, true, true>, AttnSmem<2, 0, 64>::kTotal) : launch(attn_fused_kernel<2, 0, 128, true, true, true>, AttnSmem<2, 0, 128>::kTotal);
+    if (rc) return rc;
+    SPT_LAUNCH_CHECK("attention_window");
     return 0;
 }
 

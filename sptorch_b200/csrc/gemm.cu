@@ -382,7 +382,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                     }
                     continue;
                 }
-                if (p.epilogue == EPI_GELU) {
+                if (p.epilogue == EPI_GELU || p.epilogue == EPI_GELU_MUL) {
                     if constexpr (sizeof(TOut) == 2) {
 #pragma unroll
                         for (int j = 0; j < 32; j += 2) { float2 y = gelu_fast2(make_float2(f[j], f[j + 1])); f[j] = y.x; f[j + 1] = y.y; }
@@ -393,9 +393,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
                 } else if (p.epilogue == EPI_SWIGLU) {
 #pragma unroll
                     for (int j = 0; j < 32; j++) f[j] = sizeof(TOut) == 2 ? silu_fast(f[j]) : silu_exact(f[j]);
+                } else if (p.epilogue == EPI_RELU_MUL) {
+#pragma unroll
+                    for (int j = 0; j < 32; j++) f[j] = fmaxf(f[j], 0.0f);
                 }
-                if (rbase && p.epilogue == EPI_SWIGLU) {
-                    // the R operand is the other factor: x * (g * sigmoid(g))
+                if (rbase && epilogue_multiplies(p.epilogue)) {
+                    // the R operand is the other factor: x * act(g)
                     if constexpr (sizeof(TOut) == 2) {
 #pragma unroll
                         for (int k = 0; k < NV; k++) {
@@ -572,7 +575,7 @@ bool gemm_supported(const GemmDesc& d, const char** why) {
     auto bad = [&](const char* w) { if (why) *why = w; return false; };
     if (d.mode != MM_TF32 && d.mode != MM_BF16) return bad("mode is not a tensor-core mode");
     if (d.M <= 0 || d.N <= 0 || d.K <= 0) return bad("empty problem");
-    if (d.group) return bad("block-diagonal products run on the weight-streaming kernel only");
+    if (d.group || d.act_off || d.C2) return bad("block-diagonal products, products with an activation on A and second outputs run on the weight-streaming kernel only");
     if ((reinterpret_cast<uintptr_t>(d.A) & 15) || (reinterpret_cast<uintptr_t>(d.B) & 15)) return bad("operand base not 16-byte aligned");
     if ((d.lda * es) % 16 || (d.ldb * es) % 16) return bad("operand row pitch not a multiple of 16 bytes");
     if (d.nb1 > 1 && ((d.sA1 * es) % 16 || (!d.b_broadcast && (d.sB1 * es) % 16))) return bad("batch stride not a multiple of 16 bytes");
@@ -868,8 +871,9 @@ __global__ void __launch_bounds__(256) simt_matmul_kernel(const float* __restric
             if (gm < M && gn < N) {
                 float v = acc[i][j] * alpha;
                 if (bias) v += bias[gn];
-                if (epilogue == EPI_GELU) v = gelu_exact(v);
-                if (epilogue == EPI_SWIGLU) { const float s_ = 1.0f / (1.0f + expf(-v)); v = R ? (R[(size_t)gm * st.ldc + gn] * v) * s_ : v * s_; }
+                if (epilogue == EPI_GELU || epilogue == EPI_GELU_MUL) v = gelu_exact(v);
+                if (epilogue == EPI_RELU_MUL || epilogue == EPI_GELU_MUL) v = (epilogue == EPI_RELU_MUL ? fmaxf(v, 0.0f) : v) * (R ? R[(size_t)gm * st.ldc + gn] : 1.0f);
+                else if (epilogue == EPI_SWIGLU) { const float s_ = 1.0f / (1.0f + expf(-v)); v = R ? (R[(size_t)gm * st.ldc + gn] * v) * s_ : v * s_; }
                 else if (R) v += R[(size_t)gm * st.ldc + gn];
                 C[(size_t)gm * st.ldc + gn] = v;
             }

@@ -7,7 +7,9 @@ namespace spt {
 
 enum MMMode : int { MM_TF32 = 0, MM_BF16 = 1, MM_F32 = 2 };
 // EPI_SWIGLU: C = R * g * sigmoid(g) with g = alpha * A B^T + bias (R is the other factor of the reference's swiglu(x, gate), not a residual)
-enum Epilogue : int { EPI_NONE = 0, EPI_GELU = 1, EPI_SWIGLU = 2 };
+// EPI_RELU_MUL, EPI_GELU_MUL: the same with max(g, 0) and with tanh-GELU of g
+enum Epilogue : int { EPI_NONE = 0, EPI_GELU = 1, EPI_SWIGLU = 2, EPI_RELU_MUL = 3, EPI_GELU_MUL = 4 };
+__host__ __device__ constexpr bool epilogue_multiplies(int e) { return e >= EPI_SWIGLU; }       // R is a factor, not a residual
 
 // C[z][m,n] = act(alpha * sum_k A[z][m,k] * B[z][n,k] + bias[n]) + R[z][m,n]
 // Both operands are K-major (k contiguous).  z = z1 + nb1*z2 enumerates two batch dimensions with
@@ -55,6 +57,11 @@ struct GemmDesc {
     long long group_a = 0, group_c = 0;
     const void* gate = nullptr;
     long long ld_gate = 0;
+    // Weight-streaming kernel only.  act_off: from column act_from of A on, an element a stands for a * max(A[. + act_off], 0) (a gated
+    // feed-forward whose two halves lie side by side in A).  C2: bf16 copy of an f32 output, laid out like C.
+    int act_from = 0;
+    long long act_off = 0;
+    void* C2 = nullptr;
 };
 inline int gemm_reduce_parts(int N) { return 2 * ((N + 255) / 256); }
 

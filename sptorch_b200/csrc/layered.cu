@@ -1,12 +1,17 @@
 // layered.cu -- driver of the models built from a list of layers.  Each layer has its own mixer (gated linear attention, latent
-// attention), sizes and optional feed-forward, and normalises the OUTPUT of a sublayer before it joins the residual stream:
-//   x <- x + rms(mixer(x)) w1;   x <- x + rms(mlp(x)) w2;   logits = head (rms(x) wf)
-// The residual stream x is f32; the sublayers read a copy of it in the model dtype (xb), which the kernel that updates x writes beside
+// attention, window attention), sizes and optional feed-forward.  Two ways of joining the residual stream (sptorch_layered_options):
+//   post-norm:  x <- x + rms(mixer(x)) w1;   x <- x + rms(mlp(x)) w2
+//   parallel:   h = rms(x) w1;   x <- x + mixer(h) + mlp(h);   and, with a per-layer token input e,
+//               x <- x + rms(proj (gelu(gate x) e)) ws
+// and logits = head (rms(x) wf).  The residual stream x is f32; the sublayers read a copy of it in the model dtype (xb), which the kernel that updates x writes beside
 // it.  Launches of a prompt (bf16), per layer:
 //   gated linear attention: one GEMM for q, k, v, gate and decay latent | chunk kernels (gla.cu) | W_o | post-norm
 //   latent attention: one GEMM for query latent, key/value latent and head gates | latent norms and rotation | W_uq | rotation of q |
 //                     keys and values of every position from the latents (one GEMM) | fused attention | W_o | post-norm
 //   feed-forward: W_up (+bias) | W_gate (+bias, SwiGLU product) | W_down (+bias) | post-norm
+//   parallel block with window attention: one GEMM for q, k, v, gate of the heads and W_up | W_gate (activation, product with up in place) |
+//                     convolutions, cached rows | ring | fused attention (gates in place) | one GEMM for W_o and W_down (+ f32 residual) |
+//                     side: bf16 copy of x | gate (gelu, product with e in place) | proj | post-norm together with the next layer's norm
 // A few tokens (a decode step, a short portion of a prompt) take the weight-streaming projections, the token-by-token recurrence and
 // attention over the cached latents themselves; all of these are programmatic dependents of one another, and with one or two rows the
 // projection behind a sublayer does the post-norm on the way.
@@ -23,13 +28,17 @@ namespace spt {
 bool attention_latent_supported(int D, int rot, int V, int kv_off, long long ld_q, long long ld_kv, int row);
 int attention_latent(const void* q, long long ld_q, const void* kn, const void* v, long long ld_kv, const void* kr, long long row, long long seq_stride,
                      void* out, long long ld_out, const void* gate, long long ld_gate, int B, int T, int n, int H, int D, int rot, int V, int first, float scale);
+bool attention_window_supported(int D, int V, int row, long long ld_out);
+int attention_window(const void* q, const void* rows, int row, long long seq_stride, void* out, long long ld_out, const void* gate, int B, int T, int n, int H, int G,
+                     int D, int V, int first, int window, const float* slopes, float scale);
 
 namespace {
 
-// x = embed[id] in f32 and in the model dtype; an id outside the vocabulary gives a zero row and raises the status word
+// x = embed[id] * scale in f32 and in the model dtype, and the token's row of the side table (side_ld values, 0: none); an id outside the
+// vocabulary gives zero rows and raises the status word
 template <typename T>
 __global__ void __launch_bounds__(128) embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x, T* __restrict__ xb, int vocab,
-                                                         int ld, uint32_t* status) {
+                                                         int ld, float scale, const T* __restrict__ side_table, T* __restrict__ side, int side_ld, uint32_t* status) {
     pdl_release();
     pdl_acquire();
     const int m = blockIdx.x, id = ids[m];
@@ -37,10 +46,12 @@ __global__ void __launch_bounds__(128) embed_rows_kernel(const T* __restrict__ t
     if (!ok && threadIdx.x == 0) atomicOr(status, 0x100u);
     const T* src = table + (size_t)(ok ? id : 0) * ld;
     for (int i = threadIdx.x; i < ld; i += 128) {
-        const T v = ok ? src[i] : (T)0.0f;
-        x[(size_t)m * ld + i] = (float)v;
-        xb[(size_t)m * ld + i] = v;
+        const float v = ok ? (float)src[i] * scale : 0.0f;
+        x[(size_t)m * ld + i] = v;
+        xb[(size_t)m * ld + i] = (T)v;
     }
+    const T* sr = side_table + (size_t)(ok ? id : 0) * side_ld;
+    for (int i = threadIdx.x; i < side_ld; i += 128) side[(size_t)m * side_ld + i] = ok ? sr[i] : (T)0.0f;
 }
 
 __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
@@ -178,7 +189,7 @@ int ensure(Gpt* g, LayeredScratch* s, size_t bytes) {
     return sptorch_ext_memset(s->p, 0, bytes);
 }
 
-// out[M, N] = act(a W^T + bias) (* r for the SwiGLU product); rows of a are lda apart and read for K elements, W is [N, ldw]
+// out[M, N] = act(a W^T + bias) (* r for the gated products); rows of a are lda apart and read for K elements, W is [N, ldw]
 // pend (few rows only, may be null): a is the residual stream completed on the fly; *fused tells whether that was possible, otherwise
 // nothing was launched
 int product(Gpt* g, bool few, const void* a, long long lda, const void* w, long long ldw, int K, const float* bias, const void* r, void* out, long long ldo,
@@ -195,6 +206,15 @@ int product(Gpt* g, bool few, const void* a, long long lda, const void* w, long 
     }
     if (few && linear_few_rows_supported(d)) { ProfScope ps(PROF_LINEAR); return linear_few_rows(d, nullptr, true); }
     return gemm_or_simt(d);
+}
+
+// x[M, d8] += a W^T, x f32; rows of a are lda apart, W is [d8, ldw].  Few rows: act_off as in GemmDesc, and xb gets a bf16 copy.
+GemmDesc stream_product(Gpt* g, const void* a, long long lda, const void* w, long long ldw, int K, float* x, int M) {
+    GemmDesc d;
+    d.A = a; d.B = w; d.C = x; d.R = x;
+    d.M = M; d.N = g->lay->d8; d.K = K; d.lda = lda; d.ldb = ldw; d.ldc = d.N;
+    d.mode = g->c.dtype == BF16 ? MM_BF16 : MM_F32; d.out_dtype = F32;
+    return d;
 }
 
 GlaArgs gla_args(Gpt* g, const LayeredLayer& w, int B, int T, bool cached) {
@@ -277,20 +297,113 @@ int latent_layer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const i
                             a.out, a.ld_out, (const uint8_t*)a.in + (size_t)a.c_g * 2, a.ld_in, B, T, n, a.H, a.D, a.rot, a.V, first, a.scale);
 }
 
+const LayeredLayer& kv_layer(const Gpt* g, const LayeredLayer& w) { return w.own_kv() ? w : g->lay->L[w.c.kv_from]; }
+
+WindowArgs window_args(Gpt* g, const LayeredLayer& w, int B, int T, int first, const int* pos_dev, bool cached) {
+    const LayeredLayer& kv = kv_layer(g, w);
+    uint8_t* in = (uint8_t*)g->lay->in.p;
+    WindowArgs a = {};
+    a.in = in; a.ld_in = w.n_in; a.c_q = w.c_q; a.c_k = w.c_k; a.c_v = w.c_v;
+    a.B = B; a.T = T; a.H = w.c.heads; a.G = w.c.kv_heads; a.D = w.c.dim; a.V = w.c.vdim; a.D8 = pad8(a.D); a.V8 = pad8(a.V);
+    a.taps = w.c.conv_taps; a.conv = w.conv; a.temp = w.temp; a.slopes = w.slopes;
+    a.first = first; a.pos_dev = pos_dev; a.scale = w.c.scale; a.window = w.c.window;
+    a.own_kv = w.own_kv();
+    a.ring = cached ? w.ring : nullptr; a.ring_cols = w.c_g;
+    a.rows = cached ? kv.rows : kv.kv_read ? kv.own.p : g->lay->rows.p;
+    a.row = kv.row(); a.capacity = cached ? g->cache_ctx : T; a.seq_stride = (long long)a.capacity * a.row;
+    a.q = g->lay->q.p;
+    a.out = in + (size_t)w.c_g * g->es; a.ld_out = w.n_in; a.gate = w.c.out_gate ? a.out : nullptr;
+    a.dtype = g->c.dtype;
+    return a;
+}
+
+// The heads' outputs land in the gate's columns of the projections' output.
+int window_layer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
+    const WindowArgs a = window_args(g, w, B, T, first, pos_dev, cached);
+    const bool decode = few && cached && window_decode_supported(a), fresh = decode && T == 1;
+    if (!fresh) { ProfScope ps(PROF_LATENT); if (window_prep(a, few)) return 1; }
+    ProfScope ps(PROF_ATTN_FUSED);
+    if (decode) return window_decode(a, fresh, true);
+    if (!few && g->c.dtype == BF16 && attention_window_supported(a.D, a.V, a.row, a.ld_out))
+        return attention_window(a.q, a.rows, a.row, a.seq_stride, a.out, a.ld_out, a.gate, B, T, first + T, a.H, a.G, a.D, a.V, first, a.window, a.slopes, a.scale);
+    return window_plain(a, few);
+}
+
+// Whether a few rows take the feed-forward's activation on the way into W_down: gate and up then come from one product.
+bool act_on_read(const Gpt* g, const LayeredLayer& w, int M) {
+    if (w.c.mlp != SPT_MLP_DENSE || w.c.mlp_act != SPT_ACT_RELU || w.c.mixer != SPT_MIXER_WINDOW) return false;
+    GemmDesc d = stream_product(const_cast<Gpt*>(g), g->lay->in.p, w.n_in, w.w_o, w.o_ld() + pad8(w.c.d_ff), w.o_ld() + pad8(w.c.d_ff), (float*)g->lay->x.p, M);
+    d.act_off = pad8(w.c.d_ff); d.act_from = w.o_ld();
+    return linear_few_rows_supported(d);
+}
+
+int mixer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
+    if (w.c.mixer == SPT_MIXER_GLA) return gla_layer(g, w, B, T, few, cached);
+    if (w.c.mixer == SPT_MIXER_LATENT) return latent_layer(g, w, B, T, first, pos_dev, few, cached);
+    return window_layer(g, w, B, T, first, pos_dev, few, cached);
+}
+// where a mixer leaves the heads' outputs
+const void* mixer_out(const Gpt* g, const LayeredLayer& w, long long* ld) {
+    *ld = w.c.mixer == SPT_MIXER_WINDOW ? w.n_in : w.o_ld();
+    return w.c.mixer == SPT_MIXER_WINDOW ? (const uint8_t*)g->lay->in.p + (size_t)w.c_g * g->es : (const uint8_t*)g->lay->ao.p;
+}
+
+int gated_epilogue(const LayeredLayer& w) { return w.c.mlp_act == SPT_ACT_RELU ? EPI_RELU_MUL : EPI_SWIGLU; }
+
+// A layer of a parallel block.  lay.xb holds rms(x) * norm1; afterwards x lacks only the normed lay.y (when there is a token input).
+int parallel_layer(Gpt* g, const LayeredLayer& w, int l, float* x, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
+    Layered& lay = *g->lay;
+    const int M = B * T, d8 = lay.d8, dense = w.c.mlp == SPT_MLP_DENSE, f8 = dense ? pad8(w.c.d_ff) : 0, o8 = w.o_ld();
+    const bool act = few && act_on_read(g, w, M);
+    uint8_t* in = (uint8_t*)lay.in.p;
+    if (product(g, few, lay.xb.p, d8, w.w_in, d8, d8, nullptr, nullptr, in, w.n_in, M, act ? w.n_in : w.n_in - f8, EPI_NONE)) return 1;
+    void* up = in + (size_t)w.c_up * g->es;
+    if (dense && !act && product(g, few, lay.xb.p, d8, (uint8_t*)w.w_in + (size_t)w.c_gate * d8 * g->es, d8, d8, nullptr, up, up, w.n_in, M, f8, gated_epilogue(w))) return 1;
+    if (mixer(g, w, B, T, first, pos_dev, few, cached)) return 1;
+    const bool side = lay.opt.side_dim > 0;
+    bool copied = false;
+    auto to_stream = [&](const void* a, long long lda, int col, int K, bool last) -> int {
+        GemmDesc d = stream_product(g, a, lda, (const uint8_t*)w.w_o + (size_t)col * g->es, o8 + f8, K, x, M);
+        if (act) { d.act_off = f8; d.act_from = o8; }
+        if (few) {
+            d.C2 = last && side && g->c.dtype == BF16 ? lay.xb.p : nullptr;
+            if (linear_few_rows_supported(d)) { copied = d.C2 != nullptr; ProfScope ps(PROF_LINEAR); return linear_few_rows(d, nullptr, true); }
+            d.C2 = nullptr;
+        }
+        return gemm_or_simt(d);
+    };
+    long long ld_a;
+    const void* a = mixer_out(g, w, &ld_a);
+    if (w.c.mixer == SPT_MIXER_WINDOW) { if (to_stream(a, ld_a, 0, o8 + f8, true)) return 1; }
+    else if (to_stream(a, ld_a, 0, o8, !dense) || (dense && to_stream(up, w.n_in, o8, f8, true))) return 1;
+    if (!side) return 0;
+    const int s8 = lay.side8;
+    const void* xs = x;
+    if (g->c.dtype == BF16) {
+        if (!copied && post_norm_launch(x, nullptr, nullptr, nullptr, nullptr, lay.xb.p, M, g->c.d_model, d8, g->c.eps, BF16, few)) return 1;
+        xs = lay.xb.p;
+    }
+    const long long ld_e = (long long)lay.L.size() * s8;
+    void* e = (uint8_t*)lay.side.p + (size_t)l * s8 * g->es;
+    return product(g, few, xs, d8, w.side_gate, d8, d8, nullptr, e, e, ld_e, M, s8, EPI_GELU_MUL) ||
+           product(g, few, e, ld_e, w.side_proj, s8, s8, nullptr, nullptr, lay.y.p, d8, M, d8, EPI_NONE);
+}
+
 // The launches of one step over B sequences of T new tokens at positions first .. (or pos_dev[0] ..).
 int run(Gpt* g, const void* ids, int B, int T, int first, const int* pos_dev, bool few, bool cached, void* logits, const HeadReduce* hr) {
     const sptorch_gpt_config& c = g->c;
     Layered& lay = *g->lay;
-    const int M = B * T, d8 = lay.d8, dt = c.dtype;
+    const int M = B * T, d8 = lay.d8, dt = c.dtype, side_ld = (int)lay.L.size() * lay.side8;
     float* x = (float*)lay.x.p;
     {
         ProfScope ps(PROF_EMBED);
         // an ordinary launch: it starts when everything before this step is done, so the kernels behind it may read what earlier steps
         // left in the cache before they wait for their predecessor
         if (dt == BF16) SPT_CUDA(launch_dependent(embed_rows_kernel<__nv_bfloat16>, dim3(M), dim3(128), 0, false, 1, (const __nv_bfloat16*)lay.embed, (const int*)ids, x,
-                                                  (__nv_bfloat16*)lay.xb.p, c.vocab, d8, rt().dev_status));
+                                                  (__nv_bfloat16*)lay.xb.p, c.vocab, d8, lay.opt.embed_scale, (const __nv_bfloat16*)lay.side_embed, (__nv_bfloat16*)lay.side.p,
+                                                  side_ld, rt().dev_status));
         else SPT_CUDA(launch_dependent(embed_rows_kernel<float>, dim3(M), dim3(128), 0, false, 1, (const float*)lay.embed, (const int*)ids, x, (float*)lay.xb.p, c.vocab, d8,
-                                       rt().dev_status));
+                                       lay.opt.embed_scale, (const float*)lay.side_embed, (float*)lay.side.p, side_ld, rt().dev_status));
         note_submit();
     }
     auto tap = [&](int i) -> int {
@@ -320,16 +433,25 @@ int run(Gpt* g, const void* ids, int B, int T, int first, const int* pos_dev, bo
         return settle(nullptr) || product(g, few, lay.xb.p, d8, w, d8, d8, bias, nullptr, out, N, M, N, EPI_NONE);
     };
     const int nl = (int)lay.L.size();
-    for (int l = 0; l < nl; l++) {
+    const bool parallel = lay.opt.block == SPT_BLOCK_PARALLEL;
+    if (parallel && nl > 0 && settle(lay.L[0].norm1)) return 1;
+    for (int l = 0; l < nl && parallel; l++) {
+        if (parallel_layer(g, lay.L[l], l, x, B, T, first, pos_dev, few, cached)) return 1;
+        if (lay.opt.side_dim > 0) pending = lay.L[l].side_norm;
+        if (l < nl - 1 && (settle(lay.L[l + 1].norm1) || tap(l + 1))) return 1;       // the next layer's input, too
+    }
+    for (int l = 0; l < nl && !parallel; l++) {
         const LayeredLayer& w = lay.L[l];
         if (project(w.w_in, nullptr, lay.in.p, w.n_in)) return 1;
-        if (w.c.mixer == SPT_MIXER_GLA ? gla_layer(g, w, B, T, few, cached) : latent_layer(g, w, B, T, first, pos_dev, few, cached)) return 1;
-        if (product(g, few, lay.ao.p, w.o_ld(), w.w_o, w.o_ld(), w.o_ld(), nullptr, nullptr, lay.y.p, d8, M, d8, EPI_NONE)) return 1;
+        if (mixer(g, w, B, T, first, pos_dev, few, cached)) return 1;
+        long long ld_a;
+        const void* a = mixer_out(g, w, &ld_a);
+        if (product(g, few, a, ld_a, w.w_o, w.o_ld(), w.o_ld(), nullptr, nullptr, lay.y.p, d8, M, d8, EPI_NONE)) return 1;
         pending = w.norm1;
         if (w.c.mlp == SPT_MLP_DENSE) {
             const int f8 = pad8(w.c.d_ff);
             if (project(w.w_up, w.b_up, lay.f.p, f8)) return 1;
-            if (product(g, few, lay.xb.p, d8, w.w_gate, d8, d8, w.b_gate, lay.f.p, lay.f.p, f8, M, f8, EPI_SWIGLU)) return 1;
+            if (product(g, few, lay.xb.p, d8, w.w_gate, d8, d8, w.b_gate, lay.f.p, lay.f.p, f8, M, f8, gated_epilogue(w))) return 1;
             if (product(g, few, lay.f.p, f8, w.w_down, f8, f8, w.b_down, nullptr, lay.y.p, d8, M, d8, EPI_NONE)) return 1;
             pending = w.norm2;
         }
@@ -352,15 +474,21 @@ int layered_prepare(Gpt* g, int B, int T, int first, bool cached) {
     Layered& lay = *g->lay;
     const size_t M = (size_t)B * T, es = g->es, n = (size_t)first + T;
     const bool few = cached && layered_takes_few_rows(g, (int)M, T);
-    size_t in = 0, ao = 0, cq = 0, q = 0, kv = 0, f = 0, rows = 0, qabs = 0, olat = 0, go = 0, gu = 0, gd = 0;
+    size_t in = 0, ao = 0, cq = 0, q = 0, kv = 0, f = 0, rows = 0, side = 0, qabs = 0, olat = 0, go = 0, gu = 0, gd = 0;
     auto up = [](size_t& a, size_t b) { if (b > a) a = b; };
     for (auto& w : lay.L) {
         up(in, w.n_in); up(ao, w.o_ld());
-        if (w.c.mlp == SPT_MLP_DENSE) up(f, pad8(w.c.d_ff));
+        if (w.c.mlp == SPT_MLP_DENSE && lay.opt.block != SPT_BLOCK_PARALLEL) up(f, pad8(w.c.d_ff));
         if (w.c.mixer == SPT_MIXER_GLA) {
             const GlaArgs a = gla_args(g, w, B, T, cached);
             if (!few && gla_chunked_supported(a)) { up(gu, gla_chunked_state_bytes(a)); up(gd, gla_chunked_decay_bytes(a)); }
             else up(go, M * w.c.heads * w.c.vdim * 4);
+        } else if (w.c.mixer == SPT_MIXER_WINDOW) {
+            up(q, (size_t)w.c.heads * pad8(w.c.dim));
+            if (!cached && w.own_kv()) {
+                if (!w.kv_read) up(rows, w.row());
+                else if (ensure(g, &w.own, M * w.row() * es)) return 1;
+            }
         } else {
             up(cq, pad8(w.c.q_rank)); up(q, w.q_ld());
             if (!cached) up(rows, w.row());
@@ -369,7 +497,8 @@ int layered_prepare(Gpt* g, int B, int T, int first, bool cached) {
         }
     }
     const size_t d8 = lay.d8;
-    return ensure(g, &lay.x, M * d8 * 4) || ensure(g, &lay.x2, M * d8 * 4) || ensure(g, &lay.xb, M * d8 * es) || ensure(g, &lay.y, M * d8 * es) || ensure(g, &lay.in, M * in * es) ||
+    side = lay.L.size() * lay.side8;
+    return ensure(g, &lay.side, M * side * es) || ensure(g, &lay.x, M * d8 * 4) || ensure(g, &lay.x2, M * d8 * 4) || ensure(g, &lay.xb, M * d8 * es) || ensure(g, &lay.y, M * d8 * es) || ensure(g, &lay.in, M * in * es) ||
            ensure(g, &lay.ao, M * ao * es) || ensure(g, &lay.cq, M * cq * es) || ensure(g, &lay.q, M * q * es) || ensure(g, &lay.kv, (size_t)B * n * kv * es) ||
            ensure(g, &lay.f, M * f * es) || ensure(g, &lay.rows, M * rows * es) || ensure(g, &lay.qabs, M * qabs * 4) || ensure(g, &lay.olat, M * olat * 4) ||
            ensure(g, &lay.gla_o, go) || ensure(g, &lay.gla_u, gu) || ensure(g, &lay.gla_dec, gd);
@@ -387,7 +516,13 @@ int layered_enable_cache(Gpt* g, int max_context) {
         if (w.c.mixer == SPT_MIXER_GLA) {
             w.state = (float*)galloc(g, (size_t)g->c.max_batch * w.c.heads * w.c.dim * w.c.vdim * 4);
             if (!w.state) return 1;
-        } else {
+        }
+        if (w.c.mixer == SPT_MIXER_WINDOW && w.c.conv_taps > 0) {
+            const size_t bytes = (size_t)g->c.max_batch * w.c.conv_taps * w.c_g * g->es;
+            w.ring = galloc(g, bytes);
+            if (!w.ring || sptorch_ext_memset(w.ring, 0, bytes)) return 1;
+        }
+        if (w.c.mixer == SPT_MIXER_LATENT || (w.c.mixer == SPT_MIXER_WINDOW && w.own_kv())) {
             const size_t bytes = (size_t)g->c.max_batch * max_context * w.row() * g->es;
             w.rows = galloc(g, bytes);
             if (!w.rows || sptorch_ext_memset(w.rows, 0, bytes)) return 1;
@@ -399,7 +534,7 @@ int layered_enable_cache(Gpt* g, int max_context) {
     return layered_reset_cache(g);
 }
 
-// Every sequence forgets what it has seen.  Cached rows need no clearing: a position is written before it is read.
+// Every sequence forgets what it has seen.  Cached rows and rings need no clearing: a position is written before it is read.
 int layered_reset_cache(Gpt* g) {
     for (auto& w : g->lay->L)
         if (w.state && sptorch_ext_memset(w.state, 0, (size_t)g->c.max_batch * w.c.heads * w.c.dim * w.c.vdim * 4)) return 1;
@@ -409,12 +544,17 @@ int layered_reset_cache(Gpt* g) {
 
 int layered_launches(const Gpt* g, int B, int T) {
     (void)B; (void)T;
+    const Layered& lay = *g->lay;
+    const bool parallel = lay.opt.block == SPT_BLOCK_PARALLEL, side = lay.opt.side_dim > 0;
     int n = 2;                                                        // embedding, head
-    if (g->lay->L.empty()) n++;
-    for (auto& w : g->lay->L) {
-        n += 3;                                                       // input projection, W_o, post-norm
-        n += w.c.mixer == SPT_MIXER_GLA ? (g->c.dtype == BF16 && gla_chunked_supported(gla_args(const_cast<Gpt*>(g), w, B, T, false)) ? 3 : 2) : expands(g, w) ? 5 : 5;
-        if (w.c.mlp == SPT_MLP_DENSE) n += 4;
+    if (lay.L.empty() || parallel) n++;                               // a norm of its own
+    for (auto& w : lay.L) {
+        const bool dense = w.c.mlp == SPT_MLP_DENSE;
+        if (w.c.mixer == SPT_MIXER_GLA) n += g->c.dtype == BF16 && gla_chunked_supported(gla_args(const_cast<Gpt*>(g), w, B, T, false)) ? 3 : 2;
+        else if (w.c.mixer == SPT_MIXER_LATENT) n += 5;
+        else n += 2;                                                  // convolutions, attention
+        if (!parallel) n += 3 + (dense ? 4 : 0);                      // input projection, W_o, post-norm
+        else n += 2 + (dense ? w.c.mixer == SPT_MIXER_WINDOW ? 1 : 2 : 0) + (side ? g->c.dtype == BF16 ? 4 : 3 : 1);
     }
     return n;
 }
@@ -425,7 +565,8 @@ void layered_release(Gpt* g) { delete g->lay; g->lay = nullptr; }
 namespace {
 
 // one entry per tensor: its name behind the layer's prefix, its shape, and where it goes
-struct Slot { std::string name; size_t rows, cols; void* dst; bool f32; int ld; size_t dst_row; const LayeredLayer* ukt = nullptr; };      // cols 0: a vector of `rows` values
+struct Slot { std::string name; size_t rows, cols; void* dst; bool f32; int ld; size_t dst_row; const LayeredLayer* ukt = nullptr; size_t part = 0, part_ld = 0; };
+// cols 0: a vector of `rows` values; part: a row is cut into parts of so many values, part_ld apart on the device
 
 // uk [heads*dim, kv] -> its transpose per head, [heads][kv8][dim]
 int upload_ukt(Gpt* g, const Slot& s, const float* host) {
@@ -446,16 +587,30 @@ std::vector<Slot> layer_slots(const Gpt* g, const LayeredLayer& w) {
     auto mat = [&](const char* n, size_t r, size_t k, void* dst, int ld, size_t row) { s.push_back({n, r, k, dst, false, ld, row}); };
     auto vec = [&](const char* n, size_t r, float* dst) { s.push_back({n, r, 0, dst, true, 0, 0}); };
     const bool mlp = c.mlp == SPT_MLP_DENSE;
+    const bool parallel = g->lay->opt.block == SPT_BLOCK_PARALLEL;
+    const int ld_wo = w.o_ld() + (parallel && mlp ? pad8(c.d_ff) : 0);
     vec("norm1", d, w.norm1);
-    if (mlp) vec("norm2", d, w.norm2);
+    if (mlp && !parallel) vec("norm2", d, w.norm2);
     if (c.mixer == SPT_MIXER_GLA) {
         const size_t hd = (size_t)c.heads * c.dim, hv = (size_t)c.heads * c.vdim;
         mat("mix.q", hd, d, w.w_in, d8, w.c_q); mat("mix.k", hd, d, w.w_in, d8, w.c_k); mat("mix.v", hv, d, w.w_in, d8, w.c_v); mat("mix.g", hv, d, w.w_in, d8, w.c_g);
-        mat("mix.o", d, hv, w.w_o, w.o_ld(), 0);
+        mat("mix.o", d, hv, w.w_o, ld_wo, 0);
         vec("mix.norm", c.vdim, w.head_norm);
         mat("mix.a1", c.decay_rank, d, w.w_in, d8, w.c_a);
         s.push_back({"mix.a2", hd, (size_t)c.decay_rank, w.a2, true, c.decay_rank, 0});
         vec("mix.a2.b", hd, w.a2_b);
+    } else if (c.mixer == SPT_MIXER_WINDOW) {
+        const size_t hd = (size_t)c.heads * c.dim, gd = (size_t)c.kv_heads * c.dim, gv = (size_t)c.kv_heads * c.vdim, hv = (size_t)c.heads * c.vdim;
+        const bool kv = w.own_kv();
+        mat("mix.q", hd, d, w.w_in, d8, w.c_q);
+        if (kv) { mat("mix.k", gd, d, w.w_in, d8, w.c_k); mat("mix.v", gv, d, w.w_in, d8, w.c_v); }
+        if (c.conv_taps > 0) {
+            auto taps = [&](const char* n, size_t rows, int col) { s.push_back({n, rows, (size_t)c.conv_taps, w.conv + (size_t)col * c.conv_taps, true, c.conv_taps, 0}); };
+            taps("mix.q.conv", hd, w.c_q);
+            if (kv) { taps("mix.k.conv", gd, w.c_k); taps("mix.v.conv", gv, w.c_v); }
+        }
+        if (c.out_gate) mat("mix.g", hv, d, w.w_in, d8, w.c_g);
+        mat("mix.o", d, hv, w.w_o, ld_wo, 0);
     } else {
         const int q8 = pad8(c.q_rank), kv8 = w.kv8();
         mat("mix.dq", c.q_rank, d, w.w_in, d8, w.c_dq); vec("mix.dq.norm", c.q_rank, w.dq_norm);
@@ -465,13 +620,21 @@ std::vector<Slot> layer_slots(const Gpt* g, const LayeredLayer& w) {
         if (w.w_ukt) s.back().ukt = &w;
         mat("mix.uv", (size_t)c.heads * c.vdim, c.kv_rank, w.w_ukv, kv8, w.ukv_v());
         mat("mix.g", c.heads, d, w.w_in, d8, w.c_g);
-        mat("mix.o", d, (size_t)c.heads * c.vdim, w.w_o, w.o_ld(), 0);
+        mat("mix.o", d, (size_t)c.heads * c.vdim, w.w_o, ld_wo, 0);
     }
-    if (mlp) {
+    if (mlp && parallel) {
+        mat("mlp.gate", c.d_ff, d, w.w_in, d8, w.c_gate);
+        mat("mlp.up", c.d_ff, d, w.w_in, d8, w.c_up);
+        mat("mlp.down", d, c.d_ff, (uint8_t*)w.w_o + (size_t)w.o_ld() * g->es, ld_wo, 0);
+    } else if (mlp) {
         const int f8 = pad8(c.d_ff);
-        mat("mlp.gate", c.d_ff, d, w.w_gate, d8, 0); vec("mlp.gate.b", c.d_ff, w.b_gate);
-        mat("mlp.up", c.d_ff, d, w.w_up, d8, 0); vec("mlp.up.b", c.d_ff, w.b_up);
-        mat("mlp.down", d, c.d_ff, w.w_down, f8, 0); vec("mlp.down.b", d, w.b_down);
+        mat("mlp.gate", c.d_ff, d, w.w_gate, d8, 0); if (c.mlp_bias) vec("mlp.gate.b", c.d_ff, w.b_gate);
+        mat("mlp.up", c.d_ff, d, w.w_up, d8, 0); if (c.mlp_bias) vec("mlp.up.b", c.d_ff, w.b_up);
+        mat("mlp.down", d, c.d_ff, w.w_down, f8, 0); if (c.mlp_bias) vec("mlp.down.b", d, w.b_down);
+    }
+    if (g->lay->opt.side_dim > 0) {
+        const size_t sd = g->lay->opt.side_dim;
+        mat("side.gate", sd, d, w.side_gate, d8, 0); mat("side.proj", d, sd, w.side_proj, g->lay->side8, 0); vec("side.norm", d, w.side_norm);
     }
     return s;
 }
@@ -480,10 +643,15 @@ std::vector<Slot> model_slots(const Gpt* g) {
     const size_t V = g->c.vocab, d = g->c.d_model;
     std::vector<Slot> s;
     s.push_back({"embed", V, d, g->lay->embed, false, g->lay->d8, 0});
+    const size_t L = g->lay->L.size(), sd = g->lay->opt.side_dim, s8 = g->lay->side8;
+    if (sd && L) {                                                       // a row holds sd values per layer, on the device s8
+        s.push_back({"side.embed", V, L * sd, g->lay->side_embed, false, (int)(L * s8), 0});
+        s.back().part = sd; s.back().part_ld = s8;
+    }
     for (size_t l = 0; l < g->lay->L.size(); l++)
         for (auto& e : layer_slots(g, g->lay->L[l])) { s.push_back(e); s.back().name = "l" + std::to_string(l) + "." + e.name; }
     s.push_back({"final.norm", d, 0, g->lay->final_norm, true, 0, 0});
-    s.push_back({"head", V, d, g->lay->head, false, g->lay->d8, 0});
+    if (!g->lay->opt.tied_head) s.push_back({"head", V, d, g->lay->head, false, g->lay->d8, 0});
     return s;
 }
 
@@ -505,25 +673,49 @@ int layered_set_param(Gpt* g, const char* name, const float* host, size_t n) {
         void* dst = (uint8_t*)s.dst + s.dst_row * s.ld * g->es;
         if (s.ukt && upload_ukt(g, s, host)) return 1;
         if ((size_t)s.ld == s.cols) return upload_rows(g, dst, host, n) || stream_wait();
-        std::vector<float> padded(s.rows * s.ld, 0.0f);
-        for (size_t r = 0; r < s.rows; r++) memcpy(&padded[r * s.ld], host + r * s.cols, s.cols * 4);
-        return upload_rows(g, dst, padded.data(), padded.size()) || stream_wait();
+        const size_t parts = s.part ? s.cols / s.part : 1, part = s.part ? s.part : s.cols, part_ld = s.part ? s.part_ld : (size_t)pad8((int)s.cols), wide = parts * part_ld;
+        std::vector<float> padded(s.rows * wide, 0.0f);
+        for (size_t r = 0; r < s.rows; r++)
+            for (size_t i = 0; i < parts; i++) memcpy(&padded[r * wide + i * part_ld], host + r * s.cols + i * part, part * 4);
+        if (wide == (size_t)s.ld) return upload_rows(g, dst, padded.data(), padded.size()) || stream_wait();
+        // columns of a wider matrix, whose other columns stay as they are
+        void* tight = sptorch_ext_alloc_bytes(padded.size() * g->es);
+        if (!tight) return 1;
+        int rc = upload_rows(g, tight, padded.data(), padded.size());
+        if (!rc && cudaMemcpy2DAsync(dst, (size_t)s.ld * g->es, tight, wide * g->es, wide * g->es, s.rows, cudaMemcpyDeviceToDevice, rt().stream) != cudaSuccess)
+            rc = fail("gpt_set_param(%s): copy into the fused matrix failed", name);
+        if (!rc) rc = stream_wait();
+        sptorch_free(tight);
+        return rc;
     }
     return fail("gpt_set_param: unknown parameter name '%s'", name);
 }
 
-static int check_layer(const sptorch_layer_config& c, int i) {
-    if (c.mixer != SPT_MIXER_GLA && c.mixer != SPT_MIXER_LATENT) return fail_host("layered_create: layer %d: unknown mixer %d", i, c.mixer);
+static int check_layer(const sptorch_layer_config* layers, int i, const sptorch_layered_options& opt) {
+    const sptorch_layer_config& c = layers[i];
+    if (c.mixer != SPT_MIXER_GLA && c.mixer != SPT_MIXER_LATENT && c.mixer != SPT_MIXER_WINDOW) return fail_host("layered_create: layer %d: unknown mixer %d", i, c.mixer);
     if (c.heads <= 0 || c.dim <= 0 || c.vdim <= 0) return fail_host("layered_create: layer %d: non-positive head count or size", i);
     if (c.mixer == SPT_MIXER_GLA) {
         if (c.decay_rank <= 0 || !(c.tau > 0.0f)) return fail_host("layered_create: layer %d: decay_rank and tau must be positive", i);
         if (c.dim > 512) return fail_host("layered_create: layer %d: key size %d is larger than 512", i, c.dim);
-    } else {
+    } else if (c.mixer == SPT_MIXER_LATENT) {
         if (c.kv_rank <= 0 || c.q_rank <= 0 || c.rot_dim < 0) return fail_host("layered_create: layer %d: latent sizes must be positive", i);
         if (c.rope_dims < 0 || c.rope_dims > c.rot_dim || c.rope_dims % 2) return fail_host("layered_create: layer %d: %d rotated dims of %d", i, c.rope_dims, c.rot_dim);
         if (c.rope_dims && !(c.rope_base > 0.0)) return fail_host("layered_create: layer %d: rope_base must be positive", i);
         if (pad8(c.kv_rank) + pad8(c.rot_dim) > 1280) return fail_host("layered_create: layer %d: cached rows of %d + %d values are larger than 1280", i, c.kv_rank, c.rot_dim);
+    } else {
+        if (c.dim > kWindowMaxHead || c.vdim > kWindowMaxHead) return fail_host("layered_create: layer %d: heads of %d and %d are larger than %d", i, c.dim, c.vdim, kWindowMaxHead);
+        if (c.kv_heads <= 0 || c.heads % c.kv_heads) return fail_host("layered_create: layer %d: %d query heads on %d key/value heads", i, c.heads, c.kv_heads);
+        if (c.window < 0 || c.conv_taps < 0) return fail_host("layered_create: layer %d: negative window or convolution", i);
+        if (c.kv_shared) {
+            if (c.kv_from < 0 || c.kv_from >= i) return fail_host("layered_create: layer %d: keys and values of layer %d, which does not come before it", i, c.kv_from);
+            const sptorch_layer_config& s = layers[c.kv_from];
+            if (s.mixer != SPT_MIXER_WINDOW || s.kv_shared || s.kv_heads != c.kv_heads || s.dim != c.dim || s.vdim != c.vdim)
+                return fail_host("layered_create: layer %d: layer %d has no keys and values of %d heads of %d and %d", i, c.kv_from, c.kv_heads, c.dim, c.vdim);
+        }
     }
+    if (c.mlp_act != SPT_ACT_SILU && c.mlp_act != SPT_ACT_RELU) return fail_host("layered_create: layer %d: unknown activation %d", i, c.mlp_act);
+    if (opt.block == SPT_BLOCK_PARALLEL && c.mlp == SPT_MLP_DENSE && c.mlp_bias) return fail_host("layered_create: layer %d: the feed-forward of a parallel block has no biases", i);
     if (c.mlp != SPT_MLP_NONE && c.mlp != SPT_MLP_DENSE) return fail_host("layered_create: layer %d: unknown feed-forward %d", i, c.mlp);
     if (c.mlp == SPT_MLP_DENSE && c.d_ff <= 0) return fail_host("layered_create: layer %d: non-positive d_ff", i);
     return 0;
@@ -533,7 +725,8 @@ static int check_layer(const sptorch_layer_config& c, int i) {
 
 using namespace spt;
 
-extern "C" void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const sptorch_layer_config* layers, int n_layers) {
+extern "C" void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const sptorch_layer_config* layers, int n_layers,
+                                             const sptorch_layered_options* options) {
     if (enter()) return nullptr;
     if (!cfg || (n_layers > 0 && !layers)) { fail("layered_create: null config"); return nullptr; }
     sptorch_gpt_config c = *cfg;
@@ -541,7 +734,13 @@ extern "C" void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const
     if (cfg->tp_size > 1) { fail("layered_create: no tensor parallel shards"); return nullptr; }
     if (c.vocab <= 0 || c.d_model <= 0 || n_layers < 0 || c.seq_len <= 0 || c.max_batch <= 0) { fail("layered_create: non-positive dimension"); return nullptr; }
     if (c.dtype != SPT_F32 && c.dtype != SPT_BF16) { fail("layered_create: unknown dtype %d", c.dtype); return nullptr; }
-    for (int i = 0; i < n_layers; i++) if (check_layer(layers[i], i)) return nullptr;
+    sptorch_layered_options opt = {};
+    opt.embed_scale = 1.0f;
+    if (options) opt = *options;
+    if (opt.block != SPT_BLOCK_POST_NORM && opt.block != SPT_BLOCK_PARALLEL) { fail("layered_create: unknown block %d", opt.block); return nullptr; }
+    if (opt.side_dim < 0 || (opt.side_dim > 0 && opt.block != SPT_BLOCK_PARALLEL)) { fail("layered_create: a per-layer token input needs a parallel block"); return nullptr; }
+    for (int i = 0; i < n_layers; i++) if (check_layer(layers, i, opt)) return nullptr;
+    const bool parallel = opt.block == SPT_BLOCK_PARALLEL;
     Gpt* g = new Gpt();
     g->c = c;
     g->es = c.dtype == SPT_BF16 ? 2 : 4;
@@ -553,18 +752,48 @@ extern "C" void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const
     bool ok = true;
     auto Z = [&](size_t bytes) { void* p = galloc(g, bytes); if (!p || sptorch_ext_memset(p, 0, bytes)) ok = false; return p; };
     auto F = [&](size_t n) { return (float*)Z((size_t)pad8((int)n) * 4); };
-    lay.embed = Z(V * d8 * es); lay.head = Z(V * d8 * es); lay.final_norm = F(d8);
+    lay.opt = opt;
+    lay.side8 = pad8(opt.side_dim);
+    lay.embed = Z(V * d8 * es); lay.head = opt.tied_head ? lay.embed : Z(V * d8 * es); lay.final_norm = F(d8);
+    if (opt.side_dim && n_layers) lay.side_embed = Z(V * n_layers * lay.side8 * es);
     g->head = lay.head; g->tok = lay.embed;
     std::map<std::pair<int, double>, float2*> angles;
+    std::map<std::pair<double, double>, float*> temps;
+    auto table = [&](const std::vector<float>& host) -> float* {
+        float* p = (float*)galloc(g, host.size() * 4);
+        if (!p || sptorch_ext_copy_h2d_bytes(host.data(), p, host.size() * 4) || stream_wait()) { ok = false; return nullptr; }
+        return p;
+    };
     for (int i = 0; i < n_layers && ok; i++) {
         LayeredLayer w;
         w.c = layers[i];
         const sptorch_layer_config& lc = w.c;
         auto at = [&](int& col, int width) { col = w.n_in; w.n_in += pad8(width); };
-        w.norm1 = F(d8); w.norm2 = F(d8);
+        w.norm1 = F(d8);
+        if (!parallel) w.norm2 = F(d8);
         if (lc.mixer == SPT_MIXER_GLA) {
             at(w.c_q, lc.heads * lc.dim); at(w.c_k, lc.heads * lc.dim); at(w.c_v, lc.heads * lc.vdim); at(w.c_g, lc.heads * lc.vdim); at(w.c_a, lc.decay_rank);
             w.a2 = F((size_t)lc.heads * lc.dim * lc.decay_rank); w.a2_b = F((size_t)lc.heads * lc.dim); w.head_norm = F(lc.vdim);
+        } else if (lc.mixer == SPT_MIXER_WINDOW) {
+            at(w.c_q, lc.heads * lc.dim);
+            if (w.own_kv()) { at(w.c_k, lc.kv_heads * lc.dim); at(w.c_v, lc.kv_heads * lc.vdim); }
+            at(w.c_g, lc.heads * lc.vdim);
+            if (lc.conv_taps > 0) w.conv = F((size_t)w.c_g * lc.conv_taps);
+            if (lc.q_temp_every > 0.0) {
+                float*& tab = temps[{lc.q_temp_coef, lc.q_temp_every}];
+                if (!tab) {
+                    std::vector<float> host(c.seq_len);
+                    for (int p = 0; p < c.seq_len; p++) host[p] = (float)(1.0 + lc.q_temp_coef * std::log(std::floor((p + 1.0) / lc.q_temp_every) + 1.0));
+                    tab = table(host);
+                }
+                w.temp = tab;
+            }
+            if (lc.distance_bias) {
+                std::vector<float> host(lc.heads);
+                for (int h = 0; h < lc.heads; h++) host[h] = (float)std::pow(2.0, -8.0 * (h + 1) / lc.heads);
+                w.slopes = table(host);
+            }
+            if (lc.kv_shared) lay.L[lc.kv_from].kv_read = true;
         } else {
             at(w.c_dq, lc.q_rank); at(w.c_dkv, lc.kv_rank + lc.rot_dim); at(w.c_g, lc.heads);
             w.dq_norm = F(lc.q_rank); w.dkv_norm = F(lc.kv_rank);
@@ -585,10 +814,12 @@ extern "C" void* sptorch_ext_layered_create(const sptorch_gpt_config* cfg, const
                 w.angles = tab;
             }
         }
+        const size_t f8 = lc.mlp == SPT_MLP_DENSE ? pad8(lc.d_ff) : 0;
+        if (parallel && f8) { at(w.c_up, lc.d_ff); at(w.c_gate, lc.d_ff); }
         w.w_in = Z((size_t)w.n_in * d8 * es);
-        w.w_o = Z(d8 * w.o_ld() * es);
-        if (lc.mlp == SPT_MLP_DENSE) {
-            const size_t f8 = pad8(lc.d_ff);
+        w.w_o = Z(d8 * (w.o_ld() + (parallel ? f8 : 0)) * es);
+        if (lay.side8) { w.side_gate = Z((size_t)lay.side8 * d8 * es); w.side_proj = Z(d8 * lay.side8 * es); w.side_norm = F(d8); }
+        if (f8 && !parallel) {
             w.w_gate = Z(f8 * d8 * es); w.w_up = Z(f8 * d8 * es); w.w_down = Z(d8 * f8 * es);
             w.b_gate = F(f8); w.b_up = F(f8); w.b_down = F(d8);
         }

@@ -1,5 +1,5 @@
 // layered.h -- models built from a list of layers, each with its own mixer, sizes and feed-forward: the structures of the driver
-// (layered.cu) and the launch functions of the mixers' kernels (gla.cu, latent_attention.cu).
+// (layered.cu) and the launch functions of the mixers' kernels (gla.cu, latent_attention.cu, window_attention.cu).
 //
 // Every row buffer and weight matrix is padded to a multiple of eight elements per row with zeros (pad8): a row then starts on a
 // 16-byte boundary in both dtypes, whatever the model's sizes, and a padded K adds zeros to a sum.
@@ -11,9 +11,15 @@ namespace spt {
 
 inline int pad8(int n) { return (n + 7) / 8 * 8; }
 
+// scratch grown on demand (outside any graph capture); new memory starts as zeros
+struct LayeredScratch { void* p = nullptr; size_t bytes = 0; };
+
 // One layer's weights (device), where its projections lie in the columns of its input projection's output, and what it keeps of
 // every sequence.  Gated linear attention keeps a [dim, vdim] f32 matrix per (sequence, head); latent attention keeps a row
-// [latent | rotated key part] per position.
+// [latent | rotated key part] per position; window attention keeps a row [keys | values] per position, unless it reads another layer's,
+// and a ring of its last projected rows.  Layers of a parallel block have the feed-forward's projections in w_in too, and W_o and W_down
+// side by side in w_o: the columns [gate of the heads | up] of the projections' output become [heads | feed-forward] in place, and
+// one product takes both back to the stream.
 struct LayeredLayer {
     sptorch_layer_config c;
     void* w_in = nullptr;                        // every projection that reads the layer's input, one matrix [n_in, pad8(width)]
@@ -30,26 +36,34 @@ struct LayeredLayer {
     void *w_gate = nullptr, *w_up = nullptr, *w_down = nullptr;
     float *b_gate = nullptr, *b_up = nullptr, *b_down = nullptr;
     float* state = nullptr;                      // gated linear attention: [max_batch][heads][dim][vdim]
-    void* rows = nullptr;                        // latent attention: [max_batch][cache positions][row()]
+    void* rows = nullptr;                        // latent and window attention: [max_batch][cache positions][row()]
+    int c_up = 0, c_gate = 0;                    // parallel block: columns of the feed-forward's two projections
+    float* conv = nullptr;                       // window attention: [c_g][taps], the columns of q, k and v as they lie in w_in
+    const float *temp = nullptr, *slopes = nullptr;          // ... position factors of the queries [seq_len], distance slopes [heads]
+    void* ring = nullptr;                        // ... [max_batch][taps][c_g]: projected rows of the last positions, slot = position % taps
+    LayeredScratch own;                          // ... rows of a forward without a cache
+    bool kv_read = false;                        // ... a later layer reads these keys and values
+    void *side_gate = nullptr, *side_proj = nullptr;         // per-layer token input: [pad8(side_dim), d8], [d8, pad8(side_dim)]
+    float* side_norm = nullptr;
     const float2* angles = nullptr;              // (cos, sin) of position p and pair i at [p * rope_dims / 2 + i]
 
     int q_ld() const { return pad8(c.heads * (c.dim + c.rot_dim)); }
     int kv8() const { return pad8(c.kv_rank); }
-    int row() const { return pad8(c.kv_rank) + pad8(c.rot_dim); }      // elements of a cached row
+    bool own_kv() const { return !c.kv_shared; }
+    int row() const { return c.mixer == SPT_MIXER_WINDOW ? c.kv_heads * (pad8(c.dim) + pad8(c.vdim)) : pad8(c.kv_rank) + pad8(c.rot_dim); }      // elements of a cached row
     int ukv_v() const { return pad8(c.heads * c.dim); }                // first row of the value part of w_ukv
     int ukv_ld() const { return ukv_v() + pad8(c.heads * c.vdim); }
     int o_ld() const { return pad8(c.heads * c.vdim); }
 };
 
-// scratch grown on demand (outside any graph capture); new memory starts as zeros
-struct LayeredScratch { void* p = nullptr; size_t bytes = 0; };
-
 struct Layered {
     std::vector<LayeredLayer> L;
-    int d8 = 0;                                  // pad8(width)
+    sptorch_layered_options opt = {};
+    int d8 = 0, side8 = 0;                       // pad8(width), pad8(side_dim)
+    void* side_embed = nullptr;                  // [vocab, layers * side8]
     void *embed = nullptr, *head = nullptr;      // [vocab, d8]
     float* final_norm = nullptr;
-    LayeredScratch x, x2, xb, y, in, ao, cq, q, kv, f, rows, qabs, olat, gla_o, gla_u, gla_dec;
+    LayeredScratch x, x2, xb, y, in, ao, cq, q, kv, f, rows, qabs, olat, gla_o, gla_u, gla_dec, side;
 };
 
 // ---- entry points of gpt.cu's handle for such a model ----
@@ -121,5 +135,30 @@ int latent_attention_absorbed(const LatentArgs& a, bool dependent);
 // the attention of that path for bf16 on the tensor cores: qabs [M][H * kv8] without the rotated part -> olat [M][H * kv8]
 bool latent_decode_supported(const LatentArgs& a);
 int latent_decode(const LatentArgs& a, bool dependent);
+
+// ---- window_attention.cu ----
+constexpr int kWindowMaxHead = 1024;             // largest query/key and value size of a head
+struct WindowArgs {
+    const void* in; long long ld_in;             // projections of B*T tokens: q, k, v of every head at c_q, c_k, c_v
+    int c_q, c_k, c_v;
+    int B, T, H, G, D, V, D8, V8, taps;
+    const float* conv;                           // [columns][taps] (taps 0: none)
+    const float *temp, *slopes;                  // may be null
+    int first; const int* pos_dev;               // as in LatentArgs
+    float scale; int window;                     // window 0: every earlier position
+    bool own_kv;                                 // false: the rows are another layer's, complete for this call's tokens
+    void* ring; int ring_cols;                   // null: nothing is kept, and the call starts its sequences
+    void* rows; long long seq_stride; int row, capacity;
+    void* q;                                     // out of prep: [B*T, H * D8]
+    const void* gate; void* out; long long ld_out;           // [B*T, ld_out], head h at columns h*V; gate may be out, or null
+    int dtype;
+};
+// projections -> convolved queries and cached rows; the ring's new slots
+int window_prep(const WindowArgs& a, bool dependent);
+// any sizes, from q and the rows
+int window_plain(const WindowArgs& a, bool dependent);
+// few tokens, bf16.  fresh (T = 1): window_prep has not run, the kernel does its work for the one token
+bool window_decode_supported(const WindowArgs& a);
+int window_decode(const WindowArgs& a, bool fresh, bool dependent);
 
 }  // namespace spt

@@ -1,5 +1,5 @@
 // linear_few_rows.cu -- Linear for a handful of input rows: C[m, n] = act(alpha * sum_k A[m,k] W[n,k] + bias[n]) (+ / * R[m,n]),
-// M <= 64, bf16 operands and output.  This is the shape of every projection of a decode step (M = sequences in flight;
+// M <= 64, bf16 operands, bf16 or f32 output.  This is the shape of every projection of a decode step (M = sequences in flight;
 // crates/nn/src/lib.rs:706-760 and 1119-1131 run them once per generated token).
 //
 // With so few rows the product is a stream over the weight matrix and nothing else: 2 * N * K bytes read once, a few FLOP per
@@ -53,6 +53,18 @@ constexpr int kPostNormMaxRows = 2;
 
 // GemmDesc's block-diagonal form
 struct FewRowsGroups { int group; long long group_a, group_c; const __nv_bfloat16* gate; long long ld_gate; };
+// its activation on A, f32 output and second output
+struct FewRowsExtra { int act_from; long long act_off; int c_f32; __nv_bfloat16* c2; };
+
+// a * max(g, 0) on eight bf16 values
+__device__ __forceinline__ uint4 relu_mul8(uint4 a, uint4 g) {
+    const __nv_bfloat162 zero = __float2bfloat162_rn(0.0f);
+    __nv_bfloat162* x = reinterpret_cast<__nv_bfloat162*>(&a);
+    const __nv_bfloat162* y = reinterpret_cast<const __nv_bfloat162*>(&g);
+#pragma unroll
+    for (int i = 0; i < 4; i++) x[i] = __hmul2(x[i], __hmax2(y[i], zero));
+    return a;
+}
 
 // MT: 16-row groups of A (M <= 16 MT); NT: 8-row groups of W per CTA; S: weight slices a warp has in flight.
 // NORM: A holds un-normalised rows; every CTA normalises them itself into shared memory (kind 1: LayerNorm, gamma * ((x - mean) *
@@ -64,7 +76,7 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
                                                                      const __nv_bfloat16* __restrict__ W, long long ldb,
                                                                      __nv_bfloat16* C, long long ldc, const float* __restrict__ bias,
                                                                      const __nv_bfloat16* R, int M, int N, int K, float alpha, int epilogue,
-                                                                     RowNorm nrm, int ksplit, FewRowsGroups grp) {
+                                                                     RowNorm nrm, int ksplit, FewRowsGroups grp, FewRowsExtra ext) {
     __shared__ float red[kWarps][MT * 16][NT * 8 + 1];
     extern __shared__ __align__(16) uint8_t dyn[];                       // NORM: M rows of (K + 8) bf16
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
@@ -112,7 +124,9 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
 #pragma unroll
     for (int it = 0; it < EI; it++) {
         const int e = tid + it * kWarps * 32, m = e / (NT * 8), n = n0 + e % (NT * 8);
-        rpre[it] = (R && krank == 0 && m < M && n < N) ? __bfloat162float(R[(long long)m * ldc + n]) : 0.0f;
+        rpre[it] = !(R && krank == 0 && m < M && n < N) ? 0.0f
+                   : ext.c_f32                          ? reinterpret_cast<const float*>(R)[(long long)m * ldc + n]
+                                                        : __bfloat162float(R[(long long)m * ldc + n]);
     }
 
     const long long a_ld = NORM ? (long long)(K + 8) : lda;
@@ -262,6 +276,10 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
                 const bool live = 32 * s < k_mine;
                 if (live && r0 < M) a0 = *reinterpret_cast<const uint4*>(a_base + (long long)r0 * a_ld + 32 * s + 8 * t);
                 if (live && r1 < M) a1 = *reinterpret_cast<const uint4*>(a_base + (long long)r1 * a_ld + 32 * s + 8 * t);
+                if (NORM == 0 && ext.act_off && live && 32 * s + 8 * t >= ext.act_from) {
+                    if (r0 < M) a0 = relu_mul8(a0, *reinterpret_cast<const uint4*>(a_base + (long long)r0 * a_ld + ext.act_off + 32 * s + 8 * t));
+                    if (r1 < M) a1 = relu_mul8(a1, *reinterpret_cast<const uint4*>(a_base + (long long)r1 * a_ld + ext.act_off + 32 * s + 8 * t));
+                }
 #pragma unroll
                 for (int j = 0; j < NT; j++) {
                     mma_bf16_16x8x16(acc[i][j], a0.x, a1.x, a0.y, a1.y, wv[u][j].x, wv[u][j].y);
@@ -324,11 +342,14 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
         const int m = e / (NT * 8), nn = e % (NT * 8), n = n0 + nn;
         if (m >= M || n >= N || m >= MT * 16) continue;
         float v = fmaf(tot[it], alpha, bpre[it]);
-        if (epilogue == EPI_GELU) v = gelu_fast2(make_float2(v, 0.0f)).x;
+        if (epilogue == EPI_GELU || epilogue == EPI_GELU_MUL) v = gelu_fast2(make_float2(v, 0.0f)).x;
         else if (epilogue == EPI_SWIGLU) v = silu_fast(v);
-        if (R) v = epilogue == EPI_SWIGLU ? v * rpre[it] : v + rpre[it];
+        else if (epilogue == EPI_RELU_MUL) v = fmaxf(v, 0.0f);
+        if (R) v = epilogue_multiplies(epilogue) ? v * rpre[it] : v + rpre[it];
         if (grp.gate) v *= 1.0f / (1.0f + __expf(-__bfloat162float(grp.gate[(long long)m * grp.ld_gate + gi])));
-        C[(long long)m * ldc + n] = __float2bfloat16_rn(v);
+        if (ext.c_f32) reinterpret_cast<float*>(C)[(long long)m * ldc + n] = v;
+        else C[(long long)m * ldc + n] = __float2bfloat16_rn(v);
+        if (ext.c2) ext.c2[(long long)m * ldc + n] = __float2bfloat16_rn(v);
     }
 }
 
@@ -355,7 +376,8 @@ int launch(const GemmDesc& d, const RowNorm& nrm, bool dependent) {
     SPT_CUDA(launch_dependent(kern, dim3(grid), dim3(kWarps * 32), smem, dependent, ksplit,
                               static_cast<const __nv_bfloat16*>(d.A), d.lda, static_cast<const __nv_bfloat16*>(d.B), d.ldb, static_cast<__nv_bfloat16*>(d.C), d.ldc,
                               d.bias, static_cast<const __nv_bfloat16*>(d.R), d.M, d.N, d.K, d.alpha, d.epilogue, nrm, ksplit,
-                              FewRowsGroups{d.group, d.group_a, d.group_c, static_cast<const __nv_bfloat16*>(d.gate), d.ld_gate}));
+                              FewRowsGroups{d.group, d.group_a, d.group_c, static_cast<const __nv_bfloat16*>(d.gate), d.ld_gate},
+                              FewRowsExtra{d.act_from, d.act_off, d.out_dtype == F32 ? 1 : 0, static_cast<__nv_bfloat16*>(d.C2)}));
     note_submit();
     return 0;
 }
@@ -467,12 +489,13 @@ bool linear_few_rows_supported(const GemmDesc& d) {
     // SPTORCH_B200_FEW_ROWS: the largest row count that takes this kernel (0 = never; experiments)
     static const int max_rows = [] { const char* e = getenv("SPTORCH_B200_FEW_ROWS"); const int v = e ? atoi(e) : kDefaultMaxRows; return v < 0 ? 0 : v > 64 ? 64 : v; }();
     const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    return d.mode == MM_BF16 && d.out_dtype == BF16 && d.M >= 1 && d.M <= max_rows && d.N >= 1 && d.K >= 8 && d.K % 8 == 0 && d.nb1 * d.nb2 == 1 &&
+    return d.mode == MM_BF16 && (d.out_dtype == BF16 || !d.group) && d.act_off % 8 == 0 && d.act_from % 8 == 0 && d.M >= 1 && d.M <= max_rows && d.N >= 1 && d.K >= 8 && d.K % 8 == 0 && d.nb1 * d.nb2 == 1 &&
            !d.causal_lower && !d.causal_k && !d.norm_axis && !d.reduce && d.lda % 8 == 0 && d.ldb % 8 == 0 && d.lda >= d.K && d.ldb >= d.K &&
            (d.group ? d.group > 0 && d.group % 8 == 0 && d.N % d.group == 0 && d.group_a % 8 == 0 && !d.R : d.ldc >= d.N) && al16(d.A) && al16(d.B) && d.C != nullptr;
 }
 
 bool linear_few_rows_norm_supported(const GemmDesc& d, const RowNorm& nrm) {
+    if (d.act_off) return false;
     const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     if (nrm.kind == 3)
         return linear_few_rows_supported(d) && nrm.gamma && nrm.x && nrm.y && nrm.x_out && nrm.x_out != nrm.x && nrm.xb && nrm.dim > 0 && nrm.dim <= d.K && !d.group &&

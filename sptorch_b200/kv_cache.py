@@ -82,10 +82,11 @@ def spec_of(model, max_context: int | None = None) -> KvCacheBufferSpec:
 
 @dataclass(frozen=True)
 class LayerCacheSpec:
-    """What one layer of a model built from a list of layers keeps: a row per position ("rows") or a matrix per head ("state", f32)."""
+    """What one layer of a model built from a list of layers keeps: a row per position ("rows"), a matrix per head ("state", f32) or the
+    last projected rows of its convolutions ("ring").  A layer that reads another's keys and values has no rows of its own."""
     layer: int
     kind: str
-    shape: tuple           # rows: (sequences, positions, row); state: (sequences, heads, dim, vdim)
+    shape: tuple           # rows: (sequences, positions, row); state: (sequences, heads, dim, vdim); ring: (sequences, taps, channels)
     dtype: str
 
     def elements(self) -> int:
@@ -101,11 +102,21 @@ class LayerCacheSpec:
 def layer_specs(model, max_context: int | None = None) -> list:
     """Per layer, the device buffers that sptorch_ext_gpt_enable_kv_cache allocates for a model built from a list of layers."""
     from .backend import BF16
-    ctx, out = max_context or model.cfg["seq_len"], []
+    from .layered import GLA, LATENT
+
+    def pad8(n):
+        return -(-n // 8) * 8
+
+    ctx, dtype, out = max_context or model.cfg["seq_len"], "BF16" if model.dtype == BF16 else "F32", []
     for i, c in enumerate(model.layers):
-        if c.mixer == 0:
+        if c.mixer == GLA:
             out.append(LayerCacheSpec(i, "state", (model.max_batch, c.heads, c.dim, c.vdim), "F32"))
+        elif c.mixer == LATENT:
+            out.append(LayerCacheSpec(i, "rows", (model.max_batch, ctx, pad8(c.kv_rank) + pad8(c.rot_dim)), dtype))
         else:
-            row = -(-c.kv_rank // 8) * 8 + -(-c.rot_dim // 8) * 8
-            out.append(LayerCacheSpec(i, "rows", (model.max_batch, ctx, row), "BF16" if model.dtype == BF16 else "F32"))
+            if c.conv_taps:
+                channels = pad8(c.heads * c.dim) + (0 if c.kv_shared else pad8(c.kv_heads * c.dim) + pad8(c.kv_heads * c.vdim))
+                out.append(LayerCacheSpec(i, "ring", (model.max_batch, c.conv_taps, channels), dtype))
+            if not c.kv_shared:
+                out.append(LayerCacheSpec(i, "rows", (model.max_batch, ctx, c.kv_heads * (pad8(c.dim) + pad8(c.vdim))), dtype))
     return out

@@ -7,7 +7,7 @@ import os
 from . import weights
 from .backend import BF16, FfiBackend
 from .gpt import GPT, QwenLikeGPT
-from .layered import ConfigError, LayeredGPT
+from .layered import DESIGNS, ConfigError, LayeredGPT
 
 
 def _gpt_like(cls, eps):
@@ -23,7 +23,7 @@ def _layered(backend, config, shapes, seq_len, dtype, max_batch):
     return LayeredGPT(backend, config, seq_len or int(config.get("seq_len", 4096)), dtype=dtype, max_batch=max_batch, shapes=shapes)
 
 
-ARCHITECTURES = {"GPT": _gpt_like(GPT, 1e-5), "QwenLikeGPT": _gpt_like(QwenLikeGPT, 1e-6), "Tolevik": _layered}
+ARCHITECTURES = {"GPT": _gpt_like(GPT, 1e-5), "QwenLikeGPT": _gpt_like(QwenLikeGPT, 1e-6), **{name: _layered for name in DESIGNS}}
 
 
 def read_config(folder: str) -> dict:

@@ -34,7 +34,7 @@ def test_layer_configs_refuse_what_they_do_not_know():
 
 
 def test_registry_chooses_by_architecture(tmp_path):
-    assert set(registry.ARCHITECTURES) == {"GPT", "QwenLikeGPT", "Tolevik"}
+    assert set(registry.ARCHITECTURES) == {"GPT", "QwenLikeGPT", "Tolevik", "Bulidra"}
     (tmp_path / "config.json").write_text(json.dumps({"architecture": "Nothing"}))
     with pytest.raises(ConfigError):
         registry.read_config(str(tmp_path))
