@@ -651,8 +651,9 @@ def sweep_decode(b, peaks, steps=32, emit=None, batches=(1, 8, 64)):
     return out
 
 
-# Layers of the size of real models': half gated linear attention, half latent attention, beside a Qwen-like model of equal width,
-# depth and feed-forward.  "prompt": (sequences, tokens) of a prefill; "decode": (sequences, cached positions).
+# Layers of the size of real models', beside a Qwen-like model of equal width, depth and feed-forward: half gated linear attention, half
+# latent attention ("gla", "latent"), or window attention in parallel blocks with per-layer token inputs, the last quarter of the
+# layers on the keys and values of the one before them ("window").  "prompt": (sequences, tokens) of a prefill; "decode": (sequences, cached positions).
 LAYERED_SIZES = {
     "small": dict(width=768, n_layer=8, ff=3072, n_head=12, vocab=32000, gla=dict(heads=6, dim=64, vdim=128, tau=16.0, decay_rank=16),
                   latent=dict(heads=12, dim=64, vdim=64, rot_dim=32, kv_rank=256, q_rank=384), prompts=((16, 1024), (1, 1024)), decodes=((1, 512), (8, 512), (64, 512))),
@@ -660,18 +661,30 @@ LAYERED_SIZES = {
                   latent=dict(heads=16, dim=128, vdim=128, rot_dim=64, kv_rank=512, q_rank=1024), prompts=((8, 2048), (1, 2048)), decodes=((1, 2048), (8, 2048), (64, 1024))),
     "wide_heads": dict(width=2048, n_layer=8, ff=5632, n_head=16, vocab=32000, gla=dict(heads=8, dim=128, vdim=256, tau=16.0, decay_rank=16),
                        latent=dict(heads=16, dim=64, vdim=128, rot_dim=64, kv_rank=512, q_rank=512), prompts=((8, 2048),), decodes=((8, 2048),)),
+    "window_small": dict(width=768, n_layer=8, ff=3072, n_head=12, vocab=32000, side=128, window=dict(heads=12, kv_heads=4, dim=64, vdim=64, size=512, conv=3),
+                         prompts=((16, 1024), (1, 1024)), decodes=((1, 512), (8, 512), (64, 512))),
+    "window_large": dict(width=2048, n_layer=8, ff=5632, n_head=16, vocab=32000, side=256, window=dict(heads=16, kv_heads=4, dim=128, vdim=128, size=1024, conv=3),
+                         prompts=((8, 2048), (1, 2048)), decodes=((1, 2048), (8, 2048), (64, 1024))),
+    "window_mixed": dict(width=2048, n_layer=8, ff=5632, n_head=16, vocab=32000, side=256, window=dict(heads=16, kv_heads=8, dim=96, vdim=64, size=4096, conv=4),
+                         prompts=((8, 2048), (2, 8192)), decodes=((8, 2048),)),
 }
 
 
 def layered_config(z):
-    """config.json of a layered model of size z: gated linear attention without, latent attention with a feed-forward, alternating."""
+    """config.json of a layered model of size z: gated linear attention and latent attention alternating, or window attention."""
+    if "window" in z:
+        w = z["window"]
+        m = dict(heads=w["heads"], kv_heads=w["kv_heads"], dim=w["dim"], vdim=w["vdim"], conv=w["conv"], mask=dict(size=w["size"]), q_temp=dict(coef=0.1, every=1024), scale=w["dim"] ** -0.5)
+        own = z["n_layer"] * 3 // 4
+        layers = [dict(type="attention", mixer=m if i < own else dict(m, kv_from=own - 1), mlp=dict(kind="dense", ff=z["ff"])) for i in range(z["n_layer"])]
+        return dict(architecture="Bulidra", embedding=dict(scale=z["width"] ** 0.5), layers=layers, norm=dict(eps=1e-6), token_side=dict(dim=z["side"]), vocab=z["vocab"], width=z["width"])
     la = dict(z["latent"], rot=dict(base=10000.0, dims=z["latent"]["rot_dim"]), scale=(z["latent"]["dim"] + z["latent"]["rot_dim"]) ** -0.5)
     layers = [dict(type="gla", mixer=z["gla"], mlp=dict(kind="dense", ff=z["ff"])) if i % 2 == 0 else
               dict(type="latent_attention", mixer=la, mlp=dict(kind="dense", ff=z["ff"])) for i in range(z["n_layer"])]
     return dict(architecture="Tolevik", layers=layers, norm=dict(eps=1e-5), vocab=z["vocab"], width=z["width"])
 
 
-PROF_NAMES = ["linear_gemm", "attention_gemm", "causal_softmax", "norm", "embedding", "other", "attention", "gated_linear_attention", "latent_norms_rotation"]
+PROF_NAMES = ["linear_gemm", "attention_gemm", "causal_softmax", "norm", "embedding", "other", "attention", "gated_linear_attention", "latent_norms_rotation", "short_convolution"]
 
 
 def _prof_pass(b, fn, reps):
@@ -680,9 +693,53 @@ def _prof_pass(b, fn, reps):
     for _ in range(reps):
         fn()
     b.synchronize()
-    pm, pn = (C.c_float * 9)(), (C.c_uint32 * 9)()
-    lib.sptorch_ext_prof_read(pm, pn, 9); lib.sptorch_ext_prof_enable(0)
+    n = len(PROF_NAMES)
+    pm, pn = (C.c_float * n)(), (C.c_uint32 * n)()
+    lib.sptorch_ext_prof_read(pm, pn, n); lib.sptorch_ext_prof_enable(0)
     return {n: float(pm[i]) / reps for i, n in enumerate(PROF_NAMES) if pn[i]}
+
+
+def _layered_work(z, phase, B, T):
+    """Algorithmic (FLOP, bytes) of a step per category: gated linear attention and latent attention."""
+    d, F, V, L, g, m = z["width"], z["ff"], z["vocab"], z["n_layer"], z["gla"], z["latent"]
+    M, half, w_mlp = B * T if phase == "prefill" else B, L // 2, 3 * d * F
+    gw = d * (2 * g["heads"] * g["dim"] + 2 * g["heads"] * g["vdim"] + g["decay_rank"]) + d * g["heads"] * g["vdim"]
+    lw = d * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + m["heads"]) + m["q_rank"] * m["heads"] * (m["dim"] + m["rot_dim"]) + d * m["heads"] * m["vdim"]
+    up = m["kv_rank"] * m["heads"] * (m["dim"] + m["vdim"])
+    w_lin = half * (gw + lw + 2 * w_mlp) + V * d + (half * up if phase == "prefill" else 0)
+    dk, dv, ha, row = m["dim"] + m["rot_dim"], m["vdim"], m["heads"], m["kv_rank"] + m["rot_dim"]
+    if phase == "prefill":
+        att = (B * ha * T * (T + 1.0) * (dk + dv) * half, B * T * ha * (2 * dk + 2 * dv) * 2.0 * half)
+        gla = (M * g["heads"] * (4.0 * g["dim"] * g["vdim"] + 64 * (g["dim"] + g["vdim"])) * half, M * (g["heads"] * (2 * g["dim"] + 3 * g["vdim"]) + g["decay_rank"]) * 2.0 * half)
+    else:
+        att = (2.0 * B * ha * T * (row + m["kv_rank"]) * half, (B * T * row + up) * 2.0 * half)
+        gla = (0.0, B * g["heads"] * g["dim"] * g["vdim"] * 8.0 * half)
+    return {"linear_gemm": (2.0 * M * w_lin, 2.0 * w_lin), "attention": att, "gated_linear_attention": gla, "norm": (0.0, M * d * 12.0 * 2 * L),
+            "latent_norms_rotation": (0.0, 2.0 * 2 * M * (m["q_rank"] + row + (m["heads"] * m["rot_dim"] if phase == "prefill" else 0)) * half)}
+
+
+def _window_work(z, phase, B, T):
+    """The same for window attention in parallel blocks.  Norms: 12 bytes per element for x += rms(y) w with the next layer's norm, 6 for
+    the 16-bit copy of x in front of the token input (decoding: in the projection before it)."""
+    d, F, V, L, S, w = z["width"], z["ff"], z["vocab"], z["n_layer"], z["side"], z["window"]
+    H, G, D, dv, W = w["heads"], w["kv_heads"], w["dim"], w["vdim"], w["size"]
+    M, own = B * T if phase == "prefill" else B, L * 3 // 4
+    w_lin = L * (d * (H * D + 2 * H * dv) + 3 * d * F + 2 * d * S) + own * d * G * (D + dv) + V * d
+    if phase == "prefill":
+        seen = sum(min(i + 1, W) for i in range(T))
+        att = (2.0 * B * H * seen * (D + dv) * L, B * T * (H * (D + 2 * dv) + G * (D + dv)) * 2.0 * L)
+    else:
+        att = (2.0 * B * H * min(T, W) * (D + dv) * L, B * (min(T, W) * G * (D + dv) + H * (D + 2 * dv)) * 2.0 * L)
+    conv = M * (L * H * D + own * G * (D + dv)) * 4.0
+    return {"linear_gemm": (2.0 * M * w_lin, 2.0 * w_lin), "attention": att, "norm": (0.0, M * d * (18.0 if phase == "prefill" else 12.0) * L), "short_convolution": (0.0, conv)}
+
+
+def _qwen_work(z, phase, B, T):
+    d, F, V, L = z["width"], z["ff"], z["vocab"], z["n_layer"]
+    M = B * T if phase == "prefill" else B
+    w_lin = L * (4 * d * d + 3 * d * F) + V * d
+    att = (2.0 * B * T * (T + 1.0) * d * L, 8.0 * B * T * d * L) if phase == "prefill" else (0.0, 4.0 * B * T * d * L)
+    return {"linear_gemm": (2.0 * M * w_lin, 2.0 * w_lin), "attention": att, "norm": (0.0, M * d * 4.0 * (2 * L + 1)), "other": (0.0, M * 2 * d * 4.0 * L)}
 
 
 def sweep_layered(b, peaks, iters, emit=None, sizes=None):
@@ -698,8 +755,6 @@ def sweep_layered(b, peaks, iters, emit=None, sizes=None):
     for size in sizes or LAYERED_SIZES:
         z = LAYERED_SIZES[size]
         d, F, V, L, H = z["width"], z["ff"], z["vocab"], z["n_layer"], z["n_head"]
-        g, m = z["gla"], z["latent"]
-        max_tokens = max(B * (T + 64) for B, T in tuple(z["prompts"]) + tuple(z["decodes"]))
         for kind in ("layered", "qwen_like"):
             for phase, cases in (("prefill", z["prompts"]), ("decode", z["decodes"])):
                 for B, T in cases:
@@ -732,28 +787,7 @@ def sweep_layered(b, peaks, iters, emit=None, sizes=None):
                     ms = b.timer_end() / n
                     b.synchronize()
                     parts = _prof_pass(b, step, 3)
-                    # algorithmic work per category
-                    half = L // 2
-                    w_mlp = 3 * d * F
-                    if kind == "layered":
-                        gw = d * (2 * g["heads"] * g["dim"] + 2 * g["heads"] * g["vdim"] + g["decay_rank"]) + d * g["heads"] * g["vdim"]
-                        lw = d * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + m["heads"]) + m["q_rank"] * m["heads"] * (m["dim"] + m["rot_dim"]) + d * m["heads"] * m["vdim"]
-                        up = m["kv_rank"] * m["heads"] * (m["dim"] + m["vdim"])
-                        w_lin = half * (gw + lw + 2 * w_mlp) + V * d + (half * up if phase == "prefill" else 0)
-                        dk, dv, ha, la_ = m["dim"] + m["rot_dim"], m["vdim"], m["heads"], half
-                        row = m["kv_rank"] + m["rot_dim"]
-                        if phase == "prefill":
-                            att = (B * ha * T * (T + 1.0) * (dk + dv) * la_, B * T * ha * (2 * dk + 2 * dv) * 2.0 * la_)
-                            gla = (M * g["heads"] * (4.0 * g["dim"] * g["vdim"] + 64 * (g["dim"] + g["vdim"])) * half, M * (g["heads"] * (2 * g["dim"] + 3 * g["vdim"]) + g["decay_rank"]) * 2.0 * half)
-                        else:
-                            att = (2.0 * B * ha * T * (row + m["kv_rank"]) * la_, (B * T * row + up) * 2.0 * la_)
-                            gla = (0.0, B * g["heads"] * g["dim"] * g["vdim"] * 8.0 * half)
-                        work = {"linear_gemm": (2.0 * M * w_lin, 2.0 * w_lin), "attention": att, "gated_linear_attention": gla,
-                                "norm": (0.0, M * d * 12.0 * 2 * L), "latent_norms_rotation": (0.0, 2.0 * 2 * M * (m["q_rank"] + row + (m["heads"] * m["rot_dim"] if phase == "prefill" else 0)) * half)}
-                    else:
-                        w_lin = L * (4 * d * d + w_mlp) + V * d
-                        att = (2.0 * B * T * (T + 1.0) * d * L, 8.0 * B * T * d * L) if phase == "prefill" else (0.0, 4.0 * B * T * d * L)
-                        work = {"linear_gemm": (2.0 * M * w_lin, 2.0 * w_lin), "attention": att, "norm": (0.0, M * d * 4.0 * (2 * L + 1)), "other": (0.0, M * 2 * d * 4.0 * L)}
+                    work = _window_work(z, phase, B, T) if kind == "layered" and "window" in z else _layered_work(z, phase, B, T) if kind == "layered" else _qwen_work(z, phase, B, T)
                     cats = {}
                     for name, t in parts.items():
                         e = {"ms": t}

@@ -55,7 +55,7 @@ int   sptorch_ext_flush_l2(void);                      /* overwrites a 256 MiB s
 /* per-category device timing of the GPT forward (CUDA events around each launch on the library stream).
  * categories: 0 linear GEMM, 1 attention GEMMs, 2 causal softmax, 3 layernorm, 4 embedding, 5 other, 6 fused attention (and attention
  * over cached rows), 7 gated linear attention, 8 latent attention's norms and rotations */
-#define SPT_PROF_NCAT 9
+#define SPT_PROF_NCAT 10
 int   sptorch_ext_prof_enable(int on);
 int   sptorch_ext_prof_read(float* ms, uint32_t* launches, int ncat);  /* syncs, sums since last read, clears */
 uint32_t sptorch_ext_device_status(void);              /* non-zero if a kernel's bounded wait ran out (sticky until sync) */

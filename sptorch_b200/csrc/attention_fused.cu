@@ -29,7 +29,9 @@
 // second half sits in the score columns the first leaves free), so that the weights keep close to f32 precision.
 // And window attention (WIN; window_attention.cu): several query heads read one key/value head, row i sees the last `window` keys up to
 // its own, a score carries the distance bias - slope_h (i - j), and the output is multiplied element by element with a sigmoid.  A work
-// item then starts at the first key tile that query tile 0 sees; query tile 1 starts one tile later when it sees nothing of that one.
+// item then walks the visible key tiles, and every tile's chunks, from the diagonal BACKWARDS: the bias makes near keys large and far
+// ones small, so the maxima a row starts with stay, where a forward walk would rescale at nearly every chunk.  Query tile 0 joins one
+// step late when its diagonal is one tile before query tile 1's; tile 1 leaves one step early when its window begins one tile later.
 // Algorithmic work per (sequence, head): 2 * T(T+1) * hd FLOP; HBM traffic: Q, K, V read once per query tile
 // (K/V re-reads hit L2 thanks to the work schedule below), O written once.
 #include "gemm.h"
@@ -227,21 +229,35 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const int at = k * (int)gridDim.x + (int)blockIdx.x;
         return p.sched ? __ldg(p.sched + at) : at < p.n_ptiles * BH ? at : -1;
     };
-    // work item -> (first query row, sequence, head, key tiles of query tile 0 and of query tile 1).  WIN: js is the item's first key tile,
-    // n0 and n1 count from there, and d1 is 1 when query tile 1 has no part in tile js.
-    auto decode = [&](int item, int& q0, int& bb, int& hh, int& n0, int& n1, int& js, int& d1) {
+    // work item -> (first query row, sequence, head); steps 0 .. N - 1 go over key tiles k0, k0 + dir, ..; query tile t takes part in steps
+    // b[t] .. e[t] - 1
+    struct Item { int q0, bb, hh, N, k0, dir, b[2], e[2]; };
+    auto decode = [&](int item) -> Item {
+        Item w;
         const int pt = p.n_ptiles - 1 - item / BH;
         const int bh = item % BH;
-        bb = bh / p.H; hh = bh % p.H;
-        q0 = pt * kQPair;
-        n0 = min((p.first + q0 + kQTile - 1) / kKvTile + 1, n_kv_seq);    // causal: keys 0 .. first+q0+127
-        n1 = (q0 + kQTile < p.T) ? min((p.first + q0 + 2 * kQTile - 1) / kKvTile + 1, n_kv_seq) : 0;   // second tile exists only inside the sequence
-        js = 0; d1 = 0;
+        w.bb = bh / p.H; w.hh = bh % p.H;
+        w.q0 = pt * kQPair;
+        const int last0 = min((p.first + w.q0 + kQTile - 1) / kKvTile, n_kv_seq - 1);               // causal: keys 0 .. first+q0+127
+        const int last1 = (w.q0 + kQTile < p.T) ? min((p.first + w.q0 + 2 * kQTile - 1) / kKvTile, n_kv_seq - 1) : -1;      // second tile exists only inside the sequence
+        const int last = max(last0, last1);
         if constexpr (WIN) {
-            js = max(0, p.first + q0 - p.window + 1) / kKvTile;
-            n0 -= js;
-            if (n1 > 0) { n1 -= js; d1 = max(0, p.first + q0 + kQTile - p.window + 1) / kKvTile > js ? 1 : 0; }
+            const int from0 = max(0, p.first + w.q0 - p.window + 1) / kKvTile, from1 = max(0, p.first + w.q0 + kQTile - p.window + 1) / kKvTile;
+            w.N = last - from0 + 1; w.k0 = last; w.dir = -1;
+            w.b[0] = last - last0; w.e[0] = w.N;
+            w.b[1] = 0; w.e[1] = last1 < 0 ? 0 : last - from1 + 1;
+        } else {
+            w.N = last + 1; w.k0 = 0; w.dir = 1;
+            w.b[0] = 0; w.e[0] = last0 + 1;
+            w.b[1] = 0; w.e[1] = last1 + 1;
         }
+        return w;
+    };
+    // the products of an item in issue order: step by step, query tile 0 before query tile 1 where both take part
+    auto entries = [&](const Item& w) -> int { return (w.e[0] - w.b[0]) + (w.e[1] - w.b[1]); };
+    auto entries_before = [&](const Item& w, int t, int j) -> int {
+        auto done = [&](int u, int steps) { return max(0, min(steps, w.e[u]) - w.b[u]); };
+        return done(0, t == 1 ? j + 1 : j) + done(1, j);
     };
 
     if (warp == 0) {
@@ -252,10 +268,9 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         uint32_t g = 0, it = 0;
         for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
             const int item_next = fetch(k + 1);
-            int q0, bb, hh, n0, n1, js, d1;
-            decode(item, q0, bb, hh, n0, n1, js, d1);
+            const Item w = decode(item);
             item = item_next;
-            const int nmax = max(n0, n1), kh = WIN ? hh / p.group : hh;
+            const int q0 = w.q0, bb = w.bb, hh = w.hh, nmax = w.N, kh = WIN ? hh / p.group : hh;
             ok = mbar_wait(q_free, (it & 1) ^ 1, abort_flag, p.status, kErrProducerWait);
             if (!ok) break;
             if (lane == 0) {
@@ -275,8 +290,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (lane == 0) {
                         const uint32_t dst = base + L::kK + s * L::kKBytes;
                         mbar_expect_tx(k_full + 8 * s, L::kKBytes);
-                        for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, k_full + 8 * s, kb * 64, (js + j) * kKvTile, kh, bb);
-                        for (int kb = 0; kb < KBR; kb++) tma_load_4d(dst + (KBN + kb) * (kKvTile * 128), &tmKr, k_full + 8 * s, kb * 64, j * kKvTile, 0, bb);
+                        for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, k_full + 8 * s, kb * 64, (w.k0 + w.dir * j) * kKvTile, kh, bb);
+                        for (int kb = 0; kb < KBR; kb++) tma_load_4d(dst + (KBN + kb) * (kKvTile * 128), &tmKr, k_full + 8 * s, kb * 64, (w.k0 + w.dir * j) * kKvTile, 0, bb);
                     }
                     __syncwarp();
                 }
@@ -287,7 +302,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (lane == 0) {
                         const uint32_t dst = base + L::kV + s * L::kVBytes;
                         mbar_expect_tx(v_full + 8 * s, L::kVBytes);
-                        for (int kb = 0; kb < VD / 64; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmV, v_full + 8 * s, kb * 64, (js + j - 1) * kKvTile, kh, bb);
+                        for (int kb = 0; kb < VD / 64; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmV, v_full + 8 * s, kb * 64, (w.k0 + w.dir * (j - 1)) * kKvTile, kh, bb);
                     }
                     __syncwarp();
                 }
@@ -354,13 +369,14 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             };
             for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
                 const int item_next = fetch(k + 1);
-                int q0, bb, hh, n0, n1, js, d1;
-                decode(item, q0, bb, hh, n0, n1, js, d1);
+                const Item w = decode(item);
                 item = item_next;
-                const int E = n0 + n1 - d1, nmin = min(n0, n1), t_long = n1 > n0 ? 1 : 0;
+                const int E = entries(w), both_b = w.b[0], both_e = max(both_b, min(w.e[0], w.e[1]));      // steps both tiles take part in
                 auto entry = [&](int e, int& t, int& j) {
-                    if (WIN && e > 0) e += d1;              // (tile 1, key tile 0) is left out
-                    if (e < 2 * nmin) { j = e >> 1; t = e & 1; } else { j = nmin + (e - 2 * nmin); t = t_long; }
+                    if (e < both_b) { j = e; t = 1; return; }              // b[1] is 0
+                    e -= both_b;
+                    const int two = 2 * (both_e - both_b);
+                    if (e < two) { j = both_b + (e >> 1); t = e & 1; } else { j = both_e + (e - two); t = w.e[1] > w.e[0] ? 1 : 0; }
                 };
                 ok = mbar_wait(q_full, it & 1, abort_flag, p.status, kErrMmaWait);
                 if (!ok) break;
@@ -387,38 +403,34 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     const uint32_t n = G + e, buf = n % 3;
                     ok = mbar_wait(p_full + 8 * buf, (n / 3) & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == (t ? d1 : 0)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == w.b[t]) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
                     if (ok && j > v_seen) { ok = v_ready(g + j); v_seen = j; }
                     if (!ok) break;
                     tc_fence_after();
                     int tn = 0, jn = -1;
                     if (e + 1 < E) entry(e + 1, tn, jn);
                     if (elect_one_sync()) {
-                        issue_pv3(t, g + j, n, j > (t ? d1 : 0), steps[t]);
+                        issue_pv3(t, g + j, n, j > w.b[t], steps[t]);
                         if (jn != j) mma_commit(v_empty + 8 * ((g + j) % NSV));     // every MMA that reads these values has been issued
                     }
                     __syncwarp();
                     steps[t]++;
                 }
-                g += max(n0, n1);
+                g += w.N;
                 G += E;
             }
         } else
         for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
             const int item_next = fetch(k + 1);
-            int q0, bb, hh, n0, n1, js, d1;
-            decode(item, q0, bb, hh, n0, n1, js, d1);
+            const Item w = decode(item);
             item = item_next;
-            const int nt[2] = {n0, n1};
-            const int nmax = max(n0, n1);
-            const int last_t = n1 > 0 ? 1 : 0;             // the tile whose last Q K^T is the item's last read of Q
+            const int nmax = w.N;
             ok = mbar_wait(q_full, it & 1, abort_flag, p.status, kErrMmaWait) && k_ready(g);
             if (!ok) break;
             tc_fence_after();
             if (elect_one_sync()) {
-                issue_s(0, g);
-                if (n1 > 0 && d1 == 0) issue_s(1, g);
-                if (nt[last_t] == 1) mma_commit(q_free);
+                for (int t = 0; t < 2; t++) if (w.b[t] == 0 && w.e[t] > 0) issue_s(t, g);
+                if (nmax == 1) mma_commit(q_free);          // the item's last read of Q
                 mma_commit(k_empty + 8 * (g % NSK));
             }
             __syncwarp();
@@ -426,36 +438,31 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 ok = (j + 1 >= nmax || k_ready(g + 1)) && v_ready(g);
                 if (!ok) break;
                 for (int t = 0; t < 2 && ok; t++) {
-                    if (j >= nt[t]) continue;
-                    if (WIN && t == 1 && j < d1) {             // nothing of this key tile: only the scores of the next one
-                        if (elect_one_sync()) {
-                            tc_fence_after();
-                            issue_s(1, g + 1);
-                            if (last_t == 1 && nt[1] == 2) mma_commit(q_free);
-                        }
+                    if (j >= w.e[t]) continue;
+                    if (j < w.b[t]) {                          // joins at the next step: only its first scores
+                        tc_fence_after();
+                        if (elect_one_sync()) issue_s(t, g + 1);
                         __syncwarp();
                         continue;
                     }
                     ok = mbar_wait(p_full + 8 * t, steps[t] & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == (t ? d1 : 0)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == w.b[t]) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
                     if (!ok) break;
                     steps[t]++;
                     tc_fence_after();
                     if (elect_one_sync()) {
-                        issue_pv(t, g, j > (t ? d1 : 0), steps[t] - 1);
+                        issue_pv(t, g, j > w.b[t], steps[t] - 1);
                         // the next scores of this tile go into the columns P was just read from: the tensor pipe runs the
                         // MMAs of one thread in order, so the product above has consumed P before these overwrite it
-                        if (j + 1 < nt[t]) {
-                            issue_s(t, g + 1);
-                            if (t == last_t && j + 2 == nt[t]) mma_commit(q_free);
-                        }
+                        if (j + 1 < w.e[t]) issue_s(t, g + 1);
                     }
                     __syncwarp();
                 }
                 if (ok && elect_one_sync()) {                   // every MMA that reads V_j, and K_(j+1), has been issued
                     mma_commit(v_empty + 8 * (g % NSV));
                     if (j + 1 < nmax) mma_commit(k_empty + 8 * ((g + 1) % NSK));
+                    if (j + 2 == nmax) mma_commit(q_free);
                 }
                 __syncwarp();
             }
@@ -472,26 +479,24 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         uint32_t G = 0;                                          // ROT: scores of earlier items (both tiles), as the MMA warp counts them
         for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
             const int item_next = fetch(k + 1);
-            int q0, bb, hh, n0, n1, js, d1;
-            decode(item, q0, bb, hh, n0, n1, js, d1);
+            const Item w = decode(item);
             item = item_next;
-            const int n_kv = t == 0 ? n0 : n1;
+            const int q0 = w.q0, bb = w.bb, hh = w.hh, j_first = w.b[t], n_kv = w.e[t];
             const int qrow = q0 + t * kQTile + r;
             // WIN: kUnseen until the row's first visible key (masked scores are -inf: their weights and sums are then zeros)
             constexpr float kUnseen = -1e30f;
             float m = WIN ? kUnseen : -INFINITY, l = 0.0f;
-            const int j_first = t == 1 ? d1 : 0;
             const float slope = WIN && p.slopes ? __ldg(p.slopes + hh) * 1.4426950408889634f : 0.0f;
             for (int j = j_first; j < n_kv && ok; j++, step++) {
                 // ROT: this step's scores are number G + (entries of the item before (t, j)) of the kernel, in buffer number % 3
-                const uint32_t sn = ROT ? G + (uint32_t)(min(j, n0) + min(j, n1) + ((t == 1 && j < n0) ? 1 : 0) - (WIN && j > 0 ? d1 : 0)) : step;
+                const uint32_t sn = ROT ? G + (uint32_t)entries_before(w, t, j) : step;
                 const uint32_t sbuf = ROT ? sn % 3 : (uint32_t)t;
                 const uint32_t s_addr = tmem_base + lane_off + sbuf * 128;          // scores, and P over their first 64 columns
                 ok = mbar_wait(s_full + 8 * sbuf, (ROT ? sn / 3 : sn) & 1, abort_flag, p.status, kErrEpilogueWait);
                 if (!ok) break;
                 tc_fence_after();
                 // row r of the tile sees the keys of this tile up to column r + delta
-                const int delta = p.first + q0 + t * kQTile - (js + j) * kKvTile;
+                const int delta = p.first + q0 + t * kQTile - (w.k0 + w.dir * j) * kKvTile;
                 // ... and (WIN) from column r + delta - window + 1 on
                 const bool diag = delta < kKvTile - 1 || (WIN && delta > p.window - kQTile);
                 // The 128 scores of the row are taken in four chunks of 32: the load of chunk c + 1 is in flight while chunk c is
@@ -505,12 +510,14 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 const float mul = WIN ? 1.0f : p.scale_log2;
                 const float2 c2 = make_float2(mul, mul);
                 uint32_t va[32], vb[32];
-                tmem_ld_32x32(s_addr, va);
+                tmem_ld_32x32(s_addr + (WIN ? 96 : 0), va);
                 auto chunk = [&](auto c_tag, uint32_t (&v)[32], uint32_t (&vnext)[32], auto diag_tag) -> bool {
-                    constexpr int c = decltype(c_tag)::value;
+                    constexpr int n = decltype(c_tag)::value;           // chunks before this one
+                    auto column_chunk = [](int i) { return WIN ? 3 - i : i; };
+                    constexpr int c = WIN ? 3 - n : n;
                     constexpr bool DIAG = decltype(diag_tag)::value;
                     tmem_ld_wait();
-                    if (c < 3) tmem_ld_32x32(s_addr + (c + 1) * 32, vnext);
+                    if (n < 3) tmem_ld_32x32(s_addr + column_chunk(n + 1) * 32, vnext);
                     if constexpr (WIN) {
                         const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), sl2 = make_float2(slope, slope);
                         const float b0 = slope * (float)(c * 32 - r - delta);
@@ -536,7 +543,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     }
                     const float mx = fmaxf(max3(m0, m1, m2), m3);
                     if constexpr (WIN) { if (m == kUnseen) m = fmaxf(mx, kUnseen); }     // everything accumulated so far is zero: nothing to rescale
-                    else if (j == 0 && c == 0) m = mx;               // the first chunk of a row always holds key 0: finite
+                    else if (j == 0 && n == 0) m = mx;               // the first chunk of a row always holds key 0: finite
                     const bool grow = (mx - m) * mul > 8.0f;
                     if (__any_sync(0xffffffffu, grow)) {
                         tmem_ld_wait();                          // the next chunk's registers may be moved below: they must have arrived
@@ -559,35 +566,35 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                                 tmem_st_32x32(o_addr + cc * 32, o);
                             }
                         }
-                        if (c > 0) tmem_st_wait();               // P's chunks have landed before they are read back
-                        if (c > 0 && PSPLIT) {
-                            uint32_t w[32];
+                        if (n > 0) tmem_st_wait();               // P's chunks have landed before they are read back
+                        if (n > 0 && PSPLIT) {
+                            uint32_t u[32];
 #pragma unroll
-                            for (int cc = 0; cc < c; cc++) {
-                                tmem_ld_32x32(s_addr + cc * 32, w);
+                            for (int cc = 0; cc < n; cc++) {
+                                tmem_ld_32x32(s_addr + column_chunk(cc) * 32, u);
                                 tmem_ld_wait();
 #pragma unroll
                                 for (int i = 0; i < 16; i++) {
-                                    const float lo = (__uint_as_float(w[i] << 16) + __uint_as_float(w[i + 16] << 16)) * alpha;
-                                    const float hi = (__uint_as_float(w[i] & 0xffff0000u) + __uint_as_float(w[i + 16] & 0xffff0000u)) * alpha;
-                                    split2(make_float2(lo, hi), w[i], w[i + 16]);
+                                    const float lo = (__uint_as_float(u[i] << 16) + __uint_as_float(u[i + 16] << 16)) * alpha;
+                                    const float hi = (__uint_as_float(u[i] & 0xffff0000u) + __uint_as_float(u[i + 16] & 0xffff0000u)) * alpha;
+                                    split2(make_float2(lo, hi), u[i], u[i + 16]);
                                 }
-                                tmem_st_32x32(s_addr + cc * 32, w);
+                                tmem_st_32x32(s_addr + column_chunk(cc) * 32, u);
                             }
-                        } else if (c > 0) {
+                        } else if (n > 0) {
                             // the chunks of P of this tile written so far: 16 columns (32 bf16) each
-                            uint32_t w[16];
+                            uint32_t u[16];
 #pragma unroll
-                            for (int cc = 0; cc < c; cc++) {
-                                tmem_ld_32x32b_x16(s_addr + cc * 16, w);
+                            for (int cc = 0; cc < n; cc++) {
+                                tmem_ld_32x32b_x16(s_addr + cc * 16, u);
                                 tmem_ld_wait();
 #pragma unroll
                                 for (int i = 0; i < 16; i++) {
-                                    const float lo = __uint_as_float(w[i] << 16) * alpha, hi = __uint_as_float(w[i] & 0xffff0000u) * alpha;
+                                    const float lo = __uint_as_float(u[i] << 16) * alpha, hi = __uint_as_float(u[i] & 0xffff0000u) * alpha;
                                     __nv_bfloat162 h2 = __floats2bfloat162_rn(lo, hi);
-                                    w[i] = *reinterpret_cast<uint32_t*>(&h2);
+                                    u[i] = *reinterpret_cast<uint32_t*>(&h2);
                                 }
-                                tmem_st_32x32b_x16(s_addr + cc * 16, w);
+                                tmem_st_32x32b_x16(s_addr + cc * 16, u);
                             }
                         }
                         tmem_st_wait();
@@ -627,7 +634,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 if (lane == 0) mbar_arrive(p_full + 8 * sbuf);
                 l += (sum_a.x + sum_a.y) + (sum_b.x + sum_b.y);
             }
-            G += (uint32_t)(n0 + n1 - d1);
+            G += (uint32_t)entries(w);
             if (!ok) break;
             if (n_kv > 0) {
                 float inv = 1.0f / l;

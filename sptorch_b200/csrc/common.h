@@ -106,7 +106,7 @@ __device__ __forceinline__ float2 bf16x2_to_float2(__nv_bfloat162 h) {
 }
 
 // Per-category device timing (CUDA events around launches on the library stream); off by default.
-enum ProfCat : int { PROF_LINEAR = 0, PROF_ATTN_GEMM = 1, PROF_SOFTMAX = 2, PROF_LAYERNORM = 3, PROF_EMBED = 4, PROF_OTHER = 5, PROF_ATTN_FUSED = 6, PROF_RECURRENT = 7, PROF_LATENT = 8, PROF_NCAT = 9 };
+enum ProfCat : int { PROF_LINEAR = 0, PROF_ATTN_GEMM = 1, PROF_SOFTMAX = 2, PROF_LAYERNORM = 3, PROF_EMBED = 4, PROF_OTHER = 5, PROF_ATTN_FUSED = 6, PROF_RECURRENT = 7, PROF_LATENT = 8, PROF_CONV = 9, PROF_NCAT = 10 };
 bool prof_enabled();
 void prof_begin(int cat);
 void prof_end(int cat);

@@ -321,7 +321,7 @@ WindowArgs window_args(Gpt* g, const LayeredLayer& w, int B, int T, int first, c
 int window_layer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
     const WindowArgs a = window_args(g, w, B, T, first, pos_dev, cached);
     const bool decode = few && cached && window_decode_supported(a), fresh = decode && T == 1;
-    if (!fresh) { ProfScope ps(PROF_LATENT); if (window_prep(a, few)) return 1; }
+    if (!fresh) { ProfScope ps(PROF_CONV); if (window_prep(a, few)) return 1; }
     ProfScope ps(PROF_ATTN_FUSED);
     if (decode) return window_decode(a, fresh, true);
     if (!few && g->c.dtype == BF16 && attention_window_supported(a.D, a.V, a.row, a.ld_out))
