@@ -229,9 +229,14 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const int at = k * (int)gridDim.x + (int)blockIdx.x;
         return p.sched ? __ldg(p.sched + at) : at < p.n_ptiles * BH ? at : -1;
     };
-    // work item -> (first query row, sequence, head); steps 0 .. N - 1 go over key tiles k0, k0 + dir, ..; query tile t takes part in steps
-    // b[t] .. e[t] - 1
-    struct Item { int q0, bb, hh, N, k0, dir, b[2], e[2]; };
+    // work item -> (first query row, sequence, head); steps 0 .. N - 1 go over the key tiles (WIN: from k_last down, otherwise from 0 up);
+    // query tile 0 takes part in steps b0 .. e0 - 1 (b0 = 0 without WIN), tile 1 in steps 0 .. e1 - 1
+    struct Item {
+        int q0, bb, hh, N, k_last, b0, e0, e1;
+        __device__ __forceinline__ int key_tile(int step) const { return WIN ? k_last - step : step; }
+        __device__ __forceinline__ int begin(int t) const { return WIN && t == 0 ? b0 : 0; }
+        __device__ __forceinline__ int end(int t) const { return t == 0 ? e0 : e1; }
+    };
     auto decode = [&](int item) -> Item {
         Item w;
         const int pt = p.n_ptiles - 1 - item / BH;
@@ -243,21 +248,19 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const int last = max(last0, last1);
         if constexpr (WIN) {
             const int from0 = max(0, p.first + w.q0 - p.window + 1) / kKvTile, from1 = max(0, p.first + w.q0 + kQTile - p.window + 1) / kKvTile;
-            w.N = last - from0 + 1; w.k0 = last; w.dir = -1;
-            w.b[0] = last - last0; w.e[0] = w.N;
-            w.b[1] = 0; w.e[1] = last1 < 0 ? 0 : last - from1 + 1;
+            w.N = w.e0 = last - from0 + 1; w.k_last = last; w.b0 = last - last0;
+            w.e1 = last1 < 0 ? 0 : last - from1 + 1;
         } else {
-            w.N = last + 1; w.k0 = 0; w.dir = 1;
-            w.b[0] = 0; w.e[0] = last0 + 1;
-            w.b[1] = 0; w.e[1] = last1 + 1;
+            w.N = last + 1; w.k_last = 0; w.b0 = 0;
+            w.e0 = last0 + 1; w.e1 = last1 + 1;
         }
         return w;
     };
     // the products of an item in issue order: step by step, query tile 0 before query tile 1 where both take part
-    auto entries = [&](const Item& w) -> int { return (w.e[0] - w.b[0]) + (w.e[1] - w.b[1]); };
+    auto entries = [&](const Item& w) -> int { return w.e0 - w.begin(0) + w.e1; };
     auto entries_before = [&](const Item& w, int t, int j) -> int {
-        auto done = [&](int u, int steps) { return max(0, min(steps, w.e[u]) - w.b[u]); };
-        return done(0, t == 1 ? j + 1 : j) + done(1, j);
+        if constexpr (WIN) return max(0, (t == 1 ? j + 1 : j) - w.b0) + min(j, w.e1);       // tile 0 stays to the last step
+        else return min(j, w.e0) + min(j, w.e1) + ((t == 1 && j < w.e0) ? 1 : 0);
     };
 
     if (warp == 0) {
@@ -290,8 +293,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (lane == 0) {
                         const uint32_t dst = base + L::kK + s * L::kKBytes;
                         mbar_expect_tx(k_full + 8 * s, L::kKBytes);
-                        for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, k_full + 8 * s, kb * 64, (w.k0 + w.dir * j) * kKvTile, kh, bb);
-                        for (int kb = 0; kb < KBR; kb++) tma_load_4d(dst + (KBN + kb) * (kKvTile * 128), &tmKr, k_full + 8 * s, kb * 64, (w.k0 + w.dir * j) * kKvTile, 0, bb);
+                        for (int kb = 0; kb < KBN; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmK, k_full + 8 * s, kb * 64, w.key_tile(j) * kKvTile, kh, bb);
+                        for (int kb = 0; kb < KBR; kb++) tma_load_4d(dst + (KBN + kb) * (kKvTile * 128), &tmKr, k_full + 8 * s, kb * 64, w.key_tile(j) * kKvTile, 0, bb);
                     }
                     __syncwarp();
                 }
@@ -302,7 +305,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     if (lane == 0) {
                         const uint32_t dst = base + L::kV + s * L::kVBytes;
                         mbar_expect_tx(v_full + 8 * s, L::kVBytes);
-                        for (int kb = 0; kb < VD / 64; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmV, v_full + 8 * s, kb * 64, (w.k0 + w.dir * (j - 1)) * kKvTile, kh, bb);
+                        for (int kb = 0; kb < VD / 64; kb++) tma_load_4d(dst + kb * (kKvTile * 128), &tmV, v_full + 8 * s, kb * 64, w.key_tile(j - 1) * kKvTile, kh, bb);
                     }
                     __syncwarp();
                 }
@@ -371,12 +374,12 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 const int item_next = fetch(k + 1);
                 const Item w = decode(item);
                 item = item_next;
-                const int E = entries(w), both_b = w.b[0], both_e = max(both_b, min(w.e[0], w.e[1]));      // steps both tiles take part in
+                // before joined_0 tile 1 is alone, from joined_1 on the tile that has more
+                const int E = entries(w), joined_0 = w.begin(0), joined_1 = max(joined_0, min(w.e0, w.e1)), two = 2 * joined_1 - joined_0, t_long = w.e1 > w.e0 ? 1 : 0;
                 auto entry = [&](int e, int& t, int& j) {
-                    if (e < both_b) { j = e; t = 1; return; }              // b[1] is 0
-                    e -= both_b;
-                    const int two = 2 * (both_e - both_b);
-                    if (e < two) { j = both_b + (e >> 1); t = e & 1; } else { j = both_e + (e - two); t = w.e[1] > w.e[0] ? 1 : 0; }
+                    if (WIN && e < joined_0) { j = e; t = 1; }
+                    else if (e < two) { j = (e + joined_0) >> 1; t = (e + joined_0) & 1; }
+                    else { j = joined_1 + (e - two); t = t_long; }
                 };
                 ok = mbar_wait(q_full, it & 1, abort_flag, p.status, kErrMmaWait);
                 if (!ok) break;
@@ -403,14 +406,14 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     const uint32_t n = G + e, buf = n % 3;
                     ok = mbar_wait(p_full + 8 * buf, (n / 3) & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == w.b[t]) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == w.begin(t)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
                     if (ok && j > v_seen) { ok = v_ready(g + j); v_seen = j; }
                     if (!ok) break;
                     tc_fence_after();
                     int tn = 0, jn = -1;
                     if (e + 1 < E) entry(e + 1, tn, jn);
                     if (elect_one_sync()) {
-                        issue_pv3(t, g + j, n, j > w.b[t], steps[t]);
+                        issue_pv3(t, g + j, n, j > w.begin(t), steps[t]);
                         if (jn != j) mma_commit(v_empty + 8 * ((g + j) % NSV));     // every MMA that reads these values has been issued
                     }
                     __syncwarp();
@@ -429,7 +432,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             if (!ok) break;
             tc_fence_after();
             if (elect_one_sync()) {
-                for (int t = 0; t < 2; t++) if (w.b[t] == 0 && w.e[t] > 0) issue_s(t, g);
+                for (int t = 0; t < 2; t++) if (w.begin(t) == 0 && w.end(t) > 0) issue_s(t, g);
                 if (nmax == 1) mma_commit(q_free);          // the item's last read of Q
                 mma_commit(k_empty + 8 * (g % NSK));
             }
@@ -438,8 +441,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 ok = (j + 1 >= nmax || k_ready(g + 1)) && v_ready(g);
                 if (!ok) break;
                 for (int t = 0; t < 2 && ok; t++) {
-                    if (j >= w.e[t]) continue;
-                    if (j < w.b[t]) {                          // joins at the next step: only its first scores
+                    if (j >= w.end(t)) continue;
+                    if (j < w.begin(t)) {                          // joins at the next step: only its first scores
                         tc_fence_after();
                         if (elect_one_sync()) issue_s(t, g + 1);
                         __syncwarp();
@@ -447,15 +450,15 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     }
                     ok = mbar_wait(p_full + 8 * t, steps[t] & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == w.b[t]) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == w.begin(t)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
                     if (!ok) break;
                     steps[t]++;
                     tc_fence_after();
                     if (elect_one_sync()) {
-                        issue_pv(t, g, j > w.b[t], steps[t] - 1);
+                        issue_pv(t, g, j > w.begin(t), steps[t] - 1);
                         // the next scores of this tile go into the columns P was just read from: the tensor pipe runs the
                         // MMAs of one thread in order, so the product above has consumed P before these overwrite it
-                        if (j + 1 < w.e[t]) issue_s(t, g + 1);
+                        if (j + 1 < w.end(t)) issue_s(t, g + 1);
                     }
                     __syncwarp();
                 }
@@ -481,7 +484,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             const int item_next = fetch(k + 1);
             const Item w = decode(item);
             item = item_next;
-            const int q0 = w.q0, bb = w.bb, hh = w.hh, j_first = w.b[t], n_kv = w.e[t];
+            const int q0 = w.q0, bb = w.bb, hh = w.hh, j_first = w.begin(t), n_kv = w.end(t);
             const int qrow = q0 + t * kQTile + r;
             // WIN: kUnseen until the row's first visible key (masked scores are -inf: their weights and sums are then zeros)
             constexpr float kUnseen = -1e30f;
@@ -496,7 +499,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 if (!ok) break;
                 tc_fence_after();
                 // row r of the tile sees the keys of this tile up to column r + delta
-                const int delta = p.first + q0 + t * kQTile - (w.k0 + w.dir * j) * kKvTile;
+                const int delta = p.first + q0 + t * kQTile - w.key_tile(j) * kKvTile;
                 // ... and (WIN) from column r + delta - window + 1 on
                 const bool diag = delta < kKvTile - 1 || (WIN && delta > p.window - kQTile);
                 // The 128 scores of the row are taken in four chunks of 32: the load of chunk c + 1 is in flight while chunk c is
@@ -506,32 +509,23 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 // written -- is multiplied by 2^(old - new) at that moment.  tcgen05.ld / st are warp-wide, so a warp rescales when any
                 // of its rows does (the others multiply by one).
                 float2 sum_a = make_float2(0.0f, 0.0f), sum_b = make_float2(0.0f, 0.0f);
-                // WIN: the scores become scale * s - slope * (r + delta - column) (times log2 e) before anything else is done with them
+                // WIN: m is in units of the exponent, and the maximum of a chunk is estimated as that of the unbiased scores plus the bias of the
+                // chunk's nearest key: too high by at most the bias of 31 keys (2^45), which a row sum in f32 does not notice
                 const float mul = WIN ? 1.0f : p.scale_log2;
-                const float2 c2 = make_float2(mul, mul);
+                const float2 c2 = make_float2(p.scale_log2, p.scale_log2);
                 uint32_t va[32], vb[32];
                 tmem_ld_32x32(s_addr + (WIN ? 96 : 0), va);
                 auto chunk = [&](auto c_tag, uint32_t (&v)[32], uint32_t (&vnext)[32], auto diag_tag) -> bool {
-                    constexpr int n = decltype(c_tag)::value;           // chunks before this one
+                    const int n = c_tag;                               // chunks before this one
                     auto column_chunk = [](int i) { return WIN ? 3 - i : i; };
-                    constexpr int c = WIN ? 3 - n : n;
+                    const int c = column_chunk(n);
                     constexpr bool DIAG = decltype(diag_tag)::value;
                     tmem_ld_wait();
                     if (n < 3) tmem_ld_32x32(s_addr + column_chunk(n + 1) * 32, vnext);
-                    if constexpr (WIN) {
-                        const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), sl2 = make_float2(slope, slope);
-                        const float b0 = slope * (float)(c * 32 - r - delta);
-                        const float2 b2 = make_float2(b0, b0);
-#pragma unroll
-                        for (int i = 0; i < 32; i += 2) {
-                            const float2 x = __ffma2_rn(make_float2(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), sc2, __ffma2_rn(sl2, make_float2((float)i, (float)(i + 1)), b2));
-                            v[i] = __float_as_uint(x.x); v[i + 1] = __float_as_uint(x.y);
-                        }
-                    }
                     if (DIAG) {
 #pragma unroll
                         for (int i = 0; i < 32; i++)
-                            if (c * 32 + i > r + delta || (WIN && c * 32 + i <= r + delta - p.window)) v[i] = 0xff800000u;       // -inf right of the diagonal
+                            if (i > r + delta - c * 32 || (WIN && i <= r + delta - c * 32 - p.window)) v[i] = 0xff800000u;       // -inf right of the diagonal
                     }
                     float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
 #pragma unroll
@@ -541,7 +535,9 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         m2 = max3(m2, __uint_as_float(v[i + 4]), __uint_as_float(v[i + 5]));
                         m3 = max3(m3, __uint_as_float(v[i + 6]), __uint_as_float(v[i + 7]));
                     }
-                    const float mx = fmaxf(max3(m0, m1, m2), m3);
+                    float mx = fmaxf(max3(m0, m1, m2), m3);
+                    const float bias0 = WIN ? slope * (float)(c * 32 - r - delta) : 0.0f;          // of the chunk's first key
+                    if constexpr (WIN) mx = fmaf(mx, p.scale_log2, fminf(fmaf(31.0f, slope, bias0), 0.0f));
                     if constexpr (WIN) { if (m == kUnseen) m = fmaxf(mx, kUnseen); }     // everything accumulated so far is zero: nothing to rescale
                     else if (j == 0 && n == 0) m = mx;               // the first chunk of a row always holds key 0: finite
                     const bool grow = (mx - m) * mul > 8.0f;
@@ -556,8 +552,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                             if (!mbar_wait(pv_done + 8 * (2 * t + ((step - 1) & 1)), ((step - 1) >> 1) & 1, abort_flag, p.status, kErrEpilogueWait)) return false;
                             __syncwarp();                        // the wait's lanes leave it one by one, the loads below are warp-wide
                             tc_fence_after();
-#pragma unroll
-                            for (int cc = 0; cc < VD / 32; cc++) {
+#pragma unroll 1
+                            for (int cc = 0; cc < VD / 32; cc++) {       // the rare path: small code counts for more than unrolled loops
                                 uint32_t o[32];
                                 tmem_ld_32x32(o_addr + cc * 32, o);
                                 tmem_ld_wait();
@@ -569,7 +565,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         if (n > 0) tmem_st_wait();               // P's chunks have landed before they are read back
                         if (n > 0 && PSPLIT) {
                             uint32_t u[32];
-#pragma unroll
+#pragma unroll 1
                             for (int cc = 0; cc < n; cc++) {
                                 tmem_ld_32x32(s_addr + column_chunk(cc) * 32, u);
                                 tmem_ld_wait();
@@ -584,7 +580,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         } else if (n > 0) {
                             // the chunks of P of this tile written so far: 16 columns (32 bf16) each
                             uint32_t u[16];
-#pragma unroll
+#pragma unroll 1
                             for (int cc = 0; cc < n; cc++) {
                                 tmem_ld_32x32b_x16(s_addr + cc * 16, u);
                                 tmem_ld_wait();
@@ -602,10 +598,16 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     }
                     const float mb = m * mul;
                     const float2 nmb2 = make_float2(-mb, -mb);
+                    const float2 two_slopes = make_float2(2.0f * slope, 2.0f * slope);
+                    float2 add = nmb2;                           // what the scaled scores of keys 2i, 2i + 1 lack to the exponent
                     uint32_t packed[PSPLIT ? 32 : 16];
 #pragma unroll
                     for (int i = 0; i < 16; i++) {
-                        const float2 x = __ffma2_rn(make_float2(__uint_as_float(v[2 * i]), __uint_as_float(v[2 * i + 1])), c2, nmb2);
+                        if constexpr (WIN) {
+                            if (i % 4 == 0) { add.x = fmaf(2.0f * i, slope, bias0 - mb); add.y = add.x + slope; }
+                            else add = __fadd2_rn(add, two_slopes);
+                        }
+                        const float2 x = __ffma2_rn(make_float2(__uint_as_float(v[2 * i]), __uint_as_float(v[2 * i + 1])), c2, add);
                         const float2 e = make_float2(ex2_approx(x.x), ex2_approx(x.y));
                         if (i & 1) sum_b = __fadd2_rn(sum_b, e); else sum_a = __fadd2_rn(sum_a, e);
                         if constexpr (PSPLIT) split2(e, packed[i], packed[i + 16]);
@@ -621,6 +623,12 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     return true;
                 };
                 auto tile = [&](auto diag_tag) -> bool {
+                    if constexpr (WIN) {                             // a loop of two chunks: the whole tile unrolled outgrows the instruction cache
+#pragma unroll 1
+                        for (int h = 0; h < 4; h += 2)
+                            if (!chunk(h, va, vb, diag_tag) || !chunk(h + 1, vb, va, diag_tag)) return false;
+                        return true;
+                    } else
                     return chunk(std::integral_constant<int, 0>(), va, vb, diag_tag) &&
                            chunk(std::integral_constant<int, 1>(), vb, va, diag_tag) &&
                            chunk(std::integral_constant<int, 2>(), va, vb, diag_tag) &&
@@ -639,6 +647,14 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             if (n_kv > 0) {
                 float inv = 1.0f / l;
                 if (!WIN && p.gate && qrow < p.T) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[((long long)bb * p.T + qrow) * p.ld_gate + hh])));
+                const __nv_bfloat16* grow = WIN && p.gate && qrow < p.T ? p.gate + ((long long)bb * p.T + qrow) * p.ld_gate + (long long)hh * p.V : nullptr;
+                uint4 graw[4];                                   // the next 32 columns' gates, requested ahead of the output they meet
+                auto fetch_gates = [&](int c) {
+#pragma unroll
+                    for (int i = 0; i < 4; i++)
+                        if (c * 32 + i * 8 < p.V) graw[i] = *reinterpret_cast<const uint4*>(grow + c * 32 + i * 8);
+                };
+                if (WIN && grow) fetch_gates(0);
                 // The item's last product -- after the one before it: scores run up to two ahead, so with a single query tile only the product of
                 // step - 4 is sure to be done here, and a parity wait for step - 1 could not tell step - 3 (same barrier, the phase before)
                 // from step - 1.  The product of step - 2 waits on the other barrier, one phase ahead of step - 4, and brings step - 3 with it.
@@ -653,22 +669,25 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     uint32_t o[32];
                     tmem_ld_32x32(o_addr + c * 32, o);
                     tmem_ld_wait();
+                    if constexpr (WIN) {
+                        if (grow) {
+#pragma unroll
+                            for (int i = 0; i < 4; i++) {
+                                const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&graw[i]);
+#pragma unroll
+                                for (int q = 0; q < 4; q++) {
+                                    const float2 gv = bf16x2_to_float2(gh[q]);
+                                    o[8 * i + 2 * q] = __float_as_uint(__fdividef(__uint_as_float(o[8 * i + 2 * q]), 1.0f + __expf(-gv.x)));
+                                    o[8 * i + 2 * q + 1] = __float_as_uint(__fdividef(__uint_as_float(o[8 * i + 2 * q + 1]), 1.0f + __expf(-gv.y)));
+                                }
+                            }
+                            if (c + 1 < VD / 32) fetch_gates(c + 1);
+                        }
+                    }
                     if (qrow < p.T) {
 #pragma unroll
                         for (int i = 0; i < 32; i += 8) {
                             if ((KBR > 0 || WIN) && c * 32 + i >= p.V) break;
-                            if constexpr (WIN) {
-                                if (p.gate) {
-                                    const uint4 graw = *reinterpret_cast<const uint4*>(p.gate + ((long long)bb * p.T + qrow) * p.ld_gate + (long long)hh * p.V + c * 32 + i);
-                                    const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&graw);
-#pragma unroll
-                                    for (int q = 0; q < 4; q++) {
-                                        const float2 gv = bf16x2_to_float2(gh[q]);
-                                        o[i + 2 * q] = __float_as_uint(__uint_as_float(o[i + 2 * q]) * (1.0f / (1.0f + __expf(-gv.x))));
-                                        o[i + 2 * q + 1] = __float_as_uint(__uint_as_float(o[i + 2 * q + 1]) * (1.0f / (1.0f + __expf(-gv.y))));
-                                    }
-                                }
-                            }
                             uint4 w;
                             __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&w);
 #pragma unroll

@@ -329,9 +329,11 @@ int window_layer(Gpt* g, const LayeredLayer& w, int B, int T, int first, const i
     return window_plain(a, few);
 }
 
+// Every CTA of W_down's product applies the activation to all the rows it reads, which pays while the rows are few.
+constexpr int kActOnReadRows = 16;
 // Whether a few rows take the feed-forward's activation on the way into W_down: gate and up then come from one product.
 bool act_on_read(const Gpt* g, const LayeredLayer& w, int M) {
-    if (w.c.mlp != SPT_MLP_DENSE || w.c.mlp_act != SPT_ACT_RELU || w.c.mixer != SPT_MIXER_WINDOW) return false;
+    if (w.c.mlp != SPT_MLP_DENSE || w.c.mlp_act != SPT_ACT_RELU || w.c.mixer != SPT_MIXER_WINDOW || M > kActOnReadRows) return false;
     GemmDesc d = stream_product(const_cast<Gpt*>(g), g->lay->in.p, w.n_in, w.w_o, w.o_ld() + pad8(w.c.d_ff), w.o_ld() + pad8(w.c.d_ff), (float*)g->lay->x.p, M);
     d.act_off = pad8(w.c.d_ff); d.act_from = w.o_ld();
     return linear_few_rows_supported(d);
