@@ -90,6 +90,7 @@ bool gemm_supported(const GemmDesc& d, const char** why);
 // kernel in the stream (see launch_dependent in common.h).
 // kind 3: the rows are a residual stream that still lacks the sublayer output before it, a = x + y / sqrt(mean(y^2) + eps) * gamma (x
 // f32, y bf16, rows of K elements, the mean over `dim` of them); a goes to x_out (f32, not x) and xb (bf16) too, for those who come after.
+// kind 4: the same, and the product reads a / sqrt(mean(a^2) + eps) * gamma2 (the next sublayer's norm); xb may be null.
 struct RowNorm {
     int kind = 0;
     const float* gamma = nullptr; const float* beta = nullptr;
@@ -97,6 +98,7 @@ struct RowNorm {
     int dim = 0;
     const float* x = nullptr; const __nv_bfloat16* y = nullptr;
     float* x_out = nullptr; __nv_bfloat16* xb = nullptr;
+    const float* gamma2 = nullptr;
 };
 bool linear_few_rows_supported(const GemmDesc& d);
 bool linear_few_rows_norm_supported(const GemmDesc& d, const RowNorm& nrm);

@@ -352,13 +352,25 @@ const void* mixer_out(const Gpt* g, const LayeredLayer& w, long long* ld) {
 
 int gated_epilogue(const LayeredLayer& w) { return w.c.mlp_act == SPT_ACT_RELU ? EPI_RELU_MUL : EPI_SWIGLU; }
 
-// A layer of a parallel block.  lay.xb holds rms(x) * norm1; afterwards x lacks only the normed lay.y (when there is a token input).
-int parallel_layer(Gpt* g, const LayeredLayer& w, int l, float* x, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
+// Whether the input projection of a parallel layer takes its rows as a stream to be completed (and the activation of its feed-forward is
+// left to W_down, so that nothing else reads the normed rows).
+bool parallel_takes_norm(Gpt* g, const LayeredLayer& w, const RowNorm& n, int M) {
+    if (w.c.mlp == SPT_MLP_DENSE && !act_on_read(g, w, M)) return false;
+    GemmDesc d;
+    d.A = g->lay->xb.p; d.B = w.w_in; d.C = g->lay->in.p; d.M = M; d.N = w.n_in; d.K = g->lay->d8; d.lda = d.ldb = d.K; d.ldc = w.n_in;
+    d.mode = g->c.dtype == BF16 ? MM_BF16 : MM_F32; d.out_dtype = g->c.dtype;
+    return linear_few_rows_norm_supported(d, n);
+}
+
+// A layer of a parallel block.  lay.xb holds rms(x) * norm1, or (pend) the input projection makes it from the stream that lacks the layer
+// before; afterwards x lacks only the normed lay.y (when there is a token input).
+int parallel_layer(Gpt* g, const LayeredLayer& w, int l, const RowNorm* pend, float* x, int B, int T, int first, const int* pos_dev, bool few, bool cached) {
     Layered& lay = *g->lay;
     const int M = B * T, d8 = lay.d8, dense = w.c.mlp == SPT_MLP_DENSE, f8 = dense ? pad8(w.c.d_ff) : 0, o8 = w.o_ld();
     const bool act = few && act_on_read(g, w, M);
     uint8_t* in = (uint8_t*)lay.in.p;
-    if (product(g, few, lay.xb.p, d8, w.w_in, d8, d8, nullptr, nullptr, in, w.n_in, M, act ? w.n_in : w.n_in - f8, EPI_NONE)) return 1;
+    bool fused = false;
+    if (product(g, few, lay.xb.p, d8, w.w_in, d8, d8, nullptr, nullptr, in, w.n_in, M, act ? w.n_in : w.n_in - f8, EPI_NONE, pend, &fused)) return 1;
     void* up = in + (size_t)w.c_up * g->es;
     if (dense && !act && product(g, few, lay.xb.p, d8, (uint8_t*)w.w_in + (size_t)w.c_gate * d8 * g->es, d8, d8, nullptr, up, up, w.n_in, M, f8, gated_epilogue(w))) return 1;
     if (mixer(g, w, B, T, first, pos_dev, few, cached)) return 1;
@@ -436,11 +448,16 @@ int run(Gpt* g, const void* ids, int B, int T, int first, const int* pos_dev, bo
     };
     const int nl = (int)lay.L.size();
     const bool parallel = lay.opt.block == SPT_BLOCK_PARALLEL;
-    if (parallel && nl > 0 && settle(lay.L[0].norm1)) return 1;
     for (int l = 0; l < nl && parallel; l++) {
-        if (parallel_layer(g, lay.L[l], l, x, B, T, first, pos_dev, few, cached)) return 1;
-        if (lay.opt.side_dim > 0) pending = lay.L[l].side_norm;
-        if (l < nl - 1 && (settle(lay.L[l + 1].norm1) || tap(l + 1))) return 1;       // the next layer's input, too
+        const LayeredLayer& w = lay.L[l];
+        // one or two rows: the input projection completes the stream and norms it
+        RowNorm n;
+        n.kind = 4; n.gamma = pending; n.gamma2 = w.norm1; n.eps = c.eps; n.dim = c.d_model; n.x = x; n.y = (const __nv_bfloat16*)lay.y.p; n.x_out = x_other;
+        const bool on_the_way = pending && few && !g->taps_on && parallel_takes_norm(g, w, n, M);
+        if (on_the_way) { std::swap(x, x_other); pending = nullptr; }
+        else if (settle(w.norm1) || (l > 0 && tap(l))) return 1;
+        if (parallel_layer(g, w, l, on_the_way ? &n : nullptr, x, B, T, first, pos_dev, few, cached)) return 1;
+        if (lay.opt.side_dim > 0) pending = w.side_norm;
     }
     for (int l = 0; l < nl && !parallel; l++) {
         const LayeredLayer& w = lay.L[l];
@@ -567,8 +584,9 @@ void layered_release(Gpt* g) { delete g->lay; g->lay = nullptr; }
 namespace {
 
 // one entry per tensor: its name behind the layer's prefix, its shape, and where it goes
-struct Slot { std::string name; size_t rows, cols; void* dst; bool f32; int ld; size_t dst_row; const LayeredLayer* ukt = nullptr; size_t part = 0, part_ld = 0; };
-// cols 0: a vector of `rows` values; part: a row is cut into parts of so many values, part_ld apart on the device
+struct Slot { std::string name; size_t rows, cols; void* dst; bool f32; int ld; size_t dst_row; const LayeredLayer* ukt = nullptr; size_t part = 0, part_ld = 0; bool transposed = false; };
+// cols 0: a vector of `rows` values; part: a row is cut into parts of so many values, part_ld apart on the device; transposed (f32):
+// column i of the tensor is at dst + i * ld
 
 // uk [heads*dim, kv] -> its transpose per head, [heads][kv8][dim]
 int upload_ukt(Gpt* g, const Slot& s, const float* host) {
@@ -607,7 +625,7 @@ std::vector<Slot> layer_slots(const Gpt* g, const LayeredLayer& w) {
         mat("mix.q", hd, d, w.w_in, d8, w.c_q);
         if (kv) { mat("mix.k", gd, d, w.w_in, d8, w.c_k); mat("mix.v", gv, d, w.w_in, d8, w.c_v); }
         if (c.conv_taps > 0) {
-            auto taps = [&](const char* n, size_t rows, int col) { s.push_back({n, rows, (size_t)c.conv_taps, w.conv + (size_t)col * c.conv_taps, true, c.conv_taps, 0}); };
+            auto taps = [&](const char* n, size_t rows, int col) { s.push_back({n, rows, (size_t)c.conv_taps, w.conv + col, true, w.c_g, 0}); s.back().transposed = true; };
             taps("mix.q.conv", hd, w.c_q);
             if (kv) { taps("mix.k.conv", gd, w.c_k); taps("mix.v.conv", gv, w.c_v); }
         }
@@ -671,6 +689,13 @@ int layered_set_param(Gpt* g, const char* name, const float* host, size_t n) {
         if (s.name != key) continue;
         const size_t want = s.rows * (s.cols ? s.cols : 1);
         if (n != want) return fail("gpt_set_param(%s): got %zu values, expected %zu", name, n, want);
+        if (s.transposed) {
+            std::vector<float> t(n);
+            for (size_t r = 0; r < s.rows; r++)
+                for (size_t i = 0; i < s.cols; i++) t[i * s.rows + r] = host[r * s.cols + i];
+            SPT_CUDA(cudaMemcpy2DAsync(s.dst, (size_t)s.ld * 4, t.data(), s.rows * 4, s.rows * 4, s.cols, cudaMemcpyHostToDevice, rt().stream));
+            return stream_wait();
+        }
         if (s.f32) return sptorch_ext_copy_h2d_bytes(host, s.dst, n * 4) || stream_wait();
         void* dst = (uint8_t*)s.dst + s.dst_row * s.ld * g->es;
         if (s.ukt && upload_ukt(g, s, host)) return 1;

@@ -38,7 +38,7 @@ struct LayeredLayer {
     float* state = nullptr;                      // gated linear attention: [max_batch][heads][dim][vdim]
     void* rows = nullptr;                        // latent and window attention: [max_batch][cache positions][row()]
     int c_up = 0, c_gate = 0;                    // parallel block: columns of the feed-forward's two projections
-    float* conv = nullptr;                       // window attention: [c_g][taps], the columns of q, k and v as they lie in w_in
+    float* conv = nullptr;                       // window attention: [taps][c_g], the columns of q, k and v as they lie in w_in
     const float *temp = nullptr, *slopes = nullptr;          // ... position factors of the queries [seq_len], distance slopes [heads]
     void* ring = nullptr;                        // ... [max_batch][taps][c_g]: projected rows of the last positions, slot = position % taps
     LayeredScratch own;                          // ... rows of a forward without a cache
@@ -142,7 +142,7 @@ struct WindowArgs {
     const void* in; long long ld_in;             // projections of B*T tokens: q, k, v of every head at c_q, c_k, c_v
     int c_q, c_k, c_v;
     int B, T, H, G, D, V, D8, V8, taps;
-    const float* conv;                           // [columns][taps] (taps 0: none)
+    const float* conv;                           // [taps][ring_cols] (taps 0: none)
     const float *temp, *slopes;                  // may be null
     int first; const int* pos_dev;               // as in LatentArgs
     float scale; int window;                     // window 0: every earlier position

@@ -70,7 +70,7 @@ __device__ __forceinline__ uint4 relu_mul8(uint4 a, uint4 g) {
 // NORM: A holds un-normalised rows; every CTA normalises them itself into shared memory (kind 1: LayerNorm, gamma * ((x - mean) *
 // inv) + beta with inv = 1 / sqrt(var + eps); kind 2: RMSNorm, x * inv * gamma with inv = 1 / sqrt(mean(x^2) + eps)), rounded to
 // bf16 as the stand-alone kernels store them.  M rows of K values per CTA is little work next to the launch it saves.  NORM 2: RowNorm
-// kind 3, the residual stream completed on the fly.
+// kinds 3 and 4, the residual stream completed on the fly.
 template <int MT, int NT, int S, int NORM>
 __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv_bfloat16* __restrict__ A, long long lda,
                                                                      const __nv_bfloat16* __restrict__ W, long long ldb,
@@ -132,7 +132,7 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
     const long long a_ld = NORM ? (long long)(K + 8) : lda;
     const __nv_bfloat16* a_base = NORM ? reinterpret_cast<const __nv_bfloat16*>(dyn) : A;
     if constexpr (NORM == 2) {
-        __shared__ float part[kPostNormMaxRows][kWarps];
+        __shared__ float part[kPostNormMaxRows][kWarps], part2[kPostNormMaxRows][kWarps];
         const int P = M >= 8 ? 1 : M >= 4 ? 2 : M >= 2 ? 4 : 8, RP = kWarps / P, my_p = warp % P, my_r = warp / P;
         const int nvec = K >> 3, per = (nvec + P - 1) / P, c_begin = my_p * per, c_end = min(nvec, c_begin + per);
         for (int r = my_r; r < M; r += RP) {
@@ -153,26 +153,53 @@ __global__ void __launch_bounds__(kWarps * 32) linear_few_rows_kernel(const __nv
             float tot = 0.0f;
             for (int q = 0; q < P; q++) tot += part[r][q];
             const float inv = 1.0f / sqrtf(tot / (float)nrm.dim + nrm.eps);
-            for (int c = c_begin + lane; c < c_end; c += 32) {
+            // elements 8c .. 8c + 7 of the completed row
+            auto completed = [&](int c, float (&v)[8]) {
                 const uint4 d = reinterpret_cast<const uint4*>(nrm.y + (size_t)r * K)[c];
                 const uint32_t wd[4] = {d.x, d.y, d.z, d.w};
                 const float4 x0 = reinterpret_cast<const float4*>(nrm.x + (size_t)r * K)[2 * c], x1 = reinterpret_cast<const float4*>(nrm.x + (size_t)r * K)[2 * c + 1];
                 const float4 g0 = __ldg(reinterpret_cast<const float4*>(nrm.gamma + 8 * c)), g1 = __ldg(reinterpret_cast<const float4*>(nrm.gamma + 8 * c + 4));
-                float v[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w};
-                const float gg[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+                const float xx[8] = {x0.x, x0.y, x0.z, x0.w, x1.x, x1.y, x1.z, x1.w}, gg[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    v[2 * j] = xx[2 * j] + __uint_as_float(wd[j] << 16) * inv * gg[2 * j];
+                    v[2 * j + 1] = xx[2 * j + 1] + __uint_as_float(wd[j] & 0xffff0000u) * inv * gg[2 * j + 1];
+                }
+            };
+            float sq2 = 0.0f;
+            for (int c = c_begin + lane; c < c_end; c += 32) {
+                float v[8];
+                completed(c, v);
                 uint4 o;
                 __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
 #pragma unroll
-                for (int j = 0; j < 4; j++) {
-                    v[2 * j] += __uint_as_float(wd[j] << 16) * inv * gg[2 * j];
-                    v[2 * j + 1] += __uint_as_float(wd[j] & 0xffff0000u) * inv * gg[2 * j + 1];
-                    oh[j] = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
-                }
-                reinterpret_cast<uint4*>(dyn + (size_t)r * (K + 8) * 2)[c] = o;
+                for (int j = 0; j < 4; j++) { oh[j] = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]); sq2 += v[2 * j] * v[2 * j] + v[2 * j + 1] * v[2 * j + 1]; }
+                if (!nrm.gamma2) reinterpret_cast<uint4*>(dyn + (size_t)r * (K + 8) * 2)[c] = o;
                 if (blockIdx.x == 0) {
                     reinterpret_cast<float4*>(nrm.x_out + (size_t)r * K)[2 * c] = make_float4(v[0], v[1], v[2], v[3]);
                     reinterpret_cast<float4*>(nrm.x_out + (size_t)r * K)[2 * c + 1] = make_float4(v[4], v[5], v[6], v[7]);
-                    reinterpret_cast<uint4*>(nrm.xb + (size_t)r * K)[c] = o;
+                    if (nrm.xb) reinterpret_cast<uint4*>(nrm.xb + (size_t)r * K)[c] = o;
+                }
+            }
+            if (nrm.gamma2) {
+                // one or two rows: every warp has one row (RP * P = kWarps and M divides RP or is below it), so the barrier meets all warps once
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) sq2 += __shfl_xor_sync(0xffffffffu, sq2, o);
+                if (lane == 0) part2[r][my_p] = sq2;
+                __syncthreads();
+                float tot2 = 0.0f;
+                for (int q = 0; q < P; q++) tot2 += part2[r][q];
+                const float inv2 = 1.0f / sqrtf(tot2 / (float)nrm.dim + nrm.eps);
+                for (int c = c_begin + lane; c < c_end; c += 32) {
+                    float v[8];
+                    completed(c, v);
+                    const float4 g0 = __ldg(reinterpret_cast<const float4*>(nrm.gamma2 + 8 * c)), g1 = __ldg(reinterpret_cast<const float4*>(nrm.gamma2 + 8 * c + 4));
+                    const float gg[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+                    uint4 o;
+                    __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+                    for (int j = 0; j < 4; j++) oh[j] = __floats2bfloat162_rn(v[2 * j] * inv2 * gg[2 * j], v[2 * j + 1] * inv2 * gg[2 * j + 1]);
+                    reinterpret_cast<uint4*>(dyn + (size_t)r * (K + 8) * 2)[c] = o;
                 }
             }
         }
@@ -497,8 +524,8 @@ bool linear_few_rows_supported(const GemmDesc& d) {
 bool linear_few_rows_norm_supported(const GemmDesc& d, const RowNorm& nrm) {
     if (d.act_off) return false;
     const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    if (nrm.kind == 3)
-        return linear_few_rows_supported(d) && nrm.gamma && nrm.x && nrm.y && nrm.x_out && nrm.x_out != nrm.x && nrm.xb && nrm.dim > 0 && nrm.dim <= d.K && !d.group &&
+    if (nrm.kind == 3 || nrm.kind == 4)
+        return linear_few_rows_supported(d) && (nrm.kind == 3 ? nrm.xb && !nrm.gamma2 : nrm.gamma2 && al16(nrm.gamma2)) && nrm.gamma && nrm.x && nrm.y && nrm.x_out && nrm.x_out != nrm.x && nrm.dim > 0 && nrm.dim <= d.K && !d.group &&
                al16(nrm.gamma) && al16(nrm.x) && al16(nrm.y) && al16(nrm.x_out) && al16(nrm.xb) && d.M <= kPostNormMaxRows && norm_smem(d) <= kNormSmemLimit;
     return linear_few_rows_supported(d) && (nrm.kind == 1 || nrm.kind == 2) && nrm.gamma && al16(nrm.gamma) && (nrm.kind == 2 || (nrm.beta && al16(nrm.beta))) &&
            d.M <= kNormMaxRows && norm_smem(d) <= kNormSmemLimit;
@@ -526,7 +553,7 @@ int norm_few_rows(const void* x, void* out, int rows, int K, const RowNorm& nrm,
 int linear_few_rows(const GemmDesc& d, const RowNorm* nrm, bool dependent) {
     if (nrm && nrm->kind) {
         if (!linear_few_rows_norm_supported(d, *nrm)) return fail("linear_few_rows: unsupported problem (normalised rows)");
-        return nrm->kind == 3 ? dispatch<2>(d, *nrm, dependent) : dispatch<1>(d, *nrm, dependent);
+        return nrm->kind >= 3 ? dispatch<2>(d, *nrm, dependent) : dispatch<1>(d, *nrm, dependent);
     }
     if (!linear_few_rows_supported(d)) return fail("linear_few_rows: unsupported problem");
     return dispatch<0>(d, RowNorm{}, dependent);

@@ -29,7 +29,7 @@ template <typename T>
 __device__ __forceinline__ float convolved(const WindowArgs& a, int b, int t, int pos0, int col) {
     if (a.taps == 0) return projected<T>(a, b, t, pos0, col);
     float s = 0.0f;
-    for (int j = 0; j < a.taps; j++) s = fmaf(a.conv[(size_t)col * a.taps + j], projected<T>(a, b, t - a.taps + 1 + j, pos0, col), s);
+    for (int j = 0; j < a.taps; j++) s = fmaf(a.conv[(size_t)j * a.ring_cols + col], projected<T>(a, b, t - a.taps + 1 + j, pos0, col), s);
     return s;
 }
 
@@ -53,6 +53,16 @@ __global__ void __launch_bounds__(128) window_prep_kernel(const WindowArgs a) {
     }
 }
 
+__device__ __forceinline__ void unpack(uint4 raw, float (&f)[8]) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; i++) { const float2 v = bf16x2_to_float2(h[i]); f[2 * i] = v.x; f[2 * i + 1] = v.y; }
+}
+__device__ __forceinline__ void load_taps(const float* w, float (&f)[8]) {
+    const float4 x = __ldg(reinterpret_cast<const float4*>(w)), y = __ldg(reinterpret_cast<const float4*>(w + 4));
+    f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w; f[4] = y.x; f[5] = y.y; f[6] = y.z; f[7] = y.w;
+}
+
 constexpr int kPrepTokens = 16;
 
 // bf16, head sizes multiples of eight: a thread takes eight channels of kPrepTokens consecutive tokens, the rows before the current one in
@@ -67,14 +77,7 @@ __global__ void __launch_bounds__(128) window_prep_vec_kernel(const WindowArgs a
     const int pos0 = a.pos_dev ? a.pos_dev[0] : a.first;
     float w[TAPS][8], u[TAPS][8];                               // u[j]: the row j - (TAPS - 1) tokens from the current one
 #pragma unroll
-    for (int i = 0; i < 8; i++)
-#pragma unroll
-        for (int j = 0; j < TAPS; j++) w[j][i] = __ldg(a.conv + (size_t)(c + i) * TAPS + j);
-    auto unpack = [](uint4 raw, float (&f)[8]) {
-        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-        for (int i = 0; i < 4; i++) { const float2 v = bf16x2_to_float2(h[i]); f[2 * i] = v.x; f[2 * i + 1] = v.y; }
-    };
+    for (int j = 0; j < TAPS; j++) load_taps(a.conv + (size_t)j * a.ring_cols + c, w[j]);
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + (size_t)b * a.T * a.ld_in + c;
 #pragma unroll
     for (int j = 0; j < TAPS - 1; j++) {
@@ -205,7 +208,7 @@ __host__ __device__ constexpr int wd_q_pitch(int ns) { return ns * 32 + 8; }
 __host__ __device__ constexpr int wd_o_pitch(int nb) { return nb * 64 + 4; }
 template <int NS, int NB>
 constexpr size_t wd_smem(int warps, int heads) {
-    return (size_t)kWdHeads * wd_q_pitch(NS) * 2 + (size_t)(NS * 32 + NB * 64) * 2 + (size_t)warps * kWdHeads * 8 + (size_t)warps * heads * wd_o_pitch(NB) * 4;
+    return (size_t)kWdHeads * wd_q_pitch(NS) * 2 + (size_t)(NS * 32 + NB * 64) * 2 + (size_t)warps * kWdHeads * 8 + kWdHeads * 4 + (size_t)warps * heads * wd_o_pitch(NB) * 4;
 }
 
 template <int NS, int NB, bool FRESH, int WARPS>
@@ -217,7 +220,8 @@ __global__ void __launch_bounds__(WARPS * 32) window_decode_kernel(const WindowA
     __nv_bfloat16* vf = kf + NS * 32;
     float* m_s = reinterpret_cast<float*>(vf + NB * 64);                        // [WARPS][16]
     float* l_s = m_s + WARPS * kWdHeads;
-    float* o_s = l_s + WARPS * kWdHeads;                                        // [WARPS][heads][OP]
+    float* f0_s = l_s + WARPS * kWdHeads;                                       // [16]: warp 0's factor
+    float* o_s = f0_s + kWdHeads;                                               // [WARPS][heads][OP]
     pdl_release();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     const int rank = blockIdx.x % splits, item = blockIdx.x / splits, R = a.H / a.G;
@@ -230,13 +234,15 @@ __global__ void __launch_bounds__(WARPS * 32) window_decode_kernel(const WindowA
     uint4 kr[2][NS], vr[4][NB];
     const uint4 zero4 = make_uint4(0, 0, 0, 0);
     // keys k0 + g and k0 + 8 + g; values of keys k0 + 2t, 2t + 1, 2t + 8, 2t + 9.  Positions past `last` are not read.
-    auto fetch = [&](int k0, int last) {
+    auto fetch_keys = [&](int k0, int last) {
 #pragma unroll
         for (int n = 0; n < 2; n++) {
             const int p = k0 + 8 * n + g;
 #pragma unroll
             for (int s = 0; s < NS; s++) kr[n][s] = p <= last && 32 * s + 8 * t < a.D ? *reinterpret_cast<const uint4*>(krow + (size_t)p * a.row + 32 * s + 8 * t) : zero4;
         }
+    };
+    auto fetch_values = [&](int k0, int last) {
 #pragma unroll
         for (int n = 0; n < 4; n++) {
             const int p = k0 + 2 * t + (n & 1) + 8 * (n >> 1);
@@ -248,37 +254,53 @@ __global__ void __launch_bounds__(WARPS * 32) window_decode_kernel(const WindowA
     const int last = fresh_kv ? pos - 1 : pos;               // what the cache holds
     // rows before this step's tokens were written by earlier steps: they may be requested before the kernels ahead are done
     const bool early = first + 15 < pos0;
-    if (early && first <= pos) fetch(first, last);
-    // FRESH: this CTA's share of the convolutions.  Everything but the newest projected row is there already, too.
-    pdl_acquire();
-    if (!early && first <= pos) fetch(first, last);
+    if (early && first <= pos) { fetch_keys(first, last); fetch_values(first, last); }
     if constexpr (FRESH) {
+        // this CTA's share of the convolutions, eight channels per thread: heads' queries, then (own_kv) the key and the value.  Everything
+        // but the newest projected row is there already, so only its product is left for after the wait.
         const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(a.in) + (size_t)mt * a.ld_in;
         __nv_bfloat16* ring = a.taps ? static_cast<__nv_bfloat16*>(a.ring) + (size_t)b * a.taps * a.ring_cols : nullptr;
         const int nq = heads * a.D, nk = fresh_kv ? a.D : 0, nv = fresh_kv ? a.V : 0;
-        const float temp = a.temp ? a.temp[pos] : 1.0f;
-        for (int i = tid; i < nq + nk + nv; i += WARPS * 32) {
-            const int col = i < nq ? a.c_q + h0 * a.D + i : i < nq + nk ? a.c_k + gg * a.D + (i - nq) : a.c_v + gg * a.V + (i - nq - nk);
-            const __nv_bfloat16 now = in[col];
-            float s = __bfloat162float(now);
-            if (a.taps) {
-                s *= a.conv[(size_t)col * a.taps + a.taps - 1];
+        bool acquired = false;
+        for (int i = tid * 8; i < nq + nk + nv || !acquired; i += WARPS * 256) {
+            const bool live = i < nq + nk + nv, is_q = i < nq;
+            const int col = is_q ? a.c_q + h0 * a.D + i : i < nq + nk ? a.c_k + gg * a.D + (i - nq) : a.c_v + gg * a.V + (i - nq - nk);
+            float sum[8] = {0, 0, 0, 0, 0, 0, 0, 0}, w[8] = {1, 1, 1, 1, 1, 1, 1, 1}, u[8];
+            if (live && a.taps) {
+#pragma unroll 4
                 for (int j = 1; j < a.taps; j++)
-                    if (pos - j >= 0) s = fmaf(a.conv[(size_t)col * a.taps + a.taps - 1 - j], __bfloat162float(ring[(size_t)((pos - j) % a.taps) * a.ring_cols + col]), s);
-                // no CTA reads this slot in this step
-                if (rank == 0 && (i < nq || hg == 0)) ring[(size_t)(pos % a.taps) * a.ring_cols + col] = now;
+                    if (pos - j >= 0) {
+                        load_taps(a.conv + (size_t)(a.taps - 1 - j) * a.ring_cols + col, w);
+                        unpack(*reinterpret_cast<const uint4*>(ring + (size_t)((pos - j) % a.taps) * a.ring_cols + col), u);
+#pragma unroll
+                        for (int e = 0; e < 8; e++) sum[e] = fmaf(w[e], u[e], sum[e]);
+                    }
+                load_taps(a.conv + (size_t)(a.taps - 1) * a.ring_cols + col, w);
             }
-            if (i < nq) { const int r = i / a.D; qs[r * QP + i - r * a.D] = __float2bfloat16_rn(s * temp); }
+            const float factor = is_q && a.temp ? a.temp[pos] : 1.0f;
+            if (!acquired) { pdl_acquire(); acquired = true; }
+            if (!live) break;
+            const uint4 now = *reinterpret_cast<const uint4*>(in + col);
+            unpack(now, u);
+            uint4 o;
+            __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+            for (int e = 0; e < 8; e += 2) oh[e / 2] = __floats2bfloat162_rn(fmaf(w[e], u[e], sum[e]) * factor, fmaf(w[e + 1], u[e + 1], sum[e + 1]) * factor);
+            // no CTA reads this slot of the ring in this step
+            if (a.taps && rank == 0 && (is_q || hg == 0)) *reinterpret_cast<uint4*>(ring + (size_t)(pos % a.taps) * a.ring_cols + col) = now;
+            if (is_q) { const int r = i / a.D; *reinterpret_cast<uint4*>(qs + r * QP + i - r * a.D) = o; }
             else {
-                const __nv_bfloat16 v = __float2bfloat16_rn(s);
-                if (i < nq + nk) kf[i - nq] = v; else vf[i - nq - nk] = v;
+                *reinterpret_cast<uint4*>(i < nq + nk ? kf + (i - nq) : vf + (i - nq - nk)) = o;
                 if (rank == 0 && hg == 0)
-                    static_cast<__nv_bfloat16*>(a.rows)[(size_t)b * a.seq_stride + (size_t)pos * a.row + (i < nq + nk ? gg * a.D + (i - nq) : a.G * a.D + gg * a.V + (i - nq - nk))] = v;
+                    *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.rows) + (size_t)b * a.seq_stride + (size_t)pos * a.row + (i < nq + nk ? gg * a.D + (i - nq) : a.G * a.D + gg * a.V + (i - nq - nk))) = o;
             }
         }
+        if (!early && first <= pos) { fetch_keys(first, last); fetch_values(first, last); }
         // the rest of Q: missing heads and columns
         for (int i = tid; i < kWdHeads * QP; i += WARPS * 32) { const int r = i / QP; if (r >= heads || i - r * QP >= a.D) qs[i] = __float2bfloat16_rn(0.0f); }
     } else {
+        pdl_acquire();
+        if (!early && first <= pos) { fetch_keys(first, last); fetch_values(first, last); }
         for (int i = tid; i < kWdHeads * (QP / 8); i += WARPS * 32) {
             const int r = i / (QP / 8), c = (i - r * (QP / 8)) * 8;
             *reinterpret_cast<uint4*>(qs + r * QP + c) = r < heads && c < a.D ? *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q) + ((size_t)mt * a.H + h0 + r) * a.D + c) : zero4;
@@ -294,7 +316,6 @@ __global__ void __launch_bounds__(WARPS * 32) window_decode_kernel(const WindowA
     const float sl0 = a.slopes && g < heads ? a.slopes[h0 + g] * kLog2e : 0.0f, sl1 = a.slopes && g + 8 < heads ? a.slopes[h0 + g + 8] * kLog2e : 0.0f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
     for (int k0 = first; k0 <= pos; k0 += step) {
-        if (k0 != first) fetch(k0, last);
         if (fresh_kv && pos - k0 < 16) {                     // the newest position takes its row from shared memory
             const int d = pos - k0;
 #pragma unroll
@@ -320,6 +341,7 @@ __global__ void __launch_bounds__(WARPS * 32) window_decode_kernel(const WindowA
                 mma_bf16(s[n], x.z, y.z, x.w, y.w, kr[n][i].z, kr[n][i].w);
             }
         }
+        if (k0 + step <= pos) fetch_keys(k0 + step, last);         // in flight while the softmax and P V run
         // scores of heads g (entries 0, 1) and g + 8 (2, 3), keys k0 + 8 n + 2 t + {0, 1}
         float mx0 = m0, mx1 = m1;
 #pragma unroll
@@ -361,6 +383,7 @@ __global__ void __launch_bounds__(WARPS * 32) window_decode_kernel(const WindowA
                 mma_bf16(acc[8 * sb + j], pl[0], pl[1], pl[2], pl[3], b0, b1);
             }
         }
+        if (k0 + step <= pos) fetch_values(k0 + step, last);
     }
 #pragma unroll
     for (int o = 1; o < 4; o <<= 1) { l0 += __shfl_xor_sync(0xffffffffu, l0, o); l1 += __shfl_xor_sync(0xffffffffu, l1, o); }
@@ -385,43 +408,59 @@ __global__ void __launch_bounds__(WARPS * 32) window_decode_kernel(const WindowA
     namespace cg = cooperative_groups;
     cg::cluster_group cluster = cg::this_cluster();
     __syncthreads();
-    // the CTA's own warps first: sums over the warps land in warp 0's slots
-    for (int i = tid; i < heads * a.V; i += WARPS * 32) {
+    // the CTA's own warps first: every warp's factor against the CTA's maximum, then the sums, which land in warp 0's slots
+    if (tid < kWdHeads) {
+        float tm = -INFINITY, tl = 0.0f;
+#pragma unroll
+        for (int w = 0; w < WARPS; w++) tm = fmaxf(tm, m_s[w * kWdHeads + tid]);
+#pragma unroll
+        for (int w = 0; w < WARPS; w++) {
+            const float x = m_s[w * kWdHeads + tid], f = x == -INFINITY ? 0.0f : ex2(x - tm);
+            tl = fmaf(l_s[w * kWdHeads + tid], f, tl);
+            if (w > 0) m_s[w * kWdHeads + tid] = f; else f0_s[tid] = f;
+        }
+        m_s[tid] = tm; l_s[tid] = tl;
+    }
+    __syncthreads();
+    for (int i = tid * 4; i < heads * a.V; i += WARPS * 128) {
         const int r = i / a.V, c = i - r * a.V;
-        float tm = -INFINITY, v = 0.0f;
+        float4 v = make_float4(0, 0, 0, 0);
 #pragma unroll
-        for (int w = 0; w < WARPS; w++) tm = fmaxf(tm, m_s[w * kWdHeads + r]);
-#pragma unroll
-        for (int w = 0; w < WARPS; w++) { const float ms = m_s[w * kWdHeads + r]; if (ms != -INFINITY) v = fmaf(o_s[((size_t)w * heads_max + r) * OP + c], ex2(ms - tm), v); }
-        o_s[(size_t)r * OP + c] = v;                       // this thread was the only reader of its column
+        for (int w = 0; w < WARPS; w++) {
+            const float f = w > 0 ? m_s[w * kWdHeads + r] : f0_s[r];
+            const float4 x = *reinterpret_cast<const float4*>(o_s + ((size_t)w * heads_max + r) * OP + c);
+            v.x = fmaf(x.x, f, v.x); v.y = fmaf(x.y, f, v.y); v.z = fmaf(x.z, f, v.z); v.w = fmaf(x.w, f, v.w);
+        }
+        *reinterpret_cast<float4*>(o_s + (size_t)r * OP + c) = v;              // this thread was the only reader of its columns
     }
     if (splits > 1) cluster.sync(); else __syncthreads();
-    const int per = (heads * a.V + splits - 1) / splits, i1 = min(heads * a.V, (rank + 1) * per);
+    const int quads = heads * a.V / 4, per = (quads + splits - 1) / splits, i1 = min(quads, (rank + 1) * per);
     for (int i = rank * per + tid; i < i1; i += WARPS * 32) {
-        const int r = i / a.V, c = i - r * a.V;
-        float tm = -INFINITY, tl = 0.0f, v = 0.0f;
-        for (int s = 0; s < splits; s++) {
-            const float* ms = splits > 1 ? cluster.map_shared_rank(m_s, s) : m_s;
+        const int r = i * 4 / a.V, c = i * 4 - r * a.V;
+        float tm = -INFINITY, tl = 0.0f, ms[8];
+        float4 v = make_float4(0, 0, 0, 0);
 #pragma unroll
-            for (int w = 0; w < WARPS; w++) tm = fmaxf(tm, ms[w * kWdHeads + r]);
-        }
-        for (int s = 0; s < splits; s++) {
-            const float* ms = splits > 1 ? cluster.map_shared_rank(m_s, s) : m_s;
-            const float* ls = splits > 1 ? cluster.map_shared_rank(l_s, s) : l_s;
-            const float* os = splits > 1 ? cluster.map_shared_rank(o_s, s) : o_s;
-            float cm = -INFINITY;
+        for (int s = 0; s < 8; s++) { ms[s] = s < splits ? (splits > 1 ? cluster.map_shared_rank(m_s, s) : m_s)[r] : -INFINITY; tm = fmaxf(tm, ms[s]); }
 #pragma unroll
-            for (int w = 0; w < WARPS; w++) {
-                const float x = ms[w * kWdHeads + r];
-                cm = fmaxf(cm, x);
-                if (x != -INFINITY) tl = fmaf(ls[w * kWdHeads + r], ex2(x - tm), tl);
+        for (int s = 0; s < 8; s++)
+            if (s < splits) {
+                const float f = ms[s] == -INFINITY ? 0.0f : ex2(ms[s] - tm);
+                const float4 x = *reinterpret_cast<const float4*>((splits > 1 ? cluster.map_shared_rank(o_s, s) : o_s) + (size_t)r * OP + c);
+                tl = fmaf((splits > 1 ? cluster.map_shared_rank(l_s, s) : l_s)[r], f, tl);
+                v.x = fmaf(x.x, f, v.x); v.y = fmaf(x.y, f, v.y); v.z = fmaf(x.z, f, v.z); v.w = fmaf(x.w, f, v.w);
             }
-            if (cm != -INFINITY) v = fmaf(os[(size_t)r * OP + c], ex2(cm - tm), v);
-        }
-        v /= tl;
+        const float inv = 1.0f / tl;
         const size_t at = (size_t)mt * a.ld_out + (size_t)(h0 + r) * a.V + c;
-        if (a.gate) v *= 1.0f / (1.0f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[at])));
-        static_cast<__nv_bfloat16*>(a.out)[at] = __float2bfloat16_rn(v);
+        float y[4] = {v.x * inv, v.y * inv, v.z * inv, v.w * inv};
+        if (a.gate) {
+            const uint2 graw = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(a.gate) + at);
+            const float2 g0 = bf16x2_to_float2(*reinterpret_cast<const __nv_bfloat162*>(&graw.x)), g1 = bf16x2_to_float2(*reinterpret_cast<const __nv_bfloat162*>(&graw.y));
+            y[0] *= 1.0f / (1.0f + __expf(-g0.x)); y[1] *= 1.0f / (1.0f + __expf(-g0.y)); y[2] *= 1.0f / (1.0f + __expf(-g1.x)); y[3] *= 1.0f / (1.0f + __expf(-g1.y));
+        }
+        uint2 o;
+        *reinterpret_cast<__nv_bfloat162*>(&o.x) = __floats2bfloat162_rn(y[0], y[1]);
+        *reinterpret_cast<__nv_bfloat162*>(&o.y) = __floats2bfloat162_rn(y[2], y[3]);
+        *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(a.out) + at) = o;
     }
     if (splits > 1) cluster.sync();                        // no CTA leaves while its shared memory may still be read
 }
