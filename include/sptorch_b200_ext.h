@@ -34,6 +34,8 @@ extern "C" {
 #define SPT_EPI_NONE 0
 #define SPT_EPI_GELU 1
 #define SPT_EPI_SWIGLU 2   /* out = residual * g * sigmoid(g), g = alpha x W^T + bias: swiglu(x, gate) of core-ops/src/lib.rs:1529-1541 with the gate projection fused */
+#define SPT_EPI_RELU_MUL 3 /* out = residual * max(g, 0) */
+#define SPT_EPI_GELU_MUL 4 /* out = residual * gelu(g), the tanh form */
 
 /* ---- runtime ---- */
 const char* sptorch_ext_last_error(void);              /* text of the calling thread's last failure */
@@ -54,7 +56,7 @@ int   sptorch_ext_timer_end(float* ms);                /* second event, waits fo
 int   sptorch_ext_flush_l2(void);                      /* overwrites a 256 MiB scratch (allocated on first use) */
 /* per-category device timing of the GPT forward (CUDA events around each launch on the library stream).
  * categories: 0 linear GEMM, 1 attention GEMMs, 2 causal softmax, 3 layernorm, 4 embedding, 5 other, 6 fused attention (and attention
- * over cached rows), 7 gated linear attention, 8 latent attention's norms and rotations */
+ * over cached rows), 7 gated linear attention, 8 latent attention's norms and rotations, 9 window attention's convolutions and cached rows */
 #define SPT_PROF_NCAT 10
 int   sptorch_ext_prof_enable(int on);
 int   sptorch_ext_prof_read(float* ms, uint32_t* launches, int ncat);  /* syncs, sums since last read, clears */

@@ -111,8 +111,14 @@ def latent_attention_mixer(h, p, m, eps, st):
     return o.reshape(h.shape[0], -1) @ p["o"].T
 
 
-def dense_mlp(h, p):
-    return (silu(h @ p["gate"].T + p["gate.b"]) * (h @ p["up"].T + p["up.b"])) @ p["down"].T + p["down.b"]
+def relu(z):
+    return np.maximum(z, 0.0)
+
+
+def dense_mlp(h, p, act=silu):
+    """down(act(gate h) * (up h)); the biases are left out where there are none."""
+    b = lambda name: p.get(name + ".b", 0.0)
+    return (act(h @ p["gate"].T + b("gate")) * (h @ p["up"].T + b("up"))) @ p["down"].T + b("down")
 
 
 def gelu_tanh(z):
@@ -174,21 +180,23 @@ def attention_mixer(h, p, m, st, source):
     return (o.reshape(T, H * V) * sigmoid(h @ p["g"].T)) @ p["o"].T
 
 
-def relu_mlp(h, p):
-    return (np.maximum(h @ p["gate"].T, 0.0) * (h @ p["up"].T)) @ p["down"].T
-
-
 def token_side(x, e, p, eps):
     """The per-layer token input: e [T, dim] is the layer's part of the tokens' rows in the side table."""
     y = (gelu_tanh(x @ p["gate"].T) * e) @ p["proj"].T
     return x + rms_norm(y, p["norm"], eps)
 
 
+# How the layers of an architecture join the residual stream: "parallel" or "post" (the norm behind the sublayer), the activation of the
+# feed-forward, whether the head is the embedding table, and whether the stream starts scaled and takes per-layer token inputs
+DESIGNS = {"Tolevik": dict(block="post", act=silu, tied=False, token_side=False, embedding_scale=False),
+           "Bulidra": dict(block="parallel", act=relu, tied=True, token_side=True, embedding_scale=True)}
+
+
 class LayeredOracle:
     """config: the dictionary of config.json; params: {tensor name: array}.  ``feed`` runs the next tokens of the sequence."""
 
     def __init__(self, config, params, dtype=np.float64):
-        self.c, self.dtype = config, dtype
+        self.c, self.dtype, self.design = config, dtype, DESIGNS[config["architecture"]]
         self.p = {k: np.asarray(v, dtype) for k, v in params.items()}
         self.reset()
 
@@ -211,31 +219,32 @@ class LayeredOracle:
         n = len(prefix)
         return {k[n:]: v for k, v in self.p.items() if k.startswith(prefix)}
 
+    def _mix(self, i, h):
+        la, eps = self.c["layers"][i], self.c["norm"]["eps"]
+        m, p, st = la["mixer"], self._sub(f"l{i}.mix."), self.states[i]
+        if la["type"] == "gla":
+            return gla_mixer(h, p, m, eps, st)
+        if la["type"] == "latent_attention":
+            return latent_attention_mixer(h, p, m, eps, st)
+        return attention_mixer(h, p, m, st, self.states[m["kv_from"]] if "kv_from" in m else st)
+
     def feed(self, tokens, taps=None):
-        return self._feed_bulidra(np.asarray(tokens), taps) if self.c["architecture"] == "Bulidra" else self._feed_tolevik(tokens, taps)
-
-    def _feed_bulidra(self, tokens, taps):
-        eps, dim = self.c["norm"]["eps"], self.c["token_side"]["dim"]
-        x = self.p["embed"][tokens] * self.c["embedding"]["scale"]
+        eps, d, tokens = self.c["norm"]["eps"], self.design, np.asarray(tokens)
+        x = self.p["embed"][tokens]
+        if d["embedding_scale"]:
+            x = x * self.c["embedding"]["scale"]
         for i, la in enumerate(self.c["layers"]):
-            m, st = la["mixer"], self.states[i]
-            h = rms_norm(x, self.p[f"l{i}.norm1"], eps)
-            y = attention_mixer(h, self._sub(f"l{i}.mix."), m, st, self.states[m["kv_from"]] if "kv_from" in m else st)
-            if la["mlp"] is not None:
-                y = y + relu_mlp(h, self._sub(f"l{i}.mlp."))
-            x = token_side(x + y, self.p["side.embed"][tokens][:, i * dim:(i + 1) * dim], self._sub(f"l{i}.side."), eps)
+            mlp = None if la["mlp"] is None else (lambda h: dense_mlp(h, self._sub(f"l{i}.mlp."), d["act"]))
+            if d["block"] == "parallel":
+                h = rms_norm(x, self.p[f"l{i}.norm1"], eps)
+                x = x + self._mix(i, h) + (mlp(h) if mlp else 0.0)
+            else:
+                x = x + rms_norm(self._mix(i, x), self.p[f"l{i}.norm1"], eps)
+                if mlp:
+                    x = x + rms_norm(mlp(x), self.p[f"l{i}.norm2"], eps)
+            if d["token_side"]:
+                n = self.c["token_side"]["dim"]
+                x = token_side(x, self.p["side.embed"][tokens][:, i * n:(i + 1) * n], self._sub(f"l{i}.side."), eps)
             if taps is not None:
                 taps.append(x)
-        return rms_norm(x, self.p["final.norm"], eps) @ self.p["embed"].T
-
-    def _feed_tolevik(self, tokens, taps):
-        eps = self.c["norm"]["eps"]
-        x = self.p["embed"][np.asarray(tokens)]
-        for i, la in enumerate(self.c["layers"]):
-            mix = gla_mixer if la["type"] == "gla" else latent_attention_mixer
-            x = x + rms_norm(mix(x, self._sub(f"l{i}.mix."), la["mixer"], eps, self.states[i]), self.p[f"l{i}.norm1"], eps)
-            if la["mlp"] is not None:
-                x = x + rms_norm(dense_mlp(x, self._sub(f"l{i}.mlp.")), self.p[f"l{i}.norm2"], eps)
-            if taps is not None:
-                taps.append(x)
-        return rms_norm(x, self.p["final.norm"], eps) @ self.p["head"].T
+        return rms_norm(x, self.p["final.norm"], eps) @ self.p["embed" if d["tied"] else "head"].T

@@ -21,7 +21,7 @@ from . import _lib
 
 F32, BF16 = 0, 1
 MM_TF32, MM_BF16, MM_F32 = 0, 1, 2
-EPI_NONE, EPI_GELU, EPI_SWIGLU = 0, 1, 2
+EPI_NONE, EPI_GELU, EPI_SWIGLU, EPI_RELU_MUL, EPI_GELU_MUL = 0, 1, 2, 3, 4
 
 
 class HalError(RuntimeError):

@@ -146,8 +146,9 @@ struct AttnSmem {
     static constexpr int kQ = 0;
     static constexpr int kK = kQ + 2 * kQTileBytes;
     static constexpr int kV = kK + kKStages * kKBytes;
-    static constexpr int kBars = kV + kVStages * kVBytes;     // mbarriers + TMEM slot + abort flag (256 B)
-    static constexpr int kTotal = kBars + 256;
+    static constexpr int kBars = kV + kVStages * kVBytes;     // mbarriers + TMEM slot + abort flag
+    static constexpr int kBarBytes = 320;
+    static constexpr int kTotal = kBars + kBarBytes;
     static_assert(kTotal <= 227 * 1024, "shared memory");
 };
 
@@ -183,8 +184,12 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     constexpr int NSB = ROT ? 3 : 2;                // score buffers
     constexpr uint32_t O_COL = ROT ? 384 : 256;     // first accumulator column
     constexpr uint32_t O_STRIDE = ROT ? 64 : 128;
-    const uint32_t s_full = v_empty + 8 * NSV;      // NSB (per score buffer)
-    const uint32_t p_full = s_full + 8 * 3;         // NSB
+    // Scores ready.  With rotating buffers: four barriers per query tile, taken in turn by the tile's own steps (index step & 3, phase
+    // step >> 2): up to three of a tile's scores may be complete before its softmax takes the first, and a barrier that only this
+    // tile's steps advance cannot be passed, or missed, because of what the other tile did meanwhile (an item may have no second tile).
+    // One barrier per tile otherwise.
+    const uint32_t s_full = v_empty + 8 * NSV;      // 8: [query tile][step & 3]
+    const uint32_t p_full = s_full + 8 * 8;         // NSB
     // P V products done: two barriers per query tile, taken in turn by the tile's steps (index step & 1, phase step >> 1).  With
     // rotating score buffers a tile's softmax can finish step j before P V of step j - 1 has completed, so its wait for the
     // product of step j on a single barrier would be two phases ahead -- which a parity wait cannot tell from none; on the
@@ -192,9 +197,9 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     // query tile in the item the softmax can be a step further ahead; its end has a wait of its own for that (below).
     const uint32_t pv_done = p_full + 8 * 3;        // 4: [query tile][step & 1]
     const uint32_t o_free = pv_done + 32;           // 2
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + L::kBars + 240);
-    volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + L::kBars + 244);
-    static_assert(8 * (2 + 2 * NSK + 2 * NSV + 12) <= 240, "barrier block overflows");
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(smem + L::kBars + L::kBarBytes - 16);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + L::kBars + L::kBarBytes - 12);
+    static_assert(8 * (2 + 2 * NSK + 2 * NSV + 17) <= L::kBarBytes - 16, "barrier block overflows");
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int BH = p.B * p.H;
@@ -208,10 +213,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         mbar_init(q_full, 1); mbar_init(q_free, 1);
         for (int s = 0; s < NSK; s++) { mbar_init(k_full + 8 * s, 1); mbar_init(k_empty + 8 * s, 1); }
         for (int s = 0; s < NSV; s++) { mbar_init(v_full + 8 * s, 1); mbar_init(v_empty + 8 * s, 1); }
-        for (int g = 0; g < 3; g++) {
-            mbar_init(s_full + 8 * g, 1);
-            mbar_init(p_full + 8 * g, 4);           // one arrival per softmax warp of the tile
-        }
+        for (int g = 0; g < 8; g++) mbar_init(s_full + 8 * g, 1);
+        for (int g = 0; g < 3; g++) mbar_init(p_full + 8 * g, 4);           // one arrival per softmax warp of the tile
         for (int g = 0; g < 4; g++) mbar_init(pv_done + 8 * g, 1);
         for (int g = 0; g < 2; g++) mbar_init(o_free + 8 * g, 4);
         *abort_flag = 0;
@@ -316,6 +319,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         // ---------------- MMA issuer ----------------
         bool ok = true;
         uint32_t g = 0, it = 0;                 // key tiles loaded so far (stage ring position); items so far
+        uint32_t outs[2] = {0, 0};              // items so far that each query tile had a part in (phases of o_free)
         uint32_t steps[2] = {0, 0};             // softmax steps of each query tile so far (phases of p_full)
         // 16 keys per product: 8 columns of P, or with PSPLIT 8 columns of each half (a chunk of 32 keys is 16 + 16 columns)
         auto mma_pv = [&](int t, uint32_t p_addr, uint64_t bdesc, bool accumulate) {
@@ -336,7 +340,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
                 for (int k = 0; k < 4; k++) mma_ss<false>(tmem_base + t * 128, adesc + 2 * k, bdesc + 2 * k, IDESC_S, (kb | k) != 0 ? 1u : 0u);
             }
-            mma_commit(s_full + 8 * t);
+            mma_commit(s_full + 32 * t);
         };
         // O_t (+)= P_t V with the value tile of ring position gg; P is read from the TMEM columns of S_t
         auto issue_pv = [&](int t, uint32_t gg, bool accumulate, uint32_t pvidx) {      // pvidx: which product of this tile (over the whole kernel)
@@ -352,7 +356,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             // (counted over the whole kernel) lives in buffer n % 3, which P V number n - 3 -- issued earlier by this thread, and
             // the tensor pipe runs one thread's MMAs in order -- has finished reading.
             uint32_t G = 0;                     // scores issued in earlier items
-            auto issue_s3 = [&](int t, uint32_t gg, uint32_t n) {
+            uint32_t scored[2] = {0, 0};        // scores issued so far of each query tile
+            auto issue_s3 = [&](int t, uint32_t gg, uint32_t n, uint32_t own) {
                 const uint32_t buf = n % 3;
                 const uint32_t kaddr = base + L::kK + (gg % NSK) * L::kKBytes;
 #pragma unroll
@@ -362,7 +367,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
                     for (int k = 0; k < 4; k++) mma_ss<false>(tmem_base + buf * 128, adesc + 2 * k, bdesc + 2 * k, IDESC_S, (kb | k) != 0 ? 1u : 0u);
                 }
-                mma_commit(s_full + 8 * buf);
+                mma_commit(s_full + 8 * (4 * t + (own & 3)));
             };
             auto issue_pv3 = [&](int t, uint32_t gg, uint32_t n, bool accumulate, uint32_t pvidx) {
                 const uint32_t buf = n % 3;
@@ -393,11 +398,12 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                         int tn = 0, jn = -1;
                         if (issued + 1 < E) entry(issued + 1, tn, jn);
                         if (elect_one_sync()) {
-                            issue_s3(ts, g + js, G + issued);
+                            issue_s3(ts, g + js, G + issued, ts ? scored[1] : scored[0]);
                             if (jn != js) mma_commit(k_empty + 8 * ((g + js) % NSK));            // every product that reads these keys has been issued
                             if (issued == E - 1) mma_commit(q_free);            // the item's last read of Q
                         }
                         __syncwarp();
+                        if (ts) scored[1]++; else scored[0]++;
                         issued++;
                     }
                     if (!ok) break;
@@ -406,7 +412,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     const uint32_t n = G + e, buf = n % 3;
                     ok = mbar_wait(p_full + 8 * buf, (n / 3) & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == w.begin(t)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == w.begin(t)) { ok = mbar_wait(o_free + 8 * t, ((t ? outs[1] : outs[0]) & 1) ^ 1, abort_flag, p.status, kErrMmaWait); if (t) outs[1]++; else outs[0]++; }
                     if (ok && j > v_seen) { ok = v_ready(g + j); v_seen = j; }
                     if (!ok) break;
                     tc_fence_after();
@@ -450,7 +456,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                     }
                     ok = mbar_wait(p_full + 8 * t, steps[t] & 1, abort_flag, p.status, kErrMmaWait);
                     // the item's first product overwrites the accumulator: the previous item's output must have been read
-                    if (ok && j == w.begin(t)) ok = mbar_wait(o_free + 8 * t, (it & 1) ^ 1, abort_flag, p.status, kErrMmaWait);
+                    if (ok && j == w.begin(t)) { ok = mbar_wait(o_free + 8 * t, ((t ? outs[1] : outs[0]) & 1) ^ 1, abort_flag, p.status, kErrMmaWait); if (t) outs[1]++; else outs[0]++; }
                     if (!ok) break;
                     steps[t]++;
                     tc_fence_after();
@@ -478,9 +484,9 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         const uint32_t lane_off = (uint32_t)(quarter * 32) << 16;
         const uint32_t o_addr = tmem_base + lane_off + O_COL + t * O_STRIDE;
         bool ok = true;
-        uint32_t step = 0, it = 0;                               // softmax steps of this tile so far; items so far
+        uint32_t step = 0;                                       // softmax steps of this tile so far
         uint32_t G = 0;                                          // ROT: scores of earlier items (both tiles), as the MMA warp counts them
-        for (int k = 0, item = fetch(0); item >= 0 && ok; k++, it++) {
+        for (int k = 0, item = fetch(0); item >= 0 && ok; k++) {
             const int item_next = fetch(k + 1);
             const Item w = decode(item);
             item = item_next;
@@ -495,7 +501,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
                 const uint32_t sn = ROT ? G + (uint32_t)entries_before(w, t, j) : step;
                 const uint32_t sbuf = ROT ? sn % 3 : (uint32_t)t;
                 const uint32_t s_addr = tmem_base + lane_off + sbuf * 128;          // scores, and P over their first 64 columns
-                ok = mbar_wait(s_full + 8 * sbuf, (ROT ? sn / 3 : sn) & 1, abort_flag, p.status, kErrEpilogueWait);
+                ok = mbar_wait(s_full + 8 * (4 * t + (ROT ? step & 3 : 0)), (ROT ? step >> 2 : step) & 1, abort_flag, p.status, kErrEpilogueWait);
                 if (!ok) break;
                 tc_fence_after();
                 // row r of the tile sees the keys of this tile up to column r + delta
@@ -647,7 +653,8 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             if (n_kv > 0) {
                 float inv = 1.0f / l;
                 if (!WIN && p.gate && qrow < p.T) inv *= 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[((long long)bb * p.T + qrow) * p.ld_gate + hh])));
-                const __nv_bfloat16* grow = WIN && p.gate && qrow < p.T ? p.gate + ((long long)bb * p.T + qrow) * p.ld_gate + (long long)hh * p.V : nullptr;
+                // (rows past the sequence read its last row's, so that the warp stays together: the TMEM loads below are warp-wide)
+                const __nv_bfloat16* grow = WIN && p.gate ? p.gate + ((long long)bb * p.T + min(qrow, p.T - 1)) * p.ld_gate + (long long)hh * p.V : nullptr;
                 uint4 graw[4];                                   // the next 32 columns' gates, requested ahead of the output they meet
                 auto fetch_gates = [&](int c) {
 #pragma unroll
@@ -667,6 +674,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
                 for (int c = 0; c < VD / 32; c++) {
                     uint32_t o[32];
+                    __syncwarp();                                // lanes that stored and lanes that did not
                     tmem_ld_32x32(o_addr + c * 32, o);
                     tmem_ld_wait();
                     if constexpr (WIN) {
@@ -699,7 +707,7 @@ attn_fused_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             }
             tc_fence_before();
             __syncwarp();
-            if (lane == 0) mbar_arrive(o_free + 8 * t);              // the accumulator may be overwritten by the next item
+            if (lane == 0 && n_kv > 0) mbar_arrive(o_free + 8 * t);      // the accumulator may be overwritten by the next item
         }
     }
 

@@ -1037,8 +1037,8 @@ int sptorch_ext_linear(const void* x, const void* w, const void* bias, const voi
     if (M > INT32_MAX || N > INT32_MAX || K > INT32_MAX) return fail("linear: dimension too large");
     if (ldo == 0) ldo = N;
     if (ldo < N) return fail("linear: ldo < N");
-    if (epilogue != SPT_EPI_NONE && epilogue != SPT_EPI_GELU && epilogue != SPT_EPI_SWIGLU) return fail("linear: unknown epilogue %d", epilogue);
-    if (epilogue == SPT_EPI_SWIGLU && !residual) return fail("linear: the SwiGLU epilogue multiplies by the residual operand, which is null");
+    if (epilogue < SPT_EPI_NONE || epilogue > SPT_EPI_GELU_MUL) return fail("linear: unknown epilogue %d", epilogue);
+    if (epilogue_multiplies(epilogue) && !residual) return fail("linear: a gated epilogue multiplies by the residual operand, which is null");
     if (mode == SPT_MM_F32 || K == 0) {
         if (out_dtype != SPT_F32 || ldo != N) return fail("linear: the CUDA-core f32 mode needs f32 output with ldo == N");
         return simt_matmul_f32((const float*)x, (const float*)w, (float*)out, 1, (int)M, (int)N, (int)K, false, (const float*)bias,

@@ -263,3 +263,17 @@ def test_fused_attention_when_the_last_query_tile_is_alone(backend, oracle, T):
         assert relerr(backend.attention_causal(q, k, v, H, dtype=BF16), ref) <= 2e-2
 
 
+@pytest.mark.parametrize("T", [40, 300, 600, 830])
+def test_fused_attention_items_with_and_without_a_second_query_tile(backend, oracle, T):
+    """T = 256 n + 1 .. 128 on more (sequence, head, tile pair) items than SMs: a CTA goes from an item with one query tile to items with
+    two, and the warps of the absent tile must neither start on the next item's scores early nor free its accumulator twice."""
+    rng = np.random.default_rng(T)
+    B, H, hd = 32, 12, 64
+    q, k, v = (_bf16(rng.standard_normal((B, T, H * hd)).astype(np.float32)) for _ in range(3))
+    ref = np.stack([_mha_core(oracle, q[i], k[i], v[i], H) for i in (0, B - 1)])
+    first = None
+    for _ in range(4):
+        out = np.asarray(backend.attention_causal(q, k, v, H, dtype=BF16))
+        assert relerr(out[[0, B - 1]], ref) <= 2e-2 and np.isfinite(out).all()
+        first = out if first is None else first
+        assert np.array_equal(out, first)
